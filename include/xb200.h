@@ -27,7 +27,7 @@
 extern "C" {
 #endif
 
-#define XB_ABI_VERSION 8
+#define XB_ABI_VERSION 9
 
 typedef struct xb_engine xb_engine;
 
@@ -224,15 +224,19 @@ enum {
                                  RMS-normed per head */
   XB_MIX_LATENT = 3,   /* softmax attention over a cached latent: keys and values are per-head up-projections of one
                           RMS-normed vector of m_kv_rank numbers per token, plus one rotated key part of m_rot_dim numbers
-                          that all heads share (interleaved rotary pairs on its first m_rot_dims entries, base
-                          m_rot_base); causal; the cache holds the latent and the rotated part only */
+                          that all heads share (rotary pairs on its first m_rot_dims entries, base m_rot_base, pair layout
+                          m_rot_pairs, frequencies rescaled per m_rot_scaling, cos and sin times m_rot_mult); causal; the
+                          cache holds the latent and the rotated part only.  Options: queries through a normed latent of
+                          their own of m_q_rank numbers; a window (a query sees the m_window newest keys, its own
+                          included); a sigmoid gate per head on the output (m_gate); the cache rows of an earlier layer in
+                          place of rows of its own (m_kv_from) */
   XB_MIX_GDELTA = 4,   /* delta rule with a decay and a removal rate per head and key channel:
                           S <- diag(w) S - (a*u)(u^T S) + k v^T, o = S^T r; w = exp(-e^-1/2 sigmoid(W2 tanh(W1 h) + w0))
                           (W1 of m_rank rows), a = sigmoid(.), u = unit k; read-out RMS-normed per head, weighted, gated
                           by sigmoid(g) */
   XB_MIX_LIGHTNING = 5,/* linear attention with a constant decay per head: S <- decay S + k v^T, o = S^T q, SiLU on
                           q, k, v; read-out RMS-normed over all heads together, weighted, gated by sigmoid(g) */
-  XB_MIX_SOFTMAX = 6   /* causal grouped-query softmax attention over every earlier key, keys and values of different
+  XB_MIX_SOFTMAX = 6,  /* causal grouped-query softmax attention over every earlier key, keys and values of different
                           sizes, rotary positions on the first s_rot_dims entries of each query / key head (pairs
                           (i, i + dims/2) or (2i, 2i+1), frequencies base^(-2i/dims) rescaled per XB_ROT_SCALE_*, cos and
                           sin times s_rot_mult).  Each of these is switched by its field: a learned sink per head in the
@@ -245,9 +249,12 @@ enum {
                           projection (s_v_is_k); queries multiplied by 1 + coef ln(floor((pos + 1) / every) + 1)
                           (s_qtemp_*); r1_h ln(1 + r2_h (i - j)) taken off the score of query i and key j, two numbers
                           per head (s_dist_bias) */
+  XB_MIX_GLA = 7       /* gated linear attention: S <- diag(w) S + k v^T, o = S^T q m_dim^-1/2, a decay per head and key channel
+                          w = sigmoid(W2 (W1 h) + b)^(1 / m_tau) (W1 of m_rank rows); read-out RMS-normed per head with one
+                          weight vector for all heads, gated by SiLU(g) */
 };
 
-/* how the rotary frequencies f_i = base^(-2i/dims) of XB_MIX_SOFTMAX are rescaled (l_i = 2 pi / f_i) */
+/* how the rotary frequencies f_i = base^(-2i/dims) of XB_MIX_SOFTMAX and XB_MIX_LATENT are rescaled (l_i = 2 pi / f_i) */
 enum {
   XB_ROT_SCALE_NONE = 0,
   XB_ROT_SCALE_BANDS = 1, /* f kept where l < orig / p1, f / factor where l > orig / p0, between them a blend with
@@ -260,16 +267,19 @@ enum {
 enum {
   XB_FF_RELU2 = 0,     /* down(relu(up h)^2) */
   XB_FF_GLU_CLAMP = 1, /* down(g sigmoid(1.702 g) (u + 1)), g = min(gate h, limit), u = clamp(up h, -limit, limit); biases */
+  XB_FF_GLU = 3,       /* down(act(gate h) * up h) with ff_act, no biases */
   XB_FF_MOE = 2        /* n_experts such feed-forwards without biases, each token uses `top` of them: sigmoid router scores,
                           experts in `groups` equal groups of neighbours, a group scores the sum of its two best experts and
                           only the `keep_groups` best groups stay eligible; weights = scores * route_scale; plus an
-                          always-on shared expert of width shared_ff (0 = none) */
+                          always-on shared expert of width shared_ff (0 = none), optionally times sigmoid of one
+                          number per token (shared_gate) */
 };
-/* what an expert of XB_FF_MOE computes (ff_act) */
+/* what an expert of XB_FF_MOE or the dense XB_FF_GLU computes (ff_act) */
 enum {
   XB_ACT_GLU_CLAMP = 0,   /* down(g sigmoid(1.702 g) (u + 1)) with the limits above */
   XB_ACT_SWIGLU = 1,      /* down(silu(g) u), no limits */
-  XB_ACT_GELU = 2         /* down(gelu(up h)): no gate projection, the exact (erf) form 0.5 z (1 + erf(z / sqrt 2)) */
+  XB_ACT_GELU = 2,        /* down(gelu(up h)): no gate projection, the exact (erf) form 0.5 z (1 + erf(z / sqrt 2)) */
+  XB_ACT_GEGLU = 3        /* down(gelu(g) u), gelu in the tanh form 0.5 z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3))) */
 };
 /* how the router of XB_FF_MOE turns logits into scores, what a group of experts is worth, and what weight a chosen expert
  * gets (route_score, group_score, route_norm) */
@@ -289,8 +299,9 @@ typedef struct xb_hybrid_layer {
   /* XB_MIX_LATENT / XB_MIX_GDELTA / XB_MIX_LIGHTNING: heads, per-head key size (unrotated part for LATENT), value size
    * (GDELTA: = m_dim), and for LATENT the rotated part, the latent's size and how many entries of the rotated part turn */
   int32_t m_heads, m_dim, m_vdim, m_rot_dim, m_kv_rank, m_rot_dims;
-  int32_t m_rank;                                   /* GDELTA: rows of the decay's first projection */
-  float m_scale, m_rot_base;                        /* LATENT: score scale, rotary base */
+  int32_t m_rank;                                   /* GDELTA, GLA: rows of the decay's first projection */
+  float m_scale;                                    /* LATENT: score scale */
+  double m_rot_base;                                /* LATENT: rotary base */
   int32_t ff_kind;                                  /* XB_FF_* (ff = width of the dense feed-forward or of one expert) */
   float ff_limit;
   int32_t n_experts, top, groups, keep_groups, shared_ff;   /* XB_FF_MOE; groups 0 = no group limit */
@@ -315,6 +326,18 @@ typedef struct xb_hybrid_layer {
   int32_t route_score, group_score;                 /* XB_FF_MOE: XB_ROUTE_*, XB_GROUP_* */
   int32_t route_norm;                               /* XB_FF_MOE: 1 = the chosen experts' weights are their scores divided by
                                                        the sum of the chosen scores (+ 1e-20), then times route_scale */
+  int32_t shared_gate;                              /* XB_FF_MOE: 1 = the shared expert's output is multiplied by the sigmoid
+                                                       of one number per token (row "shared.sg") */
+  float m_tau;                                      /* GLA: the decay is a sigmoid to the power 1 / m_tau */
+  int32_t m_q_rank;                                 /* LATENT: > 0 = queries are up-projections ("uq") of an RMS-normed latent
+                                                       of this size ("dq", "dq.norm"); 0 = projected directly ("q") */
+  int32_t m_window;                                 /* LATENT: a query sees the m_window newest keys; 0 = all earlier ones */
+  int32_t m_gate;                                   /* LATENT: 1 = head h's output is multiplied by sigmoid(row h of "g") */
+  int32_t m_kv_from;                                /* LATENT: >= 0 = no "dkv" of its own, the cache rows of that earlier layer
+                                                       (same latent and rotated sizes); -1: its own rows */
+  int32_t m_rot_pairs, m_rot_scaling;               /* LATENT: XB_ROPE_* pair layout, XB_ROT_SCALE_* */
+  float m_rot_mult;                                 /* LATENT: cos / sin multiplier (0 = 1) */
+  double m_rot_factor, m_rot_orig, m_rot_p0, m_rot_p1;
 } xb_hybrid_layer;
 
 typedef struct xb_hybrid_desc {
@@ -345,12 +368,20 @@ typedef struct xb_hybrid_desc {
                                         last row.  The previous token of a sequence is part of its slot's state */
   int32_t bigram_mul_prev, bigram_mul_cur;
   int32_t pos_rows;                  /* > 0: row `position` of the learned table "pos" [pos_rows, dim] joins the embedding */
+  int32_t norm_kind;                 /* XB_NORM_*: what the stream's norms compute (pre-norm blocks; others: XB_NORM_RMS) */
 } xb_hybrid_desc;
+
+enum {
+  XB_NORM_RMS = 0,
+  XB_NORM_TANH = 1        /* tanh(a x) * w + b, channel by channel, no statistics of the row: tensors "<name>" (w), "<name>.b" and
+                             the single number "<name>.alpha" */
+};
 
 enum {
   XB_BLOCK_SANDWICH = 0,  /* mixer, then feed-forward, each reading its own norm through a causal filter, each branch
                              normed before it is added; optional token side input (the Refatar layout) */
   XB_BLOCK_PARALLEL = 1,  /* one norm per layer; mixer and feed-forward read it and their sum is added: x += mix(h) + ff(h) */
+  XB_BLOCK_PRENORM = 3,   /* x += mix(norm1(x)), then x += ff(norm2(x)); plain norm weights */
   XB_BLOCK_BRANCHNORM = 2 /* no norm in front: each sublayer reads the stream itself and only its output is normed,
                              x += n1 unit(mix(x)), then x += n2 unit(ff(x)), unit(y) = y / rms(y), n1 / n2 single numbers
                              ("l<i>.norm1", ".norm2"; norm_scalar = 1); optional sigmoid gate on the output (gated_residual) */

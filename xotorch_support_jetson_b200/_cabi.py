@@ -37,7 +37,7 @@ class ModelDesc(C.Structure):
   ]
 
 
-ABI_VERSION = 8
+ABI_VERSION = 9
 
 
 def model_desc(**fields) -> ModelDesc:
@@ -45,14 +45,15 @@ def model_desc(**fields) -> ModelDesc:
   return ModelDesc(struct_size=C.sizeof(ModelDesc), **fields)
 
 
-MIX_DELTA, MIX_PARALLEL, MIX_LATENT, MIX_GDELTA, MIX_LIGHTNING, MIX_SOFTMAX = 1, 2, 3, 4, 5, 6
+MIX_DELTA, MIX_PARALLEL, MIX_LATENT, MIX_GDELTA, MIX_LIGHTNING, MIX_SOFTMAX, MIX_GLA = 1, 2, 3, 4, 5, 6, 7
 ROT_SCALE_NONE, ROT_SCALE_BANDS, ROT_SCALE_RAMP = 0, 1, 2
-ACT_GLU_CLAMP, ACT_SWIGLU, ACT_GELU = 0, 1, 2
+ACT_GLU_CLAMP, ACT_SWIGLU, ACT_GELU, ACT_GEGLU = 0, 1, 2, 3
 ROUTE_SIGMOID, ROUTE_SOFTMAX = 0, 1
 GROUP_TOP2, GROUP_MAX = 0, 1
 SINK_NONE, SINK_LEARNED, SINK_UNIT = 0, 1, 2
-FF_RELU2, FF_GLU_CLAMP, FF_MOE = 0, 1, 2
-BLOCK_SANDWICH, BLOCK_PARALLEL, BLOCK_BRANCHNORM = 0, 1, 2
+FF_RELU2, FF_GLU_CLAMP, FF_MOE, FF_GLU = 0, 1, 2, 3
+BLOCK_SANDWICH, BLOCK_PARALLEL, BLOCK_BRANCHNORM, BLOCK_PRENORM = 0, 1, 2, 3
+NORM_RMS, NORM_TANH = 0, 1
 ST_BF16, ST_F16, ST_F32 = 0, 1, 2   # element types xb_load_named accepts
 
 
@@ -66,7 +67,7 @@ class HybridLayer(C.Structure):
     ("r_heads", C.c_int32), ("r_dim", C.c_int32), ("r_vdim", C.c_int32),
     ("left_scale", C.c_float), ("right_scale", C.c_float),
     ("m_heads", C.c_int32), ("m_dim", C.c_int32), ("m_vdim", C.c_int32), ("m_rot_dim", C.c_int32), ("m_kv_rank", C.c_int32),
-    ("m_rot_dims", C.c_int32), ("m_rank", C.c_int32), ("m_scale", C.c_float), ("m_rot_base", C.c_float),
+    ("m_rot_dims", C.c_int32), ("m_rank", C.c_int32), ("m_scale", C.c_float), ("m_rot_base", C.c_double),
     ("ff_kind", C.c_int32), ("ff_limit", C.c_float),
     ("n_experts", C.c_int32), ("top", C.c_int32), ("groups", C.c_int32), ("keep_groups", C.c_int32), ("shared_ff", C.c_int32),
     ("route_scale", C.c_float), ("shared_limit", C.c_float),
@@ -81,6 +82,9 @@ class HybridLayer(C.Structure):
     ("s_qkv_bias", C.c_int32), ("s_qk_norm", C.c_int32), ("s_v_is_k", C.c_int32), ("s_dist_bias", C.c_int32),
     ("s_qtemp_every", C.c_int32), ("s_qtemp_coef", C.c_float),
     ("route_score", C.c_int32), ("group_score", C.c_int32), ("route_norm", C.c_int32),
+    ("shared_gate", C.c_int32), ("m_tau", C.c_float), ("m_q_rank", C.c_int32), ("m_window", C.c_int32), ("m_gate", C.c_int32),
+    ("m_kv_from", C.c_int32), ("m_rot_pairs", C.c_int32), ("m_rot_scaling", C.c_int32), ("m_rot_mult", C.c_float),
+    ("m_rot_factor", C.c_double), ("m_rot_orig", C.c_double), ("m_rot_p0", C.c_double), ("m_rot_p1", C.c_double),
   ]
 
 
@@ -94,7 +98,7 @@ class HybridDesc(C.Structure):
     ("norm_groups", C.c_int32), ("norm_plain", C.c_int32), ("residual_mult", C.c_float), ("tied_head", C.c_int32),
     ("ff_unfiltered", C.c_int32),
     ("gated_residual", C.c_int32), ("bigram_buckets", C.c_int32), ("bigram_mul_prev", C.c_int32), ("bigram_mul_cur", C.c_int32),
-    ("pos_rows", C.c_int32),
+    ("pos_rows", C.c_int32), ("norm_kind", C.c_int32),
   ]
 
 

@@ -14,7 +14,7 @@ CSRC = PKG / "csrc"
 LIB = PKG / "libxb200.so"
 
 NVCC_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-O3", "-lineinfo", "-std=c++17",
-              "-shared", "-Xcompiler", "-fPIC"]
+              "-shared", "-Xcompiler", "-fPIC", "--split-compile=0"]   # 0: the optimiser runs on every core
 
 
 def find_nvcc() -> str:

@@ -41,15 +41,20 @@ struct HyLayer {
   int off_dkv = 0, off_r = 0, off_w1 = 0;   // more columns of the fused input projection
   int n_up = 0, n_dn = 0;                   // rows of the fused up projection, inputs of the down projection
   bf16 *w_uk = nullptr, *w_uv = nullptr, *w_d2 = nullptr, *w_router = nullptr, *t_d2 = nullptr;
-  float *b_up = nullptr, *b_down = nullptr, *lat_norm = nullptr, *rot_freq = nullptr, *w0 = nullptr, *hdecay = nullptr;
+  float *b_up = nullptr, *b_down = nullptr, *lat_norm = nullptr, *w0 = nullptr, *hdecay = nullptr;
+  bf16 *w_uq = nullptr, *t_uq = nullptr;    // latent attention: up-projection of the queries' own latent
+  float *dq_norm = nullptr;
+  int off_dq = 0;
   int owner = -1;                           // layer whose tensors this one uses (weights_of), -1: its own
   // rotary-position attention (XB_MIX_SOFTMAX)
   float *sink = nullptr, *talk = nullptr, *vmix = nullptr;
-  double* rot_freq_d = nullptr;             // [s_rot_dims / 2] rescaled frequencies
+  double* rot_freq_d = nullptr;             // [rotating entries / 2] rescaled frequencies (softmax and latent attention)
   int vmode = 0;                            // 0: values as projected; 1: leaves its values for later layers; 2: blends with them
   bool v_all = false;                       // a value row of the pool holds every key head ([page][token][G * dv])
   // whole-projection q / k norm weights, the distance penalty's two numbers per head (XB_MIX_SOFTMAX options)
   float *qn = nullptr, *kn = nullptr, *r1 = nullptr, *r2 = nullptr;
+  // tanh norms of the stream: offset per channel and the factor on the input beside norm1 / norm2
+  float *norm1_b = nullptr, *norm1_a = nullptr, *norm2_b = nullptr, *norm2_a = nullptr;
   // gated residual: the gate's rows sit behind the mixer's in w_in (off_rg) and behind the experts' in w_up (off_rg2)
   int off_rg = -1, off_rg2 = -1;
 };
@@ -60,7 +65,7 @@ struct HyModel {
   bf16 *embed = nullptr, *side_embed = nullptr, *head = nullptr;
   bf16 *bigram = nullptr, *pos_tab = nullptr;   // hashed token-pair rows [buckets + 1, dim], learned position rows [pos_rows, dim]
   size_t st_prev = 0;                           // float offset of a slot's previous token (its bits) inside the slot's state
-  float* final_norm = nullptr;
+  float *final_norm = nullptr, *final_norm_b = nullptr, *final_norm_a = nullptr;
   float* state = nullptr;
   size_t state_floats = 0;   // per slot
   float *x = nullptr, *hn = nullptr, *P = nullptr, *c = nullptr, *o = nullptr, *m1 = nullptr, *m2 = nullptr, *beta = nullptr,
@@ -82,7 +87,7 @@ struct HyModel {
   int use_lat_mma = 1;                 // XB_HY_LAT_MMA: 0 = latent attention through the per-(token, head) kernel everywhere (A/B)
   size_t maxLatR = 0;
   float *qa = nullptr, *gw = nullptr;   // latent attention: queries in the cache's space [T, H * (rank + rot)]; experts: weights [T, E]
-  void* ah = nullptr;                  // parallel blocks: the normed stream as a Linear input (both sublayers read it)
+  void* ah = nullptr;                  // parallel and pre-norm blocks: the normed stream as a Linear input
   size_t maxQA = 0, maxE = 0, maxM = 0;   // maxM: widest matrix that passes through the m1 / m2 buffers besides the stream's width
   float* vfirst = nullptr;              // values of the first blending layer for the tokens of this step [T, G * dv]
   size_t maxGV = 0;
@@ -123,14 +128,17 @@ static void hy_name_rows(HyModel* hy, const std::string& name, bf16* base, long 
 }
 static void hy_name_vec(HyModel* hy, const std::string& name, float* dst, long long n) { hy_name(hy, name, dst, true, 1, n, n, 1); }
 
+// a latent attention layer that reads the cache rows of an earlier one has no pool of its own
+static bool hy_borrows_rows(const HyLayer& l) { return l.d.mixer == XB_MIX_LATENT && l.d.m_kv_from >= 0; }
+
 static void hy_destroy(HyModel* hy) {
   if (hy == nullptr) return;
   for (void* p : hy->allocs) cudaFree(p);
   for (HyLayer& l : hy->L) {
-    cudaFree(l.k_pool); cudaFree(l.v_pool);
+    if (!hy_borrows_rows(l)) { cudaFree(l.k_pool); cudaFree(l.v_pool); }
     if (l.owner >= 0) continue;   // the tile-major copies belong to the layer that owns the tensors
     cudaFree(l.t_in); cudaFree(l.t_o); cudaFree(l.t_o2); cudaFree(l.t_up); cudaFree(l.t_down); cudaFree(l.t_sgate); cudaFree(l.t_sproj);
-    cudaFree(l.t_d2);
+    cudaFree(l.t_d2); cudaFree(l.t_uq);
   }
   cudaFree(hy->t_head);
   cudaFree(hy->state);
@@ -143,7 +151,56 @@ static void hy_name_cols(HyModel* hy, const std::string& name, bf16* base, long 
   hy_name(hy, name, base + col0, false, rows, cols, ld, 2);
 }
 
-// Mixers of the parallel-block designs.  own: the layer has tensors of its own (else only cache / state is laid out).
+// A norm of the stream: one vector (or one number), for the tanh norm also an offset per channel and the input's factor.
+static int hy_create_norm(HyModel* hy, const std::string& name, float** w, float** b, float** a) {
+  const size_t D = hy->d.dim, nd = hy->d.norm_scalar ? 1 : D;
+  XB_TRY(hy_alloc_t(hy, w, nd));
+  hy_name_vec(hy, name, *w, nd);
+  if (hy->d.norm_kind == XB_NORM_TANH) {
+    XB_TRY(hy_alloc_t(hy, b, D)); hy_name_vec(hy, name + ".b", *b, D);
+    XB_TRY(hy_alloc_t(hy, a, 1)); hy_name_vec(hy, name + ".alpha", *a, 1);
+  }
+  return 0;
+}
+
+// Rotary frequencies f_j = base^(-2j/dims), j < dims / 2, rescaled (xb200.h: XB_ROT_SCALE_*), made in double on the host.
+static int hy_rot_frequencies(HyModel* hy, int i, int dims, double base, int scaling, double fac, double orig, double p0, double p1, double** out) {
+  const int half = dims / 2;
+  std::vector<double> fr((size_t)(half > 0 ? half : 1), 0.0);
+  const double two_pi = 6.283185307179586476925286766559;
+  XB_CHECK(half <= HY_MAX_ROT_PAIRS, "layer %d: %d rotating entries (at most %d)", i, dims, 2 * HY_MAX_ROT_PAIRS);
+  XB_CHECK(half == 0 || base > 1.0, "layer %d: rotary base %g", i, base);
+  XB_CHECK(scaling == XB_ROT_SCALE_NONE || (fac > 0.0 && orig > 0.0), "layer %d: bad rotary scaling constants", i);
+  double lo = 0.0, hi = 0.0;
+  if (scaling == XB_ROT_SCALE_RAMP && half > 0) {
+    XB_CHECK(p0 > 0.0 && p1 > 0.0, "layer %d: bad rotary ramp constants", i);
+    auto at = [&](double t) { return (double)dims * log(orig / (two_pi * t)) / (2.0 * log(base)); };
+    lo = floor(at(p0)); lo = lo < 0.0 ? 0.0 : lo;
+    hi = ceil(at(p1)); hi = hi > (double)(dims - 1) ? (double)(dims - 1) : hi;
+  }
+  for (int j = 0; j < half; ++j) {
+    double f = pow(base, -2.0 * j / (double)dims);
+    if (scaling == XB_ROT_SCALE_BANDS) {
+      XB_CHECK(p1 != p0 && p0 > 0.0 && p1 > 0.0, "layer %d: bad rotary band constants", i);
+      const double wl = two_pi / f;
+      if (wl < orig / p1) { /* kept */ }
+      else if (wl > orig / p0) f = f / fac;
+      else { const double sm = (orig / wl - p0) / (p1 - p0); f = (1.0 - sm) * f / fac + sm * f; }
+    } else if (scaling == XB_ROT_SCALE_RAMP) {
+      double r = ((double)j - lo) / (hi - lo > 0.001 ? hi - lo : 0.001);
+      r = r < 0.0 ? 0.0 : (r > 1.0 ? 1.0 : r);
+      f = f / fac * r + f * (1.0 - r);
+    } else {
+      XB_CHECK(scaling == XB_ROT_SCALE_NONE, "layer %d: unknown rotary scaling %d", i, scaling);
+    }
+    fr[j] = f;
+  }
+  XB_TRY(hy_alloc_t(hy, out, fr.size()));
+  XB_CUDA(cudaMemcpy(*out, fr.data(), fr.size() * sizeof(double), cudaMemcpyHostToDevice));
+  return 0;
+}
+
+// Mixers of the parallel-block and pre-norm designs.  own: the layer has tensors of its own (else only cache / state is laid out).
 static int hy_create_mixer(xb_engine* e, int i, bool own, size_t& st, uint64_t& wbytes, uint64_t& kvpos) {
   HyModel* hy = e->hy;
   HyLayer& l = hy->L[i];
@@ -158,8 +215,23 @@ static int hy_create_mixer(xb_engine* e, int i, bool own, size_t& st, uint64_t& 
     XB_CHECK(dr >= 0 && dv > 0 && R > 0 && R <= 512, "layer %d: bad latent attention sizes (latent of at most 512 numbers)", i);
     XB_CHECK(c.m_rot_dims >= 0 && c.m_rot_dims <= dr && c.m_rot_dims % 2 == 0, "layer %d: %d rotating entries do not fit a part of %lld", i,
              c.m_rot_dims, dr);
-    l.off_q = 0; l.off_dkv = (int)(H * (n + dr));
-    l.n_in = l.off_dkv + (int)(R + dr);
+    const long long qr = c.m_q_rank;
+    const bool rows = c.m_kv_from < 0;    // makes cache rows of its own
+    XB_CHECK(qr >= 0 && c.m_window >= 0 && c.m_scale > 0.f, "layer %d: bad latent attention constants (query rank %lld, window %d, scale %g)", i, qr,
+             c.m_window, c.m_scale);
+    XB_CHECK(c.m_rot_pairs == XB_ROPE_INTERLEAVED || c.m_rot_pairs == XB_ROPE_HALF_SPLIT, "layer %d: unknown rotary pair layout %d", i, c.m_rot_pairs);
+    XB_CHECK(own || (qr == 0 && c.m_gate == 0 && rows), "layer %d: a query latent, head gates and borrowed cache rows come with tensors of their own", i);
+    if (!rows) {
+      XB_CHECK(c.m_kv_from < i && hy->L[c.m_kv_from].d.mixer == XB_MIX_LATENT && hy->L[c.m_kv_from].d.m_kv_from < 0,
+               "layer %d: kv_from %d must name an earlier latent attention layer with rows of its own", i, c.m_kv_from);
+      const xb_hybrid_layer& o = hy->L[c.m_kv_from].d;
+      XB_CHECK(o.m_kv_rank == c.m_kv_rank && o.m_rot_dim == c.m_rot_dim, "layer %d: its cache rows are not the size of layer %d's", i, c.m_kv_from);
+    }
+    l.off_q = l.off_dq = 0;
+    l.n_in = (int)(qr > 0 ? qr : H * (n + dr));
+    l.off_dkv = rows ? l.n_in : -1;
+    if (rows) l.n_in += (int)(R + dr);
+    if (c.m_gate) { l.off_g = l.n_in; l.n_in += (int)H; }
     if (d.gated_residual) { l.off_rg = l.n_in; l.n_in += (int)D; }
     l.n_o = (int)(H * dv);
     if (own) {
@@ -169,24 +241,62 @@ static int hy_create_mixer(xb_engine* e, int i, bool own, size_t& st, uint64_t& 
       XB_TRY(hy_alloc_t(hy, &l.w_uk, (size_t)(H * n * R)));
       XB_TRY(hy_alloc_t(hy, &l.w_uv, (size_t)(H * dv * R)));
       XB_TRY(hy_alloc_t(hy, &l.lat_norm, (size_t)R));
-      hy_name_rows(hy, p + "q", l.w_in, l.off_q, H * (n + dr), D);
-      hy_name_rows(hy, p + "dkv", l.w_in, l.off_dkv, R + dr, D);
-      hy_name_vec(hy, p + "dkv.norm", l.lat_norm, R);
+      if (qr > 0) {
+        XB_TRY(hy_alloc_t(hy, &l.w_uq, (size_t)(H * (n + dr) * qr)));
+        XB_TRY(hy_alloc_t(hy, &l.dq_norm, (size_t)qr));
+        hy_name_rows(hy, p + "dq", l.w_in, l.off_dq, qr, D);
+        hy_name_vec(hy, p + "dq.norm", l.dq_norm, qr);
+        hy_name_rows(hy, p + "uq", l.w_uq, 0, H * (n + dr), qr);
+        wbytes += (size_t)(H * (n + dr) * qr) * 2;
+      } else {
+        hy_name_rows(hy, p + "q", l.w_in, l.off_q, H * (n + dr), D);
+      }
+      if (rows) {
+        hy_name_rows(hy, p + "dkv", l.w_in, l.off_dkv, R + dr, D);
+        hy_name_vec(hy, p + "dkv.norm", l.lat_norm, R);
+      }
+      if (c.m_gate) hy_name_rows(hy, p + "g", l.w_in, l.off_g, H, D);
       hy_name_rows(hy, p + "uk", l.w_uk, 0, H * n, R);
       hy_name_rows(hy, p + "uv", l.w_uv, 0, H * dv, R);
       hy_name_rows(hy, p + "o", l.w_o, 0, D, l.n_o);
-      const int half = c.m_rot_dims / 2;
-      std::vector<float> fr((size_t)(half > 0 ? half : 1), 0.f);
-      for (int j = 0; j < half; ++j) fr[j] = (float)pow((double)c.m_rot_base, -2.0 * j / (double)c.m_rot_dims);
-      XB_TRY(hy_alloc_t(hy, &l.rot_freq, fr.size()));
-      XB_CUDA(cudaMemcpy(l.rot_freq, fr.data(), fr.size() * sizeof(float), cudaMemcpyHostToDevice));
+      XB_TRY(hy_rot_frequencies(hy, i, c.m_rot_dims, c.m_rot_base, c.m_rot_scaling, c.m_rot_factor, c.m_rot_orig, c.m_rot_p0, c.m_rot_p1, &l.rot_freq_d));
       wbytes += ((size_t)l.n_in * D + D * l.n_o + (size_t)(H * (n + dv) * R)) * 2;
     }
     const size_t qa = (size_t)(H * (R + dr)), ol = (size_t)(H * R);
     if (qa > hy->maxQA) hy->maxQA = qa;
     if ((size_t)R > hy->maxLatR) hy->maxLatR = R;
     if (ol > hy->maxO) hy->maxO = ol;
-    kvpos += (uint64_t)(R + dr) * (d.compute_fp32 ? 4 : 2);
+    if (qr > 0) {
+      if ((size_t)(H * (n + dr)) > hy->maxM) hy->maxM = H * (n + dr);
+      if ((size_t)qr > hy->maxK) hy->maxK = qr;
+    }
+    if (rows) kvpos += (uint64_t)(R + dr) * (d.compute_fp32 ? 4 : 2);
+  } else if (c.mixer == XB_MIX_GLA) {
+    const long long dv = c.m_vdim, rk = c.m_rank, HK = H * n, HV = H * dv;
+    XB_CHECK(n <= HY_MAX_KDIM && dv > 0 && rk > 0 && rk <= HY_MAX_DECAY_RANK, "layer %d: bad gated linear attention sizes (key dim <= %d, decay rank <= %d)", i,
+             HY_MAX_KDIM, HY_MAX_DECAY_RANK);
+    XB_CHECK(own && c.m_tau > 0.f, "layer %d: gated linear attention keeps tensors of its own; tau %g", i, c.m_tau);
+    l.off_q = 0; l.off_k = (int)HK; l.off_v = (int)(2 * HK); l.off_g = (int)(2 * HK + HV); l.off_a = (int)(2 * HK + 2 * HV);
+    l.n_in = l.off_a + (int)rk;
+    l.n_o = (int)HV;
+    XB_TRY(hy_alloc_t(hy, &l.w_in, (size_t)l.n_in * D));
+    XB_TRY(hy_alloc_t(hy, &l.w_o, D * l.n_o));
+    XB_TRY(hy_alloc_t(hy, &l.w_d2, (size_t)(HK * rk)));
+    XB_TRY(hy_alloc_t(hy, &l.w0, (size_t)HK));
+    XB_TRY(hy_alloc_t(hy, &l.head_norm, (size_t)dv));
+    hy_name_rows(hy, p + "q", l.w_in, l.off_q, HK, D);
+    hy_name_rows(hy, p + "k", l.w_in, l.off_k, HK, D);
+    hy_name_rows(hy, p + "v", l.w_in, l.off_v, HV, D);
+    hy_name_rows(hy, p + "g", l.w_in, l.off_g, HV, D);
+    hy_name_rows(hy, p + "a1", l.w_in, l.off_a, rk, D);
+    hy_name_rows(hy, p + "a2", l.w_d2, 0, HK, rk);
+    hy_name_vec(hy, p + "a2.b", l.w0, HK);
+    hy_name_vec(hy, p + "norm", l.head_norm, dv);
+    hy_name_rows(hy, p + "o", l.w_o, 0, D, l.n_o);
+    wbytes += ((size_t)l.n_in * D + D * l.n_o + (size_t)(HK * rk)) * 2;
+    l.st_rec = st; st += (size_t)(HV * n);
+    if ((size_t)(3 * HK + HV) > hy->maxC) hy->maxC = 3 * HK + HV;
+    if ((size_t)l.n_o > hy->maxO) hy->maxO = l.n_o;
   } else if (c.mixer == XB_MIX_GDELTA) {
     const long long HN = H * n, rk = c.m_rank;
     XB_CHECK(n <= HY_MAX_KDIM && rk > 0, "layer %d: bad delta-rule sizes (key dim <= %d)", i, HY_MAX_KDIM);
@@ -266,7 +376,6 @@ static int hy_create_softmax(xb_engine* e, int i, bool own, uint64_t& wbytes, ui
   XB_CHECK(!prep2 || (size_t)((H + G) * dk) * sizeof(float) <= 48 * 1024, "layer %d: %lld query and key channels per token (at most 12288)", i, (H + G) * dk);
   XB_CHECK(c.s_qtemp_every >= 0 && c.s_sink >= XB_SINK_NONE && c.s_sink <= XB_SINK_UNIT, "layer %d: bad query temperature step %d / sink kind %d", i, c.s_qtemp_every, c.s_sink);
   XB_CHECK(rd >= 0 && rd <= dk && rd % 2 == 0, "layer %d: %lld rotating entries do not fit a head of %lld", i, rd, dk);
-  XB_CHECK(rd / 2 <= HY_MAX_ROT_PAIRS, "layer %d: %lld rotating entries (at most %d)", i, rd, 2 * HY_MAX_ROT_PAIRS);
   XB_CHECK(c.s_rot_pairs == XB_ROPE_INTERLEAVED || c.s_rot_pairs == XB_ROPE_HALF_SPLIT, "layer %d: unknown rotary pair layout %d", i, c.s_rot_pairs);
   XB_CHECK(c.s_softcap >= 0.f && c.s_scale > 0.f, "layer %d: bad score scale %g / soft cap %g", i, c.s_scale, c.s_softcap);
   l.v_all = c.s_talk != 0 && G > 1;
@@ -301,39 +410,7 @@ static int hy_create_softmax(xb_engine* e, int i, bool own, uint64_t& wbytes, ui
   if (c.s_sink == XB_SINK_UNIT) XB_TRY(hy_alloc_t(hy, &l.sink, (size_t)H));   // a sink of score 0 per head: the zeros the allocation leaves
   if (c.s_talk) { XB_TRY(hy_alloc_t(hy, &l.talk, (size_t)(H * H))); hy_name(hy, p + "talk", l.talk, true, H, H, H, 2); }
   if (c.s_vmix) { XB_TRY(hy_alloc_t(hy, &l.vmix, 1)); hy_name_vec(hy, p + "vmix", l.vmix, 1); }
-  // frequencies f_j = base^(-2j/dims), rescaled (xb200.h: XB_ROT_SCALE_*)
-  const int half = (int)(rd / 2);
-  std::vector<double> fr((size_t)(half > 0 ? half : 1), 0.0);
-  const double base = c.s_rot_base, fac = c.s_rot_factor, orig = c.s_rot_orig, p0 = c.s_rot_p0, p1 = c.s_rot_p1;
-  const double two_pi = 6.283185307179586476925286766559;
-  XB_CHECK(half == 0 || base > 1.0, "layer %d: rotary base %g", i, base);
-  XB_CHECK(c.s_rot_scaling == XB_ROT_SCALE_NONE || (fac > 0.0 && orig > 0.0), "layer %d: bad rotary scaling constants", i);
-  double lo = 0.0, hi = 0.0;
-  if (c.s_rot_scaling == XB_ROT_SCALE_RAMP && half > 0) {
-    XB_CHECK(p0 > 0.0 && p1 > 0.0, "layer %d: bad rotary ramp constants", i);
-    auto at = [&](double t) { return (double)rd * log(orig / (two_pi * t)) / (2.0 * log(base)); };
-    lo = floor(at(p0)); lo = lo < 0.0 ? 0.0 : lo;
-    hi = ceil(at(p1)); hi = hi > (double)(rd - 1) ? (double)(rd - 1) : hi;
-  }
-  for (int j = 0; j < half; ++j) {
-    double f = pow(base, -2.0 * j / (double)rd);
-    if (c.s_rot_scaling == XB_ROT_SCALE_BANDS) {
-      XB_CHECK(p1 != p0 && p0 > 0.0 && p1 > 0.0, "layer %d: bad rotary band constants", i);
-      const double wl = two_pi / f;
-      if (wl < orig / p1) { /* kept */ }
-      else if (wl > orig / p0) f = f / fac;
-      else { const double sm = (orig / wl - p0) / (p1 - p0); f = (1.0 - sm) * f / fac + sm * f; }
-    } else if (c.s_rot_scaling == XB_ROT_SCALE_RAMP) {
-      double r = ((double)j - lo) / (hi - lo > 0.001 ? hi - lo : 0.001);
-      r = r < 0.0 ? 0.0 : (r > 1.0 ? 1.0 : r);
-      f = f / fac * r + f * (1.0 - r);
-    } else {
-      XB_CHECK(c.s_rot_scaling == XB_ROT_SCALE_NONE, "layer %d: unknown rotary scaling %d", i, c.s_rot_scaling);
-    }
-    fr[j] = f;
-  }
-  XB_TRY(hy_alloc_t(hy, &l.rot_freq_d, fr.size()));
-  XB_CUDA(cudaMemcpy(l.rot_freq_d, fr.data(), fr.size() * sizeof(double), cudaMemcpyHostToDevice));
+  XB_TRY(hy_rot_frequencies(hy, i, (int)rd, c.s_rot_base, c.s_rot_scaling, c.s_rot_factor, c.s_rot_orig, c.s_rot_p0, c.s_rot_p1, &l.rot_freq_d));
   const size_t qa = (size_t)(H * dk), ol = (size_t)(H * dvo);
   if (qa > hy->maxQA) hy->maxQA = qa;
   if (ol > hy->maxO) hy->maxO = ol;
@@ -355,8 +432,10 @@ static int hy_create_ff(xb_engine* e, int i, bool own, uint64_t& wbytes) {
   const xb_hybrid_layer& c = l.d;
   const size_t D = hy->d.dim, F = c.ff;
   const std::string p = "l" + std::to_string(i) + ".mlp.";
-  XB_CHECK(hy->d.block == XB_BLOCK_PARALLEL || c.ff_kind == XB_FF_MOE, "layer %d: the dense gated feed-forward belongs to parallel blocks", i);
-  XB_CHECK(c.ff_act == XB_ACT_GLU_CLAMP || c.ff_act == XB_ACT_SWIGLU || c.ff_act == XB_ACT_GELU, "layer %d: unknown expert activation %d", i, c.ff_act);
+  XB_CHECK(hy->d.block == XB_BLOCK_PARALLEL || hy->d.block == XB_BLOCK_PRENORM || c.ff_kind == XB_FF_MOE,
+           "layer %d: the dense gated feed-forwards belong to parallel and pre-norm blocks", i);
+  XB_CHECK(c.ff_act == XB_ACT_GLU_CLAMP || c.ff_act == XB_ACT_SWIGLU || c.ff_act == XB_ACT_GELU || c.ff_act == XB_ACT_GEGLU,
+           "layer %d: unknown activation %d", i, c.ff_act);
   XB_CHECK(c.ff_act != XB_ACT_GELU || (c.ff_kind == XB_FF_MOE && !c.route_input), "layer %d: the ungated GELU form serves experts weighted on their output", i);
   XB_CHECK((c.route_score == XB_ROUTE_SIGMOID || c.route_score == XB_ROUTE_SOFTMAX) && (c.group_score == XB_GROUP_TOP2 || c.group_score == XB_GROUP_MAX),
            "layer %d: unknown router score %d / group score %d", i, c.route_score, c.group_score);
@@ -372,8 +451,18 @@ static int hy_create_ff(xb_engine* e, int i, bool own, uint64_t& wbytes) {
       hy_name_rows(hy, p + "up", l.w_up, F, F, D);     hy_name_vec(hy, p + "up.b", l.b_up + F, F);
       hy_name_rows(hy, p + "down", l.w_down, 0, D, F); hy_name_vec(hy, p + "down.b", l.b_down, D);
     }
+  } else if (c.ff_kind == XB_FF_GLU) {
+    l.n_up = (int)(2 * F); l.n_dn = (int)F;
+    if (own) {
+      XB_TRY(hy_alloc_t(hy, &l.w_up, (size_t)l.n_up * D));
+      XB_TRY(hy_alloc_t(hy, &l.w_down, D * F));
+      hy_name_rows(hy, p + "gate", l.w_up, 0, F, D);
+      hy_name_rows(hy, p + "up", l.w_up, F, F, D);
+      hy_name_rows(hy, p + "down", l.w_down, 0, D, F);
+    }
   } else if (c.ff_kind == XB_FF_MOE) {
     const size_t E = c.n_experts, S = c.shared_ff > 0 ? c.shared_ff : 0;
+    const size_t ER = E + (S > 0 && c.shared_gate ? 1 : 0);   // rows of the router's matrix: the shared expert's gate is one more
     XB_CHECK(E > 0 && c.top > 0 && (size_t)c.top <= E, "layer %d: %d experts, %d per token", i, c.n_experts, c.top);
     XB_CHECK(c.groups == 0 || (c.groups > 0 && E % c.groups == 0 && c.keep_groups > 0 && c.keep_groups <= c.groups &&
                                (size_t)c.top <= (E / c.groups) * c.keep_groups),
@@ -385,7 +474,8 @@ static int hy_create_ff(xb_engine* e, int i, bool own, uint64_t& wbytes) {
     if (own) {
       XB_TRY(hy_alloc_t(hy, &l.w_up, (size_t)l.n_up * D));
       XB_TRY(hy_alloc_t(hy, &l.w_down, D * l.n_dn));
-      XB_TRY(hy_alloc_t(hy, &l.w_router, E * D));
+      XB_TRY(hy_alloc_t(hy, &l.w_router, ER * D));
+      if (ER > E) hy_name_rows(hy, p + "shared.sg", l.w_router, E, 1, D);
       hy_name_rows(hy, p + "router", l.w_router, 0, E, D);
       for (size_t x = 0; x < E; ++x) {
         const std::string pe = p + "e" + std::to_string(x) + ".";
@@ -406,8 +496,8 @@ static int hy_create_ff(xb_engine* e, int i, bool own, uint64_t& wbytes) {
       }
       wbytes += E * D * 2;
     }
-    if (E > hy->maxE) hy->maxE = E;
-    if (E > hy->maxM) hy->maxM = E;
+    if (ER > hy->maxE) hy->maxE = ER;
+    if (ER > hy->maxM) hy->maxM = ER;
   } else {
     return xb_fail(1, "layer %d: unknown feed-forward kind %d", i, c.ff_kind);
   }
@@ -434,10 +524,13 @@ static int hy_create(xb_engine* e, const xb_hybrid_desc& d, const xb_hybrid_laye
     const xb_hybrid_layer& c = l.d;
     const std::string p = "l" + std::to_string(i) + ".";
     const bool own = c.weights_of < 0;
-    const bool sandwich = d.block == XB_BLOCK_SANDWICH, branchnorm = d.block == XB_BLOCK_BRANCHNORM;
+    const bool sandwich = d.block == XB_BLOCK_SANDWICH, branchnorm = d.block == XB_BLOCK_BRANCHNORM, prenorm = d.block == XB_BLOCK_PRENORM;
     l.owner = -1;
     XB_CHECK(!branchnorm || (own && (c.mixer == XB_MIX_SOFTMAX || c.mixer == XB_MIX_LATENT) && (c.ff == 0 || c.ff_kind == XB_FF_MOE)),
              "layer %d: branch-norm blocks take softmax or latent attention and experts, with tensors of their own", i);
+    XB_CHECK(!prenorm || (own && (c.mixer == XB_MIX_LATENT || c.mixer == XB_MIX_GLA) && (c.ff == 0 || c.ff_kind != XB_FF_RELU2)),
+             "layer %d: pre-norm blocks take latent attention or gated linear attention and gated feed-forwards, with tensors of their own", i);
+    XB_CHECK(prenorm || c.mixer != XB_MIX_GLA, "layer %d: gated linear attention belongs to pre-norm blocks", i);
     if (!own) {
       XB_CHECK(c.weights_of < d.n_layers && c.weights_of != i && layers[c.weights_of].weights_of < 0,
                "layer %d: weights_of %d must name another layer that owns its tensors", i, c.weights_of);
@@ -447,10 +540,8 @@ static int hy_create(xb_engine* e, const xb_hybrid_desc& d, const xb_hybrid_laye
       l.owner = c.weights_of;
     }
     XB_CHECK(own || (c.mixer != XB_MIX_DELTA && c.mixer != XB_MIX_PARALLEL && c.mixer != XB_MIX_SOFTMAX), "layer %d: this mixer kind keeps tensors of its own", i);
-    const size_t nd = d.norm_scalar ? 1 : D;   // numbers in a norm of the stream
     if (own) {
-      XB_TRY(hy_alloc_t(hy, &l.norm1, nd));
-      hy_name_vec(hy, p + "norm1", l.norm1, nd);
+      XB_TRY(hy_create_norm(hy, p + "norm1", &l.norm1, &l.norm1_b, &l.norm1_a));
       if (sandwich) { XB_TRY(hy_alloc_t(hy, &l.norm1b, D)); hy_name_vec(hy, p + "norm1b", l.norm1b, D); }
     }
     if (ct > 0) {
@@ -530,7 +621,7 @@ static int hy_create(xb_engine* e, const xb_hybrid_desc& d, const xb_hybrid_laye
       kvpos += (uint64_t)G * (dk + dv) * (d.compute_fp32 ? 4 : 2);
     } else if (c.mixer == XB_MIX_SOFTMAX) {
       XB_TRY(hy_create_softmax(e, i, own, wbytes, kvpos));
-    } else if (c.mixer == XB_MIX_LATENT || c.mixer == XB_MIX_GDELTA || c.mixer == XB_MIX_LIGHTNING) {
+    } else if (c.mixer == XB_MIX_LATENT || c.mixer == XB_MIX_GDELTA || c.mixer == XB_MIX_LIGHTNING || c.mixer == XB_MIX_GLA) {
       XB_TRY(hy_create_mixer(e, i, own, st, wbytes, kvpos));
     } else {
       return xb_fail(1, "layer %d: unknown mixer kind %d", i, c.mixer);
@@ -543,7 +634,7 @@ static int hy_create(xb_engine* e, const xb_hybrid_desc& d, const xb_hybrid_laye
     if ((size_t)l.n_o > hy->maxK) hy->maxK = l.n_o;
     if ((size_t)l.n_o2 > hy->maxK) hy->maxK = l.n_o2;
     if (c.ff > 0 && c.ff_kind != XB_FF_RELU2) {
-      if (branchnorm) { XB_TRY(hy_alloc_t(hy, &l.norm2, nd)); hy_name_vec(hy, p + "norm2", l.norm2, nd); }
+      if (branchnorm || prenorm) XB_TRY(hy_create_norm(hy, p + "norm2", &l.norm2, &l.norm2_b, &l.norm2_a));
       if (sandwich) {   // the feed-forward is a sublayer of its own: norm before and after, optionally the causal filter
         XB_CHECK(own && c.ff_kind == XB_FF_MOE, "layer %d: sandwich blocks take experts with tensors of their own", i);
         XB_TRY(hy_alloc_t(hy, &l.norm2, D)); hy_name_vec(hy, p + "norm2", l.norm2, D);
@@ -596,12 +687,12 @@ static int hy_create(xb_engine* e, const xb_hybrid_desc& d, const xb_hybrid_laye
     const HyLayer& o = hy->L[l.owner];
     l.w_in = o.w_in; l.b_in = o.b_in; l.w_o = o.w_o; l.w_up = o.w_up; l.w_down = o.w_down; l.norm1 = o.norm1; l.head_norm = o.head_norm;
     l.w_uk = o.w_uk; l.w_uv = o.w_uv; l.w_d2 = o.w_d2; l.w_router = o.w_router; l.b_up = o.b_up; l.b_down = o.b_down;
-    l.lat_norm = o.lat_norm; l.rot_freq = o.rot_freq; l.w0 = o.w0; l.hdecay = o.hdecay; l.canon1 = o.canon1;
+    l.lat_norm = o.lat_norm; l.rot_freq_d = o.rot_freq_d; l.w0 = o.w0; l.hdecay = o.hdecay; l.canon1 = o.canon1;
   }
   XB_TRY(hy_alloc_t(hy, &hy->embed, (size_t)d.vocab * D)); hy_name_rows(hy, "embed", hy->embed, 0, d.vocab, D);
   if (d.tied_head) hy->head = hy->embed;   // the logits are products with the embedding table itself
   else { XB_TRY(hy_alloc_t(hy, &hy->head, (size_t)d.vocab * D)); hy_name_rows(hy, "head", hy->head, 0, d.vocab, D); }
-  XB_TRY(hy_alloc_t(hy, &hy->final_norm, d.norm_scalar ? 1 : D)); hy_name_vec(hy, "final.norm", hy->final_norm, d.norm_scalar ? 1 : D);
+  XB_TRY(hy_create_norm(hy, "final.norm", &hy->final_norm, &hy->final_norm_b, &hy->final_norm_a));
   if (d.side_dim > 0) {
     const size_t w = (size_t)d.side_dim * d.n_layers;
     XB_TRY(hy_alloc_t(hy, &hy->side_embed, (size_t)d.vocab * w)); hy_name_rows(hy, "side.embed", hy->side_embed, 0, d.vocab, w);
@@ -626,7 +717,7 @@ static int hy_create(xb_engine* e, const xb_hybrid_desc& d, const xb_hybrid_laye
   XB_TRY(hy_alloc(hy, &hy->a1, Tm * hy->maxK * as));
   XB_TRY(hy_alloc(hy, &hy->a2, Tm * hy->maxK * as));
   XB_TRY(hy_alloc(hy, &hy->head_in, R * D * as));
-  if (d.block == XB_BLOCK_PARALLEL) XB_TRY(hy_alloc(hy, &hy->ah, Tm * D * as));
+  if (d.block == XB_BLOCK_PARALLEL || d.block == XB_BLOCK_PRENORM) XB_TRY(hy_alloc(hy, &hy->ah, Tm * D * as));
   {
     // the first layer that blends values leaves them for the others, whose value rows must have the same width
     long long first_gv = -1;
@@ -744,7 +835,8 @@ static int hy_finalize(xb_engine* e) {
     XB_TRY(retile(&l.t_down, l.w_down, D, n_dn));
     XB_TRY(retile(&l.t_sgate, l.w_sgate, hy->d.side_dim, D));
     XB_TRY(retile(&l.t_sproj, l.w_sproj, D, hy->d.side_dim));
-    XB_TRY(retile(&l.t_d2, l.w_d2, (size_t)l.d.m_heads * l.d.m_dim, l.d.m_rank));
+    if (l.d.mixer == XB_MIX_GDELTA) XB_TRY(retile(&l.t_d2, l.w_d2, (size_t)l.d.m_heads * l.d.m_dim, l.d.m_rank));
+    XB_TRY(retile(&l.t_uq, l.w_uq, (size_t)l.d.m_heads * (l.d.m_dim + l.d.m_rot_dim), l.d.m_q_rank));
   }
   for (HyLayer& l : hy->L) {
     if (l.owner < 0) continue;
@@ -797,6 +889,10 @@ static int hy_reserve(xb_engine* e) {
   HyModel* hy = e->hy;
   const size_t es = hy->d.compute_fp32 ? 4 : 2;
   for (HyLayer& l : hy->L) {
+    if (hy_borrows_rows(l)) {   // an earlier layer's pool (made before this one)
+      l.k_pool = hy->L[l.d.m_kv_from].k_pool;
+      continue;
+    }
     cudaFree(l.k_pool); cudaFree(l.v_pool);
     l.k_pool = l.v_pool = nullptr;
     if (l.d.mixer == XB_MIX_LATENT) {   // one pool: a row holds the latent (key and value at once) and the rotated key part
@@ -1129,9 +1225,10 @@ static int hy_sublayer_input(xb_engine* e, int T, int n_seqs, bool no_span, cons
                        reinterpret_cast<AT*>(hy->a1), (long long)D, st);
 }
 
+static int hy_latent_window(const xb_hybrid_layer& c) { return c.m_window > 0 ? c.m_window : 1 << 30; }
 // Latent attention through hy_latent_attn_mma_kernel.  0: launched; 1: not applicable (shared memory); < 0: -error.
-template <int WARPS, int DVC, int LOADW>
-static int hy_latent_mma_launch(xb_engine* e, const HyLayer& l, const BatchMeta& m, int T, int n_splits, cudaStream_t st) {
+template <int WARPS, int DVC, int LOADW, bool EXT>
+static int hy_latent_mma_launch_x(xb_engine* e, const HyLayer& l, const BatchMeta& m, int T, int n_splits, cudaStream_t st) {
   HyModel* hy = e->hy;
   const xb_hybrid_layer& c = l.d;
   const int H = c.m_heads, R = c.m_kv_rank, W = R + c.m_rot_dim, NR = T * H;
@@ -1143,18 +1240,23 @@ static int hy_latent_mma_launch(xb_engine* e, const HyLayer& l, const BatchMeta&
     int dev = 0;
     if (cudaGetDevice(&dev) != cudaSuccess || dev < 0 || dev >= XB_MAX_DEVICES) return 1;
     if (granted[dev] < smem) {
-      if (cudaFuncSetAttribute(hy_latent_attn_mma_kernel<WARPS, DVC, LOADW>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024) != cudaSuccess) return 1;
+      if (cudaFuncSetAttribute(hy_latent_attn_mma_kernel<WARPS, DVC, LOADW, EXT>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024) != cudaSuccess) return 1;
       granted[dev] = 200 * 1024;
     }
   }
   const dim3 grid((NR + 16 * WARPS - 1) / (16 * WARPS), n_splits, (R + DVC - 1) / DVC);
-  if (hy_launch(e, hy_latent_attn_mma_kernel<WARPS, DVC, LOADW>, grid, dim3(32 * LOADW), smem, st, (const float*)hy->qa, (const bf16*)l.k_pool, m, T, H, W,
-                R, c.m_scale * 1.4426950408889634f, n_splits, hy->lat_part, hy->o, (long long)H * R) != 0)
+  if (hy_launch(e, hy_latent_attn_mma_kernel<WARPS, DVC, LOADW, EXT>, grid, dim3(32 * LOADW), smem, st, (const float*)hy->qa, (const bf16*)l.k_pool, m, T, H, W,
+                R, c.m_scale * 1.4426950408889634f, n_splits, hy->lat_part, hy->o, (long long)H * R, hy_latent_window(c)) != 0)
     return -1;
   if (n_splits > 1 &&
       hy_launch(e, hy_latent_merge_kernel, dim3(NR), dim3(128), 0, st, (const float*)hy->lat_part, n_splits, NR, H, R, hy->o, (long long)H * R) != 0)
     return -1;
   return 0;
+}
+template <int WARPS, int DVC, int LOADW>
+static int hy_latent_mma_launch(xb_engine* e, const HyLayer& l, const BatchMeta& m, int T, int n_splits, cudaStream_t st) {
+  if (l.d.m_window > 0) return hy_latent_mma_launch_x<WARPS, DVC, LOADW, true>(e, l, m, T, n_splits, st);
+  return hy_latent_mma_launch_x<WARPS, DVC, LOADW, false>(e, l, m, T, n_splits, st);
 }
 static int hy_latent_mma(xb_engine* e, const HyLayer& l, const BatchMeta& m, int T, cudaStream_t st) {
   const int R = l.d.m_kv_rank, NR = T * l.d.m_heads;
@@ -1165,12 +1267,16 @@ static int hy_latent_mma(xb_engine* e, const HyLayer& l, const BatchMeta& m, int
   }
   int ns = HY_LAT_SPLIT_ROWS / 16 / tiles1;
   ns = ns < 1 ? 1 : (ns > 64 ? 64 : ns);
+  if (l.d.m_window > 0) {   // no more shares than a window has tiles
+    const int wt = (l.d.m_window + 15) / HY_LAT_KEYS + 2;
+    ns = ns > wt ? wt : ns;
+  }
   return R <= 128 ? hy_latent_mma_launch<1, 128, 4>(e, l, m, T, ns, st) : hy_latent_mma_launch<1, 256, 4>(e, l, m, T, ns, st);
 }
 
-// Latent attention of one layer: P = [q | down-projection (| other rows)] of the step's rows -> a1 = what the output
-// projection reads.  The cache row is made and appended, the queries are folded into the cache's space, the attention
-// runs over the cached latents, and the read-out goes through the value up-projection.
+// Latent attention of one layer: P = [q or the queries' latent | down-projection | head gates (| other rows)] of the step's rows
+// -> a1 = what the output projection reads.  The cache row is made and appended, the queries are folded into the cache's space,
+// the attention runs over the cached latents, and the read-out goes through the value up-projection (and the head's gate).
 template <typename AT>
 static int hy_latent_mixer(xb_engine* e, const HyLayer& l, int T, const LinOut& P, const BatchMeta& m, cudaStream_t st) {
   HyModel* hy = e->hy;
@@ -1178,13 +1284,20 @@ static int hy_latent_mixer(xb_engine* e, const HyLayer& l, int T, const LinOut& 
   const xb_hybrid_desc& d = hy->d;
   typedef typename std::conditional<std::is_same<AT, float>::value, float, bf16>::type KT;
   AT* a1 = reinterpret_cast<AT*>(hy->a1);
+  AT* a2 = reinterpret_cast<AT*>(hy->a2);
   const int H = c.m_heads, n = c.m_dim;
-  const int dr = c.m_rot_dim, dv = c.m_vdim, R = c.m_kv_rank, W = R + dr;
-  XB_TRY(hy_launch(e, hy_latent_prep_kernel<KT>, dim3(T), dim3(256), 0, st, P, l.off_q, l.off_dkv, H, n, dr, R, c.m_rot_dims,
-                   (const float*)l.rot_freq, (const float*)l.lat_norm, d.norm_eps, (KT*)l.k_pool, m, hy->qa));
+  const int dr = c.m_rot_dim, dv = c.m_vdim, R = c.m_kv_rank, W = R + dr, qr = c.m_q_rank;
+  RotArgs r;
+  r.freq = l.rot_freq_d; r.dims = c.m_rot_dims; r.half = c.m_rot_pairs == XB_ROPE_HALF_SPLIT ? 1 : 0;
+  r.mult = c.m_rot_mult != 0.f ? c.m_rot_mult : 1.f;
+  if (l.off_dkv >= 0 || qr > 0)
+    XB_TRY(hy_launch(e, hy_latent_down_kernel<AT, KT>, dim3(T), dim3(256), 0, st, P, l.off_dkv, dr, R, r, (const float*)l.lat_norm, d.norm_eps,
+                     (KT*)l.k_pool, m, l.off_dq, qr, (const float*)l.dq_norm, a2));
+  LinOut Q = P;
+  if (qr > 0) XB_TRY(hy_linear<AT>(e, a2, qr, l.w_uq, l.t_uq, nullptr, T, H * (n + dr), qr, hy->m2, hy->cap_m, st, &Q));
   const size_t mm1 = (size_t)HY_MM_ROWS * n * sizeof(float), mm2 = (size_t)HY_MM_ROWS * R * sizeof(float);
-  XB_TRY(hy_launch(e, hy_head_mm_t_kernel, dim3((T + HY_MM_ROWS - 1) / HY_MM_ROWS, H), dim3(256), mm1, st, P, l.off_q, n + dr,
-                   (const bf16*)l.w_uk, hy->qa, (long long)H * W, W, T, n, R));
+  XB_TRY(hy_launch(e, hy_latent_absorb_kernel, dim3((T + HY_MM_ROWS - 1) / HY_MM_ROWS, H), dim3(256), mm1, st, Q, l.off_q, dr,
+                   (const bf16*)l.w_uk, hy->qa, H, T, n, R, r, m.tok_pos));
   // bf16 serving at sizes the tensor-core tiles take: rows = (token, head) pairs over shared key tiles; steps of few
   // rows split every sequence's keys over blocks and merge
   bool done = false;
@@ -1194,25 +1307,67 @@ static int hy_latent_mixer(xb_engine* e, const HyLayer& l, int T, const LinOut& 
     done = rc == 0;
   }
   if (!done) {
-    const int aw = 16;   // causal: every earlier key is visible
+    const int aw = 16;   // the block's warps share out the visible keys
     const size_t asm_bytes = (size_t)(((W + 3) & ~3) + aw * (2 + R)) * sizeof(float);
-    const LinOut Q = hy_plain(hy->qa, (long long)H * W);
-    const int far = 1 << 30;
+    const LinOut QA = hy_plain(hy->qa, (long long)H * W);
+    const int far = hy_latent_window(c);
     if (R <= 256)
-      XB_TRY(hy_launch(e, hy_attn_window_kernel<KT, float, 8>, dim3(T, H), dim3(32 * aw), asm_bytes, st, Q, 0, -1, (const KT*)l.k_pool,
+      XB_TRY(hy_launch(e, hy_attn_window_kernel<KT, float, 8>, dim3(T, H), dim3(32 * aw), asm_bytes, st, QA, 0, -1, (const KT*)l.k_pool,
                        (const KT*)l.k_pool, m, H, 1, W, R, W, W, far, 0, c.m_scale, 1.0f, hy->o, (long long)H * R, AttnOpt{nullptr, 0.f, 1, 0}));
     else
-      XB_TRY(hy_launch(e, hy_attn_window_kernel<KT, float, 16>, dim3(T, H), dim3(32 * aw), asm_bytes, st, Q, 0, -1, (const KT*)l.k_pool,
+      XB_TRY(hy_launch(e, hy_attn_window_kernel<KT, float, 16>, dim3(T, H), dim3(32 * aw), asm_bytes, st, QA, 0, -1, (const KT*)l.k_pool,
                        (const KT*)l.k_pool, m, H, 1, W, R, W, W, far, 0, c.m_scale, 1.0f, hy->o, (long long)H * R, AttnOpt{nullptr, 0.f, 1, 0}));
   }
   return hy_launch(e, hy_head_mm_kernel<AT>, dim3((T + HY_MM_ROWS - 1) / HY_MM_ROWS, H), dim3(128), mm2, st, (const float*)hy->o,
-                   (long long)H * R, (const bf16*)l.w_uv, a1, (long long)l.n_o, T, R, dv);
+                   (long long)H * R, (const bf16*)l.w_uv, a1, (long long)l.n_o, T, R, dv, P, c.m_gate ? l.off_g : -1);
+}
+
+// The logits of a step: the wanted rows of the model's last norm (hn), or every sequence's last one, through the head.
+template <typename AT>
+static int hy_run_head(xb_engine* e, int n_seqs, const BatchMeta& m, cudaStream_t st) {
+  HyModel* hy = e->hy;
+  const xb_hybrid_desc& d = hy->d;
+  const int n = e->sel_rows != nullptr ? e->sel_n : n_seqs, D = d.dim;
+  if (n <= 0) return 0;
+  const int* idx = e->sel_rows != nullptr ? hy->d_rows : m.seq_last;
+  LinOut y;
+  XB_TRY(hy_launch(e, hy_gather_rows_kernel<AT>, dim3(n), dim3(256), 0, st, (const float*)hy->hn, idx, reinterpret_cast<AT*>(hy->head_in), D));
+  XB_TRY(hy_linear<AT>(e, hy->head_in, D, hy->head, hy->t_head, nullptr, n, d.vocab, D, hy->head_raw, hy->cap_head, st, &y));
+  const long long tot = (long long)n * d.vocab;
+  return hy_launch(e, hy_logits_kernel, dim3((unsigned)((tot + 255) / 256)), dim3(256), 0, st, y, d.logit_softcap, e->logits, n, d.vocab);
 }
 
 // ----------------------------------------------------------------------------- parallel blocks
 // x <- embed * scale;  per layer: h = norm(x) (made by the previous row op), x += mixer(h) + ff(h).
 // The mixers: latent attention (cache = latent + rotated key part, queries folded into the latent space so that a step
 // never rebuilds keys or values of earlier tokens), general delta rule, lightning; feed-forwards: clamped GLU, dense or experts.
+// Router of an expert layer, fp32 whatever the serving type (fp32 accumulation of the products, fp32 logits): xin -> gw.  sg: one more
+// row of the router's matrix gates the shared expert.
+template <typename AT>
+static int hy_router(xb_engine* e, const HyLayer& l, int T, const void* xin, int sg, cudaStream_t st) {
+  HyModel* hy = e->hy;
+  const xb_hybrid_layer& c = l.d;
+  const int D = hy->d.dim, NE = c.n_experts + sg;
+  const AT* x = reinterpret_cast<const AT*>(xin);
+  const int ng = c.groups > 0 ? c.groups : 1;
+  if (T <= 64 && hy->fuse_router) {   // few rows: logits and routing of a token in one block
+    const size_t rs1 = (size_t)(2 * c.n_experts + NE + ng) * sizeof(float);
+    return hy_launch(e, hy_router_route_kernel<AT>, dim3(T), dim3(256), rs1, st, x, (long long)D, (const bf16*)l.w_router, D, c.n_experts, c.top, c.groups,
+                     c.keep_groups, c.route_scale, hy->gw, c.route_score, c.group_score, c.route_norm, sg);
+  }
+  if (T <= 64) {   // few rows: a warp per (token, expert)
+    XB_TRY(hy_launch(e, hy_router_logits_kernel<AT, 1>, dim3((unsigned)(((long long)T * NE + 7) / 8)), dim3(256), 0, st, x, (long long)D,
+                     (const bf16*)l.w_router, hy->m2, T, NE, D));
+  } else {
+    const int chunks = (NE + 7) / 8;
+    XB_TRY(hy_launch(e, hy_router_logits_kernel<AT, 8>, dim3((unsigned)(((long long)T * chunks + 7) / 8)), dim3(256), 0, st, x, (long long)D,
+                     (const bf16*)l.w_router, hy->m2, T, NE, D));
+  }
+  const size_t rs = (size_t)4 * (2 * c.n_experts + ng) * sizeof(float);
+  return hy_launch(e, hy_route_kernel, dim3((T + 3) / 4), dim3(128), rs, st, (const float*)hy->m2, c.n_experts, c.top, c.groups, c.keep_groups,
+                   c.route_scale, hy->gw, T, c.route_score, c.group_score, c.route_norm, sg);
+}
+
 // xin: the normed stream as a Linear input [T, dim] of AT
 template <typename AT>
 static int hy_ff_parallel(xb_engine* e, const HyLayer& l, int T, const void* xin, cudaStream_t st, LinOut* y, LinOut* up_out = nullptr) {
@@ -1222,18 +1377,16 @@ static int hy_ff_parallel(xb_engine* e, const HyLayer& l, int T, const void* xin
   AT* a2 = reinterpret_cast<AT*>(hy->a2);
   // Steps of so few rows that at most half of the experts can have a token: read the chosen experts' rows only (two kernels
   // in place of the wide up Linear, the activation and the wide down Linear).
-  if (c.ff_kind == XB_FF_MOE && hy->use_gather && c.ff_act != XB_ACT_GELU && c.shared_ff <= 0 && l.b_up == nullptr && l.b_down == nullptr && D % 8 == 0 && c.ff % 8 == 0 &&
-      2LL * T * c.top <= c.n_experts) {
-    XB_TRY(hy_launch(e, hy_router_logits_kernel<AT, 1>, dim3((unsigned)(((long long)T * c.n_experts + 7) / 8)), dim3(256), 0, st,
-                     reinterpret_cast<const AT*>(xin), (long long)D, (const bf16*)l.w_router, hy->m2, T, c.n_experts, D));
-    const size_t rs = (size_t)4 * (2 * c.n_experts + (c.groups > 0 ? c.groups : 1)) * sizeof(float);
-    XB_TRY(hy_launch(e, hy_route_kernel, dim3((T + 3) / 4), dim3(128), rs, st, (const float*)hy->m2, c.n_experts, c.top, c.groups,
-                     c.keep_groups, c.route_scale, hy->gw, T, c.route_score, c.group_score, c.route_norm));
-    const long long nu = (long long)T * c.top * c.ff, nd = (long long)T * D;
+  const int sf = c.ff_kind == XB_FF_MOE && c.shared_ff > 0 ? c.shared_ff : 0, sg = sf > 0 && c.shared_gate ? 1 : 0;
+  const int ldg = c.n_experts + sg;   // a routing row: the experts' weights, then the shared expert's
+  if (c.ff_kind == XB_FF_MOE && hy->use_gather && c.ff_act != XB_ACT_GELU && l.b_up == nullptr && l.b_down == nullptr && D % 8 == 0 && c.ff % 8 == 0 &&
+      sf % 8 == 0 && 2LL * T * c.top <= c.n_experts) {
+    XB_TRY(hy_router<AT>(e, l, T, xin, sg, st));
+    const long long per = (long long)c.top * c.ff + sf, nu = (long long)T * per, nd = (long long)T * D;
     XB_TRY(hy_launch(e, hy_moe_gather_up_kernel<AT>, dim3((unsigned)((nu + 7) / 8)), dim3(256), 0, st, reinterpret_cast<const AT*>(xin), (long long)D,
-                     (const bf16*)l.w_up, (const float*)hy->gw, c.n_experts, c.top, c.ff, D, c.ff_limit, c.ff_act, c.route_input, a2, T));
+                     (const bf16*)l.w_up, (const float*)hy->gw, ldg, c.n_experts, c.top, c.ff, sf, D, c.ff_limit, c.shared_limit, c.ff_act, c.route_input, a2, T));
     XB_TRY(hy_launch(e, hy_moe_gather_down_kernel<AT>, dim3((unsigned)((nd + 7) / 8)), dim3(256), 0, st, (const AT*)a2, (const bf16*)l.w_down,
-                     (const float*)hy->gw, c.n_experts, c.top, c.ff, D, hy->m2, T));   // m2: the router's logits there are spent
+                     (const float*)hy->gw, ldg, c.n_experts, c.top, c.ff, sf, D, hy->m2, T));   // m2: router logits there are spent
     *y = hy_plain(hy->m2, D);
     return 0;
   }
@@ -1242,46 +1395,29 @@ static int hy_ff_parallel(xb_engine* e, const HyLayer& l, int T, const void* xin
   if (up_out != nullptr) *up_out = U;   // rows behind the experts' (a residual gate) are read by the caller
   // a bf16 matrix out of the tcgen05 Linear (prompts): the activations read and write 16 bytes per thread
   const bool vec = std::is_same<AT, bf16>::value && U.h != nullptr && U.ld % 8 == 0 && l.n_dn % 8 == 0;
-  if (c.ff_kind == XB_FF_GLU_CLAMP) {
+  if (c.ff_kind == XB_FF_GLU_CLAMP || c.ff_kind == XB_FF_GLU) {
     const long long n = (long long)T * c.ff;
+    const int act = c.ff_kind == XB_FF_GLU ? c.ff_act : XB_ACT_GLU_CLAMP;
     if (vec && c.ff % 8 == 0)
-      XB_TRY(hy_launch(e, hy_glu_clamp_vec_kernel, dim3((unsigned)((n / 8 + 255) / 256)), dim3(256), 0, st, U.h, U.ld, U.bias, c.ff, c.ff_limit,
+      XB_TRY(hy_launch(e, hy_glu_vec_kernel, dim3((unsigned)((n / 8 + 255) / 256)), dim3(256), 0, st, U.h, U.ld, U.bias, c.ff, c.ff_limit, act,
                        reinterpret_cast<bf16*>(hy->a2), (long long)l.n_dn, T));
     else
-      XB_TRY(hy_launch(e, hy_glu_clamp_kernel<AT>, dim3((unsigned)((n + 255) / 256)), dim3(256), 0, st, U, c.ff, c.ff_limit, a2, (long long)l.n_dn, T));
+      XB_TRY(hy_launch(e, hy_glu_kernel<AT>, dim3((unsigned)((n + 255) / 256)), dim3(256), 0, st, U, c.ff, c.ff_limit, act, a2, (long long)l.n_dn, T));
   } else {
-    // router in fp32 whatever the serving type: fp32 accumulation of the products, fp32 logits
-    if (T <= 64 && hy->fuse_router) {   // few rows: logits and routing of a token in one block
-      const size_t rs1 = (size_t)(3 * c.n_experts + (c.groups > 0 ? c.groups : 1)) * sizeof(float);
-      XB_TRY(hy_launch(e, hy_router_route_kernel<AT>, dim3(T), dim3(256), rs1, st, reinterpret_cast<const AT*>(xin), (long long)D, (const bf16*)l.w_router, D,
-                       c.n_experts, c.top, c.groups, c.keep_groups, c.route_scale, hy->gw, c.route_score, c.group_score, c.route_norm));
-    } else {
-      if (T <= 64) {   // few rows: a warp per (token, expert)
-        XB_TRY(hy_launch(e, hy_router_logits_kernel<AT, 1>, dim3((unsigned)(((long long)T * c.n_experts + 7) / 8)), dim3(256), 0, st,
-                         reinterpret_cast<const AT*>(xin), (long long)D, (const bf16*)l.w_router, hy->m2, T, c.n_experts, D));
-      } else {
-        const int chunks = (c.n_experts + 7) / 8;
-        XB_TRY(hy_launch(e, hy_router_logits_kernel<AT, 8>, dim3((unsigned)(((long long)T * chunks + 7) / 8)), dim3(256), 0, st,
-                         reinterpret_cast<const AT*>(xin), (long long)D, (const bf16*)l.w_router, hy->m2, T, c.n_experts, D));
-      }
-      const size_t rs = (size_t)4 * (2 * c.n_experts + (c.groups > 0 ? c.groups : 1)) * sizeof(float);
-      XB_TRY(hy_launch(e, hy_route_kernel, dim3((T + 3) / 4), dim3(128), rs, st, (const float*)hy->m2, c.n_experts, c.top, c.groups, c.keep_groups,
-                       c.route_scale, hy->gw, T, c.route_score, c.group_score, c.route_norm));
-    }
+    XB_TRY(hy_router<AT>(e, l, T, xin, sg, st));
     const long long n = (long long)T * l.n_dn;
-    const int sf = c.shared_ff > 0 ? c.shared_ff : 0;
     if (c.ff_act == XB_ACT_GELU) {   // experts without a gate projection
       if (vec && c.ff % 8 == 0 && sf % 8 == 0)
-        XB_TRY(hy_launch(e, hy_moe_act1_vec_kernel, dim3((unsigned)((n / 8 + 255) / 256)), dim3(256), 0, st, U.h, U.ld, (const float*)hy->gw, c.n_experts,
+        XB_TRY(hy_launch(e, hy_moe_act1_vec_kernel, dim3((unsigned)((n / 8 + 255) / 256)), dim3(256), 0, st, U.h, U.ld, (const float*)hy->gw, ldg, c.n_experts,
                          c.ff, sf, reinterpret_cast<bf16*>(hy->a2), (long long)l.n_dn, T));
       else
-        XB_TRY(hy_launch(e, hy_moe_act1_kernel<AT>, dim3((unsigned)((n + 255) / 256)), dim3(256), 0, st, U, (const float*)hy->gw, c.n_experts, c.ff, sf,
+        XB_TRY(hy_launch(e, hy_moe_act1_kernel<AT>, dim3((unsigned)((n + 255) / 256)), dim3(256), 0, st, U, (const float*)hy->gw, ldg, c.n_experts, c.ff, sf,
                          a2, (long long)l.n_dn, T));
     } else if (vec && c.ff % 8 == 0 && sf % 8 == 0)
-      XB_TRY(hy_launch(e, hy_moe_act_vec_kernel, dim3((unsigned)((n / 8 + 255) / 256)), dim3(256), 0, st, U.h, U.ld, (const float*)hy->gw, c.n_experts,
+      XB_TRY(hy_launch(e, hy_moe_act_vec_kernel, dim3((unsigned)((n / 8 + 255) / 256)), dim3(256), 0, st, U.h, U.ld, (const float*)hy->gw, ldg, c.n_experts,
                        c.ff, c.ff_limit, sf, c.shared_limit, c.ff_act, c.route_input, reinterpret_cast<bf16*>(hy->a2), (long long)l.n_dn, T));
     else
-      XB_TRY(hy_launch(e, hy_moe_act_kernel<AT>, dim3((unsigned)((n + 255) / 256)), dim3(256), 0, st, U, (const float*)hy->gw, c.n_experts, c.ff,
+      XB_TRY(hy_launch(e, hy_moe_act_kernel<AT>, dim3((unsigned)((n + 255) / 256)), dim3(256), 0, st, U, (const float*)hy->gw, ldg, c.n_experts, c.ff,
                        c.ff_limit, sf, c.shared_limit, c.ff_act, c.route_input, a2, (long long)l.n_dn, T));
   }
   return hy_linear<AT>(e, a2, l.n_dn, l.w_down, l.t_down, l.b_down, T, D, l.n_dn, hy->m2, hy->cap_m, st, y);
@@ -1354,18 +1490,7 @@ static int hy_run_parallel_t(xb_engine* e, int T, int n_seqs, void* const* taps,
     if (taps != nullptr && taps[li] != nullptr)
       XB_CUDA(cudaMemcpyAsync(taps[li], hy->x, (size_t)T * D * sizeof(float), cudaMemcpyDeviceToDevice, st));
   }
-  if (with_head) {
-    const int nr = e->sel_rows != nullptr ? e->sel_n : n_seqs;
-    if (nr > 0) {
-      const int* idx = e->sel_rows != nullptr ? hy->d_rows : m.seq_last;
-      LinOut y;
-      XB_TRY(hy_launch(e, hy_gather_rows_kernel<AT>, dim3(nr), dim3(256), 0, st, (const float*)hy->hn, idx, reinterpret_cast<AT*>(hy->head_in), D));
-      XB_TRY(hy_linear<AT>(e, hy->head_in, D, hy->head, hy->t_head, nullptr, nr, d.vocab, D, hy->head_raw, hy->cap_head, st, &y));
-      const long long tot = (long long)nr * d.vocab;
-      XB_TRY(hy_launch(e, hy_logits_kernel, dim3((unsigned)((tot + 255) / 256)), dim3(256), 0, st, y, d.logit_softcap, e->logits, nr, d.vocab));
-    }
-  }
-  return 0;
+  return with_head ? hy_run_head<AT>(e, n_seqs, m, st) : 0;
 }
 
 // Rotary-position softmax attention of one layer: P = [q | k | v | head gates] of the step's rows -> a1 = what the output
@@ -1542,18 +1667,96 @@ static int hy_run_branchnorm_t(xb_engine* e, int T, int n_seqs, int n_tiles, voi
     if (taps != nullptr && taps[li] != nullptr)
       XB_CUDA(cudaMemcpyAsync(taps[li], hy->x, (size_t)T * D * sizeof(float), cudaMemcpyDeviceToDevice, st));
   }
-  if (with_head) {
-    const int n = e->sel_rows != nullptr ? e->sel_n : n_seqs;
-    if (n > 0) {
-      const int* idx = e->sel_rows != nullptr ? hy->d_rows : m.seq_last;
-      LinOut y;
-      XB_TRY(hy_launch(e, hy_gather_rows_kernel<AT>, dim3(n), dim3(256), 0, st, (const float*)hy->hn, idx, reinterpret_cast<AT*>(hy->head_in), D));
-      XB_TRY(hy_linear<AT>(e, hy->head_in, D, hy->head, hy->t_head, nullptr, n, d.vocab, D, hy->head_raw, hy->cap_head, st, &y));
-      const long long tot = (long long)n * d.vocab;
-      XB_TRY(hy_launch(e, hy_logits_kernel, dim3((unsigned)((tot + 255) / 256)), dim3(256), 0, st, y, d.logit_softcap, e->logits, n, d.vocab));
+  return with_head ? hy_run_head<AT>(e, n_seqs, m, st) : 0;
+}
+
+// ----------------------------------------------------------------------------- pre-norm blocks
+// x <- embed * scale;  per layer  x += mixer(f1(x)),  x += ff(f2(x)).  Every norm rides in the kernel that last changed x: the
+// embedding kernel makes the first layer's, the residual additions the next reader's.  The tanh norm needs no statistics of the row
+// (hy_add_tanh_kernel); the RMS form is hy_row_op_kernel's plain addition.
+template <typename AT>
+static int hy_run_prenorm_t(xb_engine* e, int T, int n_seqs, void* const* taps, cudaStream_t st, int with_head) {
+  HyModel* hy = e->hy;
+  const xb_hybrid_desc& d = hy->d;
+  BatchMeta m;
+  fill_batch_meta(e, m);
+  m.page_table = e->d_page_table;
+  m.tile_start = e->d_tile_start;
+  m.tile_len = e->d_tile_len;
+  m.max_pages = e->max_pages;
+  m.page_tokens = e->page_tokens;
+  const int D = d.dim;
+  const long long SS = (long long)hy->state_floats;
+  const bool tanh_norm = d.norm_kind == XB_NORM_TANH;
+  hy->pdl_now = T <= 128;
+  AT* ah = reinterpret_cast<AT*>(hy->ah);
+  AT* a1 = reinterpret_cast<AT*>(hy->a1);
+  // x += y, then the norm that reads x next: as a Linear input, or (the model's last) in fp32
+  auto add_norm = [&](const LinOut& y, const float* w, const float* b, const float* alpha, bool final) -> int {
+    if (!tanh_norm) {
+      RowOpArgs a;
+      a.x = hy->x; a.m1 = y; a.m2 = a.m3 = hy_none(); a.s1 = 1.f; a.s2 = 0.f; a.bw = nullptr; a.bw_one = 0.f; a.nw = w; a.hn = hy->hn;
+      a.xa = nullptr; a.ha = final ? nullptr : hy->ah; a.eps = d.norm_eps; a.D = D; a.plain_add = 1; a.nw_mode = d.norm_scalar ? 2 : 1; a.groups = 1;
+      a.res_mult = 1.f; a.ext = 0;
+      return hy_row_op_launch<AT>(e, T, a, st);
     }
+    const TanhNorm n{w, b, alpha};
+    float* hn = final ? hy->hn : (float*)nullptr;
+    AT* ha = final ? (AT*)nullptr : ah;
+    if (y.h != nullptr && y.bias == nullptr && y.ld % 8 == 0 && D % 8 == 0)
+      return hy_launch(e, hy_add_tanh_vec_kernel<AT>, dim3((unsigned)(((long long)T * (D / 8) + 255) / 256)), dim3(256), 0, st, hy->x, y.h, y.ld, n, hn, ha, D, T);
+    return hy_launch(e, hy_add_tanh_kernel<AT>, dim3(T, (D + 255) / 256), dim3(256), 0, st, hy->x, y, n, hn, ha, D);
+  };
+  if (tanh_norm) {
+    const HyLayer& l0 = hy->L[0];
+    XB_TRY(hy_launch(e, hy_embed_tanh_kernel<AT>, dim3(T), dim3(256), 0, st, (const int*)e->in_tokens, (const bf16*)hy->embed, hy->x, D, d.vocab,
+                     d.embed_scale, TanhNorm{l0.norm1, l0.norm1_b, l0.norm1_a}, ah));
+  } else {
+    XB_TRY(hy_launch(e, hy_embed_kernel, dim3(T), dim3(128), 0, st, (const int*)e->in_tokens, (const bf16*)hy->embed, hy->x, D, d.vocab, d.embed_scale));
+    XB_TRY(add_norm(hy_none(), hy->L[0].norm1, nullptr, nullptr, false));
   }
-  return 0;
+  for (int li = 0; li < d.n_layers; ++li) {
+    const HyLayer& l = hy->L[li];
+    const xb_hybrid_layer& c = l.d;
+    const bool has_ff = c.ff > 0, last = li + 1 == d.n_layers;
+    const float* nw = last ? hy->final_norm : hy->L[li + 1].norm1;
+    const float* nb = last ? hy->final_norm_b : hy->L[li + 1].norm1_b;
+    const float* na = last ? hy->final_norm_a : hy->L[li + 1].norm1_a;
+    LinOut P, y1;
+    XB_TRY(hy_linear<AT>(e, ah, D, l.w_in, l.t_in, l.b_in, T, l.n_in, D, hy->P, hy->cap_P, st, &P));
+    if (c.mixer == XB_MIX_LATENT) {
+      XB_TRY(hy_latent_mixer<AT>(e, l, T, P, m, st));
+    } else {   // gated linear attention
+      const int H = c.m_heads, n = c.m_dim, dv = c.m_vdim, HK = H * n, HV = H * dv, rk = c.m_rank;
+      const long long ldc = 3LL * HK + HV;
+      const unsigned cy = (unsigned)(((HK > HV ? HK : HV) + 255) / 256);
+      const float scale = 1.0f / sqrtf((float)n), inv_tau = 1.0f / c.m_tau;
+      if (T > 64)
+        XB_TRY(hy_launch(e, hy_gla_prep_kernel<8>, dim3((T + 7) / 8, cy), dim3(256), (size_t)8 * rk * sizeof(float), st, P, l.off_q, l.off_k, l.off_v, l.off_a, rk,
+                         (const bf16*)l.w_d2, (const float*)l.w0, inv_tau, scale, hy->c, ldc, HK, HV, T));
+      else
+        XB_TRY(hy_launch(e, hy_gla_prep_kernel<1>, dim3(T, cy), dim3(256), (size_t)rk * sizeof(float), st, P, l.off_q, l.off_k, l.off_v, l.off_a, rk,
+                         (const bf16*)l.w_d2, (const float*)l.w0, inv_tau, scale, hy->c, ldc, HK, HV, T));
+      RecurIn in;
+      in.c = hy->c; in.ldc = ldc; in.qoff = 0; in.koff = HK; in.xoff[0] = 2LL * HK; in.xoff[1] = in.xoff[2] = 0; in.voff = 3LL * HK; in.q_heads = H;
+      in.beta = in.decay = in.qk = in.hdecay = nullptr;
+      XB_TRY(hy_recur<HY_REC_GLA>(e, in, hy->state + l.st_rec, SS, hy->o, (long long)l.n_o, m, n_seqs, H, n, dv, st));
+      XB_TRY(hy_launch(e, hy_head_norm_kernel<AT>, dim3(T, (H + 7) / 8), dim3(256), 0, st, (const float*)hy->o, (long long)l.n_o,
+                       (const float*)l.head_norm, P, l.off_g, d.norm_eps, 1.0f, a1, (long long)l.n_o, H, dv, 0, 0));
+    }
+    XB_TRY(hy_linear<AT>(e, a1, l.n_o, l.w_o, l.t_o, nullptr, T, D, l.n_o, hy->m1, hy->cap_m, st, &y1));
+    if (has_ff) {
+      LinOut y2;
+      XB_TRY(add_norm(y1, l.norm2, l.norm2_b, l.norm2_a, false));
+      XB_TRY(hy_ff_parallel<AT>(e, l, T, hy->ah, st, &y2));
+      XB_TRY(add_norm(y2, nw, nb, na, last));
+    } else {
+      XB_TRY(add_norm(y1, nw, nb, na, last));
+    }
+    if (taps != nullptr && taps[li] != nullptr)
+      XB_CUDA(cudaMemcpyAsync(taps[li], hy->x, (size_t)T * D * sizeof(float), cudaMemcpyDeviceToDevice, st));
+  }
+  return with_head ? hy_run_head<AT>(e, n_seqs, m, st) : 0;
 }
 
 template <typename AT>
@@ -1561,6 +1764,7 @@ static int hy_run_body_t(xb_engine* e, int T, int n_seqs, int n_tiles, void* con
   HyModel* hy = e->hy;
   const xb_hybrid_desc& d = hy->d;
   if (d.block == XB_BLOCK_PARALLEL) return hy_run_parallel_t<AT>(e, T, n_seqs, taps, st, with_head);
+  if (d.block == XB_BLOCK_PRENORM) return hy_run_prenorm_t<AT>(e, T, n_seqs, taps, st, with_head);
   if (d.block == XB_BLOCK_BRANCHNORM) return hy_run_branchnorm_t<AT>(e, T, n_seqs, n_tiles, taps, st, with_head);
   typedef typename std::conditional<std::is_same<AT, float>::value, float, bf16>::type KT;
   BatchMeta m;
@@ -1699,18 +1903,7 @@ static int hy_run_body_t(xb_engine* e, int T, int n_seqs, int n_tiles, void* con
     if (taps != nullptr && taps[li] != nullptr)
       XB_CUDA(cudaMemcpyAsync(taps[li], hy->x, (size_t)T * D * sizeof(float), cudaMemcpyDeviceToDevice, st));
   }
-  if (with_head) {
-    const int n = e->sel_rows != nullptr ? e->sel_n : n_seqs;
-    if (n > 0) {
-      const int* idx = e->sel_rows != nullptr ? hy->d_rows : m.seq_last;
-      LinOut y;
-      XB_TRY(hy_launch(e, hy_gather_rows_kernel<AT>, dim3(n), dim3(256), 0, st, (const float*)hy->hn, idx, reinterpret_cast<AT*>(hy->head_in), D));
-      XB_TRY(hy_linear<AT>(e, hy->head_in, D, hy->head, hy->t_head, nullptr, n, d.vocab, D, hy->head_raw, hy->cap_head, st, &y));
-      const long long tot = (long long)n * d.vocab;
-      XB_TRY(hy_launch(e, hy_logits_kernel, dim3((unsigned)((tot + 255) / 256)), dim3(256), 0, st, y, d.logit_softcap, e->logits, n, d.vocab));
-    }
-  }
-  return 0;
+  return with_head ? hy_run_head<AT>(e, n_seqs, m, st) : 0;
 }
 
 static int hy_run_body(xb_engine* e, int T, int n_seqs, int n_splits, int n_tiles, void* const* taps, cudaStream_t st, int with_head) {

@@ -19,12 +19,14 @@
 // programmatic-serialization attribute, the next kernel's launch overlaps this one's execution and it touches upstream
 // data only after the wait (the whole chain of earlier kernels has then completed).
 #define HY_MAX_TAPS 16   // causal filters keep taps - 1 inputs per sequence
+#define HY_MAX_DECAY_RANK 1024   // gated linear attention: rows of the decay's first projection
 #define HY_MAX_KDIM 256  // recurrent state: four lanes own one value column, up to 64 rows each
 // what one step does to a state column S_j (see hy_recur_kernel)
 #define HY_REC_HGRN 0
 #define HY_REC_DELTA 1
 #define HY_REC_GDELTA 2
 #define HY_REC_LIGHTNING 3
+#define HY_REC_GLA 4
 
 struct LinOut {
   const float* f;      // fp32 [planes][T][ld] (planes summed per column, see SplitInfo), or nullptr
@@ -87,6 +89,27 @@ __global__ void hy_embed_kernel(const int* __restrict__ tokens, const bf16* __re
   int tok = tokens[t];
   tok = tok < 0 ? 0 : (tok >= V ? V - 1 : tok);
   for (int i = threadIdx.x; i < D; i += blockDim.x) x[(long long)t * D + i] = bf2f(emb[(long long)tok * D + i]) * scale;
+}
+
+// tanh(alpha * x) * w + b: a norm of the stream without statistics of the row (one channel at a time, fp32)
+struct TanhNorm { const float *w, *b, *alpha; };
+__device__ __forceinline__ float hy_tanh_norm(const TanhNorm& n, float alpha, float x, int i) { return fmaf(tanhf(alpha * x), n.w[i], n.b[i]); }
+
+// The embedding row and the first layer's norm of it: x = emb * scale, ha = norm(x) as a Linear input.  grid (T), 256 threads.
+template <typename AT>
+__global__ void __launch_bounds__(256) hy_embed_tanh_kernel(const int* __restrict__ tokens, const bf16* __restrict__ emb, float* __restrict__ x,
+                                                            int D, int V, float scale, TanhNorm n, AT* __restrict__ ha) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int t = blockIdx.x;
+  int tok = tokens[t];
+  tok = tok < 0 ? 0 : (tok >= V ? V - 1 : tok);
+  const float alpha = n.alpha[0];
+  for (int i = threadIdx.x; i < D; i += 256) {
+    const float v = bf2f(emb[(long long)tok * D + i]) * scale;
+    x[(long long)t * D + i] = v;
+    act_store<AT>(ha + (long long)t * D + i, hy_tanh_norm(n, alpha, v, i));
+  }
 }
 
 // Embedding as a sum of three rows: the token's, a hashed row of the (previous token, token) pair and a learned position row.
@@ -431,6 +454,45 @@ __global__ void __launch_bounds__(256) hy_row_op_gated_vec_kernel(RowOpArgs a) {
   }
 }
 
+// Pre-norm blocks with the tanh norm: x += m, then the next reader's norm of it as a Linear input (ha) or, behind the last
+// layer, in fp32 (hn).  Nothing here looks across a row, so a thread owns a channel: grid (T, ceil(D / 256)), 256 threads.
+template <typename AT>
+__global__ void __launch_bounds__(256) hy_add_tanh_kernel(float* __restrict__ x, LinOut m, TanhNorm n, float* __restrict__ hn, AT* __restrict__ ha, int D) {
+  pdl_launch_dependents();
+  const int i = blockIdx.y * 256 + threadIdx.x;
+  const long long at = (long long)blockIdx.x * D + i;
+  pdl_wait();
+  if (i >= D) return;
+  const float v = x[at] + lin_at(m, blockIdx.x, i);
+  x[at] = v;
+  const float y = hy_tanh_norm(n, n.alpha[0], v, i);
+  if (hn != nullptr) hn[at] = y;
+  if (ha != nullptr) act_store<AT>(ha + at, y);
+}
+// the same for prompts whose branch is one bf16 matrix: eight channels per thread (D and the branch's pitch multiples of 8)
+template <typename AT>
+__global__ void __launch_bounds__(256) hy_add_tanh_vec_kernel(float* __restrict__ x, const bf16* __restrict__ m, long long ldm, TanhNorm n,
+                                                              float* __restrict__ hn, AT* __restrict__ ha, int D, int T) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const long long idx = (long long)blockIdx.x * 256 + threadIdx.x;
+  const int d8 = D >> 3;
+  if (idx >= (long long)T * d8) return;
+  const long long t = idx / d8;
+  const int i = (int)(idx - t * d8) << 3;
+  const float alpha = n.alpha[0];
+  float v[8], b[8];
+  hy_load8(m + t * ldm + i, nullptr, b);
+  hy_ld8f(x + t * D + i, v);
+#pragma unroll
+  for (int j = 0; j < 8; ++j) v[j] += b[j];
+  hy_st8f(x + t * D + i, v);
+#pragma unroll
+  for (int j = 0; j < 8; ++j) b[j] = hy_tanh_norm(n, alpha, v[j], i + j);
+  if (hn != nullptr) hy_st8f(hn + t * D + i, b);
+  if (ha != nullptr) hy_st8a<AT>(ha + t * D + i, b);
+}
+
 template <typename AT>
 __global__ void __launch_bounds__(256) hy_row_op_vec_kernel(RowOpArgs a) {
   pdl_launch_dependents();
@@ -753,6 +815,7 @@ __global__ void __launch_bounds__(256) hy_delta_prep_kernel(float* __restrict__ 
 //               with a = u . S_j and b = (r * w) . S_j on the OLD column: o_j = b - (r . (a * u)) a + (r . k) v_j
 //               (five row vectors per step: r * w, u, w, a * u, k; the two scalars in the beta / decay slots)
 //   lightning:  S_j <- decay S_j + k v_j;  o_j = q . S_j          (one constant decay per head)
+//   gated linear attention: S_j <- w * S_j + k v_j;  o_j = q . S_j  (a decay w per row and step: three row vectors q, k, w)
 // LPC lanes (4, 8 or 16) own one column: lane `sub` holds the rows of the 16-byte chunks sub, sub + LPC, ... (NCH chunks,
 // rows beyond dk are zero), so a dot product over the rows ends in log2(LPC) shuffles and a warp carries 32 / LPC
 // columns.  More lanes per column mean more blocks and shorter per-step chains (one long sequence), fewer mean fewer
@@ -761,13 +824,13 @@ __global__ void __launch_bounds__(256) hy_delta_prep_kernel(float* __restrict__ 
 // cp.async, one chunk of steps ahead of the arithmetic.
 // grid (n_seqs, H, ceil(dv * LPC / 128)), 128 threads; state [slot][H][dv][dk] fp32;
 // dynamic shared memory 2 * HY_TS * (NV * 4 * LPC * NCH + 128 / LPC + 4) floats, NV = hy_rec_vectors(MODE) row vectors per step.
-__host__ __device__ constexpr int hy_rec_vectors(int mode) { return mode == HY_REC_GDELTA ? 5 : 2; }
+__host__ __device__ constexpr int hy_rec_vectors(int mode) { return mode == HY_REC_GDELTA ? 5 : (mode == HY_REC_GLA ? 3 : 2); }
 #define HY_TS 16
 struct RecurIn {
   const float* c;        // [T, ldc] prepared inputs
   long long ldc;
   long long qoff, koff, voff;   // columns of head 0's q, k (or f) and v; heads follow at q_stride / k_stride / dv
-  long long xoff[3];     // HY_REC_GDELTA: columns of head 0's decay w, removal a*u and key k (qoff: r*w, koff: unit key u)
+  long long xoff[3];     // HY_REC_GLA: column of head 0's decay w (first entry); HY_REC_GDELTA: columns of head 0's decay w, removal a*u and key k (qoff: r*w, koff: unit key u)
   int q_heads;           // delta rule: heads share q / k in groups (q head = h / (H / q_heads)); others: = H
   const float *beta, *decay, *qk;   // gated delta rule: [T, H], [T, H], [T, q_heads]; HY_REC_GDELTA: beta = r.(a*u), decay = r.k, [T, H]
   const float* hdecay;   // HY_REC_LIGHTNING: [H] constant decay per head
@@ -807,10 +870,12 @@ __global__ void __launch_bounds__(128) hy_recur_kernel(RecurIn in, float* __rest
 #pragma unroll
     for (int i = 0; i < 3; ++i) cx[i] = in.c + in.xoff[i] + (long long)g * dk;
   }
+  if (MODE == HY_REC_GLA) cx[0] = in.c + in.xoff[0] + (long long)g * dk;
   const float hd = MODE == HY_REC_LIGHTNING ? in.hdecay[h] : 0.f;
   // 16-byte copies when every row piece starts on a 16-byte boundary
   bool al = ((in.ldc | in.qoff | in.koff | in.voff | dk | dv) & 3) == 0 && (reinterpret_cast<uintptr_t>(in.c) & 15) == 0;
   if (MODE == HY_REC_GDELTA) al = al && ((in.xoff[0] | in.xoff[1] | in.xoff[2]) & 3) == 0;
+  if (MODE == HY_REC_GLA) al = al && (in.xoff[0] & 3) == 0;
   for (int i = threadIdx.x; i < 2 * HY_TS * STRIDE; i += blockDim.x) stg[i] = 0.f;   // padding rows / columns stay zero
   float* st = state + (long long)sp.slot * state_stride + ((long long)h * dv + (live ? j : 0)) * dk;
   float S[4 * NCH];
@@ -931,6 +996,25 @@ __global__ void __launch_bounds__(128) hy_recur_kernel(RecurIn in, float* __rest
           S[4 * ch + 1] = fmaf(hd, S[4 * ch + 1], k4.y * v);
           S[4 * ch + 2] = fmaf(hd, S[4 * ch + 2], k4.z * v);
           S[4 * ch + 3] = fmaf(hd, S[4 * ch + 3], k4.w * v);
+          b0 = fmaf(q4.x, S[4 * ch], b0); b1 = fmaf(q4.y, S[4 * ch + 1], b1);
+          b0 = fmaf(q4.z, S[4 * ch + 2], b0); b1 = fmaf(q4.w, S[4 * ch + 3], b1);
+        }
+        float b = b0 + b1;
+#pragma unroll
+        for (int off = 1; off < LPC; off <<= 1) b += __shfl_xor_sync(0xffffffffu, b, off);
+        if (sub == 0 && live) o[orow0 + (long long)ts * ldo] = b;
+      } else if (MODE == HY_REC_GLA) {
+        float b0 = 0.f, b1 = 0.f;
+#pragma unroll
+        for (int ch = 0; ch < NCH; ++ch) {
+          const int r = (ch * LPC + sub) * 4;
+          const float4 q4 = *reinterpret_cast<const float4*>(sr + r);
+          const float4 k4 = *reinterpret_cast<const float4*>(sr + DKP + r);
+          const float4 w4 = *reinterpret_cast<const float4*>(sr + 2 * DKP + r);
+          S[4 * ch] = fmaf(w4.x, S[4 * ch], k4.x * v);
+          S[4 * ch + 1] = fmaf(w4.y, S[4 * ch + 1], k4.y * v);
+          S[4 * ch + 2] = fmaf(w4.z, S[4 * ch + 2], k4.z * v);
+          S[4 * ch + 3] = fmaf(w4.w, S[4 * ch + 3], k4.w * v);
           b0 = fmaf(q4.x, S[4 * ch], b0); b1 = fmaf(q4.y, S[4 * ch + 1], b1);
           b0 = fmaf(q4.z, S[4 * ch + 2], b0); b1 = fmaf(q4.w, S[4 * ch + 3], b1);
         }
@@ -1779,19 +1863,29 @@ __global__ void hy_logits_kernel(LinOut y, float cap, float* __restrict__ out, i
 }
 
 // ----------------------------------------------------------------------------- latent attention
-// Per token the fused projection P carries q (H heads of [dn unrotated | dr rotated]) and the down-projection
-// [R latent | dr rotated key part].  One block per token:
+// Per token the fused projection P carries the down-projection [R latent | dr rotated key part] (off_dkv, < 0: the layer reads
+// another layer's rows) and, when queries pass a latent of their own, its columns (off_dq).  One block per token:
 //   cache row  = [ latent / rms(latent) * nw  |  rot(key part) ]      -> k_pool (one "key head", row of R + dr elements)
-//   qa[t, h]   = [ (filled by hy_head_mm_t_kernel)  |  rot(q rotated part of head h) ]   fp32, rows of H * (R + dr)
-// rot: entries 2i, 2i+1 (i < rot_dims / 2) turn by the angle pos * freq[i]; the others pass.  Angles are fp32.
-template <typename KT>
-__global__ void __launch_bounds__(256) hy_latent_prep_kernel(LinOut P, int off_q, int off_dkv, int H, int dn, int dr, int R, int rot_dims,
-                                                             const float* __restrict__ freq, const float* __restrict__ nw, float eps,
-                                                             KT* __restrict__ k_pool, BatchMeta m, float* __restrict__ qa) {
+//   cq[t]      = latent query / rms * qnw, as a Linear input           (qr = 0: none)
+template <typename AT, typename KT>
+__global__ void __launch_bounds__(256) hy_latent_down_kernel(LinOut P, int off_dkv, int dr, int R, RotArgs r, const float* __restrict__ nw, float eps,
+                                                             KT* __restrict__ k_pool, BatchMeta m, int off_dq, int qr,
+                                                             const float* __restrict__ qnw, AT* __restrict__ cq) {
   pdl_launch_dependents();
   pdl_wait();
   __shared__ float red[32];
   const int row = blockIdx.x;
+  if (qr > 0) {
+    float ss = 0.f;
+    for (int i = threadIdx.x; i < qr; i += 256) {
+      const float v = lin_at(P, row, off_dq + i);
+      ss = fmaf(v, v, ss);
+    }
+    ss = block_sum<256>(ss, red);
+    const float inv = 1.0f / sqrtf(ss / (float)qr + eps);
+    for (int i = threadIdx.x; i < qr; i += 256) act_store<AT>(cq + (long long)row * qr + i, lin_at(P, row, off_dq + i) * inv * qnw[i]);
+  }
+  if (off_dkv < 0) return;
   const int s = m.tok_seq[row], pos = m.tok_pos[row];
   const int page = m.page_table[(long long)m.seq_slot[s] * m.max_pages + pos / m.page_tokens];
   KT* kr = k_pool + ((long long)page * m.page_tokens + pos % m.page_tokens) * (R + dr);
@@ -1803,68 +1897,81 @@ __global__ void __launch_bounds__(256) hy_latent_prep_kernel(LinOut P, int off_q
   ss = block_sum<256>(ss, red);
   const float inv = 1.0f / sqrtf(ss / (float)R + eps);
   for (int i = threadIdx.x; i < R; i += 256) act_store<KT>(kr + i, lin_at(P, row, off_dkv + i) * inv * nw[i]);
-  const int half = rot_dims >> 1, hp = dr - half;   // per vector: `half` pairs, then the entries that pass unchanged
-  // vector 0 = the shared key part, 1 + h = head h's rotated query part
-  for (int idx = threadIdx.x; idx < (H + 1) * hp; idx += 256) {
-    const int vec = idx / hp, i = idx - vec * hp;
-    const int src = vec == 0 ? off_dkv + R : off_q + (vec - 1) * (dn + dr) + dn;
-    float* qd = qa + (long long)row * H * (R + dr) + (long long)(vec - 1) * (R + dr) + R;
+  const int half = r.dims >> 1;   // `half` pairs, then the entries that pass unchanged
+  for (int i = threadIdx.x; i < dr - half; i += 256) {
     if (i < half) {
-      const float u = lin_at(P, row, src + 2 * i), v = lin_at(P, row, src + 2 * i + 1);
-      float sn, cs;
-      sincosf((float)pos * freq[i], &sn, &cs);
-      const float a = u * cs - v * sn, b = v * cs + u * sn;
-      if (vec == 0) { act_store<KT>(kr + R + 2 * i, a); act_store<KT>(kr + R + 2 * i + 1, b); }
-      else { qd[2 * i] = a; qd[2 * i + 1] = b; }
+      const int d0 = r.half ? i : 2 * i, d1 = r.half ? i + half : 2 * i + 1;
+      const float u = lin_at(P, row, off_dkv + R + d0), v = lin_at(P, row, off_dkv + R + d1);
+      float cs, sn;
+      hy_rot_cs(r, pos, i, &cs, &sn);
+      act_store<KT>(kr + R + d0, u * cs - v * sn);
+      act_store<KT>(kr + R + d1, v * cs + u * sn);
     } else {
-      const int j = rot_dims + (i - half);
-      const float v = lin_at(P, row, src + j);
-      if (vec == 0) act_store<KT>(kr + R + j, v);
-      else qd[j] = v;
+      act_store<KT>(kr + R + half + i, lin_at(P, row, off_dkv + R + half + i));
     }
   }
 }
 
-// Per-head products with a weight that is stored head by head.
-// "t" form (a query folded into the latent space): y[t, h * ldy + n] = sum_k X[t, xoff + h * xs + k] * W[(h * K + k) * N + n]
+// Queries in the cache's space.  Q carries H heads of [K unrotated | dr rotated] (columns from qoff); per head
+//   qa[t, h, n]     = sum_k Q[t, h, k] * W[(h * K + k) * N + n]     n < N: the query folded into the latent space
+//   qa[t, h, N + i] = rot(rotated part)[i]                          i < dr
 // grid (ceil(T / 8), H), 256 threads over n; the 8 rows' inputs sit in shared memory (8 * K floats).
 #define HY_MM_ROWS 8
-__global__ void __launch_bounds__(256) hy_head_mm_t_kernel(LinOut X, int xoff, int xs, const bf16* __restrict__ W, float* __restrict__ y,
-                                                           long long ldy_row, int ldy, int T, int K, int N) {
+__global__ void __launch_bounds__(256) hy_latent_absorb_kernel(LinOut Q, int qoff, int dr, const bf16* __restrict__ W, float* __restrict__ qa,
+                                                               int H, int T, int K, int N, RotArgs r, const int* __restrict__ tok_pos) {
   pdl_launch_dependents();
   pdl_wait();
   extern __shared__ __align__(16) float xsm[];
   const int t0 = blockIdx.x * HY_MM_ROWS, h = blockIdx.y;
   const int nt = T - t0 < HY_MM_ROWS ? T - t0 : HY_MM_ROWS;
+  const int qh = qoff + h * (K + dr), ld = N + dr;
   for (int i = threadIdx.x; i < HY_MM_ROWS * K; i += 256) {
-    const int r = i / K, k = i - r * K;
-    xsm[i] = r < nt ? lin_at(X, t0 + r, xoff + h * xs + k) : 0.f;
+    const int rr = i / K, k = i - rr * K;
+    xsm[i] = rr < nt ? lin_at(Q, t0 + rr, qh + k) : 0.f;
+  }
+  const int half = r.dims >> 1, per = dr - half;
+  for (int u = threadIdx.x; u < nt * per; u += 256) {
+    const int rr = u / per, i = u - rr * per, t = t0 + rr;
+    float* qd = qa + ((long long)t * H + h) * ld + N;
+    if (i < half) {
+      const int d0 = r.half ? i : 2 * i, d1 = r.half ? i + half : 2 * i + 1;
+      const float a = lin_at(Q, t, qh + K + d0), b = lin_at(Q, t, qh + K + d1);
+      float cs, sn;
+      hy_rot_cs(r, tok_pos[t], i, &cs, &sn);
+      qd[d0] = a * cs - b * sn;
+      qd[d1] = b * cs + a * sn;
+    } else {
+      qd[half + i] = lin_at(Q, t, qh + K + half + i);
+    }
   }
   __syncthreads();
   const bf16* Wh = W + (long long)h * K * N;
   for (int n = threadIdx.x; n < N; n += 256) {
     float acc[HY_MM_ROWS];
 #pragma unroll
-    for (int r = 0; r < HY_MM_ROWS; ++r) acc[r] = 0.f;
+    for (int rr = 0; rr < HY_MM_ROWS; ++rr) acc[rr] = 0.f;
     for (int k = 0; k < K; ++k) {
       const float w = bf2f(Wh[(long long)k * N + n]);
 #pragma unroll
-      for (int r = 0; r < HY_MM_ROWS; ++r) acc[r] = fmaf(xsm[r * K + k], w, acc[r]);
+      for (int rr = 0; rr < HY_MM_ROWS; ++rr) acc[rr] = fmaf(xsm[rr * K + k], w, acc[rr]);
     }
-    for (int r = 0; r < nt; ++r) y[(long long)(t0 + r) * ldy_row + (long long)h * ldy + n] = acc[r];
+    for (int rr = 0; rr < nt; ++rr) qa[((long long)(t0 + rr) * H + h) * ld + n] = acc[rr];
   }
 }
+// Per-head products with a weight that is stored head by head,
 // plain form (a latent read-out turned into the head's value): y[t, h * N + n] = sum_k x[t, h * K + k] * W[(h * N + n) * K + k]
 // grid (ceil(T / 8), H), 128 threads: a thread owns an output n and walks its weight row 16 bytes at a time against the 8 rows'
-// inputs in shared memory (broadcast reads, no shuffles).
+// inputs in shared memory (broadcast reads, no shuffles).  off_gate >= 0: head h is multiplied by sigmoid(G[t, off_gate + h]).
 template <typename AT>
 __global__ void __launch_bounds__(128) hy_head_mm_kernel(const float* __restrict__ x, long long ldx, const bf16* __restrict__ W,
-                                                         AT* __restrict__ y, long long ldy, int T, int K, int N) {
+                                                         AT* __restrict__ y, long long ldy, int T, int K, int N, LinOut G, int off_gate) {
   pdl_launch_dependents();
   pdl_wait();
   extern __shared__ __align__(16) float xsm[];
+  __shared__ float gate[HY_MM_ROWS];
   const int t0 = blockIdx.x * HY_MM_ROWS, h = blockIdx.y;
   const int nt = T - t0 < HY_MM_ROWS ? T - t0 : HY_MM_ROWS;
+  if (threadIdx.x < HY_MM_ROWS) gate[threadIdx.x] = off_gate >= 0 && threadIdx.x < nt ? hy_sigmoid(lin_at(G, t0 + threadIdx.x, off_gate + h)) : 1.0f;
   for (int i = threadIdx.x; i < HY_MM_ROWS * K; i += 128) {
     const int r = i / K, k = i - r * K;
     xsm[i] = r < nt ? x[(long long)(t0 + r) * ldx + (long long)h * K + k] : 0.f;
@@ -1896,7 +2003,7 @@ __global__ void __launch_bounds__(128) hy_head_mm_kernel(const float* __restrict
         for (int r = 0; r < HY_MM_ROWS; ++r) acc[r] = fmaf(xsm[r * K + k], w, acc[r]);
       }
     }
-    for (int r = 0; r < nt; ++r) act_store<AT>(y + (long long)(t0 + r) * ldy + (long long)h * N + n, acc[r]);
+    for (int r = 0; r < nt; ++r) act_store<AT>(y + (long long)(t0 + r) * ldy + (long long)h * N + n, acc[r] * gate[r]);
   }
 }
 
@@ -1975,30 +2082,94 @@ __global__ void __launch_bounds__(256) hy_gdelta_prep_kernel(LinOut P, int off_r
   }
 }
 
+// ----------------------------------------------------------------------------- gated linear attention: what the recurrence reads
+// From the fused projection P (q | k | v | gate | first decay projection of rk columns), the decay's second projection W2 [HK, rk]
+// and its bias, all fp32:
+//   z = W2 a + b,  w = sigmoid(z)^(1 / tau) = exp(-softplus(-z) / tau)
+//   c row = [ q * scale | k | w | v ]  (blocks of HK, HK, HK, HV)
+// ROWS tokens per block share the reads of W2.  grid (ceil(T / ROWS), ceil(max(HK, HV) / 256)), 256 threads, ROWS * rk floats.
+template <int ROWS>
+__global__ void __launch_bounds__(256) hy_gla_prep_kernel(LinOut P, int off_q, int off_k, int off_v, int off_a, int rk, const bf16* __restrict__ w2,
+                                                          const float* __restrict__ b2, float inv_tau, float scale, float* __restrict__ c,
+                                                          long long ldc, int HK, int HV, int T) {
+  pdl_launch_dependents();
+  pdl_wait();
+  extern __shared__ float as[];
+  const int t0 = blockIdx.x * ROWS;
+  const int nt = T - t0 < ROWS ? T - t0 : ROWS;
+  for (int i = threadIdx.x; i < ROWS * rk; i += 256) {
+    const int r = i / rk, k = i - r * rk;
+    as[i] = r < nt ? lin_at(P, t0 + r, off_a + k) : 0.f;
+  }
+  __syncthreads();
+  const int i = blockIdx.y * 256 + threadIdx.x;
+  if (i < HK) {
+    float z[ROWS];
+    const float b = b2[i];
+#pragma unroll
+    for (int r = 0; r < ROWS; ++r) z[r] = b;
+    const bf16* wr = w2 + (long long)i * rk;
+    if ((rk & 7) == 0 && (reinterpret_cast<uintptr_t>(w2) & 15) == 0) {
+      for (int k = 0; k < rk; k += 8) {
+        float wv[8];
+        hy_load8(wr + k, nullptr, wv);
+#pragma unroll
+        for (int r = 0; r < ROWS; ++r)
+#pragma unroll
+          for (int j = 0; j < 8; ++j) z[r] = fmaf(wv[j], as[r * rk + k + j], z[r]);
+      }
+    } else {
+      for (int k = 0; k < rk; ++k) {
+        const float wv = bf2f(wr[k]);
+#pragma unroll
+        for (int r = 0; r < ROWS; ++r) z[r] = fmaf(wv, as[r * rk + k], z[r]);
+      }
+    }
+#pragma unroll
+    for (int r = 0; r < ROWS; ++r) {
+      if (r >= nt) break;
+      float* row = c + (long long)(t0 + r) * ldc;
+      row[i] = lin_at(P, t0 + r, off_q + i) * scale;
+      row[HK + i] = lin_at(P, t0 + r, off_k + i);
+      row[2 * HK + i] = expf(-(fmaxf(-z[r], 0.f) + log1pf(expf(-fabsf(z[r])))) * inv_tau);
+    }
+  }
+  if (i < HV) {
+#pragma unroll
+    for (int r = 0; r < ROWS; ++r) {
+      if (r >= nt) break;
+      c[(long long)(t0 + r) * ldc + 3LL * HK + i] = lin_at(P, t0 + r, off_v + i);
+    }
+  }
+}
+
 // ----------------------------------------------------------------------------- clamped gated feed-forward, experts
 __device__ __forceinline__ float hy_glu_clamp(float g, float u, float limit) {
   g = fminf(g, limit);
   u = fminf(fmaxf(u, -limit), limit);
   return g * hy_sigmoid(1.702f * g) * (u + 1.0f);
 }
-// One channel of one expert with routing weight w.  act: XB_ACT_GLU_CLAMP or XB_ACT_SWIGLU (silu(g) u, no limits).
+// One channel of one expert with routing weight w.  act: XB_ACT_GLU_CLAMP, XB_ACT_SWIGLU (silu(g) u) or XB_ACT_GEGLU (gelu(g) u,
+// tanh form), the last two without limits.
 // on_input: the weight multiplies what the expert reads, and since both projections are linear, (w h) W^T = w (h W^T):
 // gate and up are scaled before the activation; otherwise the weight multiplies the activation (and so the output).
 __device__ __forceinline__ float hy_expert_act(float g, float u, float w, float limit, int act, int on_input) {
   if (on_input) { g *= w; u *= w; }
-  const float y = act == XB_ACT_SWIGLU ? hy_silu(g) * u : hy_glu_clamp(g, u, limit);
+  const float y = act == XB_ACT_SWIGLU ? hy_silu(g) * u : (act == XB_ACT_GEGLU ? hy_gelu_tanh(g) * u : hy_glu_clamp(g, u, limit));
   return on_input ? y : w * y;
 }
-// U carries [gate (F) | up (F)] (biases on read): out[t, i] = glu(gate_i, up_i).  grid over T * F.
+// The shared expert's weight: a routing row wider than its E experts carries it behind them, otherwise it is one.
+__device__ __forceinline__ float hy_shared_weight(const float* gwrow, int ldg, int E) { return ldg > E ? gwrow[E] : 1.0f; }
+// U carries [gate (F) | up (F)] (biases on read): out[t, i] = act(gate_i, up_i) (XB_ACT_*, see above).  grid over T * F.
 template <typename AT>
-__global__ void hy_glu_clamp_kernel(LinOut U, int F, float limit, AT* __restrict__ out, long long ld_out, int T) {
+__global__ void hy_glu_kernel(LinOut U, int F, float limit, int act, AT* __restrict__ out, long long ld_out, int T) {
   pdl_launch_dependents();
   pdl_wait();
   const long long idx = (long long)blockIdx.x * blockDim.x + threadIdx.x;
   if (idx >= (long long)T * F) return;
   const long long t = idx / F;
   const int i = (int)(idx - t * F);
-  act_store<AT>(out + t * ld_out + i, hy_glu_clamp(lin_at(U, t, i), lin_at(U, t, F + i), limit));
+  act_store<AT>(out + t * ld_out + i, hy_expert_act(lin_at(U, t, i), lin_at(U, t, F + i), 1.0f, limit, act, 0));
 }
 
 // The same two activations on a bf16 matrix (prompts: the tcgen05 Linear's output), eight neighbours per thread.
@@ -2018,8 +2189,8 @@ __device__ __forceinline__ uint4 hy_glu8(const float* g, const float* u, float l
   for (int j = 0; j < 8; ++j) y[j] = hy_expert_act(g[j], u[j], w, limit, act, on_input);
   return make_uint4(f2_to_bf2(y[0], y[1]), f2_to_bf2(y[2], y[3]), f2_to_bf2(y[4], y[5]), f2_to_bf2(y[6], y[7]));
 }
-__global__ void hy_glu_clamp_vec_kernel(const bf16* __restrict__ u, long long ld, const float* __restrict__ bias, int F, float limit,
-                                        bf16* __restrict__ out, long long ld_out, int T) {
+__global__ void hy_glu_vec_kernel(const bf16* __restrict__ u, long long ld, const float* __restrict__ bias, int F, float limit, int act,
+                                  bf16* __restrict__ out, long long ld_out, int T) {
   pdl_launch_dependents();
   pdl_wait();
   const long long idx = (long long)blockIdx.x * blockDim.x + threadIdx.x;
@@ -2030,9 +2201,9 @@ __global__ void hy_glu_clamp_vec_kernel(const bf16* __restrict__ u, long long ld
   float g[8], v[8];
   hy_load8(u + t * ld + i, bias != nullptr ? bias + i : nullptr, g);
   hy_load8(u + t * ld + F + i, bias != nullptr ? bias + F + i : nullptr, v);
-  *reinterpret_cast<uint4*>(out + t * ld_out + i) = hy_glu8(g, v, limit, 1.0f);
+  *reinterpret_cast<uint4*>(out + t * ld_out + i) = hy_glu8(g, v, limit, 1.0f, act, 0);
 }
-__global__ void hy_moe_act_vec_kernel(const bf16* __restrict__ u, long long ld, const float* __restrict__ gw, int E, int f, float limit, int sf,
+__global__ void hy_moe_act_vec_kernel(const bf16* __restrict__ u, long long ld, const float* __restrict__ gw, int ldg, int E, int f, float limit, int sf,
                                       float limit_s, int act, int on_input, bf16* __restrict__ out, long long ld_out, int T) {
   pdl_launch_dependents();
   pdl_wait();
@@ -2045,7 +2216,7 @@ __global__ void hy_moe_act_vec_kernel(const bf16* __restrict__ u, long long ld, 
   uint4 r = make_uint4(0u, 0u, 0u, 0u);
   if (i < E * f) {
     const int e = i / f, j = i - e * f;
-    const float w = gw[t * E + e];
+    const float w = gw[t * ldg + e];
     if (w != 0.f) {
       hy_load8(u + t * ld + 2 * e * f + j, nullptr, g);
       hy_load8(u + t * ld + 2 * e * f + f + j, nullptr, v);
@@ -2055,7 +2226,7 @@ __global__ void hy_moe_act_vec_kernel(const bf16* __restrict__ u, long long ld, 
     const int j = i - E * f;
     hy_load8(u + t * ld + 2 * E * f + j, nullptr, g);
     hy_load8(u + t * ld + 2 * E * f + sf + j, nullptr, v);
-    r = hy_glu8(g, v, limit_s, 1.0f, act, 0);
+    r = hy_glu8(g, v, limit_s, hy_shared_weight(gw + t * ldg, ldg, E), act, 0);
   }
   *reinterpret_cast<uint4*>(out + t * ld_out + i) = r;
 }
@@ -2119,9 +2290,9 @@ __global__ void __launch_bounds__(256) hy_router_logits_kernel(const AT* __restr
 // per warp.
 // score_mode: XB_ROUTE_SIGMOID, or XB_ROUTE_SOFTMAX = softmax of the logits over all experts.  group_mode: XB_GROUP_TOP2 as above,
 // or XB_GROUP_MAX = a group is worth its best score.  renorm: the chosen experts' scores are divided by their sum (+ 1e-20)
-// before the scale.
+// before the scale.  shared_gate: the row has one more logit, and sigmoid of it is the shared expert's weight (gwrow[E]).
 __device__ __forceinline__ void hy_route_token(const float* __restrict__ zrow, float* sc, float* el, float* gs, int E, int top, int groups, int keep,
-                                               float scale, float* __restrict__ gwrow, int score_mode, int group_mode, int renorm) {
+                                               float scale, float* __restrict__ gwrow, int score_mode, int group_mode, int renorm, int shared_gate) {
   const int lane = threadIdx.x & 31;
   if (score_mode == XB_ROUTE_SOFTMAX) {
     float mx = -INFINITY;
@@ -2160,6 +2331,7 @@ __device__ __forceinline__ void hy_route_token(const float* __restrict__ zrow, f
     __syncwarp();
   }
   for (int e = lane; e < E; e += 32) gwrow[e] = 0.f;
+  if (shared_gate && lane == 0) gwrow[E] = hy_sigmoid(zrow[E]);
   float tot = 0.f;   // sum of the chosen scores (every lane follows the same picks)
   for (int r = 0; r < top; ++r) {
     float bv = -1.f;
@@ -2184,7 +2356,7 @@ __device__ __forceinline__ void hy_route_token(const float* __restrict__ zrow, f
   }
 }
 __global__ void __launch_bounds__(128) hy_route_kernel(const float* __restrict__ z, int E, int top, int groups, int keep, float scale,
-                                                       float* __restrict__ gw, int T, int score_mode, int group_mode, int renorm) {
+                                                       float* __restrict__ gw, int T, int score_mode, int group_mode, int renorm, int shared_gate) {
   pdl_launch_dependents();
   pdl_wait();
   extern __shared__ float rsm[];
@@ -2192,15 +2364,16 @@ __global__ void __launch_bounds__(128) hy_route_kernel(const float* __restrict__
   const long long t = (long long)blockIdx.x * 4 + warp;
   if (t >= T) return;
   float* sc = rsm + (size_t)warp * (2 * E + (groups > 0 ? groups : 1));
-  hy_route_token(z + t * E, sc, sc + E, sc + 2 * E, E, top, groups, keep, scale, gw + t * E, score_mode, group_mode, renorm);
+  const int ld = E + (shared_gate ? 1 : 0);
+  hy_route_token(z + t * ld, sc, sc + E, sc + 2 * E, E, top, groups, keep, scale, gw + t * ld, score_mode, group_mode, renorm, shared_gate);
 }
 // Steps of few rows: logits and routing of a token in ONE block of eight warps.  Warp w forms the fp32 logits of experts
 // w, w + 8, ... (16-byte weight loads, fp32 sums, the order of hy_router_logits_kernel<AT, 1>), then the first warp routes.
-// Shared memory: 3 * E + groups floats.  grid (T), 256 threads.
+// Shared memory: 3 * E + groups + 1 floats.  grid (T), 256 threads.
 template <typename AT>
 __global__ void __launch_bounds__(256) hy_router_route_kernel(const AT* __restrict__ x, long long ldx, const bf16* __restrict__ w, int K, int E, int top,
                                                               int groups, int keep, float scale, float* __restrict__ gw, int score_mode, int group_mode,
-                                                              int renorm) {
+                                                              int renorm, int shared_gate) {
   pdl_launch_dependents();
   pdl_wait();
   extern __shared__ float rsm[];
@@ -2208,7 +2381,8 @@ __global__ void __launch_bounds__(256) hy_router_route_kernel(const AT* __restri
   const long long t = blockIdx.x;
   const AT* xr = x + t * ldx;
   const bool vec = (K & 7) == 0 && (reinterpret_cast<uintptr_t>(w) & 15) == 0;
-  for (int e = warp; e < E; e += 8) {
+  const int NE = E + (shared_gate ? 1 : 0);
+  for (int e = warp; e < NE; e += 8) {
     const bf16* wr = w + (long long)e * K;
     float acc = 0.f;
     if (vec) {
@@ -2225,14 +2399,14 @@ __global__ void __launch_bounds__(256) hy_router_route_kernel(const AT* __restri
     if (lane == 0) rsm[e] = acc;
   }
   __syncthreads();
-  if (warp == 0) hy_route_token(rsm, rsm + E, rsm + 2 * E, rsm + 3 * E, E, top, groups, keep, scale, gw + t * E, score_mode, group_mode, renorm);
+  if (warp == 0) hy_route_token(rsm, rsm + NE, rsm + NE + E, rsm + NE + 2 * E, E, top, groups, keep, scale, gw + t * NE, score_mode, group_mode, renorm, shared_gate);
 }
 
 // U carries, expert after expert, [gate_e (f) | up_e (f)], then the shared expert's [gate (sf) | up (sf)].
 // out[t, e * f + i] = hy_expert_act(gate, up, gw[t, e]) (zero for experts the token does not use),
 // out[t, E * f + i] = glu of the shared expert (limit_s): the input of ONE down projection over all experts' columns.
 template <typename AT>
-__global__ void hy_moe_act_kernel(LinOut U, const float* __restrict__ gw, int E, int f, float limit, int sf, float limit_s,
+__global__ void hy_moe_act_kernel(LinOut U, const float* __restrict__ gw, int ldg, int E, int f, float limit, int sf, float limit_s,
                                   int act, int on_input, AT* __restrict__ out, long long ld_out, int T) {
   pdl_launch_dependents();
   pdl_wait();
@@ -2244,11 +2418,11 @@ __global__ void hy_moe_act_kernel(LinOut U, const float* __restrict__ gw, int E,
   float v = 0.f;
   if (i < E * f) {
     const int e = i / f, j = i - e * f;
-    const float g = gw[t * E + e];
+    const float g = gw[t * ldg + e];
     if (g != 0.f) v = hy_expert_act(lin_at(U, t, 2 * e * f + j), lin_at(U, t, 2 * e * f + f + j), g, limit, act, on_input);
   } else {
     const int j = i - E * f;
-    v = hy_expert_act(lin_at(U, t, 2 * E * f + j), lin_at(U, t, 2 * E * f + sf + j), 1.0f, limit_s, act, 0);
+    v = hy_expert_act(lin_at(U, t, 2 * E * f + j), lin_at(U, t, 2 * E * f + sf + j), hy_shared_weight(gw + t * ldg, ldg, E), limit_s, act, 0);
   }
   act_store<AT>(out + t * ld_out + i, v);
 }
@@ -2258,7 +2432,7 @@ __global__ void hy_moe_act_kernel(LinOut U, const float* __restrict__ gw, int E,
 // expert: the input of ONE down projection over all experts' columns.  gelu is the exact form, 0.5 z (1 + erf(z / sqrt 2)).
 __device__ __forceinline__ float hy_gelu_erf(float z) { return 0.5f * z * (1.0f + erff(z * 0.70710678118654752f)); }
 template <typename AT>
-__global__ void hy_moe_act1_kernel(LinOut U, const float* __restrict__ gw, int E, int f, int sf, AT* __restrict__ out, long long ld_out, int T) {
+__global__ void hy_moe_act1_kernel(LinOut U, const float* __restrict__ gw, int ldg, int E, int f, int sf, AT* __restrict__ out, long long ld_out, int T) {
   pdl_launch_dependents();
   pdl_wait();
   const int W = E * f + sf;
@@ -2268,15 +2442,15 @@ __global__ void hy_moe_act1_kernel(LinOut U, const float* __restrict__ gw, int E
   const int i = (int)(idx - t * W);
   float v = 0.f;
   if (i < E * f) {
-    const float g = gw[t * E + i / f];
+    const float g = gw[t * ldg + i / f];
     if (g != 0.f) v = g * hy_gelu_erf(lin_at(U, t, i));
   } else {
-    v = hy_gelu_erf(lin_at(U, t, i));
+    v = hy_shared_weight(gw + t * ldg, ldg, E) * hy_gelu_erf(lin_at(U, t, i));
   }
   act_store<AT>(out + t * ld_out + i, v);
 }
 // the same on a bf16 matrix (prompts), eight neighbours per thread: f, sf, ld, ld_out multiples of 8
-__global__ void hy_moe_act1_vec_kernel(const bf16* __restrict__ u, long long ld, const float* __restrict__ gw, int E, int f, int sf,
+__global__ void hy_moe_act1_vec_kernel(const bf16* __restrict__ u, long long ld, const float* __restrict__ gw, int ldg, int E, int f, int sf,
                                        bf16* __restrict__ out, long long ld_out, int T) {
   pdl_launch_dependents();
   pdl_wait();
@@ -2285,7 +2459,7 @@ __global__ void hy_moe_act1_vec_kernel(const bf16* __restrict__ u, long long ld,
   if (idx >= (long long)T * W8) return;
   const long long t = idx / W8;
   const int i = (int)(idx - t * W8) << 3;
-  const float w = i < E * f ? gw[t * E + i / f] : 1.0f;
+  const float w = i < E * f ? gw[t * ldg + i / f] : hy_shared_weight(gw + t * ldg, ldg, E);
   uint4 r = make_uint4(0u, 0u, 0u, 0u);
   if (w != 0.f) {
     float v[8];
@@ -2297,10 +2471,12 @@ __global__ void hy_moe_act1_vec_kernel(const bf16* __restrict__ u, long long ld,
   *reinterpret_cast<uint4*>(out + t * ld_out + i) = r;
 }
 
-// Experts gathered: steps of so few rows that most experts have no token read only the rows of the chosen experts instead of
-// running every expert as one wide Linear.  gw [T, E] holds the routing weights (zero = not chosen; exactly `top` are not).
-// Up: a warp per (token, chosen expert j, channel r) forms the gate and the up product of that channel (16-byte weight loads,
-// fp32 sums) and applies hy_expert_act; out[t, j * F + r].  Wants D and F multiples of 8.  grid ceil(T * top * F / 8), 256 threads.
+// Experts gathered: steps of so few rows that most experts have no token read only the rows of the chosen experts (and the shared
+// one) instead of running every expert as one wide Linear.  gw [T, ldg] holds the routing weights (zero = not chosen; at most
+// `top` are not; behind them the shared expert's weight, see hy_shared_weight).
+// Up: a warp per (token, chosen expert j, channel r), then per (token, channel of the shared expert), forms the gate and the up
+// product of that channel (16-byte weight loads, fp32 sums) and applies hy_expert_act; out[t, j * F + r], out[t, top * F + r].
+// Wants D, F and S (the shared width) multiples of 8.  grid ceil(T * (top * F + S) / 8), 256 threads.
 __device__ __forceinline__ int hy_nth_chosen(const float* __restrict__ gwt, int E, int j) {
   int seen = 0;
   for (int e = 0; e < E; ++e)
@@ -2309,21 +2485,24 @@ __device__ __forceinline__ int hy_nth_chosen(const float* __restrict__ gwt, int 
 }
 template <typename AT>
 __global__ void __launch_bounds__(256) hy_moe_gather_up_kernel(const AT* __restrict__ x, long long ldx, const bf16* __restrict__ w_up,
-                                                               const float* __restrict__ gw, int E, int top, int F, int D, float limit,
-                                                               int act, int on_input, AT* __restrict__ out, int T) {
+                                                               const float* __restrict__ gw, int ldg, int E, int top, int F, int S, int D, float limit,
+                                                               float limit_s, int act, int on_input, AT* __restrict__ out, int T) {
   pdl_launch_dependents();
   pdl_wait();
   const long long wid = (long long)blockIdx.x * 8 + (threadIdx.x >> 5);
   const int lane = threadIdx.x & 31;
-  if (wid >= (long long)T * top * F) return;
-  const int t = (int)(wid / ((long long)top * F));
-  const int rem = (int)(wid - (long long)t * top * F);
-  const int j = rem / F, r = rem - j * F;
-  const int e = hy_nth_chosen(gw + (long long)t * E, E, j);
+  const int per = top * F + S;
+  if (wid >= (long long)T * per) return;
+  const int t = (int)(wid / per);
+  const int rem = (int)(wid - (long long)t * per);
+  const float* gwt = gw + (long long)t * ldg;
+  const bool shared = rem >= top * F;
+  const int j = rem / F, r = shared ? rem - top * F : rem - j * F;
+  const int e = shared ? E : hy_nth_chosen(gwt, E, j);
   float v = 0.f;
   if (e >= 0) {
     const bf16* wg = w_up + ((long long)2 * e * F + r) * D;
-    const bf16* wu = wg + (long long)F * D;
+    const bf16* wu = wg + (long long)(shared ? S : F) * D;
     const AT* xr = x + (long long)t * ldx;
     float g = 0.f, u = 0.f;
     for (int k = lane * 8; k < D; k += 256) {
@@ -2337,15 +2516,15 @@ __global__ void __launch_bounds__(256) hy_moe_gather_up_kernel(const AT* __restr
     }
     g = warp_sum(g);
     u = warp_sum(u);
-    v = hy_expert_act(g, u, gw[(long long)t * E + e], limit, act, on_input);
+    v = shared ? hy_expert_act(g, u, hy_shared_weight(gwt, ldg, E), limit_s, act, 0) : hy_expert_act(g, u, gwt[e], limit, act, on_input);
   }
-  if (lane == 0) act_store<AT>(out + (long long)t * top * F + rem, v);
+  if (lane == 0) act_store<AT>(out + (long long)t * per + rem, v);
 }
-// Down: a warp per (token, output channel d) sums over the chosen experts' column blocks of the one down matrix [D, E * F].
-// y [T, D] fp32.  grid ceil(T * D / 8), 256 threads.
+// Down: a warp per (token, output channel d) sums over the chosen experts' column blocks of the one down matrix [D, E * F + S] and
+// the shared expert's.  y [T, D] fp32.  grid ceil(T * D / 8), 256 threads.
 template <typename AT>
 __global__ void __launch_bounds__(256) hy_moe_gather_down_kernel(const AT* __restrict__ a, const bf16* __restrict__ w_down,
-                                                                 const float* __restrict__ gw, int E, int top, int F, int D,
+                                                                 const float* __restrict__ gw, int ldg, int E, int top, int F, int S, int D,
                                                                  float* __restrict__ y, int T) {
   pdl_launch_dependents();
   pdl_wait();
@@ -2353,21 +2532,25 @@ __global__ void __launch_bounds__(256) hy_moe_gather_down_kernel(const AT* __res
   const int lane = threadIdx.x & 31;
   if (wid >= (long long)T * D) return;
   const int t = (int)(wid / D), d = (int)(wid - (long long)t * D);
-  const float* gwt = gw + (long long)t * E;
-  const bf16* wrow = w_down + (long long)d * E * F;
+  const float* gwt = gw + (long long)t * ldg;
+  const bf16* wrow = w_down + (long long)d * ((long long)E * F + S);
+  const AT* at = a + (long long)t * (top * F + S);
   float acc = 0.f;
-  int j = 0;
-  for (int e = 0; e < E && j < top; ++e) {
-    if (gwt[e] == 0.f) continue;
-    const AT* ar = a + (long long)t * top * F + (long long)j * F;
-    for (int k = lane * 8; k < F; k += 256) {
+  auto add = [&](const AT* ar, const bf16* wr, int n) {
+    for (int k = lane * 8; k < n; k += 256) {
       float w[8];
-      hy_load8(wrow + (long long)e * F + k, nullptr, w);
+      hy_load8(wr + k, nullptr, w);
 #pragma unroll
       for (int i = 0; i < 8; ++i) acc = fmaf(act_load<AT>(ar + k + i), w[i], acc);
     }
+  };
+  int j = 0;
+  for (int e = 0; e < E && j < top; ++e) {
+    if (gwt[e] == 0.f) continue;
+    add(at + (long long)j * F, wrow + (long long)e * F, F);
     ++j;
   }
+  if (S > 0) add(at + (long long)top * F, wrow + (long long)E * F, S);
   acc = warp_sum(acc);
   if (lane == 0) y[(long long)t * D + d] = acc;
 }

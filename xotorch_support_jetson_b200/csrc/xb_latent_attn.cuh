@@ -4,13 +4,15 @@
 // softmax and accumulators): S = Q K^T over the whole cache row, O += P V over the latent columns of the same tile.
 //
 //   rows r = token * H + head, 16 per warp, WARPS warps per block; queries fp32 [T * H][W] (already in the cache's space:
-//   hy_head_mm_t_kernel + hy_latent_prep_kernel), rounded to bf16 in shared memory
+//   hy_latent_absorb_kernel), rounded to bf16 in shared memory
 //   pool [n_pages * page_tokens][W] bf16, W = R + rot, W and R multiples of 16
 //   grid (ceil(T * H / (16 * WARPS)), n_splits, ceil(R / DVC)): a block takes the tile's rows, one share of every
 //   sequence's keys (n_splits equal shares, whole key tiles) and DVC value columns
 //   n_splits == 1: out[t][h * R + c] = O / l;  else part[split][r][2 + R] = (m, l, O) and hy_latent_merge_kernel finishes.
 // A tile's tokens may belong to several sequences (a batch of single tokens): the block walks them one after the other,
 // rows of other sequences are masked for that walk.  Causal: row (t, h) sees keys at positions <= pos(t).
+// EXT: a window (row (t, h) sees only the `window` newest of them; tiles that no row of the block sees are not visited) and the
+// softmax weights entering O += P V as hi + lo bf16 pairs instead of one rounding.
 #pragma once
 #include "xb_attn_mma.cuh"
 
@@ -25,10 +27,10 @@ __device__ __forceinline__ void lat_cp_commit() { asm volatile("cp.async.commit_
 template <int N> __device__ __forceinline__ void lat_cp_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
 
 // LOADW >= WARPS warps per block: all of them stage queries and key tiles, the first WARPS own rows.
-template <int WARPS, int DVC, int LOADW>
+template <int WARPS, int DVC, int LOADW, bool EXT>
 __global__ void __launch_bounds__(32 * LOADW) hy_latent_attn_mma_kernel(const float* __restrict__ qa, const bf16* __restrict__ pool, BatchMeta m,
                                                                         int T, int H, int W, int R, float scale_log2, int n_splits,
-                                                                        float* __restrict__ part, float* __restrict__ out, long long ld_out) {
+                                                                        float* __restrict__ part, float* __restrict__ out, long long ld_out, int window) {
   pdl_launch_dependents();
   pdl_wait();
   extern __shared__ __align__(16) unsigned char lsm[];
@@ -72,10 +74,17 @@ __global__ void __launch_bounds__(32 * LOADW) hy_latent_attn_mma_kernel(const fl
     const int pmax = m.tok_pos[tl];
     const int* pages = m.page_table + (long long)m.seq_slot[s] * m.max_pages;
     // this block's share of keys [k_lo, k_hi): whole tiles
-    const int tiles = (pmax + HY_LAT_KEYS) / HY_LAT_KEYS;
+    int tile0 = 0;
+    if (EXT) {   // the oldest key that the tile's first token of s sees
+      int tf = t_first;
+      while (tf < tl && m.tok_seq[tf] != s) ++tf;
+      const int oldest = m.tok_pos[tf] - window + 1;
+      tile0 = oldest > 0 ? oldest / HY_LAT_KEYS : 0;
+    }
+    const int tiles = (pmax + HY_LAT_KEYS) / HY_LAT_KEYS - tile0;
     const int per = (tiles + n_splits - 1) / n_splits;
-    const int k_lo = split * per * HY_LAT_KEYS;
-    int k_hi = (split + 1) * per * HY_LAT_KEYS;
+    const int k_lo = (tile0 + split * per) * HY_LAT_KEYS;
+    int k_hi = (tile0 + (split + 1) * per) * HY_LAT_KEYS;
     k_hi = k_hi < pmax + 1 ? k_hi : pmax + 1;
     // does this warp hold a row of s
     int wt0 = wr0 / H, wt1 = (wr0 + 15 < NR ? wr0 + 15 : NR - 1) / H;
@@ -131,7 +140,7 @@ __global__ void __launch_bounds__(32 * LOADW) hy_latent_attn_mma_kernel(const fl
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
           const int j = e >> 1, kp = kb + nb * 8 + 2 * q + (e & 1);
-          const bool ok = rseq[j] == s && kp <= rpos[j];
+          const bool ok = rseq[j] == s && kp <= rpos[j] && (!EXT || rpos[j] - kp < window);
           const float v = ok ? sacc[nb][e] * scale_log2 : HY_LAT_NEG;
           sacc[nb][e] = v;
           tmax[j] = fmaxf(tmax[j], v);
@@ -146,7 +155,7 @@ __global__ void __launch_bounds__(32 * LOADW) hy_latent_attn_mma_kernel(const fl
         mx[j] = nm;
         ls[j] *= corr[j];
       }
-      uint32_t pa[KK][4];
+      uint32_t pa[KK][4], pl[EXT ? KK : 1][4];   // weights, and what their rounding to bf16 left over
 #pragma unroll
       for (int nb = 0; nb < NB; ++nb) {
         float p[4];
@@ -158,6 +167,11 @@ __global__ void __launch_bounds__(32 * LOADW) hy_latent_attn_mma_kernel(const fl
         }
         pa[nb >> 1][(nb & 1) * 2] = f2_to_bf2(p[0], p[1]);
         pa[nb >> 1][(nb & 1) * 2 + 1] = f2_to_bf2(p[2], p[3]);
+        if (EXT) {
+          const float2 h0 = bf2_to_f2(pa[nb >> 1][(nb & 1) * 2]), h1 = bf2_to_f2(pa[nb >> 1][(nb & 1) * 2 + 1]);
+          pl[EXT ? nb >> 1 : 0][(nb & 1) * 2] = f2_to_bf2(p[0] - h0.x, p[1] - h0.y);
+          pl[EXT ? nb >> 1 : 0][(nb & 1) * 2 + 1] = f2_to_bf2(p[2] - h1.x, p[3] - h1.y);
+        }
       }
 #pragma unroll
       for (int n = 0; n < NDV; ++n) {
@@ -174,6 +188,10 @@ __global__ void __launch_bounds__(32 * LOADW) hy_latent_attn_mma_kernel(const fl
             ldsm_x4_t(vaddr + (uint32_t)(kk * 16 * PITCH + n * 8) * 2, b0, b1, b2, b3);
             mma_bf16_16816(oacc[n], pa[kk], b0, b1);
             mma_bf16_16816(oacc[n + 1], pa[kk], b2, b3);
+            if (EXT) {
+              mma_bf16_16816(oacc[n], pl[EXT ? kk : 0], b0, b1);
+              mma_bf16_16816(oacc[n + 1], pl[EXT ? kk : 0], b2, b3);
+            }
           }
         }
       }

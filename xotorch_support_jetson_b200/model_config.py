@@ -28,7 +28,7 @@ _DIRECT_FIELDS = (
 _OPTIONAL_FIELDS = (("attention_dropout", "attn_dropout", 0.0), ("attention_bias", "attn_bias", False), ("hidden_act", "hidden_act", "silu"))
 
 
-HYBRID_ARCHITECTURES = ("Refatar", "Bibevik", "Pufivik", "Vusenex")
+HYBRID_ARCHITECTURES = ("Refatar", "Bibevik", "Pufivik", "Vusenex", "Rurutar")
 
 
 def is_hybrid(config: dict) -> bool:
@@ -54,6 +54,8 @@ def hybrid_model_config(raw: dict) -> dict:
     return pufivik_model_config(raw)
   if arch == "Vusenex":
     return vusenex_model_config(raw)
+  if arch == "Rurutar":
+    return rurutar_model_config(raw)
   layers = []
   for i, lc in enumerate(raw["layers"]):
     mx, kind = lc["mixer"], lc["type"]
@@ -138,14 +140,14 @@ def bibevik_model_config(raw: dict) -> dict:
 
 
 def _rotary(i: int, rot, kind: str) -> dict:
-  """The rotary part of a Pufivik mixer: how many entries of a head turn, the pair layout and the rescaling of the
-  frequencies.  ``attention`` pairs entry i with i + dims/2 and rescales in wavelength bands {factor, low, high, original};
+  """The rotary part of a mixer: how many entries of a head turn, the pair layout and the rescaling of the frequencies.
+  ``attention`` pairs entry i with i + dims/2 and rescales in wavelength bands {factor, low, high, original};
   ``attention_2`` pairs 2i with 2i + 1 and rescales along a ramp over the pair index {factor, original, fast, slow}, with
-  cos and sin multiplied by 0.1 ln(factor) + 1."""
+  cos and sin multiplied by 0.1 ln(factor) + 1; ``latent_attention`` has the pairs of the first and the ramp of the second."""
   if not rot or not int(rot.get("dims", 0)):
     return {"rot_dims": 0, "rot_pairs": "half", "rot_scaling": "none", "rot_base": 10000.0, "rot_mult": 1.0,
             "rot_factor": 1.0, "rot_orig": 1.0, "rot_p0": 0.0, "rot_p1": 0.0}
-  out = {"rot_dims": int(rot["dims"]), "rot_base": float(rot["base"]), "rot_pairs": "half" if kind == "attention" else "interleaved",
+  out = {"rot_dims": int(rot["dims"]), "rot_base": float(rot["base"]), "rot_pairs": "interleaved" if kind == "attention_2" else "half",
          "rot_scaling": "none", "rot_mult": 1.0, "rot_factor": 1.0, "rot_orig": 1.0, "rot_p0": 0.0, "rot_p1": 0.0}
   sc = rot.get("scaling")
   if sc and kind == "attention":
@@ -251,6 +253,56 @@ def vusenex_model_config(raw: dict) -> dict:
   }
 
 
+def rurutar_model_config(raw: dict) -> dict:
+  """A Rurutar ``config.json`` (``width``, ``vocab``, ``embedding.scale``, ``norm.eps``, ``logit_softcap``, ``layers`` [{type, mixer,
+  mlp}]) -> the engine's dict.  Layers are pre-norm blocks whose norm is tanh(alpha x) w + b.  Mixer kinds: ``gla`` {heads, dim,
+  vdim, tau} = linear attention with a learned decay per key channel (the rank of the decay's first projection comes from the
+  checkpoint's ``a1`` shape, see ``resolve_tensor_sizes``; the config may name it as ``rank``); ``latent_attention`` {heads, dim,
+  rot_dim, vdim, kv_rank, q_rank, scale, rot{base, dims, scaling}, mask{size}, kv_from?} = latent attention in a window with queries
+  through a latent of their own and a gate per head; ``kv_from: j`` reads layer j's cache rows.  ``mlp``: null, {kind: dense, ff}
+  (GELU-gated) or experts {expert{ff}, router{experts, top}, shared{ff}} (SiLU-gated, weights = softmax over the chosen logits,
+  the shared expert times a sigmoid per token)."""
+  layers = []
+  for i, lc in enumerate(raw["layers"]):
+    mx, kind = lc["mixer"], lc["type"]
+    if kind == "gla":
+      lay = {"mixer": "gla", "heads": int(mx["heads"]), "dim": int(mx["dim"]), "vdim": int(mx["vdim"]), "tau": float(mx["tau"]),
+             "rank": int(mx.get("rank", 0))}
+    elif kind == "latent_attention":
+      rot = mx.get("rot") or {}
+      if int(rot.get("dims", 0)) > int(mx["rot_dim"]):
+        raise ValueError(f"layer {i}: {rot['dims']} rotating entries do not fit a part of {mx['rot_dim']}")
+      lay = {"mixer": "latent", "heads": int(mx["heads"]), "dim": int(mx["dim"]), "rot_dim": int(mx["rot_dim"]), "vdim": int(mx["vdim"]),
+             "kv_rank": int(mx["kv_rank"]), "q_rank": int(mx["q_rank"]), "scale": float(mx["scale"]), "gate": True,
+             "window": int((mx.get("mask") or {}).get("size", 0)), "kv_from": int(mx["kv_from"]) if mx.get("kv_from") is not None else -1}
+      lay.update(_rotary(i, rot, kind))
+    else:
+      raise ValueError(f"layer {i}: unknown layer type {kind!r}")
+    mlp = lc.get("mlp")
+    if mlp is None:
+      lay.update({"ff": 0, "ff_kind": "none"})
+    elif mlp["kind"] == "dense":
+      lay.update({"ff": int(mlp["ff"]), "ff_kind": "glu", "ff_act": "geglu"})
+    elif mlp["kind"] == "moe":
+      rt, sh = mlp["router"], mlp.get("shared")
+      lay.update({"ff": int(mlp["expert"]["ff"]), "ff_kind": "moe", "ff_act": "swiglu", "route_input": False, "ff_limit": 0.0,
+                  "experts": int(rt["experts"]), "top": int(rt["top"]), "groups": 0, "keep_groups": 0, "route_scale": 1.0,
+                  "route_score": "softmax", "route_norm": True, "shared_ff": int(sh["ff"]) if sh else 0, "shared_limit": 0.0,
+                  "shared_gate": bool(sh)})
+    else:
+      raise ValueError(f"layer {i}: unknown feed-forward kind {mlp['kind']!r}")
+    lay["weights_of"] = -1
+    layers.append(lay)
+  return {
+    "family": "hybrid", "architecture": "Rurutar", "block": "prenorm", "norm_kind": "tanh",
+    "embed_scale": float((raw.get("embedding") or {}).get("scale", 1.0)),
+    "embed_dim": int(raw["width"]), "vocab_size": int(raw["vocab"]), "num_layers": len(layers),
+    "max_seq_len": int(raw.get("max_seq_len", 1 << 20)), "norm_eps": float(raw["norm"]["eps"]),
+    "taps": 0, "side_dim": 0, "logit_softcap": float(raw.get("logit_softcap") or 0.0), "layers": layers,
+    "torch_dtype": HF_PRECISION_STR_TO_DTYPE.get(raw.get("torch_dtype", "bfloat16"), torch.bfloat16),
+  }
+
+
 def safetensors_shapes(folder: Path) -> dict:
   """name -> shape of every tensor in the ``*.safetensors`` files of a folder, from the files' headers alone (8 bytes of
   little-endian length, then that many bytes of JSON)."""
@@ -264,15 +316,19 @@ def safetensors_shapes(folder: Path) -> dict:
   return shapes
 
 
+_DECAY_PROJECTION = {"gdelta": "w1", "gla": "a1"}   # mixer -> tensor whose row count is the decay's rank
+
+
 def resolve_tensor_sizes(cfg: dict, shapes: dict) -> dict:
-  """Sizes that a hybrid design leaves to the checkpoint: the rank of a general delta rule's first decay projection is the
-  row count of its ``l<i>.mix.w1`` (of the layer that owns the tensors).  ``shapes``: name -> shape."""
+  """Sizes that a hybrid design leaves to the checkpoint: the rank of a decay's first projection is the row count of its
+  ``l<i>.mix.w1`` (general delta rule; of the layer that owns the tensors) or ``l<i>.mix.a1`` (gated linear attention).
+  ``shapes``: name -> shape."""
   if not is_hybrid(cfg):
     return cfg
   for i, lay in enumerate(cfg["layers"]):
-    if lay.get("mixer") == "gdelta" and not lay.get("rank"):
+    if lay.get("mixer") in _DECAY_PROJECTION and not lay.get("rank"):
       src = lay["weights_of"] if lay.get("weights_of", -1) >= 0 else i
-      name = f"l{src}.mix.w1"
+      name = f"l{src}.mix.{_DECAY_PROJECTION[lay['mixer']]}"
       if name not in shapes:
         raise ValueError(f"layer {i}: neither the configuration nor a tensor {name} gives the rank of the decay projection")
       lay["rank"] = int(shapes[name][0])
@@ -286,7 +342,7 @@ def load_model_config(model_config_path: Path) -> dict:
   hf = json.loads(Path(model_config_path).read_text())
   if hf.get("architecture") in HYBRID_ARCHITECTURES:
     cfg = hybrid_model_config(hf)
-    if any(lay.get("mixer") == "gdelta" and not lay.get("rank") for lay in cfg["layers"]):
+    if any(lay.get("mixer") in _DECAY_PROJECTION and not lay.get("rank") for lay in cfg["layers"]):
       resolve_tensor_sizes(cfg, safetensors_shapes(Path(model_config_path).parent))
     if cfg.get("pos_rows"):   # a learned position table: its own row count bounds the positions
       rows = safetensors_shapes(Path(model_config_path).parent).get("pos")

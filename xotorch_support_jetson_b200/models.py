@@ -196,6 +196,50 @@ _VUSENEX_1B = _vusenex(2048, 128256, [
   (("attention", _kv_attn(32, 8, 64, coef=0.25, every=96), _gelu_experts(16, 4, 512, 4, 2, 2048)) if i % 4 in (0, 3) else
    ("latent_attention", _plain_latent(16, 64, 128, 256), _gelu_experts(16, 4, 512, 4, 2, 2048))) for i in range(16)], max_pos=8192, buckets=65521)
 
+def _rurutar(width, vocab, layers, scale=0.7, softcap=20.0, eps=1e-6):
+  """A Rurutar config.json: layers is a list of (type, mixer, mlp) entries."""
+  return {"architecture": "Rurutar", "width": width, "vocab": vocab, "embedding": {"scale": scale}, "norm": {"eps": eps}, "logit_softcap": softcap,
+          "layers": [{"type": t, "mixer": m, "mlp": f} for t, m, f in layers]}
+
+
+def _gla(heads, dim, vdim, tau=16.0, rank=None):
+  m = {"heads": heads, "dim": dim, "vdim": vdim, "tau": tau}
+  if rank:
+    m["rank"] = rank
+  return m
+
+
+def _window_latent(heads, dim, rot_dim, vdim, kv_rank, q_rank, window, kv_from=None, base=10000.0, factor=4.0, original=1024):
+  m = {"heads": heads, "dim": dim, "rot_dim": rot_dim, "vdim": vdim, "kv_rank": kv_rank, "q_rank": q_rank, "scale": (dim + rot_dim) ** -0.5,
+       "mask": {"size": window}, "rot": {"base": base, "dims": rot_dim,
+                                         "scaling": {"factor": factor, "original": original, "fast": 32.0, "slow": 1.0}}}
+  if kv_from is not None:
+    m["kv_from"] = kv_from
+  return m
+
+
+def _gated_experts(n, top, ff, shared_ff):
+  m = {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": n, "top": top}}
+  if shared_ff:
+    m["shared"] = {"ff": shared_ff}
+  return m
+
+
+_RURUTAR_TINY = _rurutar(160, 384, [
+  ("gla", _gla(3, 24, 40, tau=8.0, rank=12), {"kind": "dense", "ff": 224}),
+  ("latent_attention", _window_latent(5, 24, 16, 40, 48, 56, 37, base=20000.0), _gated_experts(6, 2, 48, 72)),
+  ("gla", _gla(5, 16, 24, rank=8), None),
+  ("latent_attention", _window_latent(3, 40, 16, 24, 48, 80, 21, kv_from=1, base=20000.0), _gated_experts(8, 3, 32, 40)),
+])
+# 1B-class geometry for throughput runs (random weights): the width, depth and vocabulary of llama-3.2-1b; three layers of gated linear
+# attention (16 heads of 128 x 128) to one of latent attention (16 heads, latent of 256, window 1024), every other latent layer on
+# the rows of the one before; 16 experts of 384 of which a token uses four beside a shared one of 2048, dense in every fourth layer
+_RURUTAR_1B = _rurutar(2048, 128256, [
+  (("latent_attention", _window_latent(16, 64, 64, 128, 256, 768, 1024, kv_from=(i - 4 if i % 8 == 7 else None), base=500000.0),
+    _gated_experts(16, 4, 384, 2048)) if i % 4 == 3 else
+   ("gla", _gla(16, 128, 128, rank=16), {"kind": "dense", "ff": 8192} if i % 4 == 0 else _gated_experts(16, 4, 384, 2048)))
+  for i in range(16)])
+
 # model id -> {layers, repo:{EngineClassName: hf repo}, hf_config}
 model_cards = {
   "llama-3.2-1b": {"layers": 16, "repo": {ENGINE_CLASS_NAME: "unsloth/Llama-3.2-1B-Instruct"},
@@ -223,6 +267,8 @@ model_cards = {
   "pufivik-1b": {"layers": 16, "repo": {ENGINE_CLASS_NAME: "synthetic/pufivik-1b"}, "hf_config": _PUFIVIK_1B},
   "vusenex-tiny": {"layers": 4, "repo": {ENGINE_CLASS_NAME: "synthetic/vusenex-tiny"}, "hf_config": _VUSENEX_TINY},
   "vusenex-1b": {"layers": 16, "repo": {ENGINE_CLASS_NAME: "synthetic/vusenex-1b"}, "hf_config": _VUSENEX_1B},
+  "rurutar-tiny": {"layers": 4, "repo": {ENGINE_CLASS_NAME: "synthetic/rurutar-tiny"}, "hf_config": _RURUTAR_TINY},
+  "rurutar-1b": {"layers": 16, "repo": {ENGINE_CLASS_NAME: "synthetic/rurutar-1b"}, "hf_config": _RURUTAR_1B},
   "mistral-tiny": {"layers": 4, "repo": {ENGINE_CLASS_NAME: "synthetic/mistral-tiny"},
                    "hf_config": _mistral(320, 5, 1, 640, 4, head_dim=64, vocab=1280)},
 }

@@ -19,6 +19,9 @@ from .model_config import has_qkv_bias, is_hybrid, load_model_config, model_fami
 from .shard import Shard
 
 
+_ROT_SCALING = {"none": _cabi.ROT_SCALE_NONE, "bands": _cabi.ROT_SCALE_BANDS, "ramp": _cabi.ROT_SCALE_RAMP}
+
+
 def _permute(t: torch.Tensor, n_heads: int, head_dim: int, dim: int) -> torch.Tensor:
   """HF half-split q/k rows -> torchtune interleaved rows (reference llm_utils.py:126-134)."""
   return t.view(n_heads, 2, head_dim // 2, dim).transpose(1, 2).reshape(head_dim * n_heads, dim)
@@ -132,12 +135,15 @@ class StageRuntime:
       L = lays[i]
       L.ff = lc["ff"]
       L.weights_of = lc.get("weights_of", -1)
-      L.ff_kind = {"relu2": _cabi.FF_RELU2, "none": _cabi.FF_RELU2, "glu_clamp": _cabi.FF_GLU_CLAMP, "moe": _cabi.FF_MOE}[lc.get("ff_kind", "relu2")]
+      L.m_kv_from = lc.get("kv_from", -1)
+      L.ff_kind = {"relu2": _cabi.FF_RELU2, "none": _cabi.FF_RELU2, "glu_clamp": _cabi.FF_GLU_CLAMP, "glu": _cabi.FF_GLU, "moe": _cabi.FF_MOE}[lc.get("ff_kind", "relu2")]
       L.ff_limit = lc.get("ff_limit", 0.0)
+      if lc.get("ff_kind") in ("moe", "glu"):
+        L.ff_act = {"glu_clamp": _cabi.ACT_GLU_CLAMP, "swiglu": _cabi.ACT_SWIGLU, "gelu": _cabi.ACT_GELU, "geglu": _cabi.ACT_GEGLU}[lc.get("ff_act", "glu_clamp")]
       if lc.get("ff_kind") == "moe":
         L.n_experts, L.top, L.groups, L.keep_groups = lc["experts"], lc["top"], lc["groups"], lc["keep_groups"]
         L.route_scale, L.shared_ff, L.shared_limit = lc["route_scale"], lc["shared_ff"], lc["shared_limit"]
-        L.ff_act = {"glu_clamp": _cabi.ACT_GLU_CLAMP, "swiglu": _cabi.ACT_SWIGLU, "gelu": _cabi.ACT_GELU}[lc.get("ff_act", "glu_clamp")]
+        L.shared_gate = int(bool(lc.get("shared_gate", False)))
         L.route_input = int(bool(lc.get("route_input", False)))
         L.route_score = {"sigmoid": _cabi.ROUTE_SIGMOID, "softmax": _cabi.ROUTE_SOFTMAX}[lc.get("route_score", "sigmoid")]
         L.group_score = {"top2": _cabi.GROUP_TOP2, "max": _cabi.GROUP_MAX}[lc.get("group_score", "top2")]
@@ -152,20 +158,26 @@ class StageRuntime:
         L.s_qtemp_coef, L.s_qtemp_every = lc.get("qtemp_coef", 0.0), lc.get("qtemp_every", 0)
         L.s_rot_dims = lc.get("rot_dims", 0)
         L.s_rot_pairs = _cabi.ROPE_HALF_SPLIT if lc.get("rot_pairs", "half") == "half" else _cabi.ROPE_INTERLEAVED
-        L.s_rot_scaling = {"none": _cabi.ROT_SCALE_NONE, "bands": _cabi.ROT_SCALE_BANDS, "ramp": _cabi.ROT_SCALE_RAMP}[lc.get("rot_scaling", "none")]
+        L.s_rot_scaling = _ROT_SCALING[lc.get("rot_scaling", "none")]
         L.s_rot_mult = lc.get("rot_mult", 1.0)
         L.s_rot_base, L.s_rot_factor, L.s_rot_orig = lc.get("rot_base", 10000.0), lc.get("rot_factor", 1.0), lc.get("rot_orig", 1.0)
         L.s_rot_p0, L.s_rot_p1 = lc.get("rot_p0", 0.0), lc.get("rot_p1", 0.0)
-      elif lc["mixer"] in ("latent", "gdelta", "lightning"):
-        L.mixer = {"latent": _cabi.MIX_LATENT, "gdelta": _cabi.MIX_GDELTA, "lightning": _cabi.MIX_LIGHTNING}[lc["mixer"]]
+      elif lc["mixer"] in ("latent", "gdelta", "lightning", "gla"):
+        L.mixer = {"latent": _cabi.MIX_LATENT, "gdelta": _cabi.MIX_GDELTA, "lightning": _cabi.MIX_LIGHTNING, "gla": _cabi.MIX_GLA}[lc["mixer"]]
         L.m_heads, L.m_dim = lc["heads"], lc["dim"]
         if lc["mixer"] == "latent":
           L.m_vdim, L.m_rot_dim, L.m_kv_rank, L.m_rot_dims = lc["vdim"], lc["rot_dim"], lc["kv_rank"], lc["rot_dims"]
           L.m_scale, L.m_rot_base = lc["scale"], lc["rot_base"]
-        elif lc["mixer"] == "gdelta":
+          L.m_q_rank, L.m_window, L.m_gate = lc.get("q_rank", 0), lc.get("window", 0), int(bool(lc.get("gate", False)))
+          L.m_rot_pairs = _cabi.ROPE_HALF_SPLIT if lc.get("rot_pairs", "interleaved") == "half" else _cabi.ROPE_INTERLEAVED
+          L.m_rot_scaling, L.m_rot_mult = _ROT_SCALING[lc.get("rot_scaling", "none")], lc.get("rot_mult", 1.0)
+          L.m_rot_factor, L.m_rot_orig = lc.get("rot_factor", 1.0), lc.get("rot_orig", 1.0)
+          L.m_rot_p0, L.m_rot_p1 = lc.get("rot_p0", 0.0), lc.get("rot_p1", 0.0)
+        elif lc["mixer"] in ("gdelta", "gla"):
           if not lc.get("rank"):
             raise ValueError(f"layer {i}: the rank of the decay projection is unknown (model_config.resolve_tensor_sizes)")
-          L.m_vdim, L.m_rank = lc["dim"], lc["rank"]
+          L.m_vdim, L.m_rank = lc.get("vdim", lc["dim"]), lc["rank"]
+          L.m_tau = lc.get("tau", 1.0)
         else:
           L.m_vdim = lc["vdim"]
       elif lc["mixer"] == "delta":
@@ -182,14 +194,15 @@ class StageRuntime:
       n_layers=nl, dim=config["embed_dim"], vocab=config["vocab_size"], taps=config["taps"], side_dim=config["side_dim"],
       norm_eps=config["norm_eps"], logit_softcap=config["logit_softcap"], compute_fp32=int(dtype == "float32"),
       max_batch_tokens=max_batch_tokens, max_seqs=max_seqs, max_logit_rows=self.max_logit_rows,
-      block={"parallel": _cabi.BLOCK_PARALLEL, "branchnorm": _cabi.BLOCK_BRANCHNORM}.get(config.get("block"), _cabi.BLOCK_SANDWICH),
+      block={"parallel": _cabi.BLOCK_PARALLEL, "branchnorm": _cabi.BLOCK_BRANCHNORM, "prenorm": _cabi.BLOCK_PRENORM}.get(config.get("block"), _cabi.BLOCK_SANDWICH),
       norm_scalar=int(bool(config.get("norm_scalar", False))), embed_scale=float(config.get("embed_scale", 1.0)),
       norm_groups=int(config.get("norm_groups", 1)), norm_plain=int(bool(config.get("norm_plain", False))),
       residual_mult=float(config.get("residual_mult", 1.0)), tied_head=int(bool(config.get("tied_head", False))),
       ff_unfiltered=int(bool(config.get("ff_unfiltered", False))),
       gated_residual=int(bool(config.get("gated_residual", False))),
       bigram_buckets=int(bg["buckets"]) if bg else 0, bigram_mul_prev=int(bg["mul_prev"]) if bg else 0,
-      bigram_mul_cur=int(bg["mul_cur"]) if bg else 0, pos_rows=int(config.get("pos_rows", 0)))
+      bigram_mul_cur=int(bg["mul_cur"]) if bg else 0, pos_rows=int(config.get("pos_rows", 0)),
+      norm_kind=_cabi.NORM_TANH if config.get("norm_kind") == "tanh" else _cabi.NORM_RMS)
     self.first_from_mlp = self.last_to_attn = False
     self.is_first = self.is_last = True
     self.desc, self._layers = d, lays

@@ -322,6 +322,76 @@ def random_vusenex_state(cfg: dict, seed: int = 0, dtype: torch.dtype = torch.bf
   return out
 
 
+def rurutar_param_shapes(cfg: dict, rank: int = 16) -> Dict[str, tuple]:
+  """name -> shape of every tensor of a Rurutar config.json.  rank: rows of the decay's first projection where the config has none."""
+  D, V = cfg["width"], cfg["vocab"]
+  sh = {"embed": (V, D), "head": (V, D)}
+
+  def norm(name):
+    sh.update({name: (D,), name + ".b": (D,), name + ".alpha": ()})
+
+  norm("final.norm")
+  for i, lc in enumerate(cfg["layers"]):
+    p, m = f"l{i}.", lc["mixer"]
+    norm(p + "norm1")
+    H, n, dv = m["heads"], m["dim"], m["vdim"]
+    if lc["type"] == "gla":
+      rk = m.get("rank", rank)
+      sh.update({p + "mix.q": (H * n, D), p + "mix.k": (H * n, D), p + "mix.v": (H * dv, D), p + "mix.g": (H * dv, D), p + "mix.o": (D, H * dv),
+                 p + "mix.norm": (dv,), p + "mix.a1": (rk, D), p + "mix.a2": (H * n, rk), p + "mix.a2.b": (H * n,)})
+    else:
+      dr, R, qr = m["rot_dim"], m["kv_rank"], m["q_rank"]
+      sh.update({p + "mix.dq": (qr, D), p + "mix.dq.norm": (qr,), p + "mix.uq": (H * (n + dr), qr), p + "mix.uk": (H * n, R),
+                 p + "mix.uv": (H * dv, R), p + "mix.g": (H, D), p + "mix.o": (D, H * dv)})
+      if m.get("kv_from") is None:
+        sh.update({p + "mix.dkv": (R + dr, D), p + "mix.dkv.norm": (R,)})
+    mlp = lc.get("mlp")
+    if not mlp:
+      continue
+    norm(p + "norm2")
+    if mlp["kind"] == "dense":
+      F = mlp["ff"]
+      sh.update({p + "mlp.gate": (F, D), p + "mlp.up": (F, D), p + "mlp.down": (D, F)})
+      continue
+    F = mlp["expert"]["ff"]
+    sh[p + "mlp.router"] = (mlp["router"]["experts"], D)
+    for e in range(mlp["router"]["experts"]):
+      sh.update({f"{p}mlp.e{e}.gate": (F, D), f"{p}mlp.e{e}.up": (F, D), f"{p}mlp.e{e}.down": (D, F)})
+    if mlp.get("shared"):
+      S = mlp["shared"]["ff"]
+      sh.update({p + "mlp.shared.gate": (S, D), p + "mlp.shared.up": (S, D), p + "mlp.shared.down": (D, S), p + "mlp.shared.sg": (1, D)})
+  return sh
+
+
+def random_rurutar_state(cfg: dict, seed: int = 0, dtype: torch.dtype = torch.bfloat16, gain: float = 1.0, device: str = "cpu",
+                         rank: int = 16) -> Dict[str, torch.Tensor]:
+  """Seeded random Rurutar weights: matrices N(0, gain^2 / in), tanh norms with factors in (0.4, 1.2), weights 1 + N(0, 0.1^2) and
+  offsets N(0, 0.1^2), plain norm weights 1 + N(0, 0.1^2), decay offsets spread over (-2, 6) so that some channels forget within
+  tokens and others keep hundreds, routers spread so that the logits differ, embedding rows N(0, 1)."""
+  out = {}
+  for idx, (name, shape) in enumerate(sorted(rurutar_param_shapes(cfg, rank).items())):
+    g = torch.Generator(device=device).manual_seed(seed * 1000003 + idx)
+    rn = lambda: torch.randn(shape, generator=g, device=device)  # noqa: E731
+    ru = lambda: torch.rand(shape, generator=g, device=device)  # noqa: E731
+    leaf = name.split(".")[-1]
+    if leaf == "alpha":
+      t = 0.4 + 0.8 * ru()
+    elif name.endswith("a2.b"):
+      t = -2.0 + 8.0 * ru()
+    elif leaf == "b":
+      t = 0.1 * rn()
+    elif leaf.startswith("norm"):
+      t = 1.0 + 0.1 * rn()
+    elif name == "embed":
+      t = rn()
+    elif leaf == "router":
+      t = 2.0 * gain * rn() / (shape[-1] ** 0.5)
+    else:
+      t = gain * rn() / (shape[-1] ** 0.5)
+    out[name] = t.to(dtype)
+  return out
+
+
 def write_random_checkpoint(path: Path, cfg: dict, seed: int = 0, std: float = 0.02,
                             norm_jitter: float = 0.0, shard_bytes: int = 4 << 30,
                             peaked_head: float = 0.0) -> Path:
@@ -338,6 +408,8 @@ def write_random_checkpoint(path: Path, cfg: dict, seed: int = 0, std: float = 0
     state = random_pufivik_state(cfg, seed=seed)
   elif cfg.get("architecture") == "Vusenex":
     state = random_vusenex_state(cfg, seed=seed)
+  elif cfg.get("architecture") == "Rurutar":
+    state = random_rurutar_state(cfg, seed=seed)
   else:
     state = random_hf_state(cfg, seed=seed, std=std, norm_jitter=norm_jitter, peaked_head=peaked_head)
   files, cur, cur_bytes = [], {}, 0
