@@ -202,14 +202,14 @@ def _rurutar(width, vocab, layers, scale=0.7, softcap=20.0, eps=1e-6):
           "layers": [{"type": t, "mixer": m, "mlp": f} for t, m, f in layers]}
 
 
-def _gla(heads, dim, vdim, tau=16.0, rank=None):
+def _gla(heads, dim, vdim, tau=20.0, rank=None):
   m = {"heads": heads, "dim": dim, "vdim": vdim, "tau": tau}
   if rank:
     m["rank"] = rank
   return m
 
 
-def _window_latent(heads, dim, rot_dim, vdim, kv_rank, q_rank, window, kv_from=None, base=10000.0, factor=4.0, original=1024):
+def _window_latent(heads, dim, rot_dim, vdim, kv_rank, q_rank, window, kv_from=None, base=10000.0, factor=8.0, original=2048):
   m = {"heads": heads, "dim": dim, "rot_dim": rot_dim, "vdim": vdim, "kv_rank": kv_rank, "q_rank": q_rank, "scale": (dim + rot_dim) ** -0.5,
        "mask": {"size": window}, "rot": {"base": base, "dims": rot_dim,
                                          "scaling": {"factor": factor, "original": original, "fast": 32.0, "slow": 1.0}}}
@@ -237,7 +237,7 @@ _RURUTAR_TINY = _rurutar(160, 384, [
 _RURUTAR_1B = _rurutar(2048, 128256, [
   (("latent_attention", _window_latent(16, 64, 64, 128, 256, 768, 1024, kv_from=(i - 4 if i % 8 == 7 else None), base=500000.0),
     _gated_experts(16, 4, 384, 2048)) if i % 4 == 3 else
-   ("gla", _gla(16, 128, 128, rank=16), {"kind": "dense", "ff": 8192} if i % 4 == 0 else _gated_experts(16, 4, 384, 2048)))
+   ("gla", _gla(16, 128, 128, rank=32), {"kind": "dense", "ff": 8192} if i % 4 == 0 else _gated_experts(16, 4, 384, 2048)))
   for i in range(16)])
 
 # model id -> {layers, repo:{EngineClassName: hf repo}, hf_config}
