@@ -10,6 +10,7 @@
 // rows x key shares that the split form of the latent attention may write: steps of fewer than num_sms / 2 tiles of 64 rows
 // use it, with at most this many (row, share) pairs
 #define HY_LAT_SPLIT_ROWS 4864
+#define HY_SEG_MIN 64   // shortest segment of a recurrence cut along the tokens
 
 struct HyTarget {
   void* dst = nullptr;
@@ -97,6 +98,10 @@ struct HyModel {
   int dec_splits = 1;                   // key splits of this step's single-token attention (hy_kv_splits)
   bool pdl_now = false;
   int recur_lpc = 0;         // XB_HY_LPC=4|8|16 pins the lanes per state column (A/B); 0: by the step's shape
+  float *seg_ws = nullptr, *seg_decay = nullptr;   // recurrences cut into segments: a state and the decays per segment
+  size_t maxSeg = 0, maxSegK = 0;                  // state numbers / key channels of the largest such layer
+  int use_seg = 1;           // XB_HY_SEG=0: recurrences always as one chain per sequence (A/B); XB_HY_SEG=n >= 64: segments of n tokens
+  int seg_len = 0;           // pinned segment length, 0: by the step's shape
   int use_tc_attn = 1;       // XB_HY_TC_ATTN=0: attention through the per-token kernel everywhere (A/B)
   int use_tc = 1;            // XB_HY_TC=0: every Linear through the plain kernels (A/B)
   size_t cap_P = 0, cap_m = 0, cap_head = 0;   // bytes of the Linear output buffers
@@ -149,6 +154,11 @@ static void hy_destroy(HyModel* hy) {
 // experts side by side are ONE matrix over all experts' activations).
 static void hy_name_cols(HyModel* hy, const std::string& name, bf16* base, long long col0, long long rows, long long cols, long long ld) {
   hy_name(hy, name, base + col0, false, rows, cols, ld, 2);
+}
+
+static void hy_segment_room(HyModel* hy, long long numbers, long long keys) {
+  if ((size_t)numbers > hy->maxSeg) hy->maxSeg = numbers;
+  if ((size_t)keys > hy->maxSegK) hy->maxSegK = keys;
 }
 
 // A norm of the stream: one vector (or one number), for the tanh norm also an offset per channel and the input's factor.
@@ -295,6 +305,7 @@ static int hy_create_mixer(xb_engine* e, int i, bool own, size_t& st, uint64_t& 
     hy_name_rows(hy, p + "o", l.w_o, 0, D, l.n_o);
     wbytes += ((size_t)l.n_in * D + D * l.n_o + (size_t)(HK * rk)) * 2;
     l.st_rec = st; st += (size_t)(HV * n);
+    hy_segment_room(hy, HV * n, HK);
     if ((size_t)(3 * HK + HV) > hy->maxC) hy->maxC = 3 * HK + HV;
     if ((size_t)l.n_o > hy->maxO) hy->maxO = l.n_o;
   } else if (c.mixer == XB_MIX_GDELTA) {
@@ -349,6 +360,7 @@ static int hy_create_mixer(xb_engine* e, int i, bool own, size_t& st, uint64_t& 
       wbytes += ((size_t)l.n_in * D + D * l.n_o) * 2;
     }
     l.st_rec = st; st += (size_t)(H * dv * n);
+    hy_segment_room(hy, H * dv * n, H * n);
     const size_t cc = (size_t)(2 * H * n + H * dv);
     if (cc > hy->maxC) hy->maxC = cc;
     if ((size_t)l.n_o > hy->maxO) hy->maxO = l.n_o;
@@ -613,6 +625,7 @@ static int hy_create(xb_engine* e, const xb_hybrid_desc& d, const xb_hybrid_laye
       l.tc_attn = !d.compute_fp32 && dk == dv && (dk == 64 || dk == 128) && H / G <= 8 && c.a_scale > 0.f;
       if (l.tc_attn && (size_t)(H * (dk + dv)) > hy->maxQG) hy->maxQG = H * (dk + dv);
       l.st_rec = st; st += (size_t)(Hr * rv * rk);
+      hy_segment_room(hy, Hr * rv * rk, Hr * rk);
       const size_t cc = (size_t)(2 * Hr * rk + Hr * rv);
       if (cc > hy->maxC) hy->maxC = cc;
       if ((size_t)l.n_o > hy->maxO) hy->maxO = l.n_o;
@@ -751,10 +764,18 @@ static int hy_create(xb_engine* e, const xb_hybrid_desc& d, const xb_hybrid_laye
     if (fr != nullptr && fr[0] == '0') hy->fuse_router = 0;
     const char* ps = getenv("XB_HY_P_SPLIT");
     if (ps != nullptr && ps[0] == '0') hy->p_split = 0;
+    const char* sl = getenv("XB_HY_SEG");
+    if (sl != nullptr) { hy->use_seg = atoi(sl) > 0 ? 1 : 0; hy->seg_len = atoi(sl) >= HY_SEG_MIN ? atoi(sl) : 0; }
     const char* lp = getenv("XB_HY_LPC");
     if (lp != nullptr && (atoi(lp) == 4 || atoi(lp) == 8 || atoi(lp) == 16)) hy->recur_lpc = atoi(lp);
   }
   XB_TRY(hy_alloc_t(hy, &hy->d_rows, R));
+  if (hy->maxSeg > 0 && Tm >= 2 * HY_SEG_MIN) {
+    // sequences of a cut step hold two segments or more on average: entries <= T / seg + sequences <= 3/2 T / seg
+    const size_t entries = Tm / HY_SEG_MIN + Tm / (2 * HY_SEG_MIN) + 2;
+    XB_TRY(hy_alloc_t(hy, &hy->seg_ws, entries * hy->maxSeg));
+    XB_TRY(hy_alloc_t(hy, &hy->seg_decay, entries * hy->maxSegK));
+  }
   if (hy->maxQG > 0) {
     XB_TRY(hy_alloc_t(hy, &hy->qg, Tm * hy->maxQG));
     std::vector<int> ones((size_t)d.max_seqs, 1);
@@ -1047,9 +1068,48 @@ static int hy_recur_l(xb_engine* e, const RecurIn& in, float* state, long long s
 #undef HY_RECUR_CASE
   return xb_fail(1, "recurrent key dim %d exceeds %d", dk, HY_MAX_KDIM);
 }
+// Prompts through the segments of hy_seg_kernel (modes whose step fades a state column entry by entry).  Segments of 128 tokens, of
+// 64 when 128 would leave the SMs with fewer than four blocks each.
+template <int NCH, int NCOL, int MODE>
+static int hy_segments_n(xb_engine* e, const RecurIn& in, float* state, long long ss, float* o, long long ldo, const BatchMeta& m, int n_seqs,
+                         int H, int dk, int dv, int T, cudaStream_t st) {
+  HyModel* hy = e->hy;
+  const int cb = (dv + 32 * NCOL - 1) / (32 * NCOL);
+  SegArgs sg;
+  sg.seg = hy->seg_len > 0 ? hy->seg_len : ((long long)(T / 128) * H * cb >= 4LL * e->num_sms ? 128 : HY_SEG_MIN);
+  sg.max_segs = (T + sg.seg - 1) / sg.seg;
+  sg.ws = hy->seg_ws;
+  sg.decay = MODE == HY_REC_LIGHTNING ? nullptr : hy->seg_decay;
+  const dim3 grid(cb, H, n_seqs * sg.max_segs);
+  constexpr size_t row = (size_t)2 * HY_SEG_TS * sizeof(float);
+  constexpr size_t s0 = row * (hy_seg_vectors(MODE, 0) * 16 * NCH + 32 * NCOL), s1 = row * (hy_seg_vectors(MODE, 1) * 16 * NCH + 32 * NCOL);
+  if (s0 > 48 * 1024) XB_SMEM_ATTR_ONCE((hy_seg_kernel<NCH, NCOL, MODE, 0>), s0);
+  if (s1 > 48 * 1024) XB_SMEM_ATTR_ONCE((hy_seg_kernel<NCH, NCOL, MODE, 1>), s1);
+  XB_TRY(hy_launch(e, hy_seg_kernel<NCH, NCOL, MODE, 0>, grid, dim3(128), s0, st, in, sg, state, ss, o, ldo, m, H, dk, dv));
+  if (sg.decay != nullptr)
+    XB_TRY(hy_launch(e, hy_seg_decay_kernel, dim3((H * dk + 255) / 256, n_seqs * sg.max_segs), dim3(256), 0, st, in.c, in.ldc,
+                     MODE == HY_REC_GLA ? in.xoff[0] : in.koff, H * dk, sg.seg, sg.max_segs, hy->seg_decay, m));
+  XB_TRY(hy_launch(e, hy_seg_scan_kernel, dim3((dv * dk + 255) / 256, H, n_seqs), dim3(256), 0, st, sg, in.hdecay, (const float*)state, ss, m, H, dk, dv));
+  return hy_launch(e, hy_seg_kernel<NCH, NCOL, MODE, 1>, grid, dim3(128), s1, st, in, sg, state, ss, o, ldo, m, H, dk, dv);
+}
+template <int MODE>
+static int hy_segments(xb_engine* e, const RecurIn& in, float* state, long long ss, float* o, long long ldo, const BatchMeta& m, int n_seqs,
+                       int H, int dk, int dv, int T, cudaStream_t st) {
+  if (dk <= 16) return hy_segments_n<1, 2, MODE>(e, in, state, ss, o, ldo, m, n_seqs, H, dk, dv, T, st);
+  if (dk <= 32) return hy_segments_n<2, 2, MODE>(e, in, state, ss, o, ldo, m, n_seqs, H, dk, dv, T, st);
+  if (dk <= 64) return hy_segments_n<4, 2, MODE>(e, in, state, ss, o, ldo, m, n_seqs, H, dk, dv, T, st);
+  if (dk <= 128) return hy_segments_n<8, 2, MODE>(e, in, state, ss, o, ldo, m, n_seqs, H, dk, dv, T, st);
+  return hy_segments_n<16, 1, MODE>(e, in, state, ss, o, ldo, m, n_seqs, H, dk, dv, T, st);
+}
+
 template <int MODE>
 static int hy_recur(xb_engine* e, const RecurIn& in, float* state, long long ss, float* o, long long ldo, const BatchMeta& m, int n_seqs,
-                    int H, int dk, int dv, cudaStream_t st) {
+                    int H, int dk, int dv, int T, cudaStream_t st) {
+  if constexpr (MODE == HY_REC_GLA || MODE == HY_REC_HGRN || MODE == HY_REC_LIGHTNING) {
+    const int least = e->hy->seg_len > 0 ? 2 * e->hy->seg_len : 4 * HY_SEG_MIN;   // average length from which it pays
+    if (e->hy->use_seg && T / n_seqs >= least && (long long)n_seqs * (T / HY_SEG_MIN + 1) <= 65535)   // grid z
+      return hy_segments<MODE>(e, in, state, ss, o, ldo, m, n_seqs, H, dk, dv, T, st);
+  }
   int lpc = e->hy->recur_lpc;
   if (lpc == 0) {
     const long long want = 2LL * e->num_sms;
@@ -1469,7 +1529,7 @@ static int hy_run_parallel_t(xb_engine* e, int T, int n_seqs, void* const* taps,
       RecurIn in;
       in.c = hy->c; in.ldc = 6LL * HN; in.qoff = 0; in.koff = HN; in.xoff[0] = 2LL * HN; in.xoff[1] = 3LL * HN; in.xoff[2] = 4LL * HN;
       in.voff = 5LL * HN; in.q_heads = H; in.beta = hy->beta; in.decay = hy->decay; in.qk = nullptr; in.hdecay = nullptr;
-      XB_TRY(hy_recur<HY_REC_GDELTA>(e, in, hy->state + l.st_rec, SS, hy->o, (long long)l.n_o, m, n_seqs, H, n, n, st));
+      XB_TRY(hy_recur<HY_REC_GDELTA>(e, in, hy->state + l.st_rec, SS, hy->o, (long long)l.n_o, m, n_seqs, H, n, n, T, st));
       XB_TRY(hy_launch(e, hy_head_norm_kernel<AT>, dim3(T, (H + 7) / 8), dim3(256), 0, st, (const float*)hy->o, (long long)l.n_o,
                        (const float*)l.head_norm, P, l.off_g, d.norm_eps, 1.0f, a1, (long long)l.n_o, H, n, n, 1));
     } else {
@@ -1480,7 +1540,7 @@ static int hy_run_parallel_t(xb_engine* e, int T, int n_seqs, void* const* taps,
       in.c = hy->c; in.ldc = nc; in.qoff = 0; in.koff = (long long)H * n; in.voff = 2LL * H * n; in.q_heads = H;
       in.xoff[0] = in.xoff[1] = in.xoff[2] = 0;
       in.beta = in.decay = in.qk = nullptr; in.hdecay = l.hdecay;
-      XB_TRY(hy_recur<HY_REC_LIGHTNING>(e, in, hy->state + l.st_rec, SS, hy->o, (long long)l.n_o, m, n_seqs, H, n, dv, st));
+      XB_TRY(hy_recur<HY_REC_LIGHTNING>(e, in, hy->state + l.st_rec, SS, hy->o, (long long)l.n_o, m, n_seqs, H, n, dv, T, st));
       XB_TRY(hy_launch(e, hy_all_heads_norm_kernel<AT>, dim3(T), dim3(256), 0, st, (const float*)hy->o, (long long)l.n_o,
                        (const float*)l.head_norm, P, l.off_g, d.norm_eps, a1, (long long)l.n_o, H * dv));
     }
@@ -1740,7 +1800,7 @@ static int hy_run_prenorm_t(xb_engine* e, int T, int n_seqs, void* const* taps, 
       RecurIn in;
       in.c = hy->c; in.ldc = ldc; in.qoff = 0; in.koff = HK; in.xoff[0] = 2LL * HK; in.xoff[1] = in.xoff[2] = 0; in.voff = 3LL * HK; in.q_heads = H;
       in.beta = in.decay = in.qk = in.hdecay = nullptr;
-      XB_TRY(hy_recur<HY_REC_GLA>(e, in, hy->state + l.st_rec, SS, hy->o, (long long)l.n_o, m, n_seqs, H, n, dv, st));
+      XB_TRY(hy_recur<HY_REC_GLA>(e, in, hy->state + l.st_rec, SS, hy->o, (long long)l.n_o, m, n_seqs, H, n, dv, T, st));
       XB_TRY(hy_launch(e, hy_head_norm_kernel<AT>, dim3(T, (H + 7) / 8), dim3(256), 0, st, (const float*)hy->o, (long long)l.n_o,
                        (const float*)l.head_norm, P, l.off_g, d.norm_eps, 1.0f, a1, (long long)l.n_o, H, dv, 0, 0));
     }
@@ -1805,7 +1865,7 @@ static int hy_run_body_t(xb_engine* e, int T, int n_seqs, int n_tiles, void* con
         in.c = hy->c; in.ldc = l.c_conv; in.qoff = 0; in.koff = (long long)G * dk; in.voff = 2LL * G * dk; in.q_heads = G;
         in.beta = hy->beta; in.decay = hy->decay; in.qk = hy->qk; in.hdecay = nullptr;
         in.xoff[0] = in.xoff[1] = in.xoff[2] = 0;
-        XB_TRY(hy_recur<HY_REC_DELTA>(e, in, hy->state + l.st_rec, SS, hy->o, (long long)l.n_o, m, n_seqs, H, dk, dv, st));
+        XB_TRY(hy_recur<HY_REC_DELTA>(e, in, hy->state + l.st_rec, SS, hy->o, (long long)l.n_o, m, n_seqs, H, dk, dv, T, st));
       }
       XB_TRY(hy_launch(e, hy_head_norm_kernel<AT>, dim3(T, (H + 7) / 8), dim3(256), 0, st, (const float*)hy->o, (long long)l.n_o,
                        (const float*)l.head_norm, P, l.off_g, d.norm_eps, 1.0f, a1, (long long)l.n_o, H, dv, 0, 0));
@@ -1855,7 +1915,7 @@ static int hy_run_body_t(xb_engine* e, int T, int n_seqs, int n_tiles, void* con
         in.c = hy->c; in.ldc = ldc; in.qoff = 0; in.koff = (long long)Hr * rk; in.voff = 2LL * Hr * rk; in.q_heads = Hr;
         in.beta = in.decay = in.qk = in.hdecay = nullptr;
         in.xoff[0] = in.xoff[1] = in.xoff[2] = 0;
-        XB_TRY(hy_recur<HY_REC_HGRN>(e, in, hy->state + l.st_rec, SS, hy->o, (long long)l.n_o2, m, n_seqs, Hr, rk, rv, st));
+        XB_TRY(hy_recur<HY_REC_HGRN>(e, in, hy->state + l.st_rec, SS, hy->o, (long long)l.n_o2, m, n_seqs, Hr, rk, rv, T, st));
       }
       XB_TRY(hy_launch(e, hy_head_norm_kernel<AT>, dim3(T, (Hr + 7) / 8), dim3(256), 0, st, (const float*)hy->o, (long long)l.n_o2,
                        (const float*)l.head_norm, P, -1, d.norm_eps, 1.0f, a2, (long long)l.n_o2, Hr, rv, 0, 0));

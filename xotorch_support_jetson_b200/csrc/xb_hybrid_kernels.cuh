@@ -1093,6 +1093,265 @@ __global__ void __launch_bounds__(128) hy_recur_kernel(RecurIn in, float* __rest
   }
 }
 
+// ----------------------------------------------------------------------------- the same recurrences, segment by segment
+// Where a step fades a state column entry by entry (HGRN2, lightning, gated linear attention), S_end = A S_start + L with A the
+// product of a segment's decays per row and L its end state from an empty start.  So a prompt is cut into segments of `seg` tokens
+// that run side by side: (1) hy_seg_kernel<PASS 0> makes L of every segment but a sequence's last, (2) hy_seg_decay_kernel makes A,
+// (3) hy_seg_scan_kernel walks the segments once and leaves every segment's start state, (4) hy_seg_kernel<PASS 1> runs the segments
+// from there and writes the outputs, the last one also the slot's new state.  All of it fp32, the same step arithmetic as
+// hy_recur_kernel; nothing is divided, so any decay (zero included) is served.
+// Workspace ws: one state [H][dv][dk] per segment; segment c of sequence s sits at entry start_row / seg + s + c (ceilings of earlier
+// sequences add up to no more than that).
+//
+// Four lanes own NCOL value columns: lane `sub` holds the rows of the 16-byte chunks sub, sub + 4, ... of each, as pairs for the packed
+// two-wide fp32 FMA.  A block's 4 warps share (segment, head) and 32 * NCOL columns; the inputs of HY_SEG_TS steps arrive in
+// shared memory by cp.async, one chunk of steps ahead.
+// grid (ceil(dv / (32 NCOL)), H, n_seqs * max_segs), 128 threads.
+#define HY_SEG_TS 8
+typedef unsigned long long hy_f2;
+__device__ __forceinline__ hy_f2 hy_f2_pack(float a, float b) {
+  hy_f2 r;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b));
+  return r;
+}
+__device__ __forceinline__ float2 hy_f2_unpack(hy_f2 v) {
+  float2 r;
+  asm("mov.b64 {%0, %1}, %2;" : "=f"(r.x), "=f"(r.y) : "l"(v));
+  return r;
+}
+__device__ __forceinline__ hy_f2 hy_f2_fma(hy_f2 a, hy_f2 b, hy_f2 c) {
+  hy_f2 r;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+  return r;
+}
+__device__ __forceinline__ hy_f2 hy_f2_mul(hy_f2 a, hy_f2 b) {
+  hy_f2 r;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+  return r;
+}
+struct SegArgs {
+  float* ws;              // [entries][H * dv * dk]
+  const float* decay;     // [entries][H * dk], or nullptr (lightning)
+  int seg, max_segs;      // tokens per segment, segments of the longest sequence a step can hold
+};
+// row vectors staged per step: k (or f), w where it is a vector of its own, q in the output pass
+__host__ __device__ constexpr int hy_seg_vectors(int mode, int pass) { return 1 + (mode == HY_REC_GLA ? 1 : 0) + (pass == 1 ? 1 : 0); }
+
+template <int NCH, int NCOL, int MODE, int PASS>
+__global__ void __launch_bounds__(128) hy_seg_kernel(RecurIn in, SegArgs sg, float* __restrict__ state, long long state_stride, float* __restrict__ o,
+                                                     long long ldo, BatchMeta m, int H, int dk, int dv) {
+  pdl_wait();
+  extern __shared__ __align__(16) float stg[];
+  constexpr int NV = hy_seg_vectors(MODE, PASS), DKP = 16 * NCH, NB = 32 * NCOL, VO = NV * DKP, STRIDE = VO + NB;
+  const int s = blockIdx.z / sg.max_segs, c = blockIdx.z - s * sg.max_segs, h = blockIdx.y, j0 = blockIdx.x * NB;
+  const SeqSpan sp = seq_span(m, s);
+  const int nseg = (sp.len + sg.seg - 1) / sg.seg;
+  if (c >= nseg || (PASS == 0 && c == nseg - 1)) return;
+  const int row0 = sp.start + c * sg.seg, len = sp.len - c * sg.seg < sg.seg ? sp.len - c * sg.seg : sg.seg;
+  float* entry = sg.ws + (long long)(sp.start / sg.seg + s + c) * H * dv * dk;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, sub = lane & 3;
+  const int jl = (warp * 8 + (lane >> 2)) * NCOL, ncv = dv - j0 < NB ? dv - j0 : NB;
+  // staged vectors in the order of the shared rows: k, (w), (q)
+  const float* src[NV];
+  src[0] = in.c + in.koff + (long long)h * dk;
+  if (MODE == HY_REC_GLA) src[1] = in.c + in.xoff[0] + (long long)h * dk;
+  if (PASS == 1) src[NV - 1] = in.c + in.qoff + (long long)h * dk;
+  const float* cv = in.c + in.voff + (long long)h * dv + j0;
+  const hy_f2 hd2 = MODE == HY_REC_LIGHTNING ? hy_f2_pack(in.hdecay[h], in.hdecay[h]) : 0ull;
+  bool al = ((in.ldc | in.qoff | in.koff | in.voff | dk | dv) & 3) == 0 && (reinterpret_cast<uintptr_t>(in.c) & 15) == 0;
+  if (MODE == HY_REC_GLA) al = al && (in.xoff[0] & 3) == 0;
+  for (int i = threadIdx.x; i < 2 * HY_SEG_TS * STRIDE; i += 128) stg[i] = 0.f;   // padding rows / columns stay zero
+  hy_f2 S[NCOL][2 * NCH];
+  const bool st_al = (dk & 3) == 0;   // entries start on 16-byte boundaries when every column does
+#pragma unroll
+  for (int n = 0; n < NCOL; ++n) {
+    const bool have = PASS == 1 && jl + n < ncv;
+    const float* st = entry + ((long long)h * dv + j0 + jl + n) * dk;
+#pragma unroll
+    for (int ch = 0; ch < NCH; ++ch) {
+      const int r = (ch * 4 + sub) * 4;
+      if (have && st_al && r < dk) {
+        const ulonglong2 v = *reinterpret_cast<const ulonglong2*>(st + r);
+        S[n][2 * ch] = v.x; S[n][2 * ch + 1] = v.y;
+      } else {
+        float e[4];
+#pragma unroll
+        for (int x = 0; x < 4; ++x) e[x] = (have && r + x < dk) ? st[r + x] : 0.f;
+        S[n][2 * ch] = hy_f2_pack(e[0], e[1]); S[n][2 * ch + 1] = hy_f2_pack(e[2], e[3]);
+      }
+    }
+  }
+  __syncthreads();
+  auto stage = [&](int t0, float* buf) {
+    const int nt = len - t0 < HY_SEG_TS ? len - t0 : HY_SEG_TS;
+    if (al) {
+      const int dq = dk >> 2, per = NV * dq + (ncv >> 2);
+      for (int idx = threadIdx.x; idx < nt * per; idx += 128) {
+        const int ts = idx / per, u = idx - ts * per;
+        const long long row = (long long)(row0 + t0 + ts) * in.ldc;
+        float* d = buf + ts * STRIDE;
+        bool done = false;
+#pragma unroll
+        for (int v = 0; v < NV; ++v)
+          if (!done && u < (v + 1) * dq) { hy_cp16(d + v * DKP + 4 * (u - v * dq), src[v] + row + 4 * (u - v * dq)); done = true; }
+        if (!done) hy_cp16(d + VO + 4 * (u - NV * dq), cv + row + 4 * (u - NV * dq));
+      }
+    } else {
+      const int per = NV * dk + ncv;
+      for (int idx = threadIdx.x; idx < nt * per; idx += 128) {
+        const int ts = idx / per, u = idx - ts * per;
+        const long long row = (long long)(row0 + t0 + ts) * in.ldc;
+        float* d = buf + ts * STRIDE;
+        bool done = false;
+#pragma unroll
+        for (int v = 0; v < NV; ++v)
+          if (!done && u < (v + 1) * dk) { hy_cp4(d + v * DKP + (u - v * dk), src[v] + row + (u - v * dk)); done = true; }
+        if (!done) hy_cp4(d + VO + (u - NV * dk), cv + row + (u - NV * dk));
+      }
+    }
+    hy_cp_commit();
+  };
+  stage(0, stg);
+  int cur = 0;
+  for (int t0 = 0; t0 < len; t0 += HY_SEG_TS, cur ^= 1) {
+    const int nt = len - t0 < HY_SEG_TS ? len - t0 : HY_SEG_TS;
+    if (t0 + HY_SEG_TS < len) { stage(t0 + HY_SEG_TS, stg + (cur ^ 1) * HY_SEG_TS * STRIDE); hy_cp_wait<1>(); }
+    else hy_cp_wait<0>();
+    __syncthreads();
+    const float* buf = stg + cur * HY_SEG_TS * STRIDE;
+    auto step = [&](int ts) {
+      const float* sr = buf + ts * STRIDE;
+      hy_f2 vv[NCOL], acc[NCOL];
+#pragma unroll
+      for (int n = 0; n < NCOL; ++n) {
+        const float v = sr[VO + jl + n];
+        vv[n] = hy_f2_pack(v, v);
+        acc[n] = 0ull;
+      }
+#pragma unroll
+      for (int ch = 0; ch < NCH; ++ch) {
+        const int r = (ch * 4 + sub) * 4;
+        const ulonglong2 k4 = *reinterpret_cast<const ulonglong2*>(sr + r);
+        hy_f2 k2[2] = {k4.x, k4.y}, w2[2], q2[2] = {0ull, 0ull};
+        if (MODE == HY_REC_GLA) {
+          const ulonglong2 w4 = *reinterpret_cast<const ulonglong2*>(sr + DKP + r);
+          w2[0] = w4.x; w2[1] = w4.y;
+        } else if (MODE == HY_REC_HGRN) {   // the k slot holds f: S <- f S + (1 - f) v
+#pragma unroll
+          for (int x = 0; x < 2; ++x) {
+            w2[x] = k2[x];
+            const float2 f = hy_f2_unpack(k2[x]);
+            k2[x] = hy_f2_pack(1.0f - f.x, 1.0f - f.y);
+          }
+        } else {
+          w2[0] = w2[1] = hd2;
+        }
+        if (PASS == 1) {
+          const ulonglong2 q4 = *reinterpret_cast<const ulonglong2*>(sr + (NV - 1) * DKP + r);
+          q2[0] = q4.x; q2[1] = q4.y;
+        }
+#pragma unroll
+        for (int n = 0; n < NCOL; ++n)
+#pragma unroll
+          for (int x = 0; x < 2; ++x) {
+            S[n][2 * ch + x] = hy_f2_fma(w2[x], S[n][2 * ch + x], hy_f2_mul(k2[x], vv[n]));
+            if (PASS == 1) acc[n] = hy_f2_fma(q2[x], S[n][2 * ch + x], acc[n]);
+          }
+      }
+      if (PASS == 1) {
+        float mine = 0.f;
+#pragma unroll
+        for (int n = 0; n < NCOL; ++n) {
+          const float2 a = hy_f2_unpack(acc[n]);
+          float b = a.x + a.y;
+          b += __shfl_xor_sync(0xffffffffu, b, 1);
+          b += __shfl_xor_sync(0xffffffffu, b, 2);
+          if (sub == n) mine = b;
+        }
+        if (sub < NCOL && jl + sub < ncv) o[(long long)(row0 + t0 + ts) * ldo + (long long)h * dv + j0 + jl + sub] = mine;
+      }
+    };
+    if (nt == HY_SEG_TS) {
+#pragma unroll 2
+      for (int ts = 0; ts < HY_SEG_TS; ++ts) step(ts);
+    } else {
+      for (int ts = 0; ts < nt; ++ts) step(ts);
+    }
+    __syncthreads();   // the buffer is refilled by the next iteration's copies
+  }
+  if (PASS == 1 && c != nseg - 1) return;
+  float* base = PASS == 0 ? entry : state + (long long)sp.slot * state_stride;
+  const bool out_al = st_al && (reinterpret_cast<uintptr_t>(base) & 15) == 0;
+#pragma unroll
+  for (int n = 0; n < NCOL; ++n) {
+    if (jl + n >= ncv) continue;
+    float* st = base + ((long long)h * dv + j0 + jl + n) * dk;
+#pragma unroll
+    for (int ch = 0; ch < NCH; ++ch) {
+      const int r = (ch * 4 + sub) * 4;
+      if (out_al && r < dk) {
+        *reinterpret_cast<ulonglong2*>(st + r) = make_ulonglong2(S[n][2 * ch], S[n][2 * ch + 1]);
+      } else {
+        const float2 a = hy_f2_unpack(S[n][2 * ch]), b = hy_f2_unpack(S[n][2 * ch + 1]);
+        const float e[4] = {a.x, a.y, b.x, b.y};
+#pragma unroll
+        for (int x = 0; x < 4; ++x)
+          if (r + x < dk) st[r + x] = e[x];
+      }
+    }
+  }
+}
+
+// decay[entry][h * dk + i] = product over the segment's tokens of column off + h * dk + i.  grid (ceil(HK / 256), n_seqs * max_segs).
+__global__ void __launch_bounds__(256) hy_seg_decay_kernel(const float* __restrict__ c, long long ldc, long long off, int HK, int seg, int max_segs,
+                                                           float* __restrict__ decay, BatchMeta m) {
+  pdl_wait();
+  const int s = blockIdx.y / max_segs, cseg = blockIdx.y - s * max_segs;
+  const SeqSpan sp = seq_span(m, s);
+  const int i = blockIdx.x * 256 + threadIdx.x;
+  if ((cseg + 1) * seg >= sp.len || i >= HK) return;   // a sequence's last segment carries nothing on
+  const float* p = c + (long long)(sp.start + cseg * seg) * ldc + off + i;
+  float a[4] = {1.f, 1.f, 1.f, 1.f};
+  int t = 0;
+  for (; t + 3 < seg; t += 4) {
+#pragma unroll
+    for (int x = 0; x < 4; ++x) a[x] *= p[(long long)(t + x) * ldc];
+  }
+  for (; t < seg; ++t) a[0] *= p[(long long)t * ldc];
+  decay[(long long)(sp.start / seg + s + cseg) * HK + i] = (a[0] * a[1]) * (a[2] * a[3]);
+}
+
+// ws entries: local end states -> start states.  A thread owns one state number and walks the segments of its sequence, four loads in
+// flight.  grid (ceil(dv * dk / 256), H, n_seqs), 256 threads.
+__global__ void __launch_bounds__(256) hy_seg_scan_kernel(SegArgs sg, const float* __restrict__ hdecay, const float* __restrict__ state,
+                                                          long long state_stride, BatchMeta m, int H, int dk, int dv) {
+  pdl_wait();
+  const int s = blockIdx.z, h = blockIdx.y, e = blockIdx.x * 256 + threadIdx.x;
+  if (e >= dv * dk) return;
+  const SeqSpan sp = seq_span(m, s);
+  const int nseg = (sp.len + sg.seg - 1) / sg.seg, i = e % dk;
+  const long long e0 = sp.start / sg.seg + s, ss = (long long)H * dv * dk, at = (long long)h * dv * dk + e;
+  float* w = sg.ws + e0 * ss + at;
+  const float* A = sg.decay != nullptr ? sg.decay + e0 * H * dk + (long long)h * dk + i : nullptr;
+  const float hp = sg.decay == nullptr ? powf(hdecay[h], (float)sg.seg) : 1.f;
+  float S = sp.pos0 > 0 ? state[(long long)sp.slot * state_stride + at] : 0.f;
+  for (int c0 = 0; c0 < nseg; c0 += 4) {
+    float L[4], a[4];
+#pragma unroll
+    for (int x = 0; x < 4; ++x) {
+      const bool in = c0 + x < nseg - 1;
+      L[x] = in ? w[(c0 + x) * ss] : 0.f;
+      a[x] = in ? (A != nullptr ? A[(long long)(c0 + x) * H * dk] : hp) : 0.f;
+    }
+#pragma unroll
+    for (int x = 0; x < 4; ++x) {
+      if (c0 + x >= nseg) break;
+      w[(c0 + x) * ss] = S;
+      S = fmaf(a[x], S, L[x]);
+    }
+  }
+}
+
 // ----------------------------------------------------------------------------- HGRN2
 // Prep: q = silu(.), f = lower + (1 - lower) sigmoid(.), v copied, into one fp32 row [q | f | v].  grid (T, ceil(n / 256)).
 __global__ void hy_hgrn_prep_kernel(LinOut P, int off_q, int off_f, int off_v, const float* __restrict__ lower, float* __restrict__ c,
