@@ -1356,8 +1356,14 @@ static int hy_latent_mixer(xb_engine* e, const HyLayer& l, int T, const LinOut& 
   LinOut Q = P;
   if (qr > 0) XB_TRY(hy_linear<AT>(e, a2, qr, l.w_uq, l.t_uq, nullptr, T, H * (n + dr), qr, hy->m2, hy->cap_m, st, &Q));
   const size_t mm1 = (size_t)HY_MM_ROWS * n * sizeof(float), mm2 = (size_t)HY_MM_ROWS * R * sizeof(float);
+  // prompts in bf16 serving whose queries came back as one bf16 matrix: both per-head products on the tensor cores
+  const bool tiles = std::is_same<AT, bf16>::value && hy->use_lat_mma && T > 64 && (n | dr | R | dv) % 8 == 0;
+  if (tiles && Q.h != nullptr && Q.bias == nullptr && Q.ld % 8 == 0 && l.off_q % 8 == 0)
+    XB_TRY(hy_launch(e, hy_latent_absorb_mma_kernel, dim3((T + HY_HG_M - 1) / HY_HG_M, H, (R + HY_HG_N - 1) / HY_HG_N), dim3(128), 0, st, Q.h + l.off_q,
+                     Q.ld, dr, (const bf16*)l.w_uk, hy->qa, H, T, n, R, r, m.tok_pos));
+  else
   XB_TRY(hy_launch(e, hy_latent_absorb_kernel, dim3((T + HY_MM_ROWS - 1) / HY_MM_ROWS, H), dim3(256), mm1, st, Q, l.off_q, dr,
-                   (const bf16*)l.w_uk, hy->qa, H, T, n, R, r, m.tok_pos));
+                     (const bf16*)l.w_uk, hy->qa, H, T, n, R, r, m.tok_pos));
   // bf16 serving at sizes the tensor-core tiles take: rows = (token, head) pairs over shared key tiles; steps of few
   // rows split every sequence's keys over blocks and merge
   bool done = false;
@@ -1378,6 +1384,9 @@ static int hy_latent_mixer(xb_engine* e, const HyLayer& l, int T, const LinOut& 
       XB_TRY(hy_launch(e, hy_attn_window_kernel<KT, float, 16>, dim3(T, H), dim3(32 * aw), asm_bytes, st, QA, 0, -1, (const KT*)l.k_pool,
                        (const KT*)l.k_pool, m, H, 1, W, R, W, W, far, 0, c.m_scale, 1.0f, hy->o, (long long)H * R, AttnOpt{nullptr, 0.f, 1, 0}));
   }
+  if (tiles)
+    return hy_launch(e, hy_head_mm_mma_kernel, dim3((T + HY_HG_M - 1) / HY_HG_M, H, (dv + HY_HG_N - 1) / HY_HG_N), dim3(128), 0, st, (const float*)hy->o,
+                     (long long)H * R, (const bf16*)l.w_uv, (bf16*)hy->a1, (long long)l.n_o, T, R, dv, P, c.m_gate ? l.off_g : -1);
   return hy_launch(e, hy_head_mm_kernel<AT>, dim3((T + HY_MM_ROWS - 1) / HY_MM_ROWS, H), dim3(128), mm2, st, (const float*)hy->o,
                    (long long)H * R, (const bf16*)l.w_uv, a1, (long long)l.n_o, T, R, dv, P, c.m_gate ? l.off_g : -1);
 }
@@ -1417,6 +1426,10 @@ static int hy_router(xb_engine* e, const HyLayer& l, int T, const void* xin, int
   }
   if (T <= 64) {   // few rows: a warp per (token, expert)
     XB_TRY(hy_launch(e, hy_router_logits_kernel<AT, 1>, dim3((unsigned)(((long long)T * NE + 7) / 8)), dim3(256), 0, st, x, (long long)D,
+                     (const bf16*)l.w_router, hy->m2, T, NE, D));
+  } else if (NE > 8 && NE % 8 == 1) {   // one row more than a multiple of eight
+    const int chunks = (NE + 8) / 9;
+    XB_TRY(hy_launch(e, hy_router_logits_kernel<AT, 9>, dim3((unsigned)(((long long)T * chunks + 7) / 8)), dim3(256), 0, st, x, (long long)D,
                      (const bf16*)l.w_router, hy->m2, T, NE, D));
   } else {
     const int chunks = (NE + 7) / 8;
@@ -1730,6 +1743,19 @@ static int hy_run_branchnorm_t(xb_engine* e, int T, int n_seqs, int n_tiles, voi
   return with_head ? hy_run_head<AT>(e, n_seqs, m, st) : 0;
 }
 
+// per-head norm of a recurrence's read-out, weighted and gated (gate_sigmoid 0: SiLU) -> a Linear input
+template <typename AT>
+static int hy_head_norm(xb_engine* e, int T, long long ldo, const float* w, const LinOut& P, int off_gate, AT* out, long long ld_out, int H, int dv,
+                        int w_hstride, int gate_sigmoid, cudaStream_t st) {
+  const int per = dv / 8;
+  if (T > 64 && off_gate >= 0 && P.h != nullptr && P.bias == nullptr && P.ld % 8 == 0 && off_gate % 8 == 0 && dv % 8 == 0 && per <= 32 && (per & (per - 1)) == 0 &&
+      ldo % 8 == 0 && ld_out % 8 == 0)
+    return hy_launch(e, hy_head_norm_vec_kernel<AT>, dim3((unsigned)(((long long)T * H * per + 255) / 256)), dim3(256), 0, st, (const float*)e->hy->o, ldo, w,
+                     P.h + off_gate, P.ld, e->hy->d.norm_eps, out, ld_out, H, dv, w_hstride, gate_sigmoid, T);
+  return hy_launch(e, hy_head_norm_kernel<AT>, dim3(T, (H + 7) / 8), dim3(256), 0, st, (const float*)e->hy->o, ldo, w, P, off_gate, e->hy->d.norm_eps, 1.0f,
+                   out, ld_out, H, dv, w_hstride, gate_sigmoid);
+}
+
 // ----------------------------------------------------------------------------- pre-norm blocks
 // x <- embed * scale;  per layer  x += mixer(f1(x)),  x += ff(f2(x)).  Every norm rides in the kernel that last changed x: the
 // embedding kernel makes the first layer's, the residual additions the next reader's.  The tanh norm needs no statistics of the row
@@ -1801,8 +1827,7 @@ static int hy_run_prenorm_t(xb_engine* e, int T, int n_seqs, void* const* taps, 
       in.c = hy->c; in.ldc = ldc; in.qoff = 0; in.koff = HK; in.xoff[0] = 2LL * HK; in.xoff[1] = in.xoff[2] = 0; in.voff = 3LL * HK; in.q_heads = H;
       in.beta = in.decay = in.qk = in.hdecay = nullptr;
       XB_TRY(hy_recur<HY_REC_GLA>(e, in, hy->state + l.st_rec, SS, hy->o, (long long)l.n_o, m, n_seqs, H, n, dv, T, st));
-      XB_TRY(hy_launch(e, hy_head_norm_kernel<AT>, dim3(T, (H + 7) / 8), dim3(256), 0, st, (const float*)hy->o, (long long)l.n_o,
-                       (const float*)l.head_norm, P, l.off_g, d.norm_eps, 1.0f, a1, (long long)l.n_o, H, dv, 0, 0));
+      XB_TRY(hy_head_norm<AT>(e, T, (long long)l.n_o, (const float*)l.head_norm, P, l.off_g, a1, (long long)l.n_o, H, dv, 0, 0, st));
     }
     XB_TRY(hy_linear<AT>(e, a1, l.n_o, l.w_o, l.t_o, nullptr, T, D, l.n_o, hy->m1, hy->cap_m, st, &y1));
     if (has_ff) {

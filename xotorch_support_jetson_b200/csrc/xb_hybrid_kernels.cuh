@@ -1401,6 +1401,35 @@ __global__ void __launch_bounds__(256) hy_head_norm_kernel(const float* __restri
   }
 }
 
+// The same for prompts whose gate is part of one bf16 matrix: eight neighbouring channels per thread, dv / 8 (a power of two up to 32)
+// neighbouring lanes per head.  off_gate, the pitches and dv are multiples of 8; no bias.  grid ceil(T * H * dv / 8 / 256), 256 threads.
+template <typename AT>
+__global__ void __launch_bounds__(256) hy_head_norm_vec_kernel(const float* __restrict__ o, long long ldo, const float* __restrict__ w, const bf16* __restrict__ g,
+                                                               long long ldg, float eps, AT* __restrict__ out, long long ld_out, int H, int dv,
+                                                               int w_hstride, int gate_sigmoid, int T) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int per = dv >> 3;
+  const long long idx = (long long)blockIdx.x * 256 + threadIdx.x, n = (long long)T * H * per;
+  const bool live = idx < n;
+  const long long th = (live ? idx : n - 1) / per;
+  const int j = (int)((live ? idx : n - 1) - th * per) << 3;
+  const long long t = th / H;
+  const int h = (int)(th - t * H);
+  float v[8], wv[8], gv[8];
+  hy_ld8f(o + t * ldo + (long long)h * dv + j, v);
+  hy_load8(g + t * ldg + (long long)h * dv + j, nullptr, gv);
+  hy_ld8f(w + (long long)h * w_hstride + j, wv);
+  float ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < 8; ++i) ss = fmaf(v[i], v[i], ss);
+  for (int off = per >> 1; off > 0; off >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, off);   // per divides 32: lanes of a head stay together
+  const float inv = 1.0f / sqrtf(ss / (float)dv + eps);
+#pragma unroll
+  for (int i = 0; i < 8; ++i) v[i] = v[i] * inv * wv[i] * (gate_sigmoid ? hy_sigmoid(gv[i]) : hy_silu(gv[i]));
+  if (live) hy_st8a<AT>(out + t * ld_out + (long long)h * dv + j, v);
+}
+
 // ----------------------------------------------------------------------------- windowed softmax attention
 // Paged pools [n_pages][G][page_tokens][d] of KT (bf16 serving, float in the all-fp32 mode).
 template <typename KT>
@@ -2266,6 +2295,71 @@ __global__ void __launch_bounds__(128) hy_head_mm_kernel(const float* __restrict
   }
 }
 
+// The two per-head products above for prompts, on the tensor cores (hy_head_tile): bf16 queries as the projection left them, the
+// read-out rounded to bf16 like every other Linear input.
+__global__ void __launch_bounds__(128) hy_latent_absorb_mma_kernel(const bf16* __restrict__ Q, long long ldq, int dr, const bf16* __restrict__ W,
+                                                                   float* __restrict__ qa, int H, int T, int K, int N, RotArgs r,
+                                                                   const int* __restrict__ tok_pos) {
+  pdl_launch_dependents();
+  pdl_wait();
+  __shared__ __align__(16) unsigned char sm[HY_HG_SMEM(true)];
+  bf16* As = reinterpret_cast<bf16*>(sm);
+  const int t0 = blockIdx.x * HY_HG_M, h = blockIdx.y, n0 = blockIdx.z * HY_HG_N, ld = N + dr;
+  const int nt = T - t0 < HY_HG_M ? T - t0 : HY_HG_M;
+  const bf16* qh = Q + (long long)t0 * ldq + (long long)h * (K + dr);
+  float acc[HY_HG_N / 8][4];
+  hy_head_tile<bf16, true>(qh, ldq, nt, W + (long long)h * K * N, n0, K, N, As, As + HY_HG_M * (HY_HG_K + 8), acc);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+#pragma unroll
+  for (int j = 0; j < 2; ++j) {
+    const int row = warp * 16 + (lane >> 2) + 8 * j;
+    if (row >= nt) continue;
+    float* dst = qa + ((long long)(t0 + row) * H + h) * ld + n0 + (lane & 3) * 2;
+#pragma unroll
+    for (int n = 0; n < HY_HG_N / 8; ++n)
+      if (n0 + n * 8 < N) *reinterpret_cast<float2*>(dst + n * 8) = make_float2(acc[n][2 * j], acc[n][2 * j + 1]);
+  }
+  if (blockIdx.z != 0) return;
+  const int half = r.dims >> 1, per = dr - half;
+  for (int u = threadIdx.x; u < nt * per; u += 128) {
+    const int rr = u / per, i = u - rr * per;
+    const bf16* src = qh + (long long)rr * ldq + K;
+    float* qd = qa + ((long long)(t0 + rr) * H + h) * ld + N;
+    if (i < half) {
+      const int d0 = r.half ? i : 2 * i, d1 = r.half ? i + half : 2 * i + 1;
+      const float a = bf2f(src[d0]), b = bf2f(src[d1]);
+      float cs, sn;
+      hy_rot_cs(r, tok_pos[t0 + rr], i, &cs, &sn);
+      qd[d0] = a * cs - b * sn;
+      qd[d1] = b * cs + a * sn;
+    } else {
+      qd[half + i] = bf2f(src[half + i]);
+    }
+  }
+}
+__global__ void __launch_bounds__(128) hy_head_mm_mma_kernel(const float* __restrict__ x, long long ldx, const bf16* __restrict__ W, bf16* __restrict__ y,
+                                                             long long ldy, int T, int K, int N, LinOut G, int off_gate) {
+  pdl_launch_dependents();
+  pdl_wait();
+  __shared__ __align__(16) unsigned char sm[HY_HG_SMEM(false)];
+  bf16* As = reinterpret_cast<bf16*>(sm);
+  const int t0 = blockIdx.x * HY_HG_M, h = blockIdx.y, n0 = blockIdx.z * HY_HG_N;
+  const int nt = T - t0 < HY_HG_M ? T - t0 : HY_HG_M;
+  float acc[HY_HG_N / 8][4];
+  hy_head_tile<float, false>(x + (long long)t0 * ldx + (long long)h * K, ldx, nt, W + (long long)h * N * K, n0, K, N, As, As + HY_HG_M * (HY_HG_K + 8), acc);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+#pragma unroll
+  for (int j = 0; j < 2; ++j) {
+    const int row = warp * 16 + (lane >> 2) + 8 * j;
+    if (row >= nt) continue;
+    const float g = off_gate >= 0 ? hy_sigmoid(lin_at(G, t0 + row, off_gate + h)) : 1.0f;
+    bf16* dst = y + (long long)(t0 + row) * ldy + (long long)h * N + n0 + (lane & 3) * 2;
+#pragma unroll
+    for (int n = 0; n < HY_HG_N / 8; ++n)
+      if (n0 + n * 8 < N) *reinterpret_cast<uint32_t*>(dst + n * 8) = f2_to_bf2(acc[n][2 * j] * g, acc[n][2 * j + 1] * g);
+  }
+}
+
 // The read-out of all heads normed as ONE vector (RMS over the n entries of a token), weighted and gated by sigmoid:
 // out[t, i] = o[t, i] / rms(o[t, :]) * w[i] * sigmoid(P[t, off_gate + i]).  grid (T), 256 threads.
 template <typename AT>
@@ -2353,7 +2447,7 @@ __global__ void __launch_bounds__(256) hy_gla_prep_kernel(LinOut P, int off_q, i
                                                           long long ldc, int HK, int HV, int T) {
   pdl_launch_dependents();
   pdl_wait();
-  extern __shared__ float as[];
+  extern __shared__ __align__(16) float as[];
   const int t0 = blockIdx.x * ROWS;
   const int nt = T - t0 < ROWS ? T - t0 : ROWS;
   for (int i = threadIdx.x; i < ROWS * rk; i += 256) {
@@ -2361,7 +2455,7 @@ __global__ void __launch_bounds__(256) hy_gla_prep_kernel(LinOut P, int off_q, i
     as[i] = r < nt ? lin_at(P, t0 + r, off_a + k) : 0.f;
   }
   __syncthreads();
-  const int i = blockIdx.y * 256 + threadIdx.x;
+  const int i0 = blockIdx.y * 256, i = i0 + threadIdx.x;
   if (i < HK) {
     float z[ROWS];
     const float b = b2[i];
@@ -2373,9 +2467,12 @@ __global__ void __launch_bounds__(256) hy_gla_prep_kernel(LinOut P, int off_q, i
         float wv[8];
         hy_load8(wr + k, nullptr, wv);
 #pragma unroll
-        for (int r = 0; r < ROWS; ++r)
+        for (int r = 0; r < ROWS; ++r) {
+          float av[8];
+          hy_ld8f(as + r * rk + k, av);
 #pragma unroll
-          for (int j = 0; j < 8; ++j) z[r] = fmaf(wv[j], as[r * rk + k + j], z[r]);
+          for (int j = 0; j < 8; ++j) z[r] = fmaf(wv[j], av[j], z[r]);
+        }
       }
     } else {
       for (int k = 0; k < rk; ++k) {
@@ -2385,20 +2482,33 @@ __global__ void __launch_bounds__(256) hy_gla_prep_kernel(LinOut P, int off_q, i
       }
     }
 #pragma unroll
-    for (int r = 0; r < ROWS; ++r) {
-      if (r >= nt) break;
-      float* row = c + (long long)(t0 + r) * ldc;
+    for (int r = 0; r < ROWS; ++r)
+      if (r < nt) c[(long long)(t0 + r) * ldc + 2LL * HK + i] = expf(-(fmaxf(-z[r], 0.f) + log1pf(expf(-fabsf(z[r])))) * inv_tau);
+  }
+  // q, k, v of the block's channels: from one bf16 matrix (prompts) eight neighbours per thread
+  const bool vec = P.h != nullptr && P.bias == nullptr && ((P.ld | off_q | off_k | off_v | ldc | HK | HV) & 7) == 0;
+  if (vec) {
+    for (int u = threadIdx.x; u < nt * 96; u += 256) {
+      const int r = u / 96, x = u - r * 96, part = x >> 5, col = i0 + ((x & 31) << 3);
+      if (col >= (part == 2 ? HV : HK)) continue;
+      float v[8];
+      hy_load8(P.h + (long long)(t0 + r) * P.ld + (part == 0 ? off_q : (part == 1 ? off_k : off_v)) + col, nullptr, v);
+      if (part == 0)
+#pragma unroll
+        for (int j = 0; j < 8; ++j) v[j] *= scale;
+      hy_st8f(c + (long long)(t0 + r) * ldc + (part == 0 ? 0 : (part == 1 ? (long long)HK : 3LL * HK)) + col, v);
+    }
+    return;
+  }
+#pragma unroll
+  for (int r = 0; r < ROWS; ++r) {
+    if (r >= nt) break;
+    float* row = c + (long long)(t0 + r) * ldc;
+    if (i < HK) {
       row[i] = lin_at(P, t0 + r, off_q + i) * scale;
       row[HK + i] = lin_at(P, t0 + r, off_k + i);
-      row[2 * HK + i] = expf(-(fmaxf(-z[r], 0.f) + log1pf(expf(-fabsf(z[r])))) * inv_tau);
     }
-  }
-  if (i < HV) {
-#pragma unroll
-    for (int r = 0; r < ROWS; ++r) {
-      if (r >= nt) break;
-      c[(long long)(t0 + r) * ldc + 3LL * HK + i] = lin_at(P, t0 + r, off_v + i);
-    }
+    if (i < HV) row[3LL * HK + i] = lin_at(P, t0 + r, off_v + i);
   }
 }
 
@@ -2490,10 +2600,13 @@ __global__ void hy_moe_act_vec_kernel(const bf16* __restrict__ u, long long ld, 
   *reinterpret_cast<uint4*>(out + t * ld_out + i) = r;
 }
 
+template <typename AT> __device__ __forceinline__ void act_load8(const AT* p, float* v);   // eight neighbours; p 16-byte aligned
+template <> __device__ __forceinline__ void act_load8<float>(const float* p, float* v) { hy_ld8f(p, v); }
+template <> __device__ __forceinline__ void act_load8<bf16>(const bf16* p, float* v) { hy_load8(p, nullptr, v); }
 // Router logits in fp32 for any number of rows: z[t, e] = sum_k x[t, k] w[e, k].  A warp takes one token and up to eight
 // experts: it reads the token's row once and streams eight weight rows (which stay in L1 / L2 across tokens).
 // grid (ceil(T * ceil(E / 8) / 8)), 256 threads.
-// EPW: experts per warp, 8 for prompts; 1 in steps of few rows, where T * E warps are what fills the GPU.
+// EPW: experts per warp, 8 for prompts (9 where that saves a pass over the rows); 1 in steps of few rows, where T * E warps are what fills the GPU.
 template <typename AT, int EPW>
 __global__ void __launch_bounds__(256) hy_router_logits_kernel(const AT* __restrict__ x, long long ldx, const bf16* __restrict__ w,
                                                                float* __restrict__ z, int T, int E, int K) {
@@ -2513,8 +2626,7 @@ __global__ void __launch_bounds__(256) hy_router_logits_kernel(const AT* __restr
   if ((K & 7) == 0 && (reinterpret_cast<uintptr_t>(w) & 15) == 0) {
     for (int k = lane * 8; k < K; k += 256) {
       float xv[8];
-#pragma unroll
-      for (int i = 0; i < 8; ++i) xv[i] = act_load<AT>(xr + k + i);
+      act_load8<AT>(xr + k, xv);
 #pragma unroll
       for (int j = 0; j < EPW; ++j) {
         if (j < ne) {
@@ -2646,10 +2758,11 @@ __global__ void __launch_bounds__(256) hy_router_route_kernel(const AT* __restri
     float acc = 0.f;
     if (vec) {
       for (int k = lane * 8; k < K; k += 256) {
-        float wv[8];
+        float wv[8], xv[8];
         hy_load8(wr + k, nullptr, wv);
+        act_load8<AT>(xr + k, xv);
 #pragma unroll
-        for (int i = 0; i < 8; ++i) acc = fmaf(act_load<AT>(xr + k + i), wv[i], acc);
+        for (int i = 0; i < 8; ++i) acc = fmaf(xv[i], wv[i], acc);
       }
     } else {
       for (int k = lane; k < K; k += 32) acc = fmaf(act_load<AT>(xr + k), bf2f(wr[k]), acc);
@@ -2766,8 +2879,7 @@ __global__ void __launch_bounds__(256) hy_moe_gather_up_kernel(const AT* __restr
     float g = 0.f, u = 0.f;
     for (int k = lane * 8; k < D; k += 256) {
       float xv[8], a[8], b[8];
-#pragma unroll
-      for (int i = 0; i < 8; ++i) xv[i] = act_load<AT>(xr + k + i);
+      act_load8<AT>(xr + k, xv);
       hy_load8(wg + k, nullptr, a);
       hy_load8(wu + k, nullptr, b);
 #pragma unroll
@@ -2797,10 +2909,11 @@ __global__ void __launch_bounds__(256) hy_moe_gather_down_kernel(const AT* __res
   float acc = 0.f;
   auto add = [&](const AT* ar, const bf16* wr, int n) {
     for (int k = lane * 8; k < n; k += 256) {
-      float w[8];
+      float w[8], av[8];
       hy_load8(wr + k, nullptr, w);
+      act_load8<AT>(ar + k, av);
 #pragma unroll
-      for (int i = 0; i < 8; ++i) acc = fmaf(act_load<AT>(ar + k + i), w[i], acc);
+      for (int i = 0; i < 8; ++i) acc = fmaf(av[i], w[i], acc);
     }
   };
   int j = 0;

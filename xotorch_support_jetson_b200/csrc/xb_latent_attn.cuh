@@ -250,3 +250,72 @@ __global__ void __launch_bounds__(128) hy_latent_merge_kernel(const float* __res
     out[(long long)t * ld_out + (long long)h * R + c] = acc * inv;
   }
 }
+
+// ----------------------------------------------------------------------------- per-head products around the attention, prompts
+// y[t, h, :] = x[t, h, :] W_h for every head on the tensor cores (mma.sync, bf16 operands, fp32 accumulation), a 64-token x 128-column
+// tile of one head per block, K in slices of 64.
+//   x: bf16 rows (XT = bf16) or fp32 rows rounded on the way into shared memory; head h starts at column h * xh
+//   W: KMAJOR ? [h][K][N] (a query folded into the latent space) : [h][N][K] (a latent read-out turned into values)
+// K and N are multiples of 8, row pitches multiples of 8 (bf16) / 4 (fp32).
+// grid (ceil(T / 64), H, ceil(N / 128)), 128 threads.
+#define HY_HG_M 64
+#define HY_HG_N 128
+#define HY_HG_K 64
+template <typename XT, bool KMAJOR>
+__device__ __forceinline__ void hy_head_tile(const XT* __restrict__ x, long long ldx, int nt, const bf16* __restrict__ w, int n0, int K, int N,
+                                             bf16* As, bf16* Bs, float (&acc)[HY_HG_N / 8][4]) {
+  constexpr int PA = HY_HG_K + 8, PB = KMAJOR ? HY_HG_N + 8 : HY_HG_K + 8;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+#pragma unroll
+  for (int n = 0; n < HY_HG_N / 8; ++n) acc[n][0] = acc[n][1] = acc[n][2] = acc[n][3] = 0.f;
+  for (int k0 = 0; k0 < K; k0 += HY_HG_K) {
+    __syncthreads();
+    for (int u = threadIdx.x; u < HY_HG_M * (HY_HG_K / 8); u += 128) {
+      const int r = u >> 3, k = k0 + ((u & 7) << 3);
+      uint4 v = make_uint4(0u, 0u, 0u, 0u);
+      if (r < nt && k < K) {
+        const XT* p = x + (long long)r * ldx + k;
+        if constexpr (sizeof(XT) == 2) {
+          v = *reinterpret_cast<const uint4*>(p);
+        } else {
+          const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
+          v = make_uint4(f2_to_bf2(a.x, a.y), f2_to_bf2(a.z, a.w), f2_to_bf2(b.x, b.y), f2_to_bf2(b.z, b.w));
+        }
+      }
+      *reinterpret_cast<uint4*>(As + r * PA + (k - k0)) = v;
+    }
+    if (KMAJOR) {
+      for (int u = threadIdx.x; u < HY_HG_K * (HY_HG_N / 8); u += 128) {
+        const int k = u >> 4, n = (u & 15) << 3;
+        const bool ok = k0 + k < K && n0 + n < N;
+        lat_cp16(smem_u32(Bs + k * PB + n), ok ? w + (long long)(k0 + k) * N + n0 + n : w, ok ? 16 : 0);
+      }
+    } else {
+      for (int u = threadIdx.x; u < HY_HG_N * (HY_HG_K / 8); u += 128) {
+        const int n = u >> 3, k = (u & 7) << 3;
+        const bool ok = k0 + k < K && n0 + n < N;
+        lat_cp16(smem_u32(Bs + n * PB + k), ok ? w + (long long)(n0 + n) * K + k0 + k : w, ok ? 16 : 0);
+      }
+    }
+    lat_cp_commit();
+    lat_cp_wait<0>();
+    __syncthreads();
+    const uint32_t aaddr = smem_u32(As + (warp * 16 + (lane & 15)) * PA + (lane >> 4) * 8);
+#pragma unroll
+    for (int ks = 0; ks < HY_HG_K; ks += 16) {
+      uint32_t a[4];
+      ldsm_x4(aaddr + ks * 2, a[0], a[1], a[2], a[3]);
+#pragma unroll
+      for (int n = 0; n < HY_HG_N / 8; n += 2) {
+        uint32_t b0, b1, b2, b3;
+        if (KMAJOR)
+          ldsm_x4_t(smem_u32(Bs + (ks + (lane & 7) + ((lane >> 3) & 1) * 8) * PB + n * 8 + ((lane >> 4) & 1) * 8), b0, b1, b2, b3);
+        else
+          ldsm_x4(smem_u32(Bs + (n * 8 + (lane & 7) + ((lane >> 4) & 1) * 8) * PB + ks + ((lane >> 3) & 1) * 8), b0, b1, b2, b3);
+        mma_bf16_16816(acc[n], a, b0, b1);
+        mma_bf16_16816(acc[n + 1], a, b2, b3);
+      }
+    }
+  }
+}
+#define HY_HG_SMEM(KMAJOR) ((HY_HG_M * (HY_HG_K + 8) + ((KMAJOR) ? HY_HG_K * (HY_HG_N + 8) : HY_HG_N * (HY_HG_K + 8))) * 2)
