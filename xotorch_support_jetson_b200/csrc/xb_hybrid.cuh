@@ -1070,11 +1070,11 @@ static int hy_recur_l(xb_engine* e, const RecurIn& in, float* state, long long s
 }
 // Prompts through the segments of hy_seg_kernel (modes whose step fades a state column entry by entry).  Segments of 128 tokens, of
 // 64 when 128 would leave the SMs with fewer than four blocks each.
-template <int NCH, int NCOL, int MODE>
+template <int NCH, int LPC, int MODE>
 static int hy_segments_n(xb_engine* e, const RecurIn& in, float* state, long long ss, float* o, long long ldo, const BatchMeta& m, int n_seqs,
                          int H, int dk, int dv, int T, cudaStream_t st) {
   HyModel* hy = e->hy;
-  const int cb = (dv + 32 * NCOL - 1) / (32 * NCOL);
+  const int cb = (dv + HY_SEG_COLS - 1) / HY_SEG_COLS;
   SegArgs sg;
   sg.seg = hy->seg_len > 0 ? hy->seg_len : ((long long)(T / 128) * H * cb >= 4LL * e->num_sms ? 128 : HY_SEG_MIN);
   sg.max_segs = (T + sg.seg - 1) / sg.seg;
@@ -1082,24 +1082,28 @@ static int hy_segments_n(xb_engine* e, const RecurIn& in, float* state, long lon
   sg.decay = MODE == HY_REC_LIGHTNING ? nullptr : hy->seg_decay;
   const dim3 grid(cb, H, n_seqs * sg.max_segs);
   constexpr size_t row = (size_t)2 * HY_SEG_TS * sizeof(float);
-  constexpr size_t s0 = row * (hy_seg_vectors(MODE, 0) * 16 * NCH + 32 * NCOL), s1 = row * (hy_seg_vectors(MODE, 1) * 16 * NCH + 32 * NCOL);
-  if (s0 > 48 * 1024) XB_SMEM_ATTR_ONCE((hy_seg_kernel<NCH, NCOL, MODE, 0>), s0);
-  if (s1 > 48 * 1024) XB_SMEM_ATTR_ONCE((hy_seg_kernel<NCH, NCOL, MODE, 1>), s1);
-  XB_TRY(hy_launch(e, hy_seg_kernel<NCH, NCOL, MODE, 0>, grid, dim3(128), s0, st, in, sg, state, ss, o, ldo, m, H, dk, dv));
+  constexpr size_t s0 = row * (hy_seg_vectors(MODE, 0) * 4 * LPC * NCH + HY_SEG_COLS), s1 = row * (hy_seg_vectors(MODE, 1) * 4 * LPC * NCH + HY_SEG_COLS);
+  if (s0 > 48 * 1024) XB_SMEM_ATTR_ONCE((hy_seg_kernel<NCH, LPC, MODE, 0>), s0);
+  if (s1 > 48 * 1024) XB_SMEM_ATTR_ONCE((hy_seg_kernel<NCH, LPC, MODE, 1>), s1);
+  XB_TRY(hy_launch(e, hy_seg_kernel<NCH, LPC, MODE, 0>, grid, dim3(128), s0, st, in, sg, state, ss, o, ldo, m, H, dk, dv));
   if (sg.decay != nullptr)
     XB_TRY(hy_launch(e, hy_seg_decay_kernel, dim3((H * dk + 255) / 256, n_seqs * sg.max_segs), dim3(256), 0, st, in.c, in.ldc,
                      MODE == HY_REC_GLA ? in.xoff[0] : in.koff, H * dk, sg.seg, sg.max_segs, hy->seg_decay, m));
-  XB_TRY(hy_launch(e, hy_seg_scan_kernel, dim3((dv * dk + 255) / 256, H, n_seqs), dim3(256), 0, st, sg, in.hdecay, (const float*)state, ss, m, H, dk, dv));
-  return hy_launch(e, hy_seg_kernel<NCH, NCOL, MODE, 1>, grid, dim3(128), s1, st, in, sg, state, ss, o, ldo, m, H, dk, dv);
+  if (dk % 4 == 0)
+    XB_TRY(hy_launch(e, hy_seg_scan_kernel<4>, dim3((dv * dk / 4 + 127) / 128, H, n_seqs), dim3(128), 0, st, sg, in.hdecay, (const float*)state, ss, m, H, dk, dv));
+  else
+    XB_TRY(hy_launch(e, hy_seg_scan_kernel<1>, dim3((dv * dk + 127) / 128, H, n_seqs), dim3(128), 0, st, sg, in.hdecay, (const float*)state, ss, m, H, dk, dv));
+  return hy_launch(e, hy_seg_kernel<NCH, LPC, MODE, 1>, grid, dim3(128), s1, st, in, sg, state, ss, o, ldo, m, H, dk, dv);
 }
 template <int MODE>
 static int hy_segments(xb_engine* e, const RecurIn& in, float* state, long long ss, float* o, long long ldo, const BatchMeta& m, int n_seqs,
                        int H, int dk, int dv, int T, cudaStream_t st) {
-  if (dk <= 16) return hy_segments_n<1, 2, MODE>(e, in, state, ss, o, ldo, m, n_seqs, H, dk, dv, T, st);
-  if (dk <= 32) return hy_segments_n<2, 2, MODE>(e, in, state, ss, o, ldo, m, n_seqs, H, dk, dv, T, st);
-  if (dk <= 64) return hy_segments_n<4, 2, MODE>(e, in, state, ss, o, ldo, m, n_seqs, H, dk, dv, T, st);
-  if (dk <= 128) return hy_segments_n<8, 2, MODE>(e, in, state, ss, o, ldo, m, n_seqs, H, dk, dv, T, st);
-  return hy_segments_n<16, 1, MODE>(e, in, state, ss, o, ldo, m, n_seqs, H, dk, dv, T, st);
+  // sixteen lanes per group of columns read less shared memory, eight pad small key dims less
+  if (dk <= 32) return hy_segments_n<1, 8, MODE>(e, in, state, ss, o, ldo, m, n_seqs, H, dk, dv, T, st);
+  if (dk <= 64) return hy_segments_n<2, 8, MODE>(e, in, state, ss, o, ldo, m, n_seqs, H, dk, dv, T, st);
+  if (dk <= 128) return hy_segments_n<2, 16, MODE>(e, in, state, ss, o, ldo, m, n_seqs, H, dk, dv, T, st);
+  if (dk <= 256) return hy_segments_n<4, 16, MODE>(e, in, state, ss, o, ldo, m, n_seqs, H, dk, dv, T, st);
+  return xb_fail(1, "recurrent key dim %d exceeds %d", dk, HY_MAX_KDIM);
 }
 
 template <int MODE>

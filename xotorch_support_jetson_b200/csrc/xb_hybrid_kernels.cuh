@@ -1103,11 +1103,13 @@ __global__ void __launch_bounds__(128) hy_recur_kernel(RecurIn in, float* __rest
 // Workspace ws: one state [H][dv][dk] per segment; segment c of sequence s sits at entry start_row / seg + s + c (ceilings of earlier
 // sequences add up to no more than that).
 //
-// Four lanes own NCOL value columns: lane `sub` holds the rows of the 16-byte chunks sub, sub + 4, ... of each, as pairs for the packed
-// two-wide fp32 FMA.  A block's 4 warps share (segment, head) and 32 * NCOL columns; the inputs of HY_SEG_TS steps arrive in
-// shared memory by cp.async, one chunk of steps ahead.
-// grid (ceil(dv / (32 NCOL)), H, n_seqs * max_segs), 128 threads.
+// LPC lanes own LPC / 2 value columns: lane `sub` holds the rows of the 16-byte chunks sub, sub + LPC, ... of each, as pairs for the
+// packed two-wide fp32 FMA.  Shared-memory reads bound this kernel: a row vector read once serves all of a lane's columns, so more
+// lanes with fewer rows and more columns each read less (with the state's registers the same).  A block's 4 warps share
+// (segment, head) and 64 columns; the inputs of HY_SEG_TS steps arrive in shared memory by cp.async, one chunk of steps ahead.
+// grid (ceil(dv / 64), H, n_seqs * max_segs), 128 threads.
 #define HY_SEG_TS 8
+#define HY_SEG_COLS 64
 typedef unsigned long long hy_f2;
 __device__ __forceinline__ hy_f2 hy_f2_pack(float a, float b) {
   hy_f2 r;
@@ -1137,20 +1139,20 @@ struct SegArgs {
 // row vectors staged per step: k (or f), w where it is a vector of its own, q in the output pass
 __host__ __device__ constexpr int hy_seg_vectors(int mode, int pass) { return 1 + (mode == HY_REC_GLA ? 1 : 0) + (pass == 1 ? 1 : 0); }
 
-template <int NCH, int NCOL, int MODE, int PASS>
+template <int NCH, int LPC, int MODE, int PASS>
 __global__ void __launch_bounds__(128) hy_seg_kernel(RecurIn in, SegArgs sg, float* __restrict__ state, long long state_stride, float* __restrict__ o,
                                                      long long ldo, BatchMeta m, int H, int dk, int dv) {
   pdl_wait();
   extern __shared__ __align__(16) float stg[];
-  constexpr int NV = hy_seg_vectors(MODE, PASS), DKP = 16 * NCH, NB = 32 * NCOL, VO = NV * DKP, STRIDE = VO + NB;
+  constexpr int NV = hy_seg_vectors(MODE, PASS), NCOL = LPC / 2, DKP = 4 * LPC * NCH, NB = HY_SEG_COLS, VO = NV * DKP, STRIDE = VO + NB;
   const int s = blockIdx.z / sg.max_segs, c = blockIdx.z - s * sg.max_segs, h = blockIdx.y, j0 = blockIdx.x * NB;
   const SeqSpan sp = seq_span(m, s);
   const int nseg = (sp.len + sg.seg - 1) / sg.seg;
   if (c >= nseg || (PASS == 0 && c == nseg - 1)) return;
   const int row0 = sp.start + c * sg.seg, len = sp.len - c * sg.seg < sg.seg ? sp.len - c * sg.seg : sg.seg;
   float* entry = sg.ws + (long long)(sp.start / sg.seg + s + c) * H * dv * dk;
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, sub = lane & 3;
-  const int jl = (warp * 8 + (lane >> 2)) * NCOL, ncv = dv - j0 < NB ? dv - j0 : NB;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, sub = lane & (LPC - 1);
+  const int jl = (warp * (32 / LPC) + lane / LPC) * NCOL, ncv = dv - j0 < NB ? dv - j0 : NB;
   // staged vectors in the order of the shared rows: k, (w), (q)
   const float* src[NV];
   src[0] = in.c + in.koff + (long long)h * dk;
@@ -1161,6 +1163,10 @@ __global__ void __launch_bounds__(128) hy_seg_kernel(RecurIn in, SegArgs sg, flo
   bool al = ((in.ldc | in.qoff | in.koff | in.voff | dk | dv) & 3) == 0 && (reinterpret_cast<uintptr_t>(in.c) & 15) == 0;
   if (MODE == HY_REC_GLA) al = al && (in.xoff[0] & 3) == 0;
   for (int i = threadIdx.x; i < 2 * HY_SEG_TS * STRIDE; i += 128) stg[i] = 0.f;   // padding rows / columns stay zero
+  int col = 0;   // the column whose sum ends up in this lane
+#pragma unroll
+  for (int off = 1; off < NCOL; off <<= 1) col += (sub & off) ? NCOL / (2 * off) : 0;
+  const bool writer = sub < LPC / 2 && jl + col < ncv;
   hy_f2 S[NCOL][2 * NCH];
   const bool st_al = (dk & 3) == 0;   // entries start on 16-byte boundaries when every column does
 #pragma unroll
@@ -1169,7 +1175,7 @@ __global__ void __launch_bounds__(128) hy_seg_kernel(RecurIn in, SegArgs sg, flo
     const float* st = entry + ((long long)h * dv + j0 + jl + n) * dk;
 #pragma unroll
     for (int ch = 0; ch < NCH; ++ch) {
-      const int r = (ch * 4 + sub) * 4;
+      const int r = (ch * LPC + sub) * 4;
       if (have && st_al && r < dk) {
         const ulonglong2 v = *reinterpret_cast<const ulonglong2*>(st + r);
         S[n][2 * ch] = v.x; S[n][2 * ch + 1] = v.y;
@@ -1183,30 +1189,32 @@ __global__ void __launch_bounds__(128) hy_seg_kernel(RecurIn in, SegArgs sg, flo
   }
   __syncthreads();
   auto stage = [&](int t0, float* buf) {
+    // a thread copies the same piece of every step's row, so its addresses advance by the row pitch alone
     const int nt = len - t0 < HY_SEG_TS ? len - t0 : HY_SEG_TS;
-    if (al) {
-      const int dq = dk >> 2, per = NV * dq + (ncv >> 2);
-      for (int idx = threadIdx.x; idx < nt * per; idx += 128) {
-        const int ts = idx / per, u = idx - ts * per;
-        const long long row = (long long)(row0 + t0 + ts) * in.ldc;
-        float* d = buf + ts * STRIDE;
-        bool done = false;
+    const int w = al ? 4 : 1, dq = dk / w, per = NV * dq + ncv / w;
+    for (int u = threadIdx.x; u < per; u += 128) {
+      const int v = u / dq;
+      const float* p;
+      float* d = buf;
+      if (v < NV) {
+        p = src[0];
 #pragma unroll
-        for (int v = 0; v < NV; ++v)
-          if (!done && u < (v + 1) * dq) { hy_cp16(d + v * DKP + 4 * (u - v * dq), src[v] + row + 4 * (u - v * dq)); done = true; }
-        if (!done) hy_cp16(d + VO + 4 * (u - NV * dq), cv + row + 4 * (u - NV * dq));
+        for (int x = 1; x < NV; ++x) p = v == x ? src[x] : p;
+        p += w * (u - v * dq);
+        d += v * DKP + w * (u - v * dq);
+      } else {
+        p = cv + w * (u - NV * dq);
+        d += VO + w * (u - NV * dq);
       }
-    } else {
-      const int per = NV * dk + ncv;
-      for (int idx = threadIdx.x; idx < nt * per; idx += 128) {
-        const int ts = idx / per, u = idx - ts * per;
-        const long long row = (long long)(row0 + t0 + ts) * in.ldc;
-        float* d = buf + ts * STRIDE;
-        bool done = false;
+      p += (long long)(row0 + t0) * in.ldc;
+      if (al && nt == HY_SEG_TS) {
 #pragma unroll
-        for (int v = 0; v < NV; ++v)
-          if (!done && u < (v + 1) * dk) { hy_cp4(d + v * DKP + (u - v * dk), src[v] + row + (u - v * dk)); done = true; }
-        if (!done) hy_cp4(d + VO + (u - NV * dk), cv + row + (u - NV * dk));
+        for (int ts = 0; ts < HY_SEG_TS; ++ts) hy_cp16(d + ts * STRIDE, p + ts * in.ldc);
+      } else {
+        for (int ts = 0; ts < nt; ++ts) {
+          if (al) hy_cp16(d + ts * STRIDE, p + ts * in.ldc);
+          else hy_cp4(d + ts * STRIDE, p + ts * in.ldc);
+        }
       }
     }
     hy_cp_commit();
@@ -1223,14 +1231,14 @@ __global__ void __launch_bounds__(128) hy_seg_kernel(RecurIn in, SegArgs sg, flo
       const float* sr = buf + ts * STRIDE;
       hy_f2 vv[NCOL], acc[NCOL];
 #pragma unroll
-      for (int n = 0; n < NCOL; ++n) {
-        const float v = sr[VO + jl + n];
-        vv[n] = hy_f2_pack(v, v);
-        acc[n] = 0ull;
+      for (int n = 0; n < NCOL; n += 4) {
+        const float4 v = *reinterpret_cast<const float4*>(sr + VO + jl + n);
+        vv[n] = hy_f2_pack(v.x, v.x); vv[n + 1] = hy_f2_pack(v.y, v.y); vv[n + 2] = hy_f2_pack(v.z, v.z); vv[n + 3] = hy_f2_pack(v.w, v.w);
+        acc[n] = acc[n + 1] = acc[n + 2] = acc[n + 3] = 0ull;
       }
 #pragma unroll
       for (int ch = 0; ch < NCH; ++ch) {
-        const int r = (ch * 4 + sub) * 4;
+        const int r = (ch * LPC + sub) * 4;
         const ulonglong2 k4 = *reinterpret_cast<const ulonglong2*>(sr + r);
         hy_f2 k2[2] = {k4.x, k4.y}, w2[2], q2[2] = {0ull, 0ull};
         if (MODE == HY_REC_GLA) {
@@ -1259,16 +1267,25 @@ __global__ void __launch_bounds__(128) hy_seg_kernel(RecurIn in, SegArgs sg, flo
           }
       }
       if (PASS == 1) {
-        float mine = 0.f;
+        // sums over the lanes: partners swap halves of their columns, so that log2(LPC) rounds leave one column per lane pair
+        float y[NCOL];
 #pragma unroll
         for (int n = 0; n < NCOL; ++n) {
           const float2 a = hy_f2_unpack(acc[n]);
-          float b = a.x + a.y;
-          b += __shfl_xor_sync(0xffffffffu, b, 1);
-          b += __shfl_xor_sync(0xffffffffu, b, 2);
-          if (sub == n) mine = b;
+          y[n] = a.x + a.y;
         }
-        if (sub < NCOL && jl + sub < ncv) o[(long long)(row0 + t0 + ts) * ldo + (long long)h * dv + j0 + jl + sub] = mine;
+#pragma unroll
+        for (int off = 1; off < NCOL; off <<= 1) {
+          const int half = NCOL / (2 * off);
+          const bool hi = (sub & off) != 0;
+#pragma unroll
+          for (int n = 0; n < half; ++n) {
+            const float keep = hi ? y[n + half] : y[n], give = hi ? y[n] : y[n + half];
+            y[n] = keep + __shfl_xor_sync(0xffffffffu, give, off);
+          }
+        }
+        const float mine = y[0] + __shfl_xor_sync(0xffffffffu, y[0], LPC / 2);
+        if (writer) o[(long long)(row0 + t0 + ts) * ldo + (long long)h * dv + j0 + jl + col] = mine;
       }
     };
     if (nt == HY_SEG_TS) {
@@ -1288,7 +1305,7 @@ __global__ void __launch_bounds__(128) hy_seg_kernel(RecurIn in, SegArgs sg, flo
     float* st = base + ((long long)h * dv + j0 + jl + n) * dk;
 #pragma unroll
     for (int ch = 0; ch < NCH; ++ch) {
-      const int r = (ch * 4 + sub) * 4;
+      const int r = (ch * LPC + sub) * 4;
       if (out_al && r < dk) {
         *reinterpret_cast<ulonglong2*>(st + r) = make_ulonglong2(S[n][2 * ch], S[n][2 * ch + 1]);
       } else {
@@ -1321,12 +1338,15 @@ __global__ void __launch_bounds__(256) hy_seg_decay_kernel(const float* __restri
   decay[(long long)(sp.start / seg + s + cseg) * HK + i] = (a[0] * a[1]) * (a[2] * a[3]);
 }
 
-// ws entries: local end states -> start states.  A thread owns one state number and walks the segments of its sequence, four loads in
-// flight.  grid (ceil(dv * dk / 256), H, n_seqs), 256 threads.
-__global__ void __launch_bounds__(256) hy_seg_scan_kernel(SegArgs sg, const float* __restrict__ hdecay, const float* __restrict__ state,
+// ws entries: local end states -> start states.  A thread owns VEC neighbouring numbers of the state (VEC = 4 wants dk a multiple of 4) and
+// walks the segments of its sequence, the loads of the next four in flight while it works on these.
+// grid (ceil(dv * dk / VEC / 128), H, n_seqs), 128 threads.
+template <int VEC>
+__global__ void __launch_bounds__(128) hy_seg_scan_kernel(SegArgs sg, const float* __restrict__ hdecay, const float* __restrict__ state,
                                                           long long state_stride, BatchMeta m, int H, int dk, int dv) {
   pdl_wait();
-  const int s = blockIdx.z, h = blockIdx.y, e = blockIdx.x * 256 + threadIdx.x;
+  constexpr int NS = 4;
+  const int s = blockIdx.z, h = blockIdx.y, e = (blockIdx.x * 128 + threadIdx.x) * VEC;
   if (e >= dv * dk) return;
   const SeqSpan sp = seq_span(m, s);
   const int nseg = (sp.len + sg.seg - 1) / sg.seg, i = e % dk;
@@ -1334,20 +1354,46 @@ __global__ void __launch_bounds__(256) hy_seg_scan_kernel(SegArgs sg, const floa
   float* w = sg.ws + e0 * ss + at;
   const float* A = sg.decay != nullptr ? sg.decay + e0 * H * dk + (long long)h * dk + i : nullptr;
   const float hp = sg.decay == nullptr ? powf(hdecay[h], (float)sg.seg) : 1.f;
-  float S = sp.pos0 > 0 ? state[(long long)sp.slot * state_stride + at] : 0.f;
-  for (int c0 = 0; c0 < nseg; c0 += 4) {
-    float L[4], a[4];
+  __align__(16) float S[VEC], L[NS][VEC], a[NS][VEC];
+  const float* st = state + (long long)sp.slot * state_stride + at;
 #pragma unroll
-    for (int x = 0; x < 4; ++x) {
-      const bool in = c0 + x < nseg - 1;
-      L[x] = in ? w[(c0 + x) * ss] : 0.f;
-      a[x] = in ? (A != nullptr ? A[(long long)(c0 + x) * H * dk] : hp) : 0.f;
+  for (int j = 0; j < VEC; ++j) S[j] = sp.pos0 > 0 ? st[j] : 0.f;
+  auto load = [&](int c0) {
+#pragma unroll
+    for (int x = 0; x < NS; ++x) {
+      if (c0 + x >= nseg - 1) continue;   // the last segment's end state is the output pass's own
+      if (VEC == 4) {
+        *reinterpret_cast<float4*>(L[x]) = *reinterpret_cast<const float4*>(w + (c0 + x) * ss);
+        if (A != nullptr) *reinterpret_cast<float4*>(a[x]) = *reinterpret_cast<const float4*>(A + (long long)(c0 + x) * H * dk);
+      } else {
+        L[x][0] = w[(c0 + x) * ss];
+        if (A != nullptr) a[x][0] = A[(long long)(c0 + x) * H * dk];
+      }
+      if (A == nullptr)
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) a[x][j] = hp;
     }
+  };
 #pragma unroll
-    for (int x = 0; x < 4; ++x) {
+  for (int x = 0; x < NS; ++x)
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) L[x][j] = a[x][j] = 0.f;
+  load(0);
+  for (int c0 = 0; c0 < nseg; c0 += NS) {
+    __align__(16) float out[NS][VEC];
+#pragma unroll
+    for (int x = 0; x < NS; ++x)
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) {
+        out[x][j] = S[j];
+        S[j] = fmaf(a[x][j], S[j], L[x][j]);
+      }
+    load(c0 + NS);
+#pragma unroll
+    for (int x = 0; x < NS; ++x) {
       if (c0 + x >= nseg) break;
-      w[(c0 + x) * ss] = S;
-      S = fmaf(a[x], S, L[x]);
+      if (VEC == 4) *reinterpret_cast<float4*>(w + (c0 + x) * ss) = *reinterpret_cast<const float4*>(out[x]);
+      else w[(c0 + x) * ss] = out[x][0];
     }
   }
 }
