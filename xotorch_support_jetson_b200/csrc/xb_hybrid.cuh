@@ -1290,7 +1290,8 @@ static int hy_sublayer_input(xb_engine* e, int T, int n_seqs, bool no_span, cons
 }
 
 static int hy_latent_window(const xb_hybrid_layer& c) { return c.m_window > 0 ? c.m_window : 1 << 30; }
-// Latent attention through hy_latent_attn_mma_kernel.  0: launched; 1: not applicable (shared memory); < 0: -error.
+// Latent attention through hy_latent_attn_mma_kernel.  0: launched; 1: not applicable (shared memory); < 0: -error.  n_splits > 1 leaves
+// the key shares in hy->lat_part.
 template <int WARPS, int DVC, int LOADW, bool EXT>
 static int hy_latent_mma_launch_x(xb_engine* e, const HyLayer& l, const BatchMeta& m, int T, int n_splits, cudaStream_t st) {
   HyModel* hy = e->hy;
@@ -1312,9 +1313,6 @@ static int hy_latent_mma_launch_x(xb_engine* e, const HyLayer& l, const BatchMet
   if (hy_launch(e, hy_latent_attn_mma_kernel<WARPS, DVC, LOADW, EXT>, grid, dim3(32 * LOADW), smem, st, (const float*)hy->qa, (const bf16*)l.k_pool, m, T, H, W,
                 R, c.m_scale * 1.4426950408889634f, n_splits, hy->lat_part, hy->o, (long long)H * R, hy_latent_window(c)) != 0)
     return -1;
-  if (n_splits > 1 &&
-      hy_launch(e, hy_latent_merge_kernel, dim3(NR), dim3(128), 0, st, (const float*)hy->lat_part, n_splits, NR, H, R, hy->o, (long long)H * R) != 0)
-    return -1;
   return 0;
 }
 template <int WARPS, int DVC, int LOADW>
@@ -1322,7 +1320,8 @@ static int hy_latent_mma_launch(xb_engine* e, const HyLayer& l, const BatchMeta&
   if (l.d.m_window > 0) return hy_latent_mma_launch_x<WARPS, DVC, LOADW, true>(e, l, m, T, n_splits, st);
   return hy_latent_mma_launch_x<WARPS, DVC, LOADW, false>(e, l, m, T, n_splits, st);
 }
-static int hy_latent_mma(xb_engine* e, const HyLayer& l, const BatchMeta& m, int T, cudaStream_t st) {
+static int hy_latent_mma(xb_engine* e, const HyLayer& l, const BatchMeta& m, int T, int* n_splits, cudaStream_t st) {
+  *n_splits = 1;
   const int R = l.d.m_kv_rank, NR = T * l.d.m_heads;
   const int tiles4 = (NR + 63) / 64, tiles1 = (NR + 15) / 16;
   const int mode = e->hy->use_lat_mma;
@@ -1335,6 +1334,7 @@ static int hy_latent_mma(xb_engine* e, const HyLayer& l, const BatchMeta& m, int
     const int wt = (l.d.m_window + 15) / HY_LAT_KEYS + 2;
     ns = ns > wt ? wt : ns;
   }
+  *n_splits = ns;
   return R <= 128 ? hy_latent_mma_launch<1, 128, 4>(e, l, m, T, ns, st) : hy_latent_mma_launch<1, 256, 4>(e, l, m, T, ns, st);
 }
 
@@ -1354,27 +1354,42 @@ static int hy_latent_mixer(xb_engine* e, const HyLayer& l, int T, const LinOut& 
   RotArgs r;
   r.freq = l.rot_freq_d; r.dims = c.m_rot_dims; r.half = c.m_rot_pairs == XB_ROPE_HALF_SPLIT ? 1 : 0;
   r.mult = c.m_rot_mult != 0.f ? c.m_rot_mult : 1.f;
-  if (l.off_dkv >= 0 || qr > 0)
-    XB_TRY(hy_launch(e, hy_latent_down_kernel<AT, KT>, dim3(T), dim3(256), 0, st, P, l.off_dkv, dr, R, r, (const float*)l.lat_norm, d.norm_eps,
-                     (KT*)l.k_pool, m, l.off_dq, qr, (const float*)l.dq_norm, a2));
+  const size_t dsm = (size_t)(qr + (l.off_dkv >= 0 ? R : 0)) * sizeof(float);
+  if (l.off_dkv >= 0 || qr > 0) {
+    if (T <= 64)
+      XB_TRY(hy_launch(e, hy_latent_down_kernel<AT, KT, 1024>, dim3(T), dim3(1024), dsm, st, P, l.off_dkv, dr, R, r, (const float*)l.lat_norm, d.norm_eps,
+                       (KT*)l.k_pool, m, l.off_dq, qr, (const float*)l.dq_norm, a2));
+    else
+      XB_TRY(hy_launch(e, hy_latent_down_kernel<AT, KT, 256>, dim3(T), dim3(256), dsm, st, P, l.off_dkv, dr, R, r, (const float*)l.lat_norm, d.norm_eps,
+                       (KT*)l.k_pool, m, l.off_dq, qr, (const float*)l.dq_norm, a2));
+  }
   LinOut Q = P;
   if (qr > 0) XB_TRY(hy_linear<AT>(e, a2, qr, l.w_uq, l.t_uq, nullptr, T, H * (n + dr), qr, hy->m2, hy->cap_m, st, &Q));
-  const size_t mm1 = (size_t)HY_MM_ROWS * n * sizeof(float), mm2 = (size_t)HY_MM_ROWS * R * sizeof(float);
+  const int mr = T <= 16 ? 1 : HY_MM_ROWS;   // tokens per block: few rows want blocks
+  const size_t mm1 = (size_t)mr * n * sizeof(float), mm2 = (size_t)HY_MM_ROWS * R * sizeof(float);
   // prompts in bf16 serving whose queries came back as one bf16 matrix: both per-head products on the tensor cores
   const bool tiles = std::is_same<AT, bf16>::value && hy->use_lat_mma && T > 64 && (n | dr | R | dv) % 8 == 0;
   if (tiles && Q.h != nullptr && Q.bias == nullptr && Q.ld % 8 == 0 && l.off_q % 8 == 0)
     XB_TRY(hy_launch(e, hy_latent_absorb_mma_kernel, dim3((T + HY_HG_M - 1) / HY_HG_M, H, (R + HY_HG_N - 1) / HY_HG_N), dim3(128), 0, st, Q.h + l.off_q,
                      Q.ld, dr, (const bf16*)l.w_uk, hy->qa, H, T, n, R, r, m.tok_pos));
+  else if (mr == 1)
+    XB_TRY(hy_launch(e, hy_latent_absorb_kernel<1>, dim3(T, H), dim3(256), mm1, st, Q, l.off_q, dr, (const bf16*)l.w_uk, hy->qa, H, T, n, R, r, m.tok_pos));
   else
-  XB_TRY(hy_launch(e, hy_latent_absorb_kernel, dim3((T + HY_MM_ROWS - 1) / HY_MM_ROWS, H), dim3(256), mm1, st, Q, l.off_q, dr,
+    XB_TRY(hy_launch(e, hy_latent_absorb_kernel<HY_MM_ROWS>, dim3((T + HY_MM_ROWS - 1) / HY_MM_ROWS, H), dim3(256), mm1, st, Q, l.off_q, dr,
                      (const bf16*)l.w_uk, hy->qa, H, T, n, R, r, m.tok_pos));
   // bf16 serving at sizes the tensor-core tiles take: rows = (token, head) pairs over shared key tiles; steps of few
   // rows split every sequence's keys over blocks and merge
   bool done = false;
   if (std::is_same<AT, bf16>::value && hy->use_lat_mma && W % 8 == 0 && R % 16 == 0) {
-    int rc = hy_latent_mma(e, l, m, T, st);
+    int ns = 1;
+    const int rc = hy_latent_mma(e, l, m, T, &ns, st);
     if (rc < 0) return -rc;
     done = rc == 0;
+    if (done && ns > 1 && T <= 16)   // few rows: merge, value up-projection and gate of a (token, head) row in one block
+      return hy_launch(e, hy_latent_readout_kernel<AT>, dim3(T, H), dim3(256), (size_t)(R + ns) * sizeof(float), st, (const float*)hy->lat_part, ns, T * H, H, R,
+                       (const bf16*)l.w_uv, a1, (long long)l.n_o, dv, P, c.m_gate ? l.off_g : -1);
+    if (done && ns > 1)
+      XB_TRY(hy_launch(e, hy_latent_merge_kernel, dim3(T * H), dim3(128), 0, st, (const float*)hy->lat_part, ns, T * H, H, R, hy->o, (long long)H * R));
   }
   if (!done) {
     const int aw = 16;   // the block's warps share out the visible keys
@@ -1425,7 +1440,7 @@ static int hy_router(xb_engine* e, const HyLayer& l, int T, const void* xin, int
   const int ng = c.groups > 0 ? c.groups : 1;
   if (T <= 64 && hy->fuse_router) {   // few rows: logits and routing of a token in one block
     const size_t rs1 = (size_t)(2 * c.n_experts + NE + ng) * sizeof(float);
-    return hy_launch(e, hy_router_route_kernel<AT>, dim3(T), dim3(256), rs1, st, x, (long long)D, (const bf16*)l.w_router, D, c.n_experts, c.top, c.groups,
+    return hy_launch(e, hy_router_route_kernel<AT>, dim3(T), dim3(32 * (NE < 32 ? (NE < 8 ? 8 : NE) : 32)), rs1, st, x, (long long)D, (const bf16*)l.w_router, D, c.n_experts, c.top, c.groups,
                      c.keep_groups, c.route_scale, hy->gw, c.route_score, c.group_score, c.route_norm, sg);
   }
   if (T <= 64) {   // few rows: a warp per (token, expert)
@@ -1821,6 +1836,11 @@ static int hy_run_prenorm_t(xb_engine* e, int T, int n_seqs, void* const* taps, 
       const long long ldc = 3LL * HK + HV;
       const unsigned cy = (unsigned)(((HK > HV ? HK : HV) + 255) / 256);
       const float scale = 1.0f / sqrtf((float)n), inv_tau = 1.0f / c.m_tau;
+      const size_t tsm = (size_t)(3 * ((n + 3) & ~3) + 3 * dv + rk) * sizeof(float);
+      if (T == n_seqs && tsm <= 48 * 1024) {   // single tokens
+        XB_TRY(hy_launch(e, hy_gla_token_kernel<AT>, dim3(n_seqs, H), dim3(512), tsm, st, P, l.off_q, l.off_k, l.off_v, l.off_g, l.off_a, rk, (const bf16*)l.w_d2,
+                         (const float*)l.w0, inv_tau, scale, hy->state + l.st_rec, SS, (const float*)l.head_norm, d.norm_eps, a1, (long long)l.n_o, m, H, n, dv));
+      } else {
       if (T > 64)
         XB_TRY(hy_launch(e, hy_gla_prep_kernel<8>, dim3((T + 7) / 8, cy), dim3(256), (size_t)8 * rk * sizeof(float), st, P, l.off_q, l.off_k, l.off_v, l.off_a, rk,
                          (const bf16*)l.w_d2, (const float*)l.w0, inv_tau, scale, hy->c, ldc, HK, HV, T));
@@ -1832,6 +1852,7 @@ static int hy_run_prenorm_t(xb_engine* e, int T, int n_seqs, void* const* taps, 
       in.beta = in.decay = in.qk = in.hdecay = nullptr;
       XB_TRY(hy_recur<HY_REC_GLA>(e, in, hy->state + l.st_rec, SS, hy->o, (long long)l.n_o, m, n_seqs, H, n, dv, T, st));
       XB_TRY(hy_head_norm<AT>(e, T, (long long)l.n_o, (const float*)l.head_norm, P, l.off_g, a1, (long long)l.n_o, H, dv, 0, 0, st));
+      }
     }
     XB_TRY(hy_linear<AT>(e, a1, l.n_o, l.w_o, l.t_o, nullptr, T, D, l.n_o, hy->m1, hy->cap_m, st, &y1));
     if (has_ff) {

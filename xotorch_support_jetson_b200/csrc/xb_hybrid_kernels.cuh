@@ -2201,38 +2201,34 @@ __global__ void hy_logits_kernel(LinOut y, float cap, float* __restrict__ out, i
 // another layer's rows) and, when queries pass a latent of their own, its columns (off_dq).  One block per token:
 //   cache row  = [ latent / rms(latent) * nw  |  rot(key part) ]      -> k_pool (one "key head", row of R + dr elements)
 //   cq[t]      = latent query / rms * qnw, as a Linear input           (qr = 0: none)
-template <typename AT, typename KT>
-__global__ void __launch_bounds__(256) hy_latent_down_kernel(LinOut P, int off_dkv, int dr, int R, RotArgs r, const float* __restrict__ nw, float eps,
-                                                             KT* __restrict__ k_pool, BatchMeta m, int off_dq, int qr,
-                                                             const float* __restrict__ qnw, AT* __restrict__ cq) {
+// Dynamic shared memory: qr + R floats (a row is read once: its split-K planes are what takes the time).  NT threads: 256 for prompts,
+// 1024 in steps of few rows.
+template <typename AT, typename KT, int NT>
+__global__ void __launch_bounds__(NT) hy_latent_down_kernel(LinOut P, int off_dkv, int dr, int R, RotArgs r, const float* __restrict__ nw, float eps,
+                                                            KT* __restrict__ k_pool, BatchMeta m, int off_dq, int qr,
+                                                            const float* __restrict__ qnw, AT* __restrict__ cq) {
   pdl_launch_dependents();
   pdl_wait();
+  extern __shared__ float dsm[];
   __shared__ float red[32];
   const int row = blockIdx.x;
+  const bool rows = off_dkv >= 0;
+  float sq = 0.f, sk = 0.f;
+  for (int i = threadIdx.x; i < qr; i += NT) { const float v = lin_at(P, row, off_dq + i); dsm[i] = v; sq = fmaf(v, v, sq); }
+  if (rows)
+    for (int i = threadIdx.x; i < R; i += NT) { const float v = lin_at(P, row, off_dkv + i); dsm[qr + i] = v; sk = fmaf(v, v, sk); }
   if (qr > 0) {
-    float ss = 0.f;
-    for (int i = threadIdx.x; i < qr; i += 256) {
-      const float v = lin_at(P, row, off_dq + i);
-      ss = fmaf(v, v, ss);
-    }
-    ss = block_sum<256>(ss, red);
-    const float inv = 1.0f / sqrtf(ss / (float)qr + eps);
-    for (int i = threadIdx.x; i < qr; i += 256) act_store<AT>(cq + (long long)row * qr + i, lin_at(P, row, off_dq + i) * inv * qnw[i]);
+    const float inv = 1.0f / sqrtf(block_sum<NT>(sq, red) / (float)qr + eps);
+    for (int i = threadIdx.x; i < qr; i += NT) act_store<AT>(cq + (long long)row * qr + i, dsm[i] * inv * qnw[i]);   // its own entries
   }
-  if (off_dkv < 0) return;
+  if (!rows) return;
   const int s = m.tok_seq[row], pos = m.tok_pos[row];
   const int page = m.page_table[(long long)m.seq_slot[s] * m.max_pages + pos / m.page_tokens];
   KT* kr = k_pool + ((long long)page * m.page_tokens + pos % m.page_tokens) * (R + dr);
-  float ss = 0.f;
-  for (int i = threadIdx.x; i < R; i += 256) {
-    const float v = lin_at(P, row, off_dkv + i);
-    ss = fmaf(v, v, ss);
-  }
-  ss = block_sum<256>(ss, red);
-  const float inv = 1.0f / sqrtf(ss / (float)R + eps);
-  for (int i = threadIdx.x; i < R; i += 256) act_store<KT>(kr + i, lin_at(P, row, off_dkv + i) * inv * nw[i]);
+  const float inv = 1.0f / sqrtf(block_sum<NT>(sk, red) / (float)R + eps);
+  for (int i = threadIdx.x; i < R; i += NT) act_store<KT>(kr + i, dsm[qr + i] * inv * nw[i]);
   const int half = r.dims >> 1;   // `half` pairs, then the entries that pass unchanged
-  for (int i = threadIdx.x; i < dr - half; i += 256) {
+  for (int i = NT - 1 - threadIdx.x; i < dr - half; i += NT) {
     if (i < half) {
       const int d0 = r.half ? i : 2 * i, d1 = r.half ? i + half : 2 * i + 1;
       const float u = lin_at(P, row, off_dkv + R + d0), v = lin_at(P, row, off_dkv + R + d1);
@@ -2249,17 +2245,18 @@ __global__ void __launch_bounds__(256) hy_latent_down_kernel(LinOut P, int off_d
 // Queries in the cache's space.  Q carries H heads of [K unrotated | dr rotated] (columns from qoff); per head
 //   qa[t, h, n]     = sum_k Q[t, h, k] * W[(h * K + k) * N + n]     n < N: the query folded into the latent space
 //   qa[t, h, N + i] = rot(rotated part)[i]                          i < dr
-// grid (ceil(T / 8), H), 256 threads over n; the 8 rows' inputs sit in shared memory (8 * K floats).
+// grid (ceil(T / ROWS), H), 256 threads over n; the rows' inputs sit in shared memory (ROWS * K floats).
 #define HY_MM_ROWS 8
+template <int ROWS>
 __global__ void __launch_bounds__(256) hy_latent_absorb_kernel(LinOut Q, int qoff, int dr, const bf16* __restrict__ W, float* __restrict__ qa,
                                                                int H, int T, int K, int N, RotArgs r, const int* __restrict__ tok_pos) {
   pdl_launch_dependents();
   pdl_wait();
   extern __shared__ __align__(16) float xsm[];
-  const int t0 = blockIdx.x * HY_MM_ROWS, h = blockIdx.y;
-  const int nt = T - t0 < HY_MM_ROWS ? T - t0 : HY_MM_ROWS;
+  const int t0 = blockIdx.x * ROWS, h = blockIdx.y;
+  const int nt = T - t0 < ROWS ? T - t0 : ROWS;
   const int qh = qoff + h * (K + dr), ld = N + dr;
-  for (int i = threadIdx.x; i < HY_MM_ROWS * K; i += 256) {
+  for (int i = threadIdx.x; i < ROWS * K; i += 256) {
     const int rr = i / K, k = i - rr * K;
     xsm[i] = rr < nt ? lin_at(Q, t0 + rr, qh + k) : 0.f;
   }
@@ -2281,13 +2278,14 @@ __global__ void __launch_bounds__(256) hy_latent_absorb_kernel(LinOut Q, int qof
   __syncthreads();
   const bf16* Wh = W + (long long)h * K * N;
   for (int n = threadIdx.x; n < N; n += 256) {
-    float acc[HY_MM_ROWS];
+    float acc[ROWS];
 #pragma unroll
-    for (int rr = 0; rr < HY_MM_ROWS; ++rr) acc[rr] = 0.f;
+    for (int rr = 0; rr < ROWS; ++rr) acc[rr] = 0.f;
+#pragma unroll 8
     for (int k = 0; k < K; ++k) {
       const float w = bf2f(Wh[(long long)k * N + n]);
 #pragma unroll
-      for (int rr = 0; rr < HY_MM_ROWS; ++rr) acc[rr] = fmaf(xsm[rr * K + k], w, acc[rr]);
+      for (int rr = 0; rr < ROWS; ++rr) acc[rr] = fmaf(xsm[rr * K + k], w, acc[rr]);
     }
     for (int rr = 0; rr < nt; ++rr) qa[((long long)(t0 + rr) * H + h) * ld + n] = acc[rr];
   }
@@ -2338,6 +2336,58 @@ __global__ void __launch_bounds__(128) hy_head_mm_kernel(const float* __restrict
       }
     }
     for (int r = 0; r < nt; ++r) act_store<AT>(y + (long long)(t0 + r) * ldy + (long long)h * N + n, acc[r] * gate[r]);
+  }
+}
+
+// Steps of few rows behind the key shares of hy_latent_attn_mma_kernel: merge of a (token, head) row's shares, its value
+// up-projection and the head's gate in one block.
+//   x = sum_s O_s 2^(m_s - M) / sum_s l_s 2^(m_s - M);  y[t, h * N + n] = sigmoid(G) * sum_k x[k] W[(h * N + n) * R + k]
+// part [n_splits][T * H][2 + R] = (m, l, O) per share.  grid (T, H), 256 threads; R + n_splits floats of shared memory.
+template <typename AT>
+__global__ void __launch_bounds__(256) hy_latent_readout_kernel(const float* __restrict__ part, int n_splits, int NR, int H, int R, const bf16* __restrict__ W,
+                                                                AT* __restrict__ y, long long ldy, int N, LinOut G, int off_gate) {
+  pdl_launch_dependents();
+  pdl_wait();
+  extern __shared__ __align__(16) float xsm[];
+  float* fac = xsm + R;
+  const int t = blockIdx.x, h = blockIdx.y, row = t * H + h;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  if (warp == 0) {
+    float M = HY_LAT_NEG;
+    for (int s = lane; s < n_splits; s += 32) M = fmaxf(M, part[((long long)s * NR + row) * (R + 2)]);
+    M = warp_max(M);
+    float L = 0.f;
+    for (int s = lane; s < n_splits; s += 32) {
+      const float* p = part + ((long long)s * NR + row) * (R + 2);
+      const float f = exp2f(p[0] - M);
+      fac[s] = f;
+      L = fmaf(p[1], f, L);
+    }
+    L = warp_sum(L);
+    for (int s = lane; s < n_splits; s += 32) fac[s] /= L;
+  }
+  __syncthreads();
+  for (int c = threadIdx.x; c < R; c += 256) {
+    float acc = 0.f;
+    const float* p = part + (long long)row * (R + 2) + 2 + c;
+#pragma unroll 8
+    for (int s = 0; s < n_splits; ++s) acc = fmaf(p[(long long)s * NR * (R + 2)], fac[s], acc);
+    xsm[c] = acc;
+  }
+  __syncthreads();
+  const float g = off_gate >= 0 ? hy_sigmoid(lin_at(G, t, off_gate + h)) : 1.0f;
+  const bf16* Wh = W + (long long)h * N * R;
+  const bool vec = (R & 7) == 0 && (reinterpret_cast<uintptr_t>(W) & 15) == 0;
+#pragma unroll 4
+  for (int n = warp; n < N; n += 8) {
+    float acc = 0.f;
+    if (vec) {
+      for (int k = lane * 8; k < R; k += 256) acc = hy_dot8(xsm + k, *reinterpret_cast<const uint4*>(Wh + (long long)n * R + k), acc);
+    } else {
+      for (int k = lane; k < R; k += 32) acc = fmaf(bf2f(Wh[(long long)n * R + k]), xsm[k], acc);
+    }
+    acc = warp_sum(acc);
+    if (lane == 0) act_store<AT>(y + (long long)t * ldy + (long long)h * N + n, acc * g);
   }
 }
 
@@ -2556,6 +2606,71 @@ __global__ void __launch_bounds__(256) hy_gla_prep_kernel(LinOut P, int off_q, i
     }
     if (i < HV) row[3LL * HK + i] = lin_at(P, t0 + r, off_v + i);
   }
+}
+
+// A step of single tokens: everything between the input and the output projection of a gated linear attention layer in one kernel, a
+// block per (sequence, head).  The head's q, k, v, gate and the decay's first projection are read once (split-K planes summed), the
+// decays formed, then a warp takes one value column after the other (state rows [dv][dk]: a column's dk numbers are neighbours):
+//   S_j <- w * S_j + k v_j,  o_j = q . S_j;  out = o / rms(o) * nw * silu(g)
+// All fp32.  Dynamic shared memory: 3 * dk + 3 * dv + rk floats.  grid (n_seqs, H), 512 threads.
+template <typename AT>
+__global__ void __launch_bounds__(512) hy_gla_token_kernel(LinOut P, int off_q, int off_k, int off_v, int off_g, int off_a, int rk, const bf16* __restrict__ w2,
+                                                           const float* __restrict__ b2, float inv_tau, float scale, float* __restrict__ state,
+                                                           long long state_stride, const float* __restrict__ nw, float eps, AT* __restrict__ out,
+                                                           long long ld_out, BatchMeta m, int H, int dk, int dv) {
+  pdl_launch_dependents();
+  pdl_wait();
+  extern __shared__ __align__(16) float gsm[];
+  __shared__ float red[32];
+  const int s = blockIdx.x, h = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nwarps = 16;
+  const int row = m.seq_last[s], dk4 = (dk + 3) & ~3;
+  float *q = gsm, *k = q + dk4, *w = k + dk4, *v = w + dk4, *g = v + dv, *o = g + dv, *a = o + dv;
+  for (int u = threadIdx.x; u < 2 * dk + 2 * dv + rk; u += 512) {
+    if (u < dk) q[u] = lin_at(P, row, off_q + h * dk + u) * scale;
+    else if (u < 2 * dk) k[u - dk] = lin_at(P, row, off_k + h * dk + u - dk);
+    else if (u < 2 * dk + dv) v[u - 2 * dk] = lin_at(P, row, off_v + h * dv + u - 2 * dk);
+    else if (u < 2 * dk + 2 * dv) g[u - 2 * dk - dv] = lin_at(P, row, off_g + h * dv + u - 2 * dk - dv);
+    else a[u - 2 * dk - 2 * dv] = lin_at(P, row, off_a + u - 2 * dk - 2 * dv);
+  }
+  __syncthreads();
+  for (int i = threadIdx.x; i < dk; i += 512) {
+    float z = b2[h * dk + i];
+    const bf16* wr = w2 + ((long long)h * dk + i) * rk;
+    for (int x = 0; x < rk; ++x) z = fmaf(bf2f(wr[x]), a[x], z);
+    w[i] = expf(-(fmaxf(-z, 0.f) + log1pf(expf(-fabsf(z)))) * inv_tau);
+  }
+  __syncthreads();
+  float* st = state + (long long)m.seq_slot[s] * state_stride + (long long)h * dv * dk;
+  const bool have = m.tok_pos[row] > 0;
+  const bool al = (dk & 3) == 0 && (reinterpret_cast<uintptr_t>(st) & 15) == 0;
+#pragma unroll 4
+  for (int j = warp; j < dv; j += nwarps) {
+    float* col = st + (long long)j * dk;
+    const float vj = v[j];
+    float acc = 0.f;
+    if (al) {
+      for (int i = lane * 4; i < dk; i += 128) {
+        float4 S = have ? *reinterpret_cast<const float4*>(col + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+        const float4 k4 = *reinterpret_cast<const float4*>(k + i), w4 = *reinterpret_cast<const float4*>(w + i), q4 = *reinterpret_cast<const float4*>(q + i);
+        S.x = fmaf(w4.x, S.x, k4.x * vj); S.y = fmaf(w4.y, S.y, k4.y * vj); S.z = fmaf(w4.z, S.z, k4.z * vj); S.w = fmaf(w4.w, S.w, k4.w * vj);
+        *reinterpret_cast<float4*>(col + i) = S;
+        acc = fmaf(q4.x, S.x, acc); acc = fmaf(q4.y, S.y, acc); acc = fmaf(q4.z, S.z, acc); acc = fmaf(q4.w, S.w, acc);
+      }
+    } else {
+      for (int i = lane; i < dk; i += 32) {
+        const float S = fmaf(w[i], have ? col[i] : 0.f, k[i] * vj);
+        col[i] = S;
+        acc = fmaf(q[i], S, acc);
+      }
+    }
+    acc = warp_sum(acc);
+    if (lane == 0) o[j] = acc;
+  }
+  __syncthreads();
+  float ss = 0.f;
+  for (int j = threadIdx.x; j < dv; j += 512) ss = fmaf(o[j], o[j], ss);
+  const float inv = 1.0f / sqrtf(block_sum<512>(ss, red) / (float)dv + eps);
+  for (int j = threadIdx.x; j < dv; j += 512) act_store<AT>(out + (long long)row * ld_out + (long long)h * dv + j, o[j] * inv * nw[j] * hy_silu(g[j]));
 }
 
 // ----------------------------------------------------------------------------- clamped gated feed-forward, experts
@@ -2784,11 +2899,10 @@ __global__ void __launch_bounds__(128) hy_route_kernel(const float* __restrict__
   const int ld = E + (shared_gate ? 1 : 0);
   hy_route_token(z + t * ld, sc, sc + E, sc + 2 * E, E, top, groups, keep, scale, gw + t * ld, score_mode, group_mode, renorm, shared_gate);
 }
-// Steps of few rows: logits and routing of a token in ONE block of eight warps.  Warp w forms the fp32 logits of experts
-// w, w + 8, ... (16-byte weight loads, fp32 sums, the order of hy_router_logits_kernel<AT, 1>), then the first warp routes.
-// Shared memory: 3 * E + groups + 1 floats.  grid (T), 256 threads.
+// Steps of few rows: logits and routing of a token in ONE block.  Warp w forms the fp32 logits of experts w, w + warps, ... (16-byte weight loads, fp32 sums, the order of hy_router_logits_kernel<AT, 1>), then the first warp routes.
+// Shared memory: 3 * E + groups + 1 floats.  grid (T), a warp per expert up to 32.
 template <typename AT>
-__global__ void __launch_bounds__(256) hy_router_route_kernel(const AT* __restrict__ x, long long ldx, const bf16* __restrict__ w, int K, int E, int top,
+__global__ void __launch_bounds__(1024) hy_router_route_kernel(const AT* __restrict__ x, long long ldx, const bf16* __restrict__ w, int K, int E, int top,
                                                               int groups, int keep, float scale, float* __restrict__ gw, int score_mode, int group_mode,
                                                               int renorm, int shared_gate) {
   pdl_launch_dependents();
@@ -2799,7 +2913,7 @@ __global__ void __launch_bounds__(256) hy_router_route_kernel(const AT* __restri
   const AT* xr = x + t * ldx;
   const bool vec = (K & 7) == 0 && (reinterpret_cast<uintptr_t>(w) & 15) == 0;
   const int NE = E + (shared_gate ? 1 : 0);
-  for (int e = warp; e < NE; e += 8) {
+  for (int e = warp; e < NE; e += blockDim.x >> 5) {
     const bf16* wr = w + (long long)e * K;
     float acc = 0.f;
     if (vec) {
