@@ -177,7 +177,8 @@ int xb_handoff_connect(xb_engine* e, const void* next_landing_handle, const void
 int xb_forward_handoff(xb_engine* e, const xb_batch* batch, int slot_in, int wait_value, int slot_out, int signal_value,
                        void* out, void* stream);
 /* xb_handoff_connect for two stages that live in ONE process (an in-process ring of per-GPU nodes, or two
- * stages on one GPU in a test): `e` stores straight into `next`'s landing buffers through their device
+ * stages on one GPU in a test; then the caller orders the consumer's stream behind the producer's, so that
+ * no kernel waits on the flag beside the kernels that set it): `e` stores straight into `next`'s landing buffers through their device
  * addresses, no CUDA IPC handle involved (xb_handoff_create may then be given NULL for both handle
  * buffers); peer access from e's device to next's is enabled when they differ.  Both stages must have
  * called xb_handoff_create with the same geometry.  `next` must outlive the connection. */

@@ -1,7 +1,8 @@
 """The decode hand-off kernels (xb_resid_send_kernel / xb_recv_norm_kernel and their flag protocol) and
 the other boundary rules of the C ABI, on ONE GPU: two pipeline stages of one process connected with
 xb_handoff_connect_local -- the same kernels and flags a multi-GPU ring runs over NVLink, with the
-next stage's landing buffer on the same device -- against the plain ``hidden=`` path bit for bit.
+next stage's landing buffer on the same device and the consumer launched behind the producer --
+against the plain ``hidden=`` path bit for bit.
 On a box with two GPUs the same test also runs with the stages on different devices (peer stores)."""
 import os
 
@@ -95,7 +96,9 @@ def test_local_handoff_equals_hidden_path_bit_for_bit(built_lib, mid, cut, devs)
           v = k + 1                                   # per-slot flag value: only grows
           with torch.cuda.stream(stream_a):
             sa.forward(slots, [1] * B, pos, tokens=tin, handoff=(-1, v, m, v))
-          with torch.cuda.stream(stream_b):           # no host synchronisation between the stages: the flag orders them
+          if devs[0] == devs[1]:                      # one GPU: a kernel that waits on the flag must not share it with the
+            stream_b.wait_stream(stream_a)            # kernels it waits for (they may not all fit at once)
+          with torch.cuda.stream(stream_b):           # two GPUs: no synchronisation between the stages, the flag orders them
             lg = sb.forward(slots, [1] * B, pos, handoff=(m, v, -1, v))
             toks[m] = sb.sample(lg, temp=0.0)
         else:

@@ -729,6 +729,8 @@ class B200ShardInferenceEngine(InferenceEngine):
   def _rows_from_ref(self, st: StageRuntime, ref: DeviceTensorRef, bsz: int, s: int):
     """What a DeviceTensorRef stands for, as input of this stage: (bf16 rows [bsz, s, D] on this GPU | None, landing)."""
     if ref.landing is not None:
+      if ref.event is not None:                       # both stages on one GPU: see _device_result
+        torch.cuda.current_stream(st.device).wait_event(ref.event)
       return None, ref.landing                        # already in this GPU's landing buffer (stored by the producer's kernel)
     if ref.recv is not None and ref.tensor is None:   # process-per-GPU ring: post the receive on this engine's stream
       buf = torch.empty((bsz * s, st.dim), dtype=torch.bfloat16, device=st.device)
@@ -746,7 +748,13 @@ class B200ShardInferenceEngine(InferenceEngine):
     st = self.stage
     shape = (bsz, s, st.dim)
     if landing_out is not None:
-      return DeviceTensorRef(shape, landing=landing_out, recv=("landed",) if self._ring_landing is not None else None)
+      ev, nxt = None, self._next_engine
+      if nxt is not None and nxt.stage is not None and nxt.stage.device == st.device:
+        # two stages on ONE GPU: a consumer kernel that waits on the flag, and the blocks parked behind it, could hold the SMs
+        # the producer still needs; the stream dependency keeps it off the GPU until the flag is set
+        ev = torch.cuda.Event()
+        ev.record(torch.cuda.current_stream(st.device))
+      return DeviceTensorRef(shape, event=ev, landing=landing_out, recv=("landed",) if self._ring_landing is not None else None)
     if self._ring is not None:
       self._ring.send_rows(out.reshape(bsz * s, -1))    # enqueued on this stream, right behind the forward
       return DeviceTensorRef(shape, tensor=out, recv=("sent",))

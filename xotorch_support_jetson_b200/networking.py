@@ -41,7 +41,8 @@ class DeviceTensorRef:
 
   ``tensor``: bf16 CUDA tensor ``[B*s, D]`` + ``event`` (recorded on the producing stream), or None when
   the rows went through a landing buffer: then ``landing = (slot, flag_value)`` names the consumer-side
-  slot the producer's last kernel stored them into, and -- across processes -- ``recv = (src_rank,)``
+  slot the producer's last kernel stored them into (stages that share one GPU also carry ``event``: the consumer's
+  kernels start behind it instead of waiting on the flag beside the producer's), and -- across processes -- ``recv = (src_rank,)``
   says that the rows still have to be received from that rank (posted by the consuming engine on its
   own stream).  ``np.asarray(ref)`` materialises what the reference would have shipped (fp32 numpy)."""
   ndim = 3
