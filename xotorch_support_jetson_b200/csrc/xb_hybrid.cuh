@@ -229,6 +229,8 @@ static int hy_create_mixer(xb_engine* e, int i, bool own, size_t& st, uint64_t& 
     const bool rows = c.m_kv_from < 0;    // makes cache rows of its own
     XB_CHECK(qr >= 0 && c.m_window >= 0 && c.m_scale > 0.f, "layer %d: bad latent attention constants (query rank %lld, window %d, scale %g)", i, qr,
              c.m_window, c.m_scale);
+    XB_CHECK(qr + R <= 12288 && n <= 1536, "layer %d: query latent %lld + latent %lld (at most 12288) or key size %lld (at most 1536) exceed a block's shared memory", i, qr,
+             R, n);
     XB_CHECK(c.m_rot_pairs == XB_ROPE_INTERLEAVED || c.m_rot_pairs == XB_ROPE_HALF_SPLIT, "layer %d: unknown rotary pair layout %d", i, c.m_rot_pairs);
     XB_CHECK(own || (qr == 0 && c.m_gate == 0 && rows), "layer %d: a query latent, head gates and borrowed cache rows come with tensors of their own", i);
     if (!rows) {
@@ -1841,17 +1843,17 @@ static int hy_run_prenorm_t(xb_engine* e, int T, int n_seqs, void* const* taps, 
         XB_TRY(hy_launch(e, hy_gla_token_kernel<AT>, dim3(n_seqs, H), dim3(512), tsm, st, P, l.off_q, l.off_k, l.off_v, l.off_g, l.off_a, rk, (const bf16*)l.w_d2,
                          (const float*)l.w0, inv_tau, scale, hy->state + l.st_rec, SS, (const float*)l.head_norm, d.norm_eps, a1, (long long)l.n_o, m, H, n, dv));
       } else {
-      if (T > 64)
-        XB_TRY(hy_launch(e, hy_gla_prep_kernel<8>, dim3((T + 7) / 8, cy), dim3(256), (size_t)8 * rk * sizeof(float), st, P, l.off_q, l.off_k, l.off_v, l.off_a, rk,
-                         (const bf16*)l.w_d2, (const float*)l.w0, inv_tau, scale, hy->c, ldc, HK, HV, T));
-      else
-        XB_TRY(hy_launch(e, hy_gla_prep_kernel<1>, dim3(T, cy), dim3(256), (size_t)rk * sizeof(float), st, P, l.off_q, l.off_k, l.off_v, l.off_a, rk,
-                         (const bf16*)l.w_d2, (const float*)l.w0, inv_tau, scale, hy->c, ldc, HK, HV, T));
-      RecurIn in;
-      in.c = hy->c; in.ldc = ldc; in.qoff = 0; in.koff = HK; in.xoff[0] = 2LL * HK; in.xoff[1] = in.xoff[2] = 0; in.voff = 3LL * HK; in.q_heads = H;
-      in.beta = in.decay = in.qk = in.hdecay = nullptr;
-      XB_TRY(hy_recur<HY_REC_GLA>(e, in, hy->state + l.st_rec, SS, hy->o, (long long)l.n_o, m, n_seqs, H, n, dv, T, st));
-      XB_TRY(hy_head_norm<AT>(e, T, (long long)l.n_o, (const float*)l.head_norm, P, l.off_g, a1, (long long)l.n_o, H, dv, 0, 0, st));
+        if (T > 64)
+          XB_TRY(hy_launch(e, hy_gla_prep_kernel<8>, dim3((T + 7) / 8, cy), dim3(256), (size_t)8 * rk * sizeof(float), st, P, l.off_q, l.off_k, l.off_v, l.off_a, rk,
+                           (const bf16*)l.w_d2, (const float*)l.w0, inv_tau, scale, hy->c, ldc, HK, HV, T));
+        else
+          XB_TRY(hy_launch(e, hy_gla_prep_kernel<1>, dim3(T, cy), dim3(256), (size_t)rk * sizeof(float), st, P, l.off_q, l.off_k, l.off_v, l.off_a, rk,
+                           (const bf16*)l.w_d2, (const float*)l.w0, inv_tau, scale, hy->c, ldc, HK, HV, T));
+        RecurIn in;
+        in.c = hy->c; in.ldc = ldc; in.qoff = 0; in.koff = HK; in.xoff[0] = 2LL * HK; in.xoff[1] = in.xoff[2] = 0; in.voff = 3LL * HK; in.q_heads = H;
+        in.beta = in.decay = in.qk = in.hdecay = nullptr;
+        XB_TRY(hy_recur<HY_REC_GLA>(e, in, hy->state + l.st_rec, SS, hy->o, (long long)l.n_o, m, n_seqs, H, n, dv, T, st));
+        XB_TRY(hy_head_norm<AT>(e, T, (long long)l.n_o, (const float*)l.head_norm, P, l.off_g, a1, (long long)l.n_o, H, dv, 0, 0, st));
       }
     }
     XB_TRY(hy_linear<AT>(e, a1, l.n_o, l.w_o, l.t_o, nullptr, T, D, l.n_o, hy->m1, hy->cap_m, st, &y1));
