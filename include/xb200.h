@@ -27,7 +27,7 @@
 extern "C" {
 #endif
 
-#define XB_ABI_VERSION 9
+#define XB_ABI_VERSION 10
 
 typedef struct xb_engine xb_engine;
 
@@ -249,7 +249,16 @@ enum {
                           channel (s_qk_norm); values that are the keys as projected, before that norm, with no value
                           projection (s_v_is_k); queries multiplied by 1 + coef ln(floor((pos + 1) / every) + 1)
                           (s_qtemp_*); r1_h ln(1 + r2_h (i - j)) taken off the score of query i and key j, two numbers
-                          per head (s_dist_bias) */
+                          per head (s_dist_bias); a causal filter of s_taps taps per channel of the projected q, k, v, before
+                          norm and rotation (s_taps, "q.conv" ...; the last s_taps - 1 projected rows are state of the slot);
+                          query and key heads divided by their root mean square after the rotation, no weight (s_head_norm);
+                          a bias on the output projection (s_o_bias); a window (i - j < s_window) and / or chunks counted
+                          from position 0 (i / s_chunk = j / s_chunk); a second mixer on the same input, whose tensors sit
+                          under ".right." while this one's sit under ".left.": left_scale * this + right_scale * second */
+  XB_MIX_MLSTM = 8,    /* matrix memory: S <- e^(f + m' - m) S + e^(i - m) k v^T with log gates i = cap tanh(zi / cap),
+                          f = logsigmoid(cap tanh(zf / cap)) per head (cap = m_gate_cap) and m = max(f + m', i) from m = 0 on; a normaliser n
+                          of m_dim numbers the same way with k alone; o = S^T q m_dim^-1/2 / (max(|n . q m_dim^-1/2|, e^-m) + 1e-6);
+                          read-out RMS-normed per head, a weight per channel of all heads, gated by sigmoid(g) */
   XB_MIX_GLA = 7       /* gated linear attention: S <- diag(w) S + k v^T, o = S^T q m_dim^-1/2, a decay per head and key channel
                           w = sigmoid(W2 (W1 h) + b)^(1 / m_tau) (W1 of m_rank rows); read-out RMS-normed per head with one
                           weight vector for all heads, gated by SiLU(g) */
@@ -280,6 +289,7 @@ enum {
   XB_ACT_GLU_CLAMP = 0,   /* down(g sigmoid(1.702 g) (u + 1)) with the limits above */
   XB_ACT_SWIGLU = 1,      /* down(silu(g) u), no limits */
   XB_ACT_GELU = 2,        /* down(gelu(up h)): no gate projection, the exact (erf) form 0.5 z (1 + erf(z / sqrt 2)) */
+  XB_ACT_RELU2 = 4,       /* XB_FF_MOE: down(relu(up h)^2), no gate projection */
   XB_ACT_GEGLU = 3        /* down(gelu(g) u), gelu in the tanh form 0.5 z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3))) */
 };
 /* how the router of XB_FF_MOE turns logits into scores, what a group of experts is worth, and what weight a chosen expert
@@ -339,6 +349,14 @@ typedef struct xb_hybrid_layer {
   int32_t m_rot_pairs, m_rot_scaling;               /* LATENT: XB_ROPE_* pair layout, XB_ROT_SCALE_* */
   float m_rot_mult;                                 /* LATENT: cos / sin multiplier (0 = 1) */
   double m_rot_factor, m_rot_orig, m_rot_p0, m_rot_p1;
+  int32_t s_taps, s_head_norm, s_o_bias, s_window, s_chunk;   /* XB_MIX_SOFTMAX, see there; 0 = none */
+  int32_t second;                                   /* SOFTMAX: XB_MIX_MLSTM (its m_* fields) beside it, scaled by right_scale,
+                                                       this one by left_scale; 0 = none */
+  float m_gate_cap;                                 /* MLSTM */
+  int32_t identity;                                 /* XB_FF_MOE: router outputs behind the n_experts that hand the input on, times
+                                                       their weight; they compete like experts and have no tensors */
+  int32_t route_bias;                               /* XB_FF_MOE: 1 = experts are chosen by score + "correction" (per router
+                                                       output); the weights use the score alone */
 } xb_hybrid_layer;
 
 typedef struct xb_hybrid_desc {
@@ -370,10 +388,14 @@ typedef struct xb_hybrid_desc {
   int32_t bigram_mul_prev, bigram_mul_cur;
   int32_t pos_rows;                  /* > 0: row `position` of the learned table "pos" [pos_rows, dim] joins the embedding */
   int32_t norm_kind;                 /* XB_NORM_*: what the stream's norms compute (pre-norm blocks; others: XB_NORM_RMS) */
+  int32_t streams;                   /* pre-norm blocks: > 0 = the stream is this many copies x_1 .. x_s of one row (hyper-connections): a
+                                        sublayer q (1 mixer, 2 feed-forward) reads u = sum_i hc<q>.in[i] x_i and its output y joins as
+                                        x_j <- sum_i hc<q>.mix[i, j] x_i + hc<q>.out[j] y; the model's last norm reads sum_i x_i */
 } xb_hybrid_desc;
 
 enum {
   XB_NORM_RMS = 0,
+  XB_NORM_LAYER = 2,      /* (x - mean) / sqrt(mean squared deviation + eps) * w, no offset */
   XB_NORM_TANH = 1        /* tanh(a x) * w + b, channel by channel, no statistics of the row: tensors "<name>" (w), "<name>.b" and
                              the single number "<name>.alpha" */
 };

@@ -37,7 +37,7 @@ class ModelDesc(C.Structure):
   ]
 
 
-ABI_VERSION = 9
+ABI_VERSION = 10
 
 
 def model_desc(**fields) -> ModelDesc:
@@ -45,15 +45,15 @@ def model_desc(**fields) -> ModelDesc:
   return ModelDesc(struct_size=C.sizeof(ModelDesc), **fields)
 
 
-MIX_DELTA, MIX_PARALLEL, MIX_LATENT, MIX_GDELTA, MIX_LIGHTNING, MIX_SOFTMAX, MIX_GLA = 1, 2, 3, 4, 5, 6, 7
+MIX_DELTA, MIX_PARALLEL, MIX_LATENT, MIX_GDELTA, MIX_LIGHTNING, MIX_SOFTMAX, MIX_GLA, MIX_MLSTM = 1, 2, 3, 4, 5, 6, 7, 8
 ROT_SCALE_NONE, ROT_SCALE_BANDS, ROT_SCALE_RAMP = 0, 1, 2
-ACT_GLU_CLAMP, ACT_SWIGLU, ACT_GELU, ACT_GEGLU = 0, 1, 2, 3
+ACT_GLU_CLAMP, ACT_SWIGLU, ACT_GELU, ACT_GEGLU, ACT_RELU2 = 0, 1, 2, 3, 4
 ROUTE_SIGMOID, ROUTE_SOFTMAX = 0, 1
 GROUP_TOP2, GROUP_MAX = 0, 1
 SINK_NONE, SINK_LEARNED, SINK_UNIT = 0, 1, 2
 FF_RELU2, FF_GLU_CLAMP, FF_MOE, FF_GLU = 0, 1, 2, 3
 BLOCK_SANDWICH, BLOCK_PARALLEL, BLOCK_BRANCHNORM, BLOCK_PRENORM = 0, 1, 2, 3
-NORM_RMS, NORM_TANH = 0, 1
+NORM_RMS, NORM_TANH, NORM_LAYER = 0, 1, 2
 ST_BF16, ST_F16, ST_F32 = 0, 1, 2   # element types xb_load_named accepts
 
 
@@ -85,6 +85,8 @@ class HybridLayer(C.Structure):
     ("shared_gate", C.c_int32), ("m_tau", C.c_float), ("m_q_rank", C.c_int32), ("m_window", C.c_int32), ("m_gate", C.c_int32),
     ("m_kv_from", C.c_int32), ("m_rot_pairs", C.c_int32), ("m_rot_scaling", C.c_int32), ("m_rot_mult", C.c_float),
     ("m_rot_factor", C.c_double), ("m_rot_orig", C.c_double), ("m_rot_p0", C.c_double), ("m_rot_p1", C.c_double),
+    ("s_taps", C.c_int32), ("s_head_norm", C.c_int32), ("s_o_bias", C.c_int32), ("s_window", C.c_int32), ("s_chunk", C.c_int32),
+    ("second", C.c_int32), ("m_gate_cap", C.c_float), ("identity", C.c_int32), ("route_bias", C.c_int32),
   ]
 
 
@@ -98,7 +100,7 @@ class HybridDesc(C.Structure):
     ("norm_groups", C.c_int32), ("norm_plain", C.c_int32), ("residual_mult", C.c_float), ("tied_head", C.c_int32),
     ("ff_unfiltered", C.c_int32),
     ("gated_residual", C.c_int32), ("bigram_buckets", C.c_int32), ("bigram_mul_prev", C.c_int32), ("bigram_mul_cur", C.c_int32),
-    ("pos_rows", C.c_int32), ("norm_kind", C.c_int32),
+    ("pos_rows", C.c_int32), ("norm_kind", C.c_int32), ("streams", C.c_int32),
   ]
 
 

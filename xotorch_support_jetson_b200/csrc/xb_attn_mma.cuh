@@ -47,13 +47,14 @@ __device__ __forceinline__ uint32_t att_tile_off(int r, int c16) {
 //   sK, sV  : shared-memory byte addresses of the K / V tile
 //   krow0   : first key row (inside the tile) this warp handles; it handles NKB*16 rows
 //   key_abs0: absolute position of tile row 0;  lim0/lim1: last visible key of the thread's two rows
+//   lo      : first visible key (a window or a chunk), 0 = all earlier ones
 //   dist    : nullptr, or {r1, r2} of row 0 then of row 1: r1 * ln(1 + r2 * (lim - key)) is taken off the scaled score
 //             (lim = the row's own position), in log2 units r1 * log2(1 + r2 * distance)
 template <int HD, int NKB>
 __device__ __forceinline__ void att_warp_block(const uint32_t (*qf)[4], uint32_t sK, uint32_t sV, int krow0, int key_abs0,
                                                int lim0, int lim1, float scale_log2, float (&mrow)[2],
                                                float (&lrow)[2], float (*o)[4], float softcap = 0.f, bool p_split = false,
-                                               const float* dist = nullptr) {
+                                               const float* dist = nullptr, int lo = 0) {
   constexpr int KS = HD / 16;   // k-steps over the head dim
   constexpr int DT = HD / 8;    // output n-tiles over the head dim
   constexpr int NT = NKB * 2;   // score n-tiles (8 keys each)
@@ -100,6 +101,10 @@ __device__ __forceinline__ void att_warp_block(const uint32_t (*qf)[4], uint32_t
     if (k0 + 1 > lim0) s[j][1] = -INFINITY;
     if (k0 > lim1) s[j][2] = -INFINITY;
     if (k0 + 1 > lim1) s[j][3] = -INFINITY;
+    if (lo > key_abs0) {   // the tile straddles the oldest visible key
+      if (k0 < lo) s[j][0] = s[j][2] = -INFINITY;
+      if (k0 + 1 < lo) s[j][1] = s[j][3] = -INFINITY;
+    }
     mx0 = fmaxf(mx0, fmaxf(s[j][0], s[j][1]));
     mx1 = fmaxf(mx1, fmaxf(s[j][2], s[j][3]));
   }
@@ -168,8 +173,9 @@ __device__ __forceinline__ void att_issue_tile(const CUtensorMap* tmK, const CUt
     const int pi = key / P;
     const int page = pt[pi < max_pages ? pi : max_pages - 1];   // rows past the context are masked
     const int row = (page * KV + kvh) * P + (key % P);
-    // v_wide: a value row holds every key head's values side by side; this block reads head vh of it
-    const int vrow = v_wide ? page * P + (key % P) : row, vx0 = v_wide ? vh * HD : 0;
+    // v_wide 1: a value row holds every key head's values side by side, this block reads head vh of it; 2: a value row is several
+    // pieces of HD channels, this block reads piece vh
+    const int vrow = v_wide == 1 ? page * P + (key % P) : row, vx0 = v_wide ? vh * HD : 0;
 #pragma unroll
     for (int db = 0; db < HD / 64; ++db) {
       tma_load_2d(sK + db * (XB_ATT_TILE * 128) + rg * BR * 128, tmK, bar, db * 64, row);
@@ -201,7 +207,9 @@ struct AttDecCfg {
 // Options of the decode kernel beyond plain causal attention (all zero = none): a sink per head in the softmax denominator,
 // a cap on the scores, wide value rows (grid y = KV * KV: block y reads keys of head y % KV and values of head y / KV and
 // writes to out + (token * H + head) * out_head_stride + (y / KV) * HD; out_head_stride 0 = HD).  With wide value rows the
-// splits are merged inside a cluster or not made at all (the global partial buffers are not laid out for them).
+// splits are merged inside a cluster or not made at all (the global partial buffers are not laid out for them).  v_wide 2: value heads
+// wider than HD in pieces of HD channels (grid y = KV * pieces, block y: head y % KV, piece y / KV, output as above).
+// window / chunk > 0: keys i - j < window / of the query's own chunk of positions only.
 struct AttDecOpt {
   const float* sink;
   float softcap;
@@ -210,6 +218,7 @@ struct AttDecOpt {
   int p_split;   // 1: the softmax weights enter the value product as hi + lo bf16 pairs (fp32-grade weights)
   const float* r1;   // both or neither, one number per head: r1 * ln(1 + r2 * (position - key position)) is taken off the score
   const float* r2;
+  int window, chunk;
 };
 struct QkvFin {
   const float* part;
@@ -258,8 +267,14 @@ __global__ void __launch_bounds__(160) xb_attn_decode_mma_kernel(
   const int slot = m.seq_slot[m.tok_seq[t]];
   const int* pt = m.page_table + (long long)slot * m.max_pages;
   const int n_tiles = pos / XB_ATT_TILE + 1;
-  const int kt0 = (int)(((long long)sp * n_tiles) / n_splits);
-  const int kt1 = (int)(((long long)(sp + 1) * n_tiles) / n_splits);
+  int lo = 0;   // oldest visible key
+  if (!FUSED) {
+    if (opt.window > 0 && pos - opt.window + 1 > 0) lo = pos - opt.window + 1;
+    if (opt.chunk > 0 && pos - pos % opt.chunk > lo) lo = pos - pos % opt.chunk;
+  }
+  const int ktf = lo / XB_ATT_TILE;
+  const int kt0 = ktf + (int)(((long long)sp * (n_tiles - ktf)) / n_splits);
+  const int kt1 = ktf + (int)(((long long)(sp + 1) * (n_tiles - ktf)) / n_splits);
 
   if (threadIdx.x == 0) {
     for (int i = 0; i < NST; ++i) {
@@ -370,7 +385,7 @@ __global__ void __launch_bounds__(160) xb_attn_decode_mma_kernel(
       }
       if (key_abs0 + warp * 16 <= pos) {
         const uint32_t sK = smem_u32(stages + stage * Cfg::STAGE_BYTES);
-        att_warp_block<HD, 1>(qf, sK, sK + Cfg::TILE_BYTES, warp * 16, key_abs0, pos, pos, scale_log2, mrow, lrow, o, opt.softcap, opt.p_split != 0, distp);
+        att_warp_block<HD, 1>(qf, sK, sK + Cfg::TILE_BYTES, warp * 16, key_abs0, pos, pos, scale_log2, mrow, lrow, o, opt.softcap, opt.p_split != 0, distp, lo);
       }
       __syncwarp();
       if (lane == 0) mbar_arrive(&empty_bar[stage]);
@@ -586,9 +601,10 @@ struct AttTcCfg {
 };
 
 // Which keys a query sees besides j <= i.  window > 0: only i - j < window, plus the first `keep_first` keys of the
-// sequence (kept at their true positions); window <= 0: every earlier key (plain causal attention).
+// sequence (kept at their true positions); window <= 0: every earlier key (plain causal attention).  chunk > 0 (EXT kernels): only keys
+// of the query's own chunk of positions, floor(i / chunk) = floor(j / chunk) (keep_first = 0 then).
 struct AttMask {
-  int window, keep_first;
+  int window, keep_first, chunk;
 };
 // Where the query rows come from and what the epilogue does besides the normalisation.  q row of (token t, head h):
 // q + t * ldq + h * HD (+ qbias[h * HD + .] added in fp32 before the bf16 rounding when qbias != nullptr);
@@ -597,7 +613,7 @@ struct AttMask {
 // cap * tanh(s / cap) before the softmax.  v_wide: a row of the value pool holds every key head's values side by side
 // ([page][token][KV * HD]); block z then reads value head z whatever its key head is and writes to
 // out + (token * H + head) * out_head_stride + z * HD, so that every query head meets every value head (grid z = KV).
-// out_head_stride 0 = HD.
+// out_head_stride 0 = HD.  v_wide 2: value heads wider than HD in pieces of HD channels; block z reads piece z of its own head.
 struct AttIo {
   long long ldq;
   const float* qbias;
@@ -665,6 +681,7 @@ __global__ void __launch_bounds__(192, 2) xb_attn_prefill_tc_kernel(
     nkf = kf_tiles < w0 ? kf_tiles : w0;
     skip = w0 - nkf;
   }
+  if (EXT && mk.chunk > 0 && (pos0 - pos0 % mk.chunk) / XB_ATT_TILE > skip) skip = (pos0 - pos0 % mk.chunk) / XB_ATT_TILE;
   const int n_kt = last_pos / XB_ATT_TILE + 1 - skip;
   auto tile_of = [&](int i) { return i < nkf ? i : i + skip; };
 
@@ -722,7 +739,7 @@ __global__ void __launch_bounds__(192, 2) xb_attn_prefill_tc_kernel(
           int page;
           if (i < XB_ATT_PG_CACHE) page = s_pages[i];
           else { const int pi = key / P; page = pt[pi < m.max_pages ? pi : m.max_pages - 1]; }
-          const int row = (EXT && wide) ? page * P + (key % P) : (page * KV + kvh) * P + (key % P);
+          const int row = (EXT && wide && io.v_wide == 1) ? page * P + (key % P) : (page * KV + kvh) * P + (key % P);
 #pragma unroll
           for (int db = 0; db < HD / 64; ++db) tma_load_2d(dst + db * (XB_ATT_TILE * 128) + rg * BR * 128, tm, bar, x0 + db * 64, row);
         }
@@ -831,6 +848,9 @@ __global__ void __launch_bounds__(192, 2) xb_attn_prefill_tc_kernel(
     const float sl2 = (EXT && (io.softcap > 0.f || dist)) ? 1.0f : scale_log2;             // what turns a score in v[] into log2 units
     const float cl2 = io.softcap * 1.4426950408889634f;
     const float cap_k = io.softcap > 0.f ? 2.0f * scale_log2 / io.softcap : 0.f;  // raw product -> 2 s / cap in log2 units
+    // first key of this row's chunk and of the last row's
+    const int chunk_row = (EXT && mk.chunk > 0 && lim > 0) ? lim - lim % mk.chunk : 0;
+    const int chunk_last = (EXT && mk.chunk > 0) ? last_pos - last_pos % mk.chunk : 0;
     for (int kt = 0; kt < n_kt; ++kt) {
       mbar_wait(&s_full[kt & 1], (kt >> 1) & 1);
       tc_fence_after();
@@ -865,8 +885,9 @@ __global__ void __launch_bounds__(192, 2) xb_attn_prefill_tc_kernel(
       }
       // only tiles that reach past the first row's position, or (with a window) back beyond the last row's window,
       // need per-element masks.  The row sees key k when k <= lim and (k >= lo_row or k < kf).
-      const bool masked = key0 + XB_ATT_TILE - 1 > pos0 || (mk.window > 0 && last_pos - key0 >= mk.window);
-      const int lo_row = (mk.window > 0 && lim - mk.window + 1 > 0) ? lim - mk.window + 1 : 0;
+      const bool masked = key0 + XB_ATT_TILE - 1 > pos0 || (mk.window > 0 && last_pos - key0 >= mk.window) || (EXT && key0 < chunk_last);
+      int lo_row = (mk.window > 0 && lim - mk.window + 1 > 0) ? lim - mk.window + 1 : 0;
+      if (EXT) lo_row = max(lo_row, chunk_row);
       const int kf = mk.window > 0 ? mk.keep_first : 0;
       auto vis = [&](int k) { return k <= lim && (k >= lo_row || k < kf); };
       float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};   // independent chains (ILP)

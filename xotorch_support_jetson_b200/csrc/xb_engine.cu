@@ -1304,8 +1304,10 @@ extern "C" int xb_engine_create_hybrid(const xb_hybrid_desc* desc, const xb_hybr
            "a gated residual, a token-pair table and a learned position table are options of branch-norm blocks");
   XB_CHECK(h.bigram_buckets >= 0 && h.pos_rows >= 0 && (h.bigram_buckets == 0 || (h.bigram_mul_prev >= 0 && h.bigram_mul_cur >= 0)),
            "bad token-pair table constants (%d buckets, multipliers %d / %d) or position rows %d", h.bigram_buckets, h.bigram_mul_prev, h.bigram_mul_cur, h.pos_rows);
-  XB_CHECK(h.norm_kind == XB_NORM_RMS || (h.norm_kind == XB_NORM_TANH && h.block == XB_BLOCK_PRENORM && h.norm_scalar == 0),
-           "norm kind %d: the tanh norm belongs to pre-norm blocks, with a weight per channel", h.norm_kind);
+  XB_CHECK(h.norm_kind == XB_NORM_RMS || ((h.norm_kind == XB_NORM_TANH || h.norm_kind == XB_NORM_LAYER) && h.block == XB_BLOCK_PRENORM && h.norm_scalar == 0),
+           "norm kind %d: the tanh and the layer norm belong to pre-norm blocks, with a weight per channel", h.norm_kind);
+  XB_CHECK(h.streams >= 0 && h.streams <= HY_MAX_STREAMS && (h.streams == 0 || (h.block == XB_BLOCK_PRENORM && h.norm_kind != XB_NORM_TANH)),
+           "%d copies of the stream (at most %d): an option of pre-norm blocks with an RMS or layer norm", h.streams, HY_MAX_STREAMS);
   XB_CHECK(h.norm_groups >= 0 && h.norm_groups <= HY_MAX_NORM_GROUPS && (h.norm_groups <= 1 || h.dim % h.norm_groups == 0),
            "norm groups %d must divide dim %d (at most %d)", h.norm_groups, h.dim, HY_MAX_NORM_GROUPS);
   XB_CHECK(h.block == XB_BLOCK_SANDWICH || (h.norm_groups <= 1 && h.norm_plain == 0 && (h.residual_mult == 0.f || h.residual_mult == 1.f) && h.ff_unfiltered == 0),

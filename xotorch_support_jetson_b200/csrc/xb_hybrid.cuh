@@ -56,6 +56,15 @@ struct HyLayer {
   float *qn = nullptr, *kn = nullptr, *r1 = nullptr, *r2 = nullptr;
   // tanh norms of the stream: offset per channel and the factor on the input beside norm1 / norm2
   float *norm1_b = nullptr, *norm1_a = nullptr, *norm2_b = nullptr, *norm2_a = nullptr;
+  // options of softmax attention (xb_qkv_prep.cuh) and the matrix memory, alone or as its second mixer
+  bool prep3 = false;                       // q | k | v reach cache and attention through hy_qkv_prep_kernel
+  int kp = 0, vp = 0, vpieces = 1;          // entries of a key and a value row in the pools; pieces of a value row a tensor-core block reads
+  float *b_o = nullptr, *qkv_conv = nullptr;
+  size_t st_qkv = 0, st_m = 0;              // filter tail of q | k | v, running maxima of the matrix memory
+  int off_mq = 0, off_mk = 0, off_mv = 0, off_mg = 0, off_mi = 0, off_mf = 0, n_left = 0;   // n_left: columns of a1 in front of the second mixer's
+  float *m_norm = nullptr, *choice = nullptr;   // read-out norm of the matrix memory; the router's correction
+  // several copies of the stream: read / write weights and mixing matrix of both sublayers
+  float *hc_in[2] = {nullptr, nullptr}, *hc_out[2] = {nullptr, nullptr}, *hc_mix[2] = {nullptr, nullptr};
   // gated residual: the gate's rows sit behind the mixer's in w_in (off_rg) and behind the experts' in w_up (off_rg2)
   int off_rg = -1, off_rg2 = -1;
 };
@@ -370,21 +379,68 @@ static int hy_create_mixer(xb_engine* e, int i, bool own, size_t& st, uint64_t& 
   return 0;
 }
 
+static int hy_experts_rows(const xb_hybrid_layer& c) { return c.n_experts + c.identity; }   // outputs of the router
+
+// Matrix memory: rows q | k | v | gate of the input matrix at the current end of it (the i and f rows follow when the caller is ready
+// for rows that do not come in eights), state [H][columns][m_dim] and the running maxima.  dst: its output projection's columns.
+static int hy_create_mlstm(xb_engine* e, int i, size_t& st) {
+  HyModel* hy = e->hy;
+  HyLayer& l = hy->L[i];
+  const xb_hybrid_layer& c = l.d;
+  const long long H = c.m_heads, n = c.m_dim, dv = c.m_vdim, dvp = hy_mlstm_cols((int)dv);
+  XB_CHECK(H > 0 && n > 0 && n <= HY_MAX_KDIM && dv > 0 && c.m_gate_cap > 0.f, "layer %d: bad matrix memory sizes (key dim <= %d) or gate cap %g", i, HY_MAX_KDIM,
+           c.m_gate_cap);
+  l.off_mq = l.n_in; l.off_mk = l.off_mq + (int)(H * n); l.off_mv = l.off_mk + (int)(H * n); l.off_mg = l.off_mv + (int)(H * dv);
+  l.n_in = l.off_mg + (int)(H * dv);
+  l.st_rec = st; st += (size_t)(H * dvp * n);
+  l.st_m = st; st += (size_t)((H + 3) & ~3LL);
+  hy_segment_room(hy, H * dvp * n, H);
+  if ((size_t)H > hy->maxH) hy->maxH = H;
+  if ((size_t)(2 * H * n + H * dvp) > hy->maxC) hy->maxC = 2 * H * n + H * dvp;
+  if ((size_t)(H * dvp) > hy->maxO) hy->maxO = H * dvp;
+  return 0;
+}
+// its tensors, once the input matrix has its size; the output projection is columns [n_left, n_o) of w_o
+static int hy_name_mlstm(xb_engine* e, int i, const std::string& p) {
+  HyModel* hy = e->hy;
+  HyLayer& l = hy->L[i];
+  const xb_hybrid_layer& c = l.d;
+  const long long D = hy->d.dim, H = c.m_heads, n = c.m_dim, dv = c.m_vdim;
+  XB_TRY(hy_alloc_t(hy, &l.m_norm, (size_t)(H * dv)));
+  hy_name_rows(hy, p + "q", l.w_in, l.off_mq, H * n, D);
+  hy_name_rows(hy, p + "k", l.w_in, l.off_mk, H * n, D);
+  hy_name_rows(hy, p + "v", l.w_in, l.off_mv, H * dv, D);
+  hy_name_rows(hy, p + "g", l.w_in, l.off_mg, H * dv, D);
+  hy_name_rows(hy, p + "i", l.w_in, l.off_mi, H, D);   hy_name_vec(hy, p + "i.b", l.b_in + l.off_mi, H);
+  hy_name_rows(hy, p + "f", l.w_in, l.off_mf, H, D);   hy_name_vec(hy, p + "f.b", l.b_in + l.off_mf, H);
+  hy_name_vec(hy, p + "norm", l.m_norm, H * dv);
+  hy_name_cols(hy, p + "o", l.w_o, l.n_left, D, H * dv, l.n_o);
+  return 0;
+}
+
 // Rotary-position softmax attention: q | k | v | head gates are the rows of one input matrix; sink, head-mixing matrix and
 // blend factor are fp32 vectors; the rescaled rotary frequencies are made here, in double, from the layer's constants.
-static int hy_create_softmax(xb_engine* e, int i, bool own, uint64_t& wbytes, uint64_t& kvpos) {
+static int hy_create_softmax(xb_engine* e, int i, bool own, size_t& st, uint64_t& wbytes, uint64_t& kvpos) {
   HyModel* hy = e->hy;
   HyLayer& l = hy->L[i];
   const xb_hybrid_layer& c = l.d;
   const xb_hybrid_desc& d = hy->d;
   const size_t D = d.dim;
-  const std::string p = "l" + std::to_string(i) + ".mix.";
+  const bool pair = c.second != 0;
+  const std::string pm = "l" + std::to_string(i) + ".mix.", p = pair ? pm + "left." : pm;
   const long long H = c.s_heads, G = c.s_kv_heads, dk = c.s_dim, dv = c.s_vdim, rd = c.s_rot_dims;
-  XB_CHECK(own, "layer %d: an attention layer keeps tensors of its own", i);
-  XB_CHECK(d.block == XB_BLOCK_SANDWICH || d.block == XB_BLOCK_BRANCHNORM, "layer %d: softmax attention belongs to sandwich or branch-norm blocks", i);
+  XB_CHECK(own || (d.block == XB_BLOCK_PRENORM && !c.s_vmix), "layer %d: an attention layer keeps tensors of its own (outside pre-norm blocks, or when it blends values)", i);
+  XB_CHECK(d.block == XB_BLOCK_SANDWICH || d.block == XB_BLOCK_BRANCHNORM || d.block == XB_BLOCK_PRENORM, "layer %d: softmax attention belongs to sandwich, branch-norm or pre-norm blocks", i);
+  XB_CHECK(c.second == 0 || (c.second == XB_MIX_MLSTM && d.block == XB_BLOCK_PRENORM), "layer %d: the second mixer %d of a layer is a matrix memory, in pre-norm blocks", i, c.second);
+  XB_CHECK(c.s_o_bias == 0 || d.block == XB_BLOCK_PRENORM, "layer %d: a bias on the output projection is an option of pre-norm blocks", i);
+  XB_CHECK(c.s_taps >= 0 && c.s_taps <= HY_MAX_TAPS && c.s_window >= 0 && c.s_chunk >= 0, "layer %d: bad filter taps %d (0..%d), window %d or chunk %d", i, c.s_taps, HY_MAX_TAPS,
+           c.s_window, c.s_chunk);
   XB_CHECK(H > 0 && G > 0 && H % G == 0 && dk > 0 && dv > 0, "layer %d: bad attention sizes", i);
   const bool vk = c.s_v_is_k != 0;
-  const bool prep2 = c.s_qk_norm != 0 || vk || c.s_qtemp_every > 0;   // hy_qk_prep_kernel in place of the rotation kernel
+  l.prep3 = pair || c.s_taps > 0 || c.s_head_norm != 0 || c.s_window > 0 || c.s_chunk > 0 || (c.s_qk_norm != 0 && rd > 0) || d.block == XB_BLOCK_PRENORM;
+  XB_CHECK(!l.prep3 || (!vk && !c.s_vmix && !c.s_talk), "layer %d: a filter, unit heads, a window, chunks or a second mixer come without blended values, mixed heads and key values", i);
+  XB_CHECK(!l.prep3 || (size_t)((H + G) * (dk + 1) + rd) * sizeof(float) <= 48 * 1024, "layer %d: %lld query and key channels per token (at most 12032)", i, (H + G) * dk);
+  const bool prep2 = !l.prep3 && (c.s_qk_norm != 0 || vk || c.s_qtemp_every > 0);   // hy_qk_prep_kernel in place of the rotation kernel
   XB_CHECK(!vk || (dv == dk && !c.s_vmix && !c.s_talk), "layer %d: values that are the keys need equal sizes and neither blending nor mixed heads", i);
   XB_CHECK(!prep2 || (rd == 0 && !c.s_vmix && !c.s_talk), "layer %d: whole-projection norms, key values and the query temperature come without rotation, blending or mixed heads", i);
   XB_CHECK(!prep2 || (size_t)((H + G) * dk) * sizeof(float) <= 48 * 1024, "layer %d: %lld query and key channels per token (at most 12288)", i, (H + G) * dk);
@@ -393,20 +449,56 @@ static int hy_create_softmax(xb_engine* e, int i, bool own, uint64_t& wbytes, ui
   XB_CHECK(c.s_rot_pairs == XB_ROPE_INTERLEAVED || c.s_rot_pairs == XB_ROPE_HALF_SPLIT, "layer %d: unknown rotary pair layout %d", i, c.s_rot_pairs);
   XB_CHECK(c.s_softcap >= 0.f && c.s_scale > 0.f, "layer %d: bad score scale %g / soft cap %g", i, c.s_scale, c.s_softcap);
   l.v_all = c.s_talk != 0 && G > 1;
-  const long long dvo = l.v_all ? G * dv : dv;   // value channels one (token, head) block of the attention kernel carries
+  // bf16 serving, key and value heads of one size (64 or 128), at most 8 query heads per key head: prompts run through the
+  // engine's tcgen05 attention (sink, score cap and the wide value rows of mixed heads as its options).  Behind hy_qkv_prep_kernel any sizes
+  // do: rows are padded to 64 or 128 entries, wider value heads are read in pieces.
+  l.tc_attn = !d.compute_fp32 && dk == dv && (dk == 64 || dk == 128) && H / G <= 8;
+  l.kp = (int)dk; l.vp = (int)dv; l.vpieces = 1;
+  if (l.prep3 && !d.compute_fp32 && dk <= 128 && dv <= 512 && H / G <= 8) {
+    l.tc_attn = true;
+    l.kp = dk <= 64 && dv <= 64 ? 64 : 128;
+    l.vpieces = (int)((dv + l.kp - 1) / l.kp);
+    l.vp = l.vpieces * l.kp;
+  }
+  const long long dvo = l.v_all ? G * dv : l.vp;   // value channels one (token, head) block of the attention kernel carries
   // values that are the keys as projected: no value rows, the value columns ARE the key columns
   l.off_q = 0; l.off_k = (int)(H * dk); l.off_v = vk ? l.off_k : l.off_k + (int)(G * dk); l.off_g = l.off_v + (int)(G * dv);
-  l.n_in = l.off_g + (c.s_gate ? (int)H : 0);
+  l.n_o = l.n_left = (int)(H * dv);
+  if (l.prep3) {   // what comes in eights first, then single rows per head; the matrix ends on a multiple of eight rows
+    l.n_in = l.off_g;
+    if (pair) { XB_TRY(hy_create_mlstm(e, i, st)); l.n_o += c.m_heads * c.m_vdim; }
+    if (c.s_gate) { l.off_g = l.n_in; l.n_in += (int)H; }
+    if (pair) { l.off_mi = l.n_in; l.off_mf = l.off_mi + c.m_heads; l.n_in = l.off_mf + c.m_heads; }
+    l.n_in = (l.n_in + 7) & ~7;
+    if (c.s_taps > 0) { l.st_qkv = st; st += (size_t)(c.s_taps - 1) * (H * dk + G * (dk + dv)); }
+  } else {
+    l.n_in = l.off_g + (c.s_gate ? (int)H : 0);
+  }
   if (d.gated_residual) { l.off_rg = l.n_in; l.n_in += (int)D; }
-  l.n_o = (int)(H * dv);
+  const size_t qa = (size_t)(H * (dk > l.kp ? dk : l.kp)), ol = (size_t)(H * dvo);
+  if (qa > hy->maxQA) hy->maxQA = qa;
+  if (ol > hy->maxO) hy->maxO = ol;
+  if (c.s_vmix && (size_t)(G * dv) > hy->maxGV) hy->maxGV = (size_t)(G * dv);
+  if (l.tc_attn && qa > hy->maxQG) hy->maxQG = qa;
+  kvpos += (uint64_t)G * (l.kp + l.vp) * (d.compute_fp32 ? 4 : 2);
+  if (!own) return 0;   // another layer's tensors
   XB_TRY(hy_alloc_t(hy, &l.w_in, (size_t)l.n_in * D));
   XB_TRY(hy_alloc_t(hy, &l.w_o, D * l.n_o));
   hy_name_rows(hy, p + "q", l.w_in, l.off_q, H * dk, D);
   hy_name_rows(hy, p + "k", l.w_in, l.off_k, G * dk, D);
   if (!vk) hy_name_rows(hy, p + "v", l.w_in, l.off_v, G * dv, D);
   if (c.s_gate) hy_name_rows(hy, p + "g", l.w_in, l.off_g, H, D);
-  hy_name_rows(hy, p + "o", l.w_o, 0, D, l.n_o);
-  if (c.s_qkv_bias || d.gated_residual) XB_TRY(hy_alloc_t(hy, &l.b_in, (size_t)l.n_in));
+  hy_name_cols(hy, p + "o", l.w_o, 0, D, l.n_left, l.n_o);
+  if (c.s_qkv_bias || d.gated_residual || pair) XB_TRY(hy_alloc_t(hy, &l.b_in, (size_t)l.n_in));
+  if (pair) XB_TRY(hy_name_mlstm(e, i, pm + "right."));
+  if (c.s_o_bias) { XB_TRY(hy_alloc_t(hy, &l.b_o, D)); hy_name_vec(hy, p + "o.b", l.b_o, D); }
+  if (c.s_taps > 0) {
+    const long long tp = c.s_taps;
+    XB_TRY(hy_alloc_t(hy, &l.qkv_conv, (size_t)((H * dk + G * (dk + dv)) * tp)));
+    hy_name(hy, p + "q.conv", l.qkv_conv, true, H * dk, tp, tp, 2);
+    hy_name(hy, p + "k.conv", l.qkv_conv + (H * dk) * tp, true, G * dk, tp, tp, 2);
+    hy_name(hy, p + "v.conv", l.qkv_conv + (H * dk + G * dk) * tp, true, G * dv, tp, tp, 2);
+  }
   if (c.s_qkv_bias) {
     hy_name_vec(hy, p + "q.b", l.b_in + l.off_q, H * dk);
     hy_name_vec(hy, p + "k.b", l.b_in + l.off_k, G * dk);
@@ -425,21 +517,13 @@ static int hy_create_softmax(xb_engine* e, int i, bool own, uint64_t& wbytes, ui
   if (c.s_talk) { XB_TRY(hy_alloc_t(hy, &l.talk, (size_t)(H * H))); hy_name(hy, p + "talk", l.talk, true, H, H, H, 2); }
   if (c.s_vmix) { XB_TRY(hy_alloc_t(hy, &l.vmix, 1)); hy_name_vec(hy, p + "vmix", l.vmix, 1); }
   XB_TRY(hy_rot_frequencies(hy, i, (int)rd, c.s_rot_base, c.s_rot_scaling, c.s_rot_factor, c.s_rot_orig, c.s_rot_p0, c.s_rot_p1, &l.rot_freq_d));
-  const size_t qa = (size_t)(H * dk), ol = (size_t)(H * dvo);
-  if (qa > hy->maxQA) hy->maxQA = qa;
-  if (ol > hy->maxO) hy->maxO = ol;
-  if (c.s_vmix && (size_t)(G * dv) > hy->maxGV) hy->maxGV = (size_t)(G * dv);
-  // bf16 serving, key and value heads of one size (64 or 128), at most 8 query heads per key head: prompts run through the
-  // engine's tcgen05 attention (sink, score cap and the wide value rows of mixed heads as its options)
-  l.tc_attn = !d.compute_fp32 && dk == dv && (dk == 64 || dk == 128) && H / G <= 8;
-  if (l.tc_attn && qa > hy->maxQG) hy->maxQG = qa;
   wbytes += ((size_t)l.n_in * D + D * l.n_o) * 2;
-  kvpos += (uint64_t)G * (dk + dv) * (d.compute_fp32 ? 4 : 2);
   return 0;
 }
 
 // Gated feed-forwards: dense (gate | up rows of one matrix, biases) or experts (every expert's gate | up rows, then the
 // shared expert's, in one matrix; every expert's down projection side by side as the columns of one matrix).
+static bool hy_ff_gated(const xb_hybrid_layer& c) { return c.ff_act != XB_ACT_GELU && c.ff_act != XB_ACT_RELU2; }
 static int hy_create_ff(xb_engine* e, int i, bool own, uint64_t& wbytes) {
   HyModel* hy = e->hy;
   HyLayer& l = hy->L[i];
@@ -448,9 +532,9 @@ static int hy_create_ff(xb_engine* e, int i, bool own, uint64_t& wbytes) {
   const std::string p = "l" + std::to_string(i) + ".mlp.";
   XB_CHECK(hy->d.block == XB_BLOCK_PARALLEL || hy->d.block == XB_BLOCK_PRENORM || c.ff_kind == XB_FF_MOE,
            "layer %d: the dense gated feed-forwards belong to parallel and pre-norm blocks", i);
-  XB_CHECK(c.ff_act == XB_ACT_GLU_CLAMP || c.ff_act == XB_ACT_SWIGLU || c.ff_act == XB_ACT_GELU || c.ff_act == XB_ACT_GEGLU,
+  XB_CHECK(c.ff_act == XB_ACT_GLU_CLAMP || c.ff_act == XB_ACT_SWIGLU || c.ff_act == XB_ACT_GELU || c.ff_act == XB_ACT_GEGLU || c.ff_act == XB_ACT_RELU2,
            "layer %d: unknown activation %d", i, c.ff_act);
-  XB_CHECK(c.ff_act != XB_ACT_GELU || (c.ff_kind == XB_FF_MOE && !c.route_input), "layer %d: the ungated GELU form serves experts weighted on their output", i);
+  XB_CHECK(hy_ff_gated(c) || (c.ff_kind == XB_FF_MOE && !c.route_input), "layer %d: the ungated forms serve experts weighted on their output", i);
   XB_CHECK((c.route_score == XB_ROUTE_SIGMOID || c.route_score == XB_ROUTE_SOFTMAX) && (c.group_score == XB_GROUP_TOP2 || c.group_score == XB_GROUP_MAX),
            "layer %d: unknown router score %d / group score %d", i, c.route_score, c.group_score);
   const bool rg = hy->d.gated_residual != 0;
@@ -476,12 +560,14 @@ static int hy_create_ff(xb_engine* e, int i, bool own, uint64_t& wbytes) {
     }
   } else if (c.ff_kind == XB_FF_MOE) {
     const size_t E = c.n_experts, S = c.shared_ff > 0 ? c.shared_ff : 0;
-    const size_t ER = E + (S > 0 && c.shared_gate ? 1 : 0);   // rows of the router's matrix: the shared expert's gate is one more
-    XB_CHECK(E > 0 && c.top > 0 && (size_t)c.top <= E, "layer %d: %d experts, %d per token", i, c.n_experts, c.top);
+    XB_CHECK(E > 0 && c.identity >= 0 && c.top > 0 && c.top <= hy_experts_rows(c), "layer %d: %d experts and %d identity outputs, %d per token", i, c.n_experts, c.identity, c.top);
+    XB_CHECK(c.identity == 0 || (c.groups == 0 && hy->d.norm_kind == XB_NORM_LAYER), "layer %d: identity outputs come without groups, in blocks with a layer norm", i);
+    const size_t EI = hy_experts_rows(c);
+    const size_t ER = EI + (S > 0 && c.shared_gate ? 1 : 0);   // rows of the router's matrix: the shared expert's gate is one more
     XB_CHECK(c.groups == 0 || (c.groups > 0 && E % c.groups == 0 && c.keep_groups > 0 && c.keep_groups <= c.groups &&
                                (size_t)c.top <= (E / c.groups) * c.keep_groups),
              "layer %d: %d groups (%d kept) do not fit %d experts with %d per token", i, c.groups, c.keep_groups, c.n_experts, c.top);
-    const bool gated = c.ff_act != XB_ACT_GELU;   // ungated experts: up rows only, expert after expert, then the shared expert's
+    const bool gated = hy_ff_gated(c);   // ungated experts: up rows only, expert after expert, then the shared expert's
     const size_t U = gated ? 2 : 1;
     l.n_up = (int)(U * (E * F + S)); l.n_dn = (int)(E * F + S);
     if (rg) { l.off_rg2 = l.n_up; l.n_up += (int)D; }   // the residual gate reads what the experts read: its rows follow theirs
@@ -489,8 +575,9 @@ static int hy_create_ff(xb_engine* e, int i, bool own, uint64_t& wbytes) {
       XB_TRY(hy_alloc_t(hy, &l.w_up, (size_t)l.n_up * D));
       XB_TRY(hy_alloc_t(hy, &l.w_down, D * l.n_dn));
       XB_TRY(hy_alloc_t(hy, &l.w_router, ER * D));
-      if (ER > E) hy_name_rows(hy, p + "shared.sg", l.w_router, E, 1, D);
-      hy_name_rows(hy, p + "router", l.w_router, 0, E, D);
+      if (ER > EI) hy_name_rows(hy, p + "shared.sg", l.w_router, EI, 1, D);
+      hy_name_rows(hy, p + "router", l.w_router, 0, EI, D);
+      if (c.route_bias) { XB_TRY(hy_alloc_t(hy, &l.choice, EI)); hy_name_vec(hy, p + "correction", l.choice, EI); }
       for (size_t x = 0; x < E; ++x) {
         const std::string pe = p + "e" + std::to_string(x) + ".";
         if (gated) hy_name_rows(hy, pe + "gate", l.w_up, 2 * x * F, F, D);
@@ -542,9 +629,10 @@ static int hy_create(xb_engine* e, const xb_hybrid_desc& d, const xb_hybrid_laye
     l.owner = -1;
     XB_CHECK(!branchnorm || (own && (c.mixer == XB_MIX_SOFTMAX || c.mixer == XB_MIX_LATENT) && (c.ff == 0 || c.ff_kind == XB_FF_MOE)),
              "layer %d: branch-norm blocks take softmax or latent attention and experts, with tensors of their own", i);
-    XB_CHECK(!prenorm || (own && (c.mixer == XB_MIX_LATENT || c.mixer == XB_MIX_GLA) && (c.ff == 0 || c.ff_kind != XB_FF_RELU2)),
-             "layer %d: pre-norm blocks take latent attention or gated linear attention and gated feed-forwards, with tensors of their own", i);
-    XB_CHECK(prenorm || c.mixer != XB_MIX_GLA, "layer %d: gated linear attention belongs to pre-norm blocks", i);
+    XB_CHECK(!prenorm || c.mixer == XB_MIX_SOFTMAX || c.mixer == XB_MIX_MLSTM || (own && (c.mixer == XB_MIX_LATENT || c.mixer == XB_MIX_GLA)),
+             "layer %d: pre-norm blocks take softmax attention, a matrix memory, latent attention or gated linear attention (the last two with tensors of their own)", i);
+    XB_CHECK(!prenorm || c.ff == 0 || c.ff_kind != XB_FF_RELU2, "layer %d: the dense squared-ReLU feed-forward belongs to sandwich blocks", i);
+    XB_CHECK(prenorm || (c.mixer != XB_MIX_GLA && c.mixer != XB_MIX_MLSTM), "layer %d: gated linear attention and the matrix memory belong to pre-norm blocks", i);
     if (!own) {
       XB_CHECK(c.weights_of < d.n_layers && c.weights_of != i && layers[c.weights_of].weights_of < 0,
                "layer %d: weights_of %d must name another layer that owns its tensors", i, c.weights_of);
@@ -553,7 +641,7 @@ static int hy_create(xb_engine* e, const xb_hybrid_desc& d, const xb_hybrid_laye
                i, c.weights_of);
       l.owner = c.weights_of;
     }
-    XB_CHECK(own || (c.mixer != XB_MIX_DELTA && c.mixer != XB_MIX_PARALLEL && c.mixer != XB_MIX_SOFTMAX), "layer %d: this mixer kind keeps tensors of its own", i);
+    XB_CHECK(own || (c.mixer != XB_MIX_DELTA && c.mixer != XB_MIX_PARALLEL), "layer %d: this mixer kind keeps tensors of its own", i);
     if (own) {
       XB_TRY(hy_create_norm(hy, p + "norm1", &l.norm1, &l.norm1_b, &l.norm1_a));
       if (sandwich) { XB_TRY(hy_alloc_t(hy, &l.norm1b, D)); hy_name_vec(hy, p + "norm1b", l.norm1b, D); }
@@ -635,7 +723,20 @@ static int hy_create(xb_engine* e, const xb_hybrid_desc& d, const xb_hybrid_laye
       wbytes += ((size_t)l.n_in * D + D * l.n_o + D * l.n_o2) * 2;
       kvpos += (uint64_t)G * (dk + dv) * (d.compute_fp32 ? 4 : 2);
     } else if (c.mixer == XB_MIX_SOFTMAX) {
-      XB_TRY(hy_create_softmax(e, i, own, wbytes, kvpos));
+      XB_TRY(hy_create_softmax(e, i, own, st, wbytes, kvpos));
+    } else if (c.mixer == XB_MIX_MLSTM) {
+      l.n_in = 0;
+      XB_TRY(hy_create_mlstm(e, i, st));
+      l.n_o = c.m_heads * c.m_vdim;
+      l.off_mi = l.n_in; l.off_mf = l.off_mi + c.m_heads;
+      l.n_in = (l.off_mf + c.m_heads + 7) & ~7;
+      if (own) {
+        XB_TRY(hy_alloc_t(hy, &l.w_in, (size_t)l.n_in * D));
+        XB_TRY(hy_alloc_t(hy, &l.b_in, (size_t)l.n_in));
+        XB_TRY(hy_alloc_t(hy, &l.w_o, D * l.n_o));
+        XB_TRY(hy_name_mlstm(e, i, p + "mix."));
+        wbytes += ((size_t)l.n_in * D + D * l.n_o) * 2;
+      }
     } else if (c.mixer == XB_MIX_LATENT || c.mixer == XB_MIX_GDELTA || c.mixer == XB_MIX_LIGHTNING || c.mixer == XB_MIX_GLA) {
       XB_TRY(hy_create_mixer(e, i, own, st, wbytes, kvpos));
     } else {
@@ -649,7 +750,7 @@ static int hy_create(xb_engine* e, const xb_hybrid_desc& d, const xb_hybrid_laye
     if ((size_t)l.n_o > hy->maxK) hy->maxK = l.n_o;
     if ((size_t)l.n_o2 > hy->maxK) hy->maxK = l.n_o2;
     if (c.ff > 0 && c.ff_kind != XB_FF_RELU2) {
-      if (branchnorm || prenorm) XB_TRY(hy_create_norm(hy, p + "norm2", &l.norm2, &l.norm2_b, &l.norm2_a));
+      if (branchnorm || (prenorm && own)) XB_TRY(hy_create_norm(hy, p + "norm2", &l.norm2, &l.norm2_b, &l.norm2_a));
       if (sandwich) {   // the feed-forward is a sublayer of its own: norm before and after, optionally the causal filter
         XB_CHECK(own && c.ff_kind == XB_FF_MOE, "layer %d: sandwich blocks take experts with tensors of their own", i);
         XB_TRY(hy_alloc_t(hy, &l.norm2, D)); hy_name_vec(hy, p + "norm2", l.norm2, D);
@@ -675,6 +776,14 @@ static int hy_create(xb_engine* e, const xb_hybrid_desc& d, const xb_hybrid_laye
       if (F > hy->maxK) hy->maxK = F;
       wbytes += 2 * F * D * 2;
     }
+    if (d.streams > 0 && own)
+      for (int q = 0; q < (c.ff > 0 ? 2 : 1); ++q) {
+        const std::string ph = p + (q == 0 ? "hc1." : "hc2.");
+        const size_t s = d.streams;
+        XB_TRY(hy_alloc_t(hy, &l.hc_in[q], s));       hy_name_vec(hy, ph + "in", l.hc_in[q], s);
+        XB_TRY(hy_alloc_t(hy, &l.hc_out[q], s));      hy_name_vec(hy, ph + "out", l.hc_out[q], s);
+        XB_TRY(hy_alloc_t(hy, &l.hc_mix[q], s * s));  hy_name(hy, ph + "mix", l.hc_mix[q], true, s, s, s, 2);
+      }
     if (d.side_dim > 0) {
       const size_t sd = d.side_dim;
       XB_TRY(hy_alloc_t(hy, &l.w_sgate, sd * D)); hy_name_rows(hy, p + "side.gate", l.w_sgate, 0, sd, D);
@@ -702,6 +811,11 @@ static int hy_create(xb_engine* e, const xb_hybrid_desc& d, const xb_hybrid_laye
     const HyLayer& o = hy->L[l.owner];
     l.w_in = o.w_in; l.b_in = o.b_in; l.w_o = o.w_o; l.w_up = o.w_up; l.w_down = o.w_down; l.norm1 = o.norm1; l.head_norm = o.head_norm;
     l.w_uk = o.w_uk; l.w_uv = o.w_uv; l.w_d2 = o.w_d2; l.w_router = o.w_router; l.b_up = o.b_up; l.b_down = o.b_down;
+    XB_CHECK(l.n_in == o.n_in && l.n_o == o.n_o && l.n_up == o.n_up && l.n_dn == o.n_dn && l.kp == o.kp && l.vp == o.vp,
+             "layer %d: its sizes differ from layer %d's, whose tensors it uses", i, l.owner);
+    l.norm2 = o.norm2; l.b_o = o.b_o; l.qkv_conv = o.qkv_conv; l.qn = o.qn; l.kn = o.kn; l.sink = o.sink; l.talk = o.talk; l.r1 = o.r1; l.r2 = o.r2;
+    l.m_norm = o.m_norm; l.choice = o.choice;
+    for (int q = 0; q < 2; ++q) { l.hc_in[q] = o.hc_in[q]; l.hc_out[q] = o.hc_out[q]; l.hc_mix[q] = o.hc_mix[q]; }
     l.lat_norm = o.lat_norm; l.rot_freq_d = o.rot_freq_d; l.w0 = o.w0; l.hdecay = o.hdecay; l.canon1 = o.canon1;
   }
   XB_TRY(hy_alloc_t(hy, &hy->embed, (size_t)d.vocab * D)); hy_name_rows(hy, "embed", hy->embed, 0, d.vocab, D);
@@ -715,7 +829,7 @@ static int hy_create(xb_engine* e, const xb_hybrid_desc& d, const xb_hybrid_laye
   wbytes += (size_t)d.vocab * D * 2;
   const size_t as = d.compute_fp32 ? 4 : 2;
   const size_t R = (size_t)(d.max_logit_rows > d.max_seqs ? d.max_logit_rows : d.max_seqs);
-  XB_TRY(hy_alloc_t(hy, &hy->x, Tm * D));
+  XB_TRY(hy_alloc_t(hy, &hy->x, Tm * D * (d.streams > 1 ? d.streams : 1)));
   XB_TRY(hy_alloc_t(hy, &hy->hn, Tm * D));
   const size_t ws_min = d.compute_fp32 ? 0 : ((size_t)32 << 20);   // room for the split-K planes of decode-sized batches
   hy->cap_P = Tm * hy->maxN * 4 > ws_min ? Tm * hy->maxN * 4 : ws_min;
@@ -925,8 +1039,8 @@ static int hy_reserve(xb_engine* e) {
       continue;
     }
     if (l.d.mixer == XB_MIX_SOFTMAX) {   // keys [page][G][token][dk]; values the same way, or [page][token][G * dv] (v_all)
-      const size_t kb = (size_t)e->n_pages * l.d.s_kv_heads * e->page_tokens * l.d.s_dim * es;
-      const size_t vb = (size_t)e->n_pages * l.d.s_kv_heads * e->page_tokens * l.d.s_vdim * es;
+      const size_t kb = (size_t)e->n_pages * l.d.s_kv_heads * e->page_tokens * l.kp * es;
+      const size_t vb = (size_t)e->n_pages * l.d.s_kv_heads * e->page_tokens * l.vp * es;
       XB_TRY(dmalloc(&l.k_pool, kb));
       XB_TRY(dmalloc(&l.v_pool, vb));
       XB_CUDA(cudaMemset(l.k_pool, 0, kb));
@@ -934,9 +1048,9 @@ static int hy_reserve(xb_engine* e) {
       if (l.tc_attn) {
         const long long G = l.d.s_kv_heads, pool_rows = (long long)e->n_pages * G * e->page_tokens;
         const int box_rows = e->page_tokens < 64 ? e->page_tokens : 64;
-        XB_TRY(xb_make_tmap(&l.tmK, l.k_pool, pool_rows, l.d.s_dim, l.d.s_dim, box_rows));
+        XB_TRY(xb_make_tmap(&l.tmK, l.k_pool, pool_rows, l.kp, l.kp, box_rows));
         if (l.v_all) XB_TRY(xb_make_tmap(&l.tmV, l.v_pool, pool_rows / G, G * l.d.s_vdim, G * l.d.s_vdim, box_rows));
-        else XB_TRY(xb_make_tmap(&l.tmV, l.v_pool, pool_rows, l.d.s_vdim, l.d.s_vdim, box_rows));
+        else XB_TRY(xb_make_tmap(&l.tmV, l.v_pool, pool_rows, l.vp, l.vp, box_rows));
       }
       continue;
     }
@@ -1082,13 +1196,18 @@ static int hy_segments_n(xb_engine* e, const RecurIn& in, float* state, long lon
   sg.max_segs = (T + sg.seg - 1) / sg.seg;
   sg.ws = hy->seg_ws;
   sg.decay = MODE == HY_REC_LIGHTNING ? nullptr : hy->seg_decay;
+  sg.per_head = MODE == HY_REC_MLSTM ? 1 : 0;
   const dim3 grid(cb, H, n_seqs * sg.max_segs);
   constexpr size_t row = (size_t)2 * HY_SEG_TS * sizeof(float);
-  constexpr size_t s0 = row * (hy_seg_vectors(MODE, 0) * 4 * LPC * NCH + HY_SEG_COLS), s1 = row * (hy_seg_vectors(MODE, 1) * 4 * LPC * NCH + HY_SEG_COLS);
+  constexpr int ex = MODE == HY_REC_MLSTM ? 4 : 0;
+  constexpr size_t s0 = row * (hy_seg_vectors(MODE, 0) * 4 * LPC * NCH + HY_SEG_COLS + ex), s1 = row * (hy_seg_vectors(MODE, 1) * 4 * LPC * NCH + HY_SEG_COLS + ex);
   if (s0 > 48 * 1024) XB_SMEM_ATTR_ONCE((hy_seg_kernel<NCH, LPC, MODE, 0>), s0);
   if (s1 > 48 * 1024) XB_SMEM_ATTR_ONCE((hy_seg_kernel<NCH, LPC, MODE, 1>), s1);
   XB_TRY(hy_launch(e, hy_seg_kernel<NCH, LPC, MODE, 0>, grid, dim3(128), s0, st, in, sg, state, ss, o, ldo, m, H, dk, dv));
-  if (sg.decay != nullptr)
+  if (sg.per_head)
+    XB_TRY(hy_launch(e, hy_seg_decay_kernel, dim3((H + 255) / 256, n_seqs * sg.max_segs), dim3(256), 0, st, in.decay, (long long)H, 0LL, H, sg.seg, sg.max_segs,
+                     hy->seg_decay, m));
+  else if (sg.decay != nullptr)
     XB_TRY(hy_launch(e, hy_seg_decay_kernel, dim3((H * dk + 255) / 256, n_seqs * sg.max_segs), dim3(256), 0, st, in.c, in.ldc,
                      MODE == HY_REC_GLA ? in.xoff[0] : in.koff, H * dk, sg.seg, sg.max_segs, hy->seg_decay, m));
   if (dk % 4 == 0)
@@ -1111,7 +1230,7 @@ static int hy_segments(xb_engine* e, const RecurIn& in, float* state, long long 
 template <int MODE>
 static int hy_recur(xb_engine* e, const RecurIn& in, float* state, long long ss, float* o, long long ldo, const BatchMeta& m, int n_seqs,
                     int H, int dk, int dv, int T, cudaStream_t st) {
-  if constexpr (MODE == HY_REC_GLA || MODE == HY_REC_HGRN || MODE == HY_REC_LIGHTNING) {
+  if constexpr (MODE == HY_REC_GLA || MODE == HY_REC_HGRN || MODE == HY_REC_LIGHTNING || MODE == HY_REC_MLSTM) {
     const int least = e->hy->seg_len > 0 ? 2 * e->hy->seg_len : 4 * HY_SEG_MIN;   // average length from which it pays
     if (e->hy->use_seg && T / n_seqs >= least && (long long)n_seqs * (T / HY_SEG_MIN + 1) <= 65535)   // grid z
       return hy_segments<MODE>(e, in, state, ss, o, ldo, m, n_seqs, H, dk, dv, T, st);
@@ -1199,10 +1318,11 @@ template <int HD, int GRP>
 static int hy_attn_tc_any_g(xb_engine* e, const HyLayer& l, const BatchMeta& m, const HyAttnIn& in, bf16* out, int H, int KV, float scale, int gz,
                             cudaStream_t st) {
   using Cfg = AttTcCfg<HD>;
+  const AttMask mk{l.d.s_window, 0, l.d.s_chunk};
   XB_SMEM_ATTR_ONCE((xb_attn_prefill_tc_kernel<HD, GRP, true>), Cfg::SMEM_BYTES);
   e->c.tc_attention++;
   return hy_launch(e, xb_attn_prefill_tc_kernel<HD, GRP, true>, dim3(in.n_tiles, KV, gz), dim3(192), Cfg::SMEM_BYTES, st, l.tmK, l.tmV, in.q, m,
-                   in.tile_start, in.tile_len, out, H, KV, scale * 1.4426950408889634f, AttMask{0, 0}, in.io);
+                   in.tile_start, in.tile_len, out, H, KV, scale * 1.4426950408889634f, mk, in.io);
 }
 template <int HD>
 static int hy_attn_tc_any(xb_engine* e, const HyLayer& l, const BatchMeta& m, const HyAttnIn& in, bf16* out, int H, int KV, float scale, int gz,
@@ -1229,7 +1349,7 @@ static int hy_attn_dec_g(xb_engine* e, const HyLayer& l, const BatchMeta& m, int
   using Cfg = AttDecCfg<HD, GRP, NST>;
   auto kern = xb_attn_decode_mma_kernel<HD, GRP, NST, false>;
   XB_SMEM_ATTR_ONCE(kern, Cfg::SMEM_BYTES);
-  const dim3 grid(T, opt.v_wide ? KV * KV : KV, n_splits);
+  const dim3 grid(T, opt.v_wide == 1 ? KV * KV : (opt.v_wide == 2 ? KV * (int)(opt.out_head_stride / HD) : KV), n_splits);
   return launch_kc(e, kern, grid, dim3(160), Cfg::SMEM_BYTES, st, dim3(1, 1, n_splits), l.tmK, l.tmV, q, m, (float*)nullptr, (float*)nullptr, out,
                    H, KV, n_splits, scale * 1.4426950408889634f, QkvFin{}, n_splits > 1 ? 1 : 0, opt);
 }
@@ -1437,13 +1557,14 @@ template <typename AT>
 static int hy_router(xb_engine* e, const HyLayer& l, int T, const void* xin, int sg, cudaStream_t st) {
   HyModel* hy = e->hy;
   const xb_hybrid_layer& c = l.d;
-  const int D = hy->d.dim, NE = c.n_experts + sg;
+  const int D = hy->d.dim, EI = hy_experts_rows(c), NE = EI + sg;
   const AT* x = reinterpret_cast<const AT*>(xin);
+  const float* choice = l.choice;
   const int ng = c.groups > 0 ? c.groups : 1;
   if (T <= 64 && hy->fuse_router) {   // few rows: logits and routing of a token in one block
-    const size_t rs1 = (size_t)(2 * c.n_experts + NE + ng) * sizeof(float);
-    return hy_launch(e, hy_router_route_kernel<AT>, dim3(T), dim3(32 * (NE < 32 ? (NE < 8 ? 8 : NE) : 32)), rs1, st, x, (long long)D, (const bf16*)l.w_router, D, c.n_experts, c.top, c.groups,
-                     c.keep_groups, c.route_scale, hy->gw, c.route_score, c.group_score, c.route_norm, sg);
+    const size_t rs1 = (size_t)(2 * EI + NE + ng) * sizeof(float);
+    return hy_launch(e, hy_router_route_kernel<AT>, dim3(T), dim3(32 * (NE < 32 ? (NE < 8 ? 8 : NE) : 32)), rs1, st, x, (long long)D, (const bf16*)l.w_router, D, EI, c.top, c.groups,
+                     c.keep_groups, c.route_scale, hy->gw, c.route_score, c.group_score, c.route_norm, sg, choice);
   }
   if (T <= 64) {   // few rows: a warp per (token, expert)
     XB_TRY(hy_launch(e, hy_router_logits_kernel<AT, 1>, dim3((unsigned)(((long long)T * NE + 7) / 8)), dim3(256), 0, st, x, (long long)D,
@@ -1457,9 +1578,9 @@ static int hy_router(xb_engine* e, const HyLayer& l, int T, const void* xin, int
     XB_TRY(hy_launch(e, hy_router_logits_kernel<AT, 8>, dim3((unsigned)(((long long)T * chunks + 7) / 8)), dim3(256), 0, st, x, (long long)D,
                      (const bf16*)l.w_router, hy->m2, T, NE, D));
   }
-  const size_t rs = (size_t)4 * (2 * c.n_experts + ng) * sizeof(float);
-  return hy_launch(e, hy_route_kernel, dim3((T + 3) / 4), dim3(128), rs, st, (const float*)hy->m2, c.n_experts, c.top, c.groups, c.keep_groups,
-                   c.route_scale, hy->gw, T, c.route_score, c.group_score, c.route_norm, sg);
+  const size_t rs = (size_t)4 * (2 * EI + ng) * sizeof(float);
+  return hy_launch(e, hy_route_kernel, dim3((T + 3) / 4), dim3(128), rs, st, (const float*)hy->m2, EI, c.top, c.groups, c.keep_groups,
+                   c.route_scale, hy->gw, T, c.route_score, c.group_score, c.route_norm, sg, choice);
 }
 
 // xin: the normed stream as a Linear input [T, dim] of AT
@@ -1472,13 +1593,15 @@ static int hy_ff_parallel(xb_engine* e, const HyLayer& l, int T, const void* xin
   // Steps of so few rows that at most half of the experts can have a token: read the chosen experts' rows only (two kernels
   // in place of the wide up Linear, the activation and the wide down Linear).
   const int sf = c.ff_kind == XB_FF_MOE && c.shared_ff > 0 ? c.shared_ff : 0, sg = sf > 0 && c.shared_gate ? 1 : 0;
-  const int ldg = c.n_experts + sg;   // a routing row: the experts' weights, then the shared expert's
-  if (c.ff_kind == XB_FF_MOE && hy->use_gather && c.ff_act != XB_ACT_GELU && l.b_up == nullptr && l.b_down == nullptr && D % 8 == 0 && c.ff % 8 == 0 &&
+  const int ldg = hy_experts_rows(c) + sg;   // a routing row: the weights of the router's outputs, then the shared expert's
+  const int sg_at = sg ? hy_experts_rows(c) : -1;
+  if (c.ff_kind == XB_FF_MOE && hy->use_gather && l.b_up == nullptr && l.b_down == nullptr && D % 8 == 0 && c.ff % 8 == 0 &&
       sf % 8 == 0 && 2LL * T * c.top <= c.n_experts) {
     XB_TRY(hy_router<AT>(e, l, T, xin, sg, st));
     const long long per = (long long)c.top * c.ff + sf, nu = (long long)T * per, nd = (long long)T * D;
-    XB_TRY(hy_launch(e, hy_moe_gather_up_kernel<AT>, dim3((unsigned)((nu + 7) / 8)), dim3(256), 0, st, reinterpret_cast<const AT*>(xin), (long long)D,
-                     (const bf16*)l.w_up, (const float*)hy->gw, ldg, c.n_experts, c.top, c.ff, sf, D, c.ff_limit, c.shared_limit, c.ff_act, c.route_input, a2, T));
+    auto up = hy_ff_gated(c) ? hy_moe_gather_up_kernel<AT, true> : hy_moe_gather_up_kernel<AT, false>;
+    XB_TRY(hy_launch(e, up, dim3((unsigned)((nu + 7) / 8)), dim3(256), 0, st, reinterpret_cast<const AT*>(xin), (long long)D,
+                     (const bf16*)l.w_up, (const float*)hy->gw, ldg, sg_at, c.n_experts, c.top, c.ff, sf, D, c.ff_limit, c.shared_limit, c.ff_act, c.route_input, a2, T));
     XB_TRY(hy_launch(e, hy_moe_gather_down_kernel<AT>, dim3((unsigned)((nd + 7) / 8)), dim3(256), 0, st, (const AT*)a2, (const bf16*)l.w_down,
                      (const float*)hy->gw, ldg, c.n_experts, c.top, c.ff, sf, D, hy->m2, T));   // m2: router logits there are spent
     *y = hy_plain(hy->m2, D);
@@ -1500,18 +1623,18 @@ static int hy_ff_parallel(xb_engine* e, const HyLayer& l, int T, const void* xin
   } else {
     XB_TRY(hy_router<AT>(e, l, T, xin, sg, st));
     const long long n = (long long)T * l.n_dn;
-    if (c.ff_act == XB_ACT_GELU) {   // experts without a gate projection
+    if (!hy_ff_gated(c)) {   // experts without a gate projection
       if (vec && c.ff % 8 == 0 && sf % 8 == 0)
-        XB_TRY(hy_launch(e, hy_moe_act1_vec_kernel, dim3((unsigned)((n / 8 + 255) / 256)), dim3(256), 0, st, U.h, U.ld, (const float*)hy->gw, ldg, c.n_experts,
-                         c.ff, sf, reinterpret_cast<bf16*>(hy->a2), (long long)l.n_dn, T));
+        XB_TRY(hy_launch(e, hy_moe_act1_vec_kernel, dim3((unsigned)((n / 8 + 255) / 256)), dim3(256), 0, st, U.h, U.ld, (const float*)hy->gw, ldg, sg_at, c.n_experts,
+                         c.ff, sf, c.ff_act, reinterpret_cast<bf16*>(hy->a2), (long long)l.n_dn, T));
       else
-        XB_TRY(hy_launch(e, hy_moe_act1_kernel<AT>, dim3((unsigned)((n + 255) / 256)), dim3(256), 0, st, U, (const float*)hy->gw, ldg, c.n_experts, c.ff, sf,
+        XB_TRY(hy_launch(e, hy_moe_act1_kernel<AT>, dim3((unsigned)((n + 255) / 256)), dim3(256), 0, st, U, (const float*)hy->gw, ldg, sg_at, c.n_experts, c.ff, sf, c.ff_act,
                          a2, (long long)l.n_dn, T));
     } else if (vec && c.ff % 8 == 0 && sf % 8 == 0)
-      XB_TRY(hy_launch(e, hy_moe_act_vec_kernel, dim3((unsigned)((n / 8 + 255) / 256)), dim3(256), 0, st, U.h, U.ld, (const float*)hy->gw, ldg, c.n_experts,
+      XB_TRY(hy_launch(e, hy_moe_act_vec_kernel, dim3((unsigned)((n / 8 + 255) / 256)), dim3(256), 0, st, U.h, U.ld, (const float*)hy->gw, ldg, sg_at, c.n_experts,
                        c.ff, c.ff_limit, sf, c.shared_limit, c.ff_act, c.route_input, reinterpret_cast<bf16*>(hy->a2), (long long)l.n_dn, T));
     else
-      XB_TRY(hy_launch(e, hy_moe_act_kernel<AT>, dim3((unsigned)((n + 255) / 256)), dim3(256), 0, st, U, (const float*)hy->gw, ldg, c.n_experts, c.ff,
+      XB_TRY(hy_launch(e, hy_moe_act_kernel<AT>, dim3((unsigned)((n + 255) / 256)), dim3(256), 0, st, U, (const float*)hy->gw, ldg, sg_at, c.n_experts, c.ff,
                        c.ff_limit, sf, c.shared_limit, c.ff_act, c.route_input, a2, (long long)l.n_dn, T));
   }
   return hy_linear<AT>(e, a2, l.n_dn, l.w_down, l.t_down, l.b_down, T, D, l.n_dn, hy->m2, hy->cap_m, st, y);
@@ -1597,12 +1720,14 @@ static int hy_heads_mix_bf16(xb_engine* e, const HyLayer& l, int T, const LinOut
   const xb_hybrid_layer& c = l.d;
   const int H = c.s_heads, G = l.v_all ? c.s_kv_heads : 1, dv = c.s_vdim;
   const float* talk = c.s_talk ? (const float*)l.talk : (const float*)nullptr;
+  const int ohs = l.prep3 ? l.vp : dv;
+  const float os = c.second ? c.left_scale : 1.0f;
   AT* a1 = reinterpret_cast<AT*>(hy->a1);
   if (dv % 8 == 0)
     return hy_launch(e, hy_heads_mix_vec_kernel<AT>, dim3(T, (H * dv / 8 + 255) / 256), dim3(256), 0, st, (const bf16*)hy->o, talk, P,
-                     c.s_gate ? l.off_g : -1, H, G, dv, a1, (long long)l.n_o);
+                     c.s_gate ? l.off_g : -1, H, G, dv, a1, (long long)l.n_o, ohs, os);
   return hy_launch(e, hy_heads_mix_kernel<AT, bf16>, dim3(T, (H * dv + 255) / 256), dim3(256), 0, st, (const bf16*)hy->o, talk, P,
-                   c.s_gate ? l.off_g : -1, H, G, dv, a1, (long long)l.n_o);
+                   c.s_gate ? l.off_g : -1, H, G, dv, a1, (long long)l.n_o, ohs, os);
 }
 
 template <typename AT>
@@ -1624,7 +1749,31 @@ static int hy_softmax_mixer(xb_engine* e, const HyLayer& l, int T, int n_seqs, i
   const int rope_by = T >= 512 ? 1 : (units + 255) / 256;
   const bool rope_vec = tc && P.h != nullptr && P.bias == nullptr && P.ld % 8 == 0 && dk % 8 == 0 && dv % 8 == 0 &&
                         c.s_rot_dims % (r.half ? 16 : 8) == 0 && (G * dv) % 8 == 0;
-  if (c.s_qk_norm != 0 || c.s_v_is_k != 0 || c.s_qtemp_every > 0) {   // no rotation: whole-projection norms, temperature, append
+  if (l.prep3) {   // filter, norms, rotation, unit heads, append
+    QkvPrep a;
+    a.off_q = l.off_q; a.H = H; a.G = G; a.dk = dk; a.dv = dv; a.kp = l.kp; a.vp = l.vp;
+    a.taps = c.s_taps; a.conv_w = l.qkv_conv; a.tail = c.s_taps > 1 ? hy->state + l.st_qkv : nullptr; a.tail_stride = (long long)hy->state_floats;
+    a.write_tail = c.s_taps > 1 && T == n_seqs ? 1 : 0;
+    a.qn = c.s_qk_norm ? l.qn : nullptr; a.kn = c.s_qk_norm ? l.kn : nullptr; a.eps = hy->d.norm_eps;
+    a.temp_coef = c.s_qtemp_coef; a.temp_every = c.s_qtemp_every;
+    a.rot = r; a.head_norm = c.s_head_norm;
+    a.qa = (tc || dec) ? (float*)nullptr : hy->qa;
+    a.qg = (tc || dec) ? hy->qg : (bf16*)nullptr;
+    const size_t sm = (size_t)((H + G) * (dk + 1) + c.s_rot_dims) * sizeof(float);
+    bool vec8 = false;
+    if constexpr (std::is_same<KT, bf16>::value) vec8 = T > 64 && P.h != nullptr && P.ld % 8 == 0 && dk % 8 == 0 && dv % 8 == 0 && l.off_q % 8 == 0;
+    if (vec8) {
+      if constexpr (std::is_same<KT, bf16>::value)
+        XB_TRY(hy_launch(e, hy_qkv_prep_kernel<KT, 256, 8>, dim3(T), dim3(256), sm, st, P, a, (KT*)l.k_pool, (KT*)l.v_pool, m));
+    } else if (T <= 64)
+      XB_TRY(hy_launch(e, hy_qkv_prep_kernel<KT, 1024, 1>, dim3(T), dim3(1024), sm, st, P, a, (KT*)l.k_pool, (KT*)l.v_pool, m));
+    else
+      XB_TRY(hy_launch(e, hy_qkv_prep_kernel<KT, 256, 1>, dim3(T), dim3(256), sm, st, P, a, (KT*)l.k_pool, (KT*)l.v_pool, m));
+    if (c.s_taps > 1 && !a.write_tail) {
+      const int C = H * dk + G * (dk + dv);
+      XB_TRY(hy_launch(e, hy_tail_update_kernel, dim3(n_seqs, (C + 255) / 256), dim3(256), 0, st, P, l.off_q, C, c.s_taps, a.tail, a.tail_stride, m));
+    }
+  } else if (c.s_qk_norm != 0 || c.s_v_is_k != 0 || c.s_qtemp_every > 0) {   // no rotation: whole-projection norms, temperature, append
     const float* qn = c.s_qk_norm ? (const float*)l.qn : (const float*)nullptr;
     const float* kn = c.s_qk_norm ? (const float*)l.kn : (const float*)nullptr;
     float* qa = (tc || dec) ? (float*)nullptr : hy->qa;          // fp32 queries for the per-(token, head) kernel only
@@ -1652,17 +1801,23 @@ static int hy_softmax_mixer(xb_engine* e, const HyLayer& l, int T, int n_seqs, i
   XB_TRY(hy_launch(e, hy_rope_append_kernel<KT>, dim3(T, rope_by), dim3(256), 0, st, P, l.off_q, l.off_k, l.off_v, H, G, dk, dv, r,
                    hy->qa, (tc || dec) ? hy->qg : (bf16*)nullptr, (KT*)l.k_pool, (KT*)l.v_pool, l.v_all ? 1 : 0, (const float*)l.vmix, hy->vfirst,
                    l.vmode, m));
-  const int dvo = l.v_all ? G * dv : dv;
+  const int dvo = l.v_all ? G * dv : dv;   // value channels of a (token, head) block of the per-token kernel
   const int vch = dvo > 512 ? 512 : 0;   // wider value rows: blocks along z take 512 channels each
-  const AttnOpt opt{c.s_sink ? l.sink : nullptr, c.s_softcap, l.v_all ? 1 : G, vch, c.s_dist_bias ? l.r1 : nullptr, c.s_dist_bias ? l.r2 : nullptr};
-  const bool post = c.s_talk != 0 || c.s_gate != 0;
+  const AttnOpt opt{c.s_sink ? l.sink : nullptr, c.s_softcap, l.v_all ? 1 : G, vch, c.s_dist_bias ? l.r1 : nullptr, c.s_dist_bias ? l.r2 : nullptr, c.s_chunk};
+  // padded rows and a second mixer's columns beside this one's go through the head kernel as well
+  const bool post = c.s_talk != 0 || c.s_gate != 0 || c.second != 0 || ((tc || dec) && l.vp != dv);
+  const int wide = l.v_all ? 1 : (l.vpieces > 1 ? 2 : 0);
+  const long long ohs = l.v_all ? (long long)G * dv : l.vp;
+  const int HD = l.kp;
   if (dec) {
     // mixed heads multiply the blocks by the key heads: fewer splits keep the grid near one wave
     int ns = l.v_all ? hy->dec_splits / G : hy->dec_splits;
+    const int span = c.s_window > 0 && (c.s_chunk <= 0 || c.s_window < c.s_chunk) ? c.s_window : c.s_chunk;   // most keys a query sees, 0 = all
+    if (span > 0 && ns > (span + XB_ATT_TILE - 2) / XB_ATT_TILE + 1) ns = (span + XB_ATT_TILE - 2) / XB_ATT_TILE + 1;
     ns = ns < 1 ? 1 : ns;
-    const AttDecOpt dopt{c.s_sink ? l.sink : nullptr, c.s_softcap, l.v_all ? 1 : 0, (long long)dvo, hy->p_split, opt.r1, opt.r2};
+    const AttDecOpt dopt{c.s_sink ? l.sink : nullptr, c.s_softcap, wide, ohs, hy->p_split, opt.r1, opt.r2, c.s_window, c.s_chunk};
     bf16* dst = post ? reinterpret_cast<bf16*>(hy->o) : reinterpret_cast<bf16*>(hy->a1);
-    if (dk == 128) XB_TRY(hy_attn_dec<128>(e, l, m, T, hy->qg, dst, H, G, c.s_scale, ns, dopt, st));
+    if (HD == 128) XB_TRY(hy_attn_dec<128>(e, l, m, T, hy->qg, dst, H, G, c.s_scale, ns, dopt, st));
     else XB_TRY(hy_attn_dec<64>(e, l, m, T, hy->qg, dst, H, G, c.s_scale, ns, dopt, st));
     if (post) XB_TRY(hy_heads_mix_bf16<AT>(e, l, T, P, st));
     return 0;
@@ -1670,14 +1825,16 @@ static int hy_softmax_mixer(xb_engine* e, const HyLayer& l, int T, int n_seqs, i
   if (tc) {
     HyAttnIn in;
     in.tile_start = m.tile_start; in.tile_len = m.tile_len; in.n_tiles = n_tiles; in.q = hy->qg;
-    in.io = AttIo{(long long)H * dk, nullptr, nullptr, 0, c.s_sink ? l.sink : nullptr, c.s_softcap, l.v_all ? 1 : 0, (long long)dvo, hy->p_split, opt.r1, opt.r2};
+    in.io = AttIo{(long long)H * l.kp, nullptr, nullptr, 0, c.s_sink ? l.sink : nullptr, c.s_softcap, wide, ohs, hy->p_split, opt.r1, opt.r2};
     bf16* dst = post ? reinterpret_cast<bf16*>(hy->o) : reinterpret_cast<bf16*>(hy->a1);
-    if (dk == 128) XB_TRY(hy_attn_tc_any<128>(e, l, m, in, dst, H, G, c.s_scale, l.v_all ? G : 1, st));
-    else XB_TRY(hy_attn_tc_any<64>(e, l, m, in, dst, H, G, c.s_scale, l.v_all ? G : 1, st));
+    if (HD == 128) XB_TRY(hy_attn_tc_any<128>(e, l, m, in, dst, H, G, c.s_scale, l.v_all ? G : l.vpieces, st));
+    else XB_TRY(hy_attn_tc_any<64>(e, l, m, in, dst, H, G, c.s_scale, l.v_all ? G : l.vpieces, st));
     if (post) XB_TRY(hy_heads_mix_bf16<AT>(e, l, T, P, st));
     return 0;
   }
-  const int aw = 16, far = 1 << 30;   // causal over the whole sequence: the block's warps share out all earlier keys
+  const int far = c.s_window > 0 ? c.s_window : 1 << 30;   // no window: the block's warps share out all earlier keys
+  const int most = c.s_chunk > 0 && c.s_chunk < far ? c.s_chunk : far;
+  const int aw = most >= 512 ? 16 : (most + 31) / 32;
   const size_t asm_bytes = (size_t)(((dk + 3) & ~3) + aw * (2 + (vch ? vch : dvo))) * sizeof(float);
   const LinOut Q = hy_plain(hy->qa, (long long)H * dk);
   const KT* kp = (const KT*)l.k_pool;
@@ -1685,19 +1842,20 @@ static int hy_softmax_mixer(xb_engine* e, const HyLayer& l, int T, int n_seqs, i
   const dim3 grid(T, H, vch ? (dvo + vch - 1) / vch : 1), block(32 * aw);
   if (post) {
     if (dvo <= 256)
-      XB_TRY(hy_launch(e, hy_attn_window_kernel<KT, float, 8>, grid, block, asm_bytes, st, Q, 0, -1, kp, vp, m, H, G, dk, dvo, dk, dvo, far, 0,
+      XB_TRY(hy_launch(e, hy_attn_window_kernel<KT, float, 8>, grid, block, asm_bytes, st, Q, 0, -1, kp, vp, m, H, G, dk, dvo, l.kp, l.v_all ? dvo : l.vp, far, 0,
                        c.s_scale, 1.0f, hy->o, (long long)H * dvo, opt));
     else
-      XB_TRY(hy_launch(e, hy_attn_window_kernel<KT, float, 16>, grid, block, asm_bytes, st, Q, 0, -1, kp, vp, m, H, G, dk, dvo, dk, dvo, far, 0,
+      XB_TRY(hy_launch(e, hy_attn_window_kernel<KT, float, 16>, grid, block, asm_bytes, st, Q, 0, -1, kp, vp, m, H, G, dk, dvo, l.kp, l.v_all ? dvo : l.vp, far, 0,
                        c.s_scale, 1.0f, hy->o, (long long)H * dvo, opt));
     XB_TRY(hy_launch(e, hy_heads_mix_kernel<AT, float>, dim3(T, (H * dv + 255) / 256), dim3(256), 0, st, (const float*)hy->o,
-                     c.s_talk ? (const float*)l.talk : (const float*)nullptr, P, c.s_gate ? l.off_g : -1, H, l.v_all ? G : 1, dv, a1, (long long)l.n_o));
+                     c.s_talk ? (const float*)l.talk : (const float*)nullptr, P, c.s_gate ? l.off_g : -1, H, l.v_all ? G : 1, dv, a1, (long long)l.n_o, dvo,
+                     c.second ? c.left_scale : 1.0f));
   } else {
     if (dvo <= 256)
-      XB_TRY(hy_launch(e, hy_attn_window_kernel<KT, AT, 8>, grid, block, asm_bytes, st, Q, 0, -1, kp, vp, m, H, G, dk, dvo, dk, dvo, far, 0,
+      XB_TRY(hy_launch(e, hy_attn_window_kernel<KT, AT, 8>, grid, block, asm_bytes, st, Q, 0, -1, kp, vp, m, H, G, dk, dvo, l.kp, l.v_all ? dvo : l.vp, far, 0,
                        c.s_scale, 1.0f, a1, (long long)l.n_o, opt));
     else
-      XB_TRY(hy_launch(e, hy_attn_window_kernel<KT, AT, 16>, grid, block, asm_bytes, st, Q, 0, -1, kp, vp, m, H, G, dk, dvo, dk, dvo, far, 0,
+      XB_TRY(hy_launch(e, hy_attn_window_kernel<KT, AT, 16>, grid, block, asm_bytes, st, Q, 0, -1, kp, vp, m, H, G, dk, dvo, l.kp, l.v_all ? dvo : l.vp, far, 0,
                        c.s_scale, 1.0f, a1, (long long)l.n_o, opt));
   }
   return 0;
@@ -1777,12 +1935,59 @@ static int hy_head_norm(xb_engine* e, int T, long long ldo, const float* w, cons
                    out, ld_out, H, dv, w_hstride, gate_sigmoid);
 }
 
+// The stream as several copies (or one) with the norm that reads it next: hy_hyper_kernel, four channels per thread where rows and branch allow.
+template <typename AT>
+static int hy_hyper(xb_engine* e, int T, const HyperArgs& a, cudaStream_t st) {
+  const int D = a.D, n = a.n;
+  const size_t sm = (size_t)D * sizeof(float);
+  const bool plain = a.y.f == nullptr || a.y.si.splits == 0;
+  const bool vec = D % 4 == 0 && plain && ((a.y.f == nullptr && a.y.h == nullptr) || a.y.ld % 4 == 0);
+  if (T <= 64 && D >= 1024 && !vec) {   // few rows out of split-K planes: more threads per row keep more loads in flight
+    if (n <= 4) return hy_launch(e, hy_hyper_kernel<AT, 1024, 4, 1>, dim3(T), dim3(1024), sm, st, a);
+    return hy_launch(e, hy_hyper_kernel<AT, 1024, HY_MAX_STREAMS, 1>, dim3(T), dim3(1024), sm, st, a);
+  }
+  if (n <= 4) {
+    if (vec) return hy_launch(e, hy_hyper_kernel<AT, 256, 4, 4>, dim3(T), dim3(256), sm, st, a);
+    return hy_launch(e, hy_hyper_kernel<AT, 256, 4, 1>, dim3(T), dim3(256), sm, st, a);
+  }
+  return hy_launch(e, hy_hyper_kernel<AT, 256, HY_MAX_STREAMS, 1>, dim3(T), dim3(256), sm, st, a);
+}
+
+// Matrix memory of one layer, from its columns of the projection to columns [n_left, n_o) of a1, times `scale`.
+template <typename AT>
+static int hy_mlstm_mixer(xb_engine* e, const HyLayer& l, int T, int n_seqs, const LinOut& P, float out_scale, const BatchMeta& m, cudaStream_t st) {
+  HyModel* hy = e->hy;
+  const xb_hybrid_layer& c = l.d;
+  const int H = c.m_heads, n = c.m_dim, dv = c.m_vdim, dvp = hy_mlstm_cols(dv), HK = H * n;
+  const long long SS = (long long)hy->state_floats, ldo = (long long)H * dvp, ldc = 2LL * HK + ldo;
+  const float scale = 1.0f / sqrtf((float)n), eps = hy->d.norm_eps;
+  AT* out = reinterpret_cast<AT*>(hy->a1) + (c.mixer == XB_MIX_MLSTM ? 0 : l.n_left);
+  float *rec = hy->state + l.st_rec, *ms = hy->state + l.st_m;
+  const size_t tsm = (size_t)(2 * ((n + 3) & ~3) + 3 * dv + 1) * sizeof(float);
+  if (T == n_seqs && tsm <= 48 * 1024)   // single tokens
+    return hy_launch(e, hy_mlstm_token_kernel<AT>, dim3(n_seqs, H), dim3(512), tsm, st, P, l.off_mq, l.off_mk, l.off_mv, l.off_mg, l.off_mi, l.off_mf, c.m_gate_cap,
+                     scale, rec, ms, SS, (const float*)l.m_norm, eps, out_scale, out, (long long)l.n_o, m, H, n, dv);
+  XB_TRY(hy_launch(e, hy_mlstm_gates_kernel, dim3(H, n_seqs), dim3(256), 0, st, P, l.off_mi, l.off_mf, c.m_gate_cap, ms, SS, hy->decay, hy->beta, hy->qk, H, m));
+  const bool vec = P.h != nullptr && ((P.ld | l.off_mq | l.off_mk | l.off_mv | n | dv) & 7) == 0;
+  const int units = vec ? (2 * HK + H * dv) / 8 + H : 2 * HK + H * dv + H;
+  auto prep = vec ? hy_mlstm_prep_kernel<8> : hy_mlstm_prep_kernel<1>;
+  XB_TRY(hy_launch(e, prep, dim3(T, (units + 255) / 256), dim3(256), 0, st, P, l.off_mq, l.off_mk, l.off_mv, scale, (const float*)hy->beta, hy->c, ldc, H, n, dv));
+  RecurIn in;
+  in.c = hy->c; in.ldc = ldc; in.qoff = 0; in.koff = HK; in.voff = 2LL * HK; in.q_heads = H;
+  in.xoff[0] = in.xoff[1] = in.xoff[2] = 0;
+  in.beta = in.qk = in.hdecay = nullptr; in.decay = hy->decay;
+  XB_TRY(hy_recur<HY_REC_MLSTM>(e, in, rec, SS, hy->o, ldo, m, n_seqs, H, n, dvp, T, st));
+  return hy_launch(e, hy_mlstm_out_kernel<AT>, dim3((unsigned)(((long long)T * H + 7) / 8)), dim3(256), 0, st, (const float*)hy->o, (const float*)hy->qk,
+                   (const float*)l.m_norm, P, l.off_mg, eps, out_scale, out, (long long)l.n_o, T, H, dv);
+}
+
 // ----------------------------------------------------------------------------- pre-norm blocks
 // x <- embed * scale;  per layer  x += mixer(f1(x)),  x += ff(f2(x)).  Every norm rides in the kernel that last changed x: the
 // embedding kernel makes the first layer's, the residual additions the next reader's.  The tanh norm needs no statistics of the row
-// (hy_add_tanh_kernel); the RMS form is hy_row_op_kernel's plain addition.
+// (hy_add_tanh_kernel); the RMS form is hy_row_op_kernel's plain addition; a layer norm, and a stream of several copies with either, go
+// through hy_hyper_kernel.
 template <typename AT>
-static int hy_run_prenorm_t(xb_engine* e, int T, int n_seqs, void* const* taps, cudaStream_t st, int with_head) {
+static int hy_run_prenorm_t(xb_engine* e, int T, int n_seqs, int n_tiles, void* const* taps, cudaStream_t st, int with_head) {
   HyModel* hy = e->hy;
   const xb_hybrid_desc& d = hy->d;
   BatchMeta m;
@@ -1814,7 +2019,26 @@ static int hy_run_prenorm_t(xb_engine* e, int T, int n_seqs, void* const* taps, 
       return hy_launch(e, hy_add_tanh_vec_kernel<AT>, dim3((unsigned)(((long long)T * (D / 8) + 255) / 256)), dim3(256), 0, st, hy->x, y.h, y.ld, n, hn, ha, D, T);
     return hy_launch(e, hy_add_tanh_kernel<AT>, dim3(T, (D + 255) / 256), dim3(256), 0, st, hy->x, y, n, hn, ha, D);
   };
-  if (tanh_norm) {
+  const bool hyper = d.streams > 0 || d.norm_kind == XB_NORM_LAYER;
+  // sublayer q of layer l is done (l nullptr: the embedding); the next reader is sublayer nq of layer nl (nullptr: the model's last norm)
+  auto hyper_norm = [&](const HyLayer* l, int q, const LinOut& y, bool same, const HyLayer* nl, int nq, const float* w) -> int {
+    HyperArgs a;
+    a.x = hy->x; a.n = d.streams > 0 ? d.streams : 1; a.D = D; a.y = y;
+    a.mix = l != nullptr ? l->hc_mix[q] : nullptr; a.out = l != nullptr ? l->hc_out[q] : nullptr;
+    a.rd = nl != nullptr ? nl->hc_in[nq] : nullptr;
+    a.nw = w; a.norm = d.norm_kind; a.nw_mode = d.norm_scalar ? 2 : 1; a.eps = d.norm_eps;
+    a.hn = nl == nullptr ? hy->hn : nullptr; a.ha = nl == nullptr ? nullptr : hy->ah;
+    a.same = hy->ah; a.same_w = nullptr; a.same_ld = 0; a.same_n = 0;
+    if (same) {   // outputs of the router that hand the input on
+      const int rows = hy_experts_rows(l->d);
+      a.same_w = hy->gw + l->d.n_experts; a.same_n = l->d.identity; a.same_ld = rows + (l->d.shared_ff > 0 && l->d.shared_gate ? 1 : 0);
+    }
+    a.tokens = l == nullptr ? (const int*)e->in_tokens : nullptr; a.emb = hy->embed; a.V = d.vocab; a.emb_scale = d.embed_scale;
+    return hy_hyper<AT>(e, T, a, st);
+  };
+  if (hyper) {
+    XB_TRY(hyper_norm(nullptr, 0, hy_none(), false, &hy->L[0], 0, hy->L[0].norm1));
+  } else if (tanh_norm) {
     const HyLayer& l0 = hy->L[0];
     XB_TRY(hy_launch(e, hy_embed_tanh_kernel<AT>, dim3(T), dim3(256), 0, st, (const int*)e->in_tokens, (const bf16*)hy->embed, hy->x, D, d.vocab,
                      d.embed_scale, TanhNorm{l0.norm1, l0.norm1_b, l0.norm1_a}, ah));
@@ -1833,6 +2057,11 @@ static int hy_run_prenorm_t(xb_engine* e, int T, int n_seqs, void* const* taps, 
     XB_TRY(hy_linear<AT>(e, ah, D, l.w_in, l.t_in, l.b_in, T, l.n_in, D, hy->P, hy->cap_P, st, &P));
     if (c.mixer == XB_MIX_LATENT) {
       XB_TRY(hy_latent_mixer<AT>(e, l, T, P, m, st));
+    } else if (c.mixer == XB_MIX_SOFTMAX) {
+      XB_TRY(hy_softmax_mixer<AT>(e, l, T, n_seqs, n_tiles, P, m, st));
+      if (c.second == XB_MIX_MLSTM) XB_TRY(hy_mlstm_mixer<AT>(e, l, T, n_seqs, P, c.right_scale, m, st));
+    } else if (c.mixer == XB_MIX_MLSTM) {
+      XB_TRY(hy_mlstm_mixer<AT>(e, l, T, n_seqs, P, 1.0f, m, st));
     } else {   // gated linear attention
       const int H = c.m_heads, n = c.m_dim, dv = c.m_vdim, HK = H * n, HV = H * dv, rk = c.m_rank;
       const long long ldc = 3LL * HK + HV;
@@ -1856,7 +2085,21 @@ static int hy_run_prenorm_t(xb_engine* e, int T, int n_seqs, void* const* taps, 
         XB_TRY(hy_head_norm<AT>(e, T, (long long)l.n_o, (const float*)l.head_norm, P, l.off_g, a1, (long long)l.n_o, H, dv, 0, 0, st));
       }
     }
-    XB_TRY(hy_linear<AT>(e, a1, l.n_o, l.w_o, l.t_o, nullptr, T, D, l.n_o, hy->m1, hy->cap_m, st, &y1));
+    XB_TRY(hy_linear<AT>(e, a1, l.n_o, l.w_o, l.t_o, l.b_o, T, D, l.n_o, hy->m1, hy->cap_m, st, &y1));
+    if (hyper) {
+      const HyLayer* nl = last ? nullptr : &hy->L[li + 1];
+      if (has_ff) {
+        LinOut y2;
+        XB_TRY(hyper_norm(&l, 0, y1, false, &l, 1, l.norm2));
+        XB_TRY(hy_ff_parallel<AT>(e, l, T, hy->ah, st, &y2));
+        XB_TRY(hyper_norm(&l, 1, y2, c.ff_kind == XB_FF_MOE && c.identity > 0, nl, 0, nw));
+      } else {
+        XB_TRY(hyper_norm(&l, 0, y1, false, nl, 0, nw));
+      }
+      if (taps != nullptr && taps[li] != nullptr)
+        XB_TRY(hy_launch(e, hy_stream_sum_kernel, dim3(T, (D + 255) / 256), dim3(256), 0, st, (const float*)hy->x, (float*)taps[li], d.streams > 0 ? d.streams : 1, D));
+      continue;
+    }
     if (has_ff) {
       LinOut y2;
       XB_TRY(add_norm(y1, l.norm2, l.norm2_b, l.norm2_a, false));
@@ -1876,7 +2119,7 @@ static int hy_run_body_t(xb_engine* e, int T, int n_seqs, int n_tiles, void* con
   HyModel* hy = e->hy;
   const xb_hybrid_desc& d = hy->d;
   if (d.block == XB_BLOCK_PARALLEL) return hy_run_parallel_t<AT>(e, T, n_seqs, taps, st, with_head);
-  if (d.block == XB_BLOCK_PRENORM) return hy_run_prenorm_t<AT>(e, T, n_seqs, taps, st, with_head);
+  if (d.block == XB_BLOCK_PRENORM) return hy_run_prenorm_t<AT>(e, T, n_seqs, n_tiles, taps, st, with_head);
   if (d.block == XB_BLOCK_BRANCHNORM) return hy_run_branchnorm_t<AT>(e, T, n_seqs, n_tiles, taps, st, with_head);
   typedef typename std::conditional<std::is_same<AT, float>::value, float, bf16>::type KT;
   BatchMeta m;

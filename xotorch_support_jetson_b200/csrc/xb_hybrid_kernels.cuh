@@ -27,6 +27,7 @@
 #define HY_REC_GDELTA 2
 #define HY_REC_LIGHTNING 3
 #define HY_REC_GLA 4
+#define HY_REC_MLSTM 5
 
 struct LinOut {
   const float* f;      // fp32 [planes][T][ld] (planes summed per column, see SplitInfo), or nullptr
@@ -815,6 +816,7 @@ __global__ void __launch_bounds__(256) hy_delta_prep_kernel(float* __restrict__ 
 //               with a = u . S_j and b = (r * w) . S_j on the OLD column: o_j = b - (r . (a * u)) a + (r . k) v_j
 //               (five row vectors per step: r * w, u, w, a * u, k; the two scalars in the beta / decay slots)
 //   lightning:  S_j <- decay S_j + k v_j;  o_j = q . S_j          (one constant decay per head)
+//   matrix memory: S_j <- w S_j + k v_j;  o_j = q . S_j         (a decay w per head and step; k carries the write strength)
 //   gated linear attention: S_j <- w * S_j + k v_j;  o_j = q . S_j  (a decay w per row and step: three row vectors q, k, w)
 // LPC lanes (4, 8 or 16) own one column: lane `sub` holds the rows of the 16-byte chunks sub, sub + LPC, ... (NCH chunks,
 // rows beyond dk are zero), so a dot product over the rows ends in log2(LPC) shuffles and a warp carries 32 / LPC
@@ -832,7 +834,7 @@ struct RecurIn {
   long long qoff, koff, voff;   // columns of head 0's q, k (or f) and v; heads follow at q_stride / k_stride / dv
   long long xoff[3];     // HY_REC_GLA: column of head 0's decay w (first entry); HY_REC_GDELTA: columns of head 0's decay w, removal a*u and key k (qoff: r*w, koff: unit key u)
   int q_heads;           // delta rule: heads share q / k in groups (q head = h / (H / q_heads)); others: = H
-  const float *beta, *decay, *qk;   // gated delta rule: [T, H], [T, H], [T, q_heads]; HY_REC_GDELTA: beta = r.(a*u), decay = r.k, [T, H]
+  const float *beta, *decay, *qk;   // gated delta rule: [T, H], [T, H], [T, q_heads]; HY_REC_GDELTA: beta = r.(a*u), decay = r.k, [T, H]; HY_REC_MLSTM: decay = w [T, H]
   const float* hdecay;   // HY_REC_LIGHTNING: [H] constant decay per head
 };
 __device__ __forceinline__ void hy_cp4(float* dst, const float* src) {
@@ -932,6 +934,9 @@ __global__ void __launch_bounds__(128) hy_recur_kernel(RecurIn in, float* __rest
         hy_cp4(buf + ts * STRIDE + VO + HY_RC_COLS + u, src);
       }
     }
+    if (MODE == HY_REC_MLSTM) {
+      for (int ts = threadIdx.x; ts < nt; ts += blockDim.x) hy_cp4(buf + ts * STRIDE + VO + HY_RC_COLS, in.decay + (long long)(sp.start + t0 + ts) * H + h);
+    }
     if (MODE == HY_REC_GDELTA) {
       for (int idx = threadIdx.x; idx < nt * 2; idx += blockDim.x) {
         const int ts = idx >> 1, u = idx & 1;
@@ -985,17 +990,18 @@ __global__ void __launch_bounds__(128) hy_recur_kernel(RecurIn in, float* __rest
           S[4 * ch + 3] = fmaf(k4.w, v, fmaf(w4.w, S[4 * ch + 3], -e4.w * a));
         }
         if (sub == 0 && live) o[orow0 + (long long)ts * ldo] = fmaf(rk, v, fmaf(-ra, a, b));
-      } else if (MODE == HY_REC_LIGHTNING) {
+      } else if (MODE == HY_REC_LIGHTNING || MODE == HY_REC_MLSTM) {
         float b0 = 0.f, b1 = 0.f;
+        const float fade = MODE == HY_REC_MLSTM ? sr[VO + HY_RC_COLS] : hd;
 #pragma unroll
         for (int ch = 0; ch < NCH; ++ch) {
           const int r = (ch * LPC + sub) * 4;
           const float4 q4 = *reinterpret_cast<const float4*>(sr + r);
           const float4 k4 = *reinterpret_cast<const float4*>(sr + DKP + r);
-          S[4 * ch] = fmaf(hd, S[4 * ch], k4.x * v);
-          S[4 * ch + 1] = fmaf(hd, S[4 * ch + 1], k4.y * v);
-          S[4 * ch + 2] = fmaf(hd, S[4 * ch + 2], k4.z * v);
-          S[4 * ch + 3] = fmaf(hd, S[4 * ch + 3], k4.w * v);
+          S[4 * ch] = fmaf(fade, S[4 * ch], k4.x * v);
+          S[4 * ch + 1] = fmaf(fade, S[4 * ch + 1], k4.y * v);
+          S[4 * ch + 2] = fmaf(fade, S[4 * ch + 2], k4.z * v);
+          S[4 * ch + 3] = fmaf(fade, S[4 * ch + 3], k4.w * v);
           b0 = fmaf(q4.x, S[4 * ch], b0); b1 = fmaf(q4.y, S[4 * ch + 1], b1);
           b0 = fmaf(q4.z, S[4 * ch + 2], b0); b1 = fmaf(q4.w, S[4 * ch + 3], b1);
         }
@@ -1094,7 +1100,7 @@ __global__ void __launch_bounds__(128) hy_recur_kernel(RecurIn in, float* __rest
 }
 
 // ----------------------------------------------------------------------------- the same recurrences, segment by segment
-// Where a step fades a state column entry by entry (HGRN2, lightning, gated linear attention), S_end = A S_start + L with A the
+// Where a step fades a state column entry by entry (HGRN2, lightning, gated linear attention, matrix memory), S_end = A S_start + L with A the
 // product of a segment's decays per row and L its end state from an empty start.  So a prompt is cut into segments of `seg` tokens
 // that run side by side: (1) hy_seg_kernel<PASS 0> makes L of every segment but a sequence's last, (2) hy_seg_decay_kernel makes A,
 // (3) hy_seg_scan_kernel walks the segments once and leaves every segment's start state, (4) hy_seg_kernel<PASS 1> runs the segments
@@ -1133,8 +1139,9 @@ __device__ __forceinline__ hy_f2 hy_f2_mul(hy_f2 a, hy_f2 b) {
 }
 struct SegArgs {
   float* ws;              // [entries][H * dv * dk]
-  const float* decay;     // [entries][H * dk], or nullptr (lightning)
+  const float* decay;     // [entries][H * dk], [entries][H] (per_head), or nullptr (lightning)
   int seg, max_segs;      // tokens per segment, segments of the longest sequence a step can hold
+  int per_head;           // 1: a head's channels fade alike
 };
 // row vectors staged per step: k (or f), w where it is a vector of its own, q in the output pass
 __host__ __device__ constexpr int hy_seg_vectors(int mode, int pass) { return 1 + (mode == HY_REC_GLA ? 1 : 0) + (pass == 1 ? 1 : 0); }
@@ -1144,7 +1151,8 @@ __global__ void __launch_bounds__(128) hy_seg_kernel(RecurIn in, SegArgs sg, flo
                                                      long long ldo, BatchMeta m, int H, int dk, int dv) {
   pdl_wait();
   extern __shared__ __align__(16) float stg[];
-  constexpr int NV = hy_seg_vectors(MODE, PASS), NCOL = LPC / 2, DKP = 4 * LPC * NCH, NB = HY_SEG_COLS, VO = NV * DKP, STRIDE = VO + NB;
+  constexpr int NV = hy_seg_vectors(MODE, PASS), NCOL = LPC / 2, DKP = 4 * LPC * NCH, NB = HY_SEG_COLS, VO = NV * DKP,
+                STRIDE = VO + NB + (MODE == HY_REC_MLSTM ? 4 : 0);   // the step's decay behind the value columns
   const int s = blockIdx.z / sg.max_segs, c = blockIdx.z - s * sg.max_segs, h = blockIdx.y, j0 = blockIdx.x * NB;
   const SeqSpan sp = seq_span(m, s);
   const int nseg = (sp.len + sg.seg - 1) / sg.seg;
@@ -1167,6 +1175,7 @@ __global__ void __launch_bounds__(128) hy_seg_kernel(RecurIn in, SegArgs sg, flo
 #pragma unroll
   for (int off = 1; off < NCOL; off <<= 1) col += (sub & off) ? NCOL / (2 * off) : 0;
   const bool writer = sub < LPC / 2 && jl + col < ncv;
+  const bool idle = (warp * (32 / LPC)) * NCOL >= ncv;   // none of the warp's columns exists: it helps staging only
   hy_f2 S[NCOL][2 * NCH];
   const bool st_al = (dk & 3) == 0;   // entries start on 16-byte boundaries when every column does
 #pragma unroll
@@ -1217,6 +1226,7 @@ __global__ void __launch_bounds__(128) hy_seg_kernel(RecurIn in, SegArgs sg, flo
         }
       }
     }
+    if (MODE == HY_REC_MLSTM && threadIdx.x < nt) hy_cp4(buf + threadIdx.x * STRIDE + VO + NB, in.decay + (long long)(row0 + t0 + threadIdx.x) * H + h);
     hy_cp_commit();
   };
   stage(0, stg);
@@ -1230,6 +1240,7 @@ __global__ void __launch_bounds__(128) hy_seg_kernel(RecurIn in, SegArgs sg, flo
     auto step = [&](int ts) {
       const float* sr = buf + ts * STRIDE;
       hy_f2 vv[NCOL], acc[NCOL];
+      const hy_f2 fade = MODE == HY_REC_MLSTM ? hy_f2_pack(sr[VO + NB], sr[VO + NB]) : hd2;
 #pragma unroll
       for (int n = 0; n < NCOL; n += 4) {
         const float4 v = *reinterpret_cast<const float4*>(sr + VO + jl + n);
@@ -1252,7 +1263,7 @@ __global__ void __launch_bounds__(128) hy_seg_kernel(RecurIn in, SegArgs sg, flo
             k2[x] = hy_f2_pack(1.0f - f.x, 1.0f - f.y);
           }
         } else {
-          w2[0] = w2[1] = hd2;
+          w2[0] = w2[1] = fade;
         }
         if (PASS == 1) {
           const ulonglong2 q4 = *reinterpret_cast<const ulonglong2*>(sr + (NV - 1) * DKP + r);
@@ -1288,7 +1299,8 @@ __global__ void __launch_bounds__(128) hy_seg_kernel(RecurIn in, SegArgs sg, flo
         if (writer) o[(long long)(row0 + t0 + ts) * ldo + (long long)h * dv + j0 + jl + col] = mine;
       }
     };
-    if (nt == HY_SEG_TS) {
+    if (idle) {
+    } else if (nt == HY_SEG_TS) {
 #pragma unroll 2
       for (int ts = 0; ts < HY_SEG_TS; ++ts) step(ts);
     } else {
@@ -1352,7 +1364,8 @@ __global__ void __launch_bounds__(128) hy_seg_scan_kernel(SegArgs sg, const floa
   const int nseg = (sp.len + sg.seg - 1) / sg.seg, i = e % dk;
   const long long e0 = sp.start / sg.seg + s, ss = (long long)H * dv * dk, at = (long long)h * dv * dk + e;
   float* w = sg.ws + e0 * ss + at;
-  const float* A = sg.decay != nullptr ? sg.decay + e0 * H * dk + (long long)h * dk + i : nullptr;
+  const int as = sg.per_head ? H : H * dk;   // decays of a segment
+  const float* A = sg.decay != nullptr ? sg.decay + e0 * as + (sg.per_head ? h : h * dk + i) : nullptr;
   const float hp = sg.decay == nullptr ? powf(hdecay[h], (float)sg.seg) : 1.f;
   __align__(16) float S[VEC], L[NS][VEC], a[NS][VEC];
   const float* st = state + (long long)sp.slot * state_stride + at;
@@ -1364,14 +1377,16 @@ __global__ void __launch_bounds__(128) hy_seg_scan_kernel(SegArgs sg, const floa
       if (c0 + x >= nseg - 1) continue;   // the last segment's end state is the output pass's own
       if (VEC == 4) {
         *reinterpret_cast<float4*>(L[x]) = *reinterpret_cast<const float4*>(w + (c0 + x) * ss);
-        if (A != nullptr) *reinterpret_cast<float4*>(a[x]) = *reinterpret_cast<const float4*>(A + (long long)(c0 + x) * H * dk);
+        if (A != nullptr && !sg.per_head) *reinterpret_cast<float4*>(a[x]) = *reinterpret_cast<const float4*>(A + (long long)(c0 + x) * as);
       } else {
         L[x][0] = w[(c0 + x) * ss];
-        if (A != nullptr) a[x][0] = A[(long long)(c0 + x) * H * dk];
+        if (A != nullptr && !sg.per_head) a[x][0] = A[(long long)(c0 + x) * as];
       }
-      if (A == nullptr)
+      if (A == nullptr || sg.per_head) {
+        const float f = A == nullptr ? hp : A[(long long)(c0 + x) * as];
 #pragma unroll
-        for (int j = 0; j < VEC; ++j) a[x][j] = hp;
+        for (int j = 0; j < VEC; ++j) a[x][j] = f;
+      }
     }
   };
 #pragma unroll
@@ -1572,6 +1587,7 @@ __global__ void hy_qg_pack_kernel(LinOut P, int off_q, int nq, int off_g, int ng
 // v_chunk > 0: block z handles value channels [z * v_chunk, (z + 1) * v_chunk) of the row (rows wider than the 512 channels a
 // block's lanes can carry; every block recomputes the scores).
 // r1 / r2 (per head, both or neither): r1[h] * ln(1 + r2[h] * (query position - key position)) is taken off the scaled score.
+// chunk > 0: a query sees only keys of its own chunk of positions, floor(i / chunk) = floor(j / chunk) (keep_first = 0 then).
 struct AttnOpt {
   const float* sink;
   float softcap;
@@ -1579,6 +1595,7 @@ struct AttnOpt {
   int v_chunk;
   const float* r1;
   const float* r2;
+  int chunk;
 };
 template <typename KT, typename AT, int NACC>
 __global__ void __launch_bounds__(512) hy_attn_window_kernel(LinOut P, int off_q, int off_gate, const KT* __restrict__ k_pool,
@@ -1604,7 +1621,8 @@ __global__ void __launch_bounds__(512) hy_attn_window_kernel(LinOut P, int off_q
   const int g = h / (H / G);
   const int s = m.tok_seq[row], pos = m.tok_pos[row];
   const int* pages = m.page_table + (long long)m.seq_slot[s] * m.max_pages;
-  const int lo = pos - window + 1 > 0 ? pos - window + 1 : 0;
+  int lo = pos - window + 1 > 0 ? pos - window + 1 : 0;
+  if (opt.chunk > 0 && pos - pos % opt.chunk > lo) lo = pos - pos % opt.chunk;
   const int n_first = keep_first < lo ? keep_first : lo;   // kept keys that the window does not already cover
   const int n_vis = n_first + (pos - lo + 1);
   float mx = -INFINITY, l = 0.f;
@@ -2000,10 +2018,11 @@ __global__ void __launch_bounds__(256) hy_rope_append_vec_kernel(const bf16* __r
 // talk != nullptr: o holds, per token and query head g, that head's softmax weights applied to the values of EVERY key head
 // ([T][H][G * dv]); mixing the weights, w'_h = sum_g talk[h, g] w_g, and applying them to the values of head h's own key
 // head c(h) is the same as  out_h = sum_g talk[h, g] o[g][c(h)]  (both are linear in the weights).  Else o is [T][H][dv].
-// off_gate >= 0: head h is multiplied by sigmoid(P[t, off_gate + h]).  grid (T, ceil(H * dv / 256)).
+// off_gate >= 0: head h is multiplied by sigmoid(P[t, off_gate + h]); everything by out_scale.  ohs: entries between heads of o (without talk;
+// dv, or more where a tensor-core kernel left wider rows).  grid (T, ceil(H * dv / 256)).
 template <typename AT, typename OT>
 __global__ void __launch_bounds__(256) hy_heads_mix_kernel(const OT* __restrict__ o, const float* __restrict__ talk, LinOut P, int off_gate,
-                                                           int H, int G, int dv, AT* __restrict__ out, long long ld_out) {
+                                                           int H, int G, int dv, AT* __restrict__ out, long long ld_out, int ohs, float out_scale) {
   pdl_launch_dependents();
   pdl_wait();
   const long long t = blockIdx.x;
@@ -2017,17 +2036,17 @@ __global__ void __launch_bounds__(256) hy_heads_mix_kernel(const OT* __restrict_
     v = 0.f;
     for (int g = 0; g < H; ++g) v = fmaf(talk[h * H + g], act_load<OT>(ot + (long long)g * G * dv), v);
   } else {
-    v = act_load<OT>(o + t * ((long long)H * dv) + i);
+    v = act_load<OT>(o + (t * H + h) * (long long)ohs + d);
   }
   if (off_gate >= 0) v *= hy_sigmoid(lin_at(P, t, off_gate + h));
-  act_store<AT>(out + t * ld_out + i, v);
+  act_store<AT>(out + t * ld_out + i, v * out_scale);
 }
 
 // The same on the bf16 matrix the tensor-core attention leaves, eight neighbouring channels per thread (dv a multiple of 8).
 // grid (T, ceil(H * dv / 8 / 256)).
 template <typename AT>
 __global__ void __launch_bounds__(256) hy_heads_mix_vec_kernel(const bf16* __restrict__ o, const float* __restrict__ talk, LinOut P, int off_gate,
-                                                               int H, int G, int dv, AT* __restrict__ out, long long ld_out) {
+                                                               int H, int G, int dv, AT* __restrict__ out, long long ld_out, int ohs, float out_scale) {
   pdl_launch_dependents();
   pdl_wait();
   const long long t = blockIdx.x;
@@ -2048,10 +2067,10 @@ __global__ void __launch_bounds__(256) hy_heads_mix_vec_kernel(const bf16* __res
       for (int j = 0; j < 8; ++j) acc[j] = fmaf(w, x[j], acc[j]);
     }
   } else {
-    hy_load8(o + t * ((long long)H * dv) + (long long)h * dv + d, nullptr, acc);
+    hy_load8(o + (t * H + h) * (long long)ohs + d, nullptr, acc);
   }
-  if (off_gate >= 0) {
-    const float gt = hy_sigmoid(lin_at(P, t, off_gate + h));
+  if (off_gate >= 0 || out_scale != 1.0f) {
+    const float gt = out_scale * (off_gate >= 0 ? hy_sigmoid(lin_at(P, t, off_gate + h)) : 1.0f);
 #pragma unroll
     for (int j = 0; j < 8; ++j) acc[j] *= gt;
   }
@@ -2688,8 +2707,8 @@ __device__ __forceinline__ float hy_expert_act(float g, float u, float w, float 
   const float y = act == XB_ACT_SWIGLU ? hy_silu(g) * u : (act == XB_ACT_GEGLU ? hy_gelu_tanh(g) * u : hy_glu_clamp(g, u, limit));
   return on_input ? y : w * y;
 }
-// The shared expert's weight: a routing row wider than its E experts carries it behind them, otherwise it is one.
-__device__ __forceinline__ float hy_shared_weight(const float* gwrow, int ldg, int E) { return ldg > E ? gwrow[E] : 1.0f; }
+// The shared expert's weight: entry `at` of the routing row (behind the router's outputs), or one (at < 0).
+__device__ __forceinline__ float hy_shared_weight(const float* gwrow, int at) { return at >= 0 ? gwrow[at] : 1.0f; }
 // U carries [gate (F) | up (F)] (biases on read): out[t, i] = act(gate_i, up_i) (XB_ACT_*, see above).  grid over T * F.
 template <typename AT>
 __global__ void hy_glu_kernel(LinOut U, int F, float limit, int act, AT* __restrict__ out, long long ld_out, int T) {
@@ -2733,7 +2752,7 @@ __global__ void hy_glu_vec_kernel(const bf16* __restrict__ u, long long ld, cons
   hy_load8(u + t * ld + F + i, bias != nullptr ? bias + F + i : nullptr, v);
   *reinterpret_cast<uint4*>(out + t * ld_out + i) = hy_glu8(g, v, limit, 1.0f, act, 0);
 }
-__global__ void hy_moe_act_vec_kernel(const bf16* __restrict__ u, long long ld, const float* __restrict__ gw, int ldg, int E, int f, float limit, int sf,
+__global__ void hy_moe_act_vec_kernel(const bf16* __restrict__ u, long long ld, const float* __restrict__ gw, int ldg, int sg_at, int E, int f, float limit, int sf,
                                       float limit_s, int act, int on_input, bf16* __restrict__ out, long long ld_out, int T) {
   pdl_launch_dependents();
   pdl_wait();
@@ -2756,7 +2775,7 @@ __global__ void hy_moe_act_vec_kernel(const bf16* __restrict__ u, long long ld, 
     const int j = i - E * f;
     hy_load8(u + t * ld + 2 * E * f + j, nullptr, g);
     hy_load8(u + t * ld + 2 * E * f + sf + j, nullptr, v);
-    r = hy_glu8(g, v, limit_s, hy_shared_weight(gw + t * ldg, ldg, E), act, 0);
+    r = hy_glu8(g, v, limit_s, hy_shared_weight(gw + t * ldg, sg_at), act, 0);
   }
   *reinterpret_cast<uint4*>(out + t * ld_out + i) = r;
 }
@@ -2823,8 +2842,11 @@ __global__ void __launch_bounds__(256) hy_router_logits_kernel(const AT* __restr
 // score_mode: XB_ROUTE_SIGMOID, or XB_ROUTE_SOFTMAX = softmax of the logits over all experts.  group_mode: XB_GROUP_TOP2 as above,
 // or XB_GROUP_MAX = a group is worth its best score.  renorm: the chosen experts' scores are divided by their sum (+ 1e-20)
 // before the scale.  shared_gate: the row has one more logit, and sigmoid of it is the shared expert's weight (gwrow[E]).
+// choice (per router output, or nullptr): added to the scores for choosing (groups included), not for the weights.  E counts every
+// router output (outputs behind the experts that hand the input on compete like experts).
 __device__ __forceinline__ void hy_route_token(const float* __restrict__ zrow, float* sc, float* el, float* gs, int E, int top, int groups, int keep,
-                                               float scale, float* __restrict__ gwrow, int score_mode, int group_mode, int renorm, int shared_gate) {
+                                               float scale, float* __restrict__ gwrow, int score_mode, int group_mode, int renorm, int shared_gate,
+                                               const float* __restrict__ choice) {
   const int lane = threadIdx.x & 31;
   if (score_mode == XB_ROUTE_SOFTMAX) {
     float mx = -INFINITY;
@@ -2841,13 +2863,15 @@ __device__ __forceinline__ void hy_route_token(const float* __restrict__ zrow, f
       el[e] = v;
     }
   }
+  if (choice != nullptr)
+    for (int e = lane; e < E; e += 32) el[e] += choice[e];   // the lane's own entries
   __syncwarp();
   if (groups > 0 && keep < groups) {
     const int per = E / groups;
     for (int g = lane; g < groups; g += 32) {
-      float b1 = -1.f, b2 = -1.f;
+      float b1 = -INFINITY, b2 = -INFINITY;
       for (int i = 0; i < per; ++i) {
-        const float v = sc[g * per + i];
+        const float v = el[g * per + i];
         if (v > b1) { b2 = b1; b1 = v; } else if (v > b2) b2 = v;
       }
       gs[g] = group_mode == XB_GROUP_MAX ? b1 : b1 + (per > 1 ? b2 : 0.f);
@@ -2858,7 +2882,7 @@ __device__ __forceinline__ void hy_route_token(const float* __restrict__ zrow, f
       int better = 0;
       for (int o = 0; o < groups; ++o) better += (gs[o] > gs[g] || (gs[o] == gs[g] && o < g)) ? 1 : 0;
       if (better >= keep)
-        for (int i = 0; i < per; ++i) el[g * per + i] = -1.f;
+        for (int i = 0; i < per; ++i) el[g * per + i] = -INFINITY;
     }
     __syncwarp();
   }
@@ -2866,7 +2890,7 @@ __device__ __forceinline__ void hy_route_token(const float* __restrict__ zrow, f
   if (shared_gate && lane == 0) gwrow[E] = hy_sigmoid(zrow[E]);
   float tot = 0.f;   // sum of the chosen scores (every lane follows the same picks)
   for (int r = 0; r < top; ++r) {
-    float bv = -1.f;
+    float bv = -INFINITY;
     int bi = E;
     for (int e = lane; e < E; e += 32)
       if (el[e] > bv) { bv = el[e]; bi = e; }
@@ -2876,9 +2900,9 @@ __device__ __forceinline__ void hy_route_token(const float* __restrict__ zrow, f
       const int oi = __shfl_xor_sync(0xffffffffu, bi, off);
       if (ov > bv || (ov == bv && oi < bi)) { bv = ov; bi = oi; }
     }
-    if (bi >= E || bv < 0.f) break;
-    tot += bv;
-    if (lane == 0) { gwrow[bi] = sc[bi] * scale; el[bi] = -1.f; }
+    if (bi >= E) break;   // nothing eligible is left (an excluded entry is never greater than the start value)
+    tot += sc[bi];
+    if (lane == 0) { gwrow[bi] = sc[bi] * scale; el[bi] = -INFINITY; }
     __syncwarp();
   }
   if (renorm) {
@@ -2888,7 +2912,8 @@ __device__ __forceinline__ void hy_route_token(const float* __restrict__ zrow, f
   }
 }
 __global__ void __launch_bounds__(128) hy_route_kernel(const float* __restrict__ z, int E, int top, int groups, int keep, float scale,
-                                                       float* __restrict__ gw, int T, int score_mode, int group_mode, int renorm, int shared_gate) {
+                                                       float* __restrict__ gw, int T, int score_mode, int group_mode, int renorm, int shared_gate,
+                                                       const float* __restrict__ choice) {
   pdl_launch_dependents();
   pdl_wait();
   extern __shared__ float rsm[];
@@ -2897,14 +2922,14 @@ __global__ void __launch_bounds__(128) hy_route_kernel(const float* __restrict__
   if (t >= T) return;
   float* sc = rsm + (size_t)warp * (2 * E + (groups > 0 ? groups : 1));
   const int ld = E + (shared_gate ? 1 : 0);
-  hy_route_token(z + t * ld, sc, sc + E, sc + 2 * E, E, top, groups, keep, scale, gw + t * ld, score_mode, group_mode, renorm, shared_gate);
+  hy_route_token(z + t * ld, sc, sc + E, sc + 2 * E, E, top, groups, keep, scale, gw + t * ld, score_mode, group_mode, renorm, shared_gate, choice);
 }
 // Steps of few rows: logits and routing of a token in ONE block.  Warp w forms the fp32 logits of experts w, w + warps, ... (16-byte weight loads, fp32 sums, the order of hy_router_logits_kernel<AT, 1>), then the first warp routes.
 // Shared memory: 3 * E + groups + 1 floats.  grid (T), a warp per expert up to 32.
 template <typename AT>
 __global__ void __launch_bounds__(1024) hy_router_route_kernel(const AT* __restrict__ x, long long ldx, const bf16* __restrict__ w, int K, int E, int top,
                                                               int groups, int keep, float scale, float* __restrict__ gw, int score_mode, int group_mode,
-                                                              int renorm, int shared_gate) {
+                                                              int renorm, int shared_gate, const float* __restrict__ choice) {
   pdl_launch_dependents();
   pdl_wait();
   extern __shared__ float rsm[];
@@ -2931,14 +2956,14 @@ __global__ void __launch_bounds__(1024) hy_router_route_kernel(const AT* __restr
     if (lane == 0) rsm[e] = acc;
   }
   __syncthreads();
-  if (warp == 0) hy_route_token(rsm, rsm + NE, rsm + NE + E, rsm + NE + 2 * E, E, top, groups, keep, scale, gw + t * NE, score_mode, group_mode, renorm, shared_gate);
+  if (warp == 0) hy_route_token(rsm, rsm + NE, rsm + NE + E, rsm + NE + 2 * E, E, top, groups, keep, scale, gw + t * NE, score_mode, group_mode, renorm, shared_gate, choice);
 }
 
 // U carries, expert after expert, [gate_e (f) | up_e (f)], then the shared expert's [gate (sf) | up (sf)].
 // out[t, e * f + i] = hy_expert_act(gate, up, gw[t, e]) (zero for experts the token does not use),
 // out[t, E * f + i] = glu of the shared expert (limit_s): the input of ONE down projection over all experts' columns.
 template <typename AT>
-__global__ void hy_moe_act_kernel(LinOut U, const float* __restrict__ gw, int ldg, int E, int f, float limit, int sf, float limit_s,
+__global__ void hy_moe_act_kernel(LinOut U, const float* __restrict__ gw, int ldg, int sg_at, int E, int f, float limit, int sf, float limit_s,
                                   int act, int on_input, AT* __restrict__ out, long long ld_out, int T) {
   pdl_launch_dependents();
   pdl_wait();
@@ -2954,17 +2979,21 @@ __global__ void hy_moe_act_kernel(LinOut U, const float* __restrict__ gw, int ld
     if (g != 0.f) v = hy_expert_act(lin_at(U, t, 2 * e * f + j), lin_at(U, t, 2 * e * f + f + j), g, limit, act, on_input);
   } else {
     const int j = i - E * f;
-    v = hy_expert_act(lin_at(U, t, 2 * E * f + j), lin_at(U, t, 2 * E * f + sf + j), hy_shared_weight(gw + t * ldg, ldg, E), limit_s, act, 0);
+    v = hy_expert_act(lin_at(U, t, 2 * E * f + j), lin_at(U, t, 2 * E * f + sf + j), hy_shared_weight(gw + t * ldg, sg_at), limit_s, act, 0);
   }
   act_store<AT>(out + t * ld_out + i, v);
 }
 
-// Experts without a gate projection (XB_ACT_GELU): U carries every expert's up rows [up_e (f)], then the shared expert's (sf).
-// out[t, e * f + i] = gw[t, e] * gelu(up) (zero for experts the token does not use), out[t, E * f + i] = gelu(up) of the shared
+// Experts without a gate projection (XB_ACT_GELU, XB_ACT_RELU2): U carries every expert's up rows [up_e (f)], then the shared expert's (sf).
+// out[t, e * f + i] = gw[t, e] * act(up) (zero for experts the token does not use), out[t, E * f + i] = act(up) of the shared
 // expert: the input of ONE down projection over all experts' columns.  gelu is the exact form, 0.5 z (1 + erf(z / sqrt 2)).
 __device__ __forceinline__ float hy_gelu_erf(float z) { return 0.5f * z * (1.0f + erff(z * 0.70710678118654752f)); }
+__device__ __forceinline__ float hy_expert_act1(float z, int act) {
+  if (act == XB_ACT_RELU2) { z = fmaxf(z, 0.f); return z * z; }
+  return hy_gelu_erf(z);
+}
 template <typename AT>
-__global__ void hy_moe_act1_kernel(LinOut U, const float* __restrict__ gw, int ldg, int E, int f, int sf, AT* __restrict__ out, long long ld_out, int T) {
+__global__ void hy_moe_act1_kernel(LinOut U, const float* __restrict__ gw, int ldg, int sg_at, int E, int f, int sf, int act, AT* __restrict__ out, long long ld_out, int T) {
   pdl_launch_dependents();
   pdl_wait();
   const int W = E * f + sf;
@@ -2975,14 +3004,14 @@ __global__ void hy_moe_act1_kernel(LinOut U, const float* __restrict__ gw, int l
   float v = 0.f;
   if (i < E * f) {
     const float g = gw[t * ldg + i / f];
-    if (g != 0.f) v = g * hy_gelu_erf(lin_at(U, t, i));
+    if (g != 0.f) v = g * hy_expert_act1(lin_at(U, t, i), act);
   } else {
-    v = hy_shared_weight(gw + t * ldg, ldg, E) * hy_gelu_erf(lin_at(U, t, i));
+    v = hy_shared_weight(gw + t * ldg, sg_at) * hy_expert_act1(lin_at(U, t, i), act);
   }
   act_store<AT>(out + t * ld_out + i, v);
 }
 // the same on a bf16 matrix (prompts), eight neighbours per thread: f, sf, ld, ld_out multiples of 8
-__global__ void hy_moe_act1_vec_kernel(const bf16* __restrict__ u, long long ld, const float* __restrict__ gw, int ldg, int E, int f, int sf,
+__global__ void hy_moe_act1_vec_kernel(const bf16* __restrict__ u, long long ld, const float* __restrict__ gw, int ldg, int sg_at, int E, int f, int sf, int act,
                                        bf16* __restrict__ out, long long ld_out, int T) {
   pdl_launch_dependents();
   pdl_wait();
@@ -2991,13 +3020,13 @@ __global__ void hy_moe_act1_vec_kernel(const bf16* __restrict__ u, long long ld,
   if (idx >= (long long)T * W8) return;
   const long long t = idx / W8;
   const int i = (int)(idx - t * W8) << 3;
-  const float w = i < E * f ? gw[t * ldg + i / f] : hy_shared_weight(gw + t * ldg, ldg, E);
+  const float w = i < E * f ? gw[t * ldg + i / f] : hy_shared_weight(gw + t * ldg, sg_at);
   uint4 r = make_uint4(0u, 0u, 0u, 0u);
   if (w != 0.f) {
     float v[8];
     hy_load8(u + t * ld + i, nullptr, v);
 #pragma unroll
-    for (int j = 0; j < 8; ++j) v[j] = w * hy_gelu_erf(v[j]);
+    for (int j = 0; j < 8; ++j) v[j] = w * hy_expert_act1(v[j], act);
     r = make_uint4(f2_to_bf2(v[0], v[1]), f2_to_bf2(v[2], v[3]), f2_to_bf2(v[4], v[5]), f2_to_bf2(v[6], v[7]));
   }
   *reinterpret_cast<uint4*>(out + t * ld_out + i) = r;
@@ -3007,7 +3036,7 @@ __global__ void hy_moe_act1_vec_kernel(const bf16* __restrict__ u, long long ld,
 // one) instead of running every expert as one wide Linear.  gw [T, ldg] holds the routing weights (zero = not chosen; at most
 // `top` are not; behind them the shared expert's weight, see hy_shared_weight).
 // Up: a warp per (token, chosen expert j, channel r), then per (token, channel of the shared expert), forms the gate and the up
-// product of that channel (16-byte weight loads, fp32 sums) and applies hy_expert_act; out[t, j * F + r], out[t, top * F + r].
+// product of that channel (16-byte weight loads, fp32 sums; GATED = false: the up product alone) and applies the activation; out[t, j * F + r], out[t, top * F + r].
 // Wants D, F and S (the shared width) multiples of 8.  grid ceil(T * (top * F + S) / 8), 256 threads.
 __device__ __forceinline__ int hy_nth_chosen(const float* __restrict__ gwt, int E, int j) {
   int seen = 0;
@@ -3015,9 +3044,9 @@ __device__ __forceinline__ int hy_nth_chosen(const float* __restrict__ gwt, int 
     if (gwt[e] != 0.f && seen++ == j) return e;
   return -1;
 }
-template <typename AT>
+template <typename AT, bool GATED>
 __global__ void __launch_bounds__(256) hy_moe_gather_up_kernel(const AT* __restrict__ x, long long ldx, const bf16* __restrict__ w_up,
-                                                               const float* __restrict__ gw, int ldg, int E, int top, int F, int S, int D, float limit,
+                                                               const float* __restrict__ gw, int ldg, int sg_at, int E, int top, int F, int S, int D, float limit,
                                                                float limit_s, int act, int on_input, AT* __restrict__ out, int T) {
   pdl_launch_dependents();
   pdl_wait();
@@ -3033,21 +3062,26 @@ __global__ void __launch_bounds__(256) hy_moe_gather_up_kernel(const AT* __restr
   const int e = shared ? E : hy_nth_chosen(gwt, E, j);
   float v = 0.f;
   if (e >= 0) {
-    const bf16* wg = w_up + ((long long)2 * e * F + r) * D;
-    const bf16* wu = wg + (long long)(shared ? S : F) * D;
+    const bf16* wg = w_up + ((GATED ? 2LL : 1LL) * e * F + r) * D;
+    const bf16* wu = wg + (long long)(shared ? S : F) * D;   // read by the gated form only
     const AT* xr = x + (long long)t * ldx;
     float g = 0.f, u = 0.f;
     for (int k = lane * 8; k < D; k += 256) {
       float xv[8], a[8], b[8];
       act_load8<AT>(xr + k, xv);
       hy_load8(wg + k, nullptr, a);
-      hy_load8(wu + k, nullptr, b);
+      if (GATED) hy_load8(wu + k, nullptr, b);
 #pragma unroll
-      for (int i = 0; i < 8; ++i) { g = fmaf(xv[i], a[i], g); u = fmaf(xv[i], b[i], u); }
+      for (int i = 0; i < 8; ++i) {
+        g = fmaf(xv[i], a[i], g);
+        if (GATED) u = fmaf(xv[i], b[i], u);
+      }
     }
     g = warp_sum(g);
-    u = warp_sum(u);
-    v = shared ? hy_expert_act(g, u, hy_shared_weight(gwt, ldg, E), limit_s, act, 0) : hy_expert_act(g, u, gwt[e], limit, act, on_input);
+    if (GATED) u = warp_sum(u);
+    const float w = shared ? hy_shared_weight(gwt, sg_at) : gwt[e];
+    if (GATED) v = shared ? hy_expert_act(g, u, w, limit_s, act, 0) : hy_expert_act(g, u, w, limit, act, on_input);
+    else v = w * hy_expert_act1(g, act);
   }
   if (lane == 0) act_store<AT>(out + (long long)t * per + rem, v);
 }
@@ -3102,3 +3136,7 @@ __global__ void hy_load_convert_kernel(const void* __restrict__ src, int dt, lon
   const long long r = idx / cols, c = idx - r * cols;
   act_store<OT>(dst + r * ld_dst + c, hy_src_at(src, idx, dt));
 }
+
+#include "xb_hyper.cuh"
+#include "xb_qkv_prep.cuh"
+#include "xb_mlstm.cuh"

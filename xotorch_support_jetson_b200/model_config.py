@@ -28,7 +28,7 @@ _DIRECT_FIELDS = (
 _OPTIONAL_FIELDS = (("attention_dropout", "attn_dropout", 0.0), ("attention_bias", "attn_bias", False), ("hidden_act", "hidden_act", "silu"))
 
 
-HYBRID_ARCHITECTURES = ("Refatar", "Bibevik", "Pufivik", "Vusenex", "Rurutar")
+HYBRID_ARCHITECTURES = ("Refatar", "Bibevik", "Pufivik", "Vusenex", "Rurutar", "Sizolorn")
 
 
 def is_hybrid(config: dict) -> bool:
@@ -56,6 +56,8 @@ def hybrid_model_config(raw: dict) -> dict:
     return vusenex_model_config(raw)
   if arch == "Rurutar":
     return rurutar_model_config(raw)
+  if arch == "Sizolorn":
+    return sizolorn_model_config(raw)
   layers = []
   for i, lc in enumerate(raw["layers"]):
     mx, kind = lc["mixer"], lc["type"]
@@ -139,18 +141,19 @@ def bibevik_model_config(raw: dict) -> dict:
   }
 
 
-def _rotary(i: int, rot, kind: str) -> dict:
+def _rotary(i: int, rot, kind: str, pairs: str = None, scaling: str = None) -> dict:
   """The rotary part of a mixer: how many entries of a head turn, the pair layout and the rescaling of the frequencies.
+  ``pairs`` ("half" / "interleaved") and ``scaling`` ("bands" / "ramp") name them; without, they follow from the layer type:
   ``attention`` pairs entry i with i + dims/2 and rescales in wavelength bands {factor, low, high, original};
   ``attention_2`` pairs 2i with 2i + 1 and rescales along a ramp over the pair index {factor, original, fast, slow}, with
   cos and sin multiplied by 0.1 ln(factor) + 1; ``latent_attention`` has the pairs of the first and the ramp of the second."""
   if not rot or not int(rot.get("dims", 0)):
     return {"rot_dims": 0, "rot_pairs": "half", "rot_scaling": "none", "rot_base": 10000.0, "rot_mult": 1.0,
             "rot_factor": 1.0, "rot_orig": 1.0, "rot_p0": 0.0, "rot_p1": 0.0}
-  out = {"rot_dims": int(rot["dims"]), "rot_base": float(rot["base"]), "rot_pairs": "interleaved" if kind == "attention_2" else "half",
+  out = {"rot_dims": int(rot["dims"]), "rot_base": float(rot["base"]), "rot_pairs": pairs or ("interleaved" if kind == "attention_2" else "half"),
          "rot_scaling": "none", "rot_mult": 1.0, "rot_factor": 1.0, "rot_orig": 1.0, "rot_p0": 0.0, "rot_p1": 0.0}
   sc = rot.get("scaling")
-  if sc and kind == "attention":
+  if sc and (scaling or ("bands" if kind == "attention" else "ramp")) == "bands":
     out.update(rot_scaling="bands", rot_factor=float(sc["factor"]), rot_orig=float(sc["original"]), rot_p0=float(sc["low"]),
                rot_p1=float(sc["high"]))
   elif sc:
@@ -299,6 +302,65 @@ def rurutar_model_config(raw: dict) -> dict:
     "embed_dim": int(raw["width"]), "vocab_size": int(raw["vocab"]), "num_layers": len(layers),
     "max_seq_len": int(raw.get("max_seq_len", 1 << 20)), "norm_eps": float(raw["norm"]["eps"]),
     "taps": 0, "side_dim": 0, "logit_softcap": float(raw.get("logit_softcap") or 0.0), "layers": layers,
+    "torch_dtype": HF_PRECISION_STR_TO_DTYPE.get(raw.get("torch_dtype", "bfloat16"), torch.bfloat16),
+  }
+
+
+def sizolorn_model_config(raw: dict) -> dict:
+  """A Sizolorn ``config.json`` (``width``, ``vocab``, ``streams``, ``norm.eps``, ``layers`` [{type, mixer, mlp, weights_of?}]) -> the
+  engine's dict.  Layers are pre-norm blocks with a layer norm (a weight, no offset) on a stream of several copies
+  (hyper-connections), a tied head.  Mixer kinds: ``attention`` {heads, kv_heads, dim, vdim, scale, conv, rot{base, dims, scaling},
+  mask{size}} = grouped-query softmax attention in chunks of mask.size positions with biases, a short causal filter of ``conv`` taps on q, k
+  and v, whole-projection q / k norms, neighbour rotary pairs rescaled in bands and a gate per head; ``attention_2`` {heads, kv_heads, dim,
+  vdim, scale, rot, mask{size}} = the same in chunks with biases and unit query / key heads after the rotation, without filter and gate;
+  ``parallel`` {left, right, left_scale, right_scale}: left = windowed grouped-query attention with half-split rotary pairs and a gate per
+  head, right {heads, dim, vdim, gate_cap} = the matrix memory of xLSTM.  ``mlp``: null or experts {expert{ff}, router{experts,
+  top, identity?}, shared{ff}?} of the squared-ReLU form: softmax scores over experts and identity outputs, chosen by score plus a learned
+  correction, weights renormalised, the shared expert times a sigmoid per token.  ``weights_of: j``: layer j's tensors."""
+  def softmax(i, mx, pairs, mask):
+    m = mx.get("mask") or {}
+    rot = mx.get("rot")
+    if rot and int(rot.get("dims", 0)) > int(mx["dim"]):
+      raise ValueError(f"layer {i}: {rot['dims']} rotating entries do not fit a head of {mx['dim']}")
+    lay = {"mixer": "softmax", "heads": int(mx["heads"]), "kv_heads": int(mx["kv_heads"]), "dim": int(mx["dim"]), "vdim": int(mx["vdim"]),
+           "scale": float(mx["scale"]), mask: int(m.get("size", 0))}
+    lay.update(_rotary(i, rot, "", pairs=pairs, scaling="bands"))
+    return lay
+
+  layers = []
+  for i, lc in enumerate(raw["layers"]):
+    mx, kind = lc["mixer"], lc["type"]
+    if kind == "attention":
+      lay = softmax(i, mx, "interleaved", "chunk")
+      lay.update(taps=int(mx.get("conv") or 0), qkv_bias=True, o_bias=True, qk_norm=True, gate=True)
+    elif kind == "attention_2":
+      lay = softmax(i, mx, "interleaved", "chunk")
+      lay.update(qkv_bias=True, o_bias=True, head_norm=True)
+    elif kind == "parallel":
+      ri = mx["right"]
+      lay = softmax(i, mx["left"], "half", "window")
+      lay.update(gate=True, left_scale=float(mx["left_scale"]), right_scale=float(mx["right_scale"]),
+                 second={"mixer": "mlstm", "heads": int(ri["heads"]), "dim": int(ri["dim"]), "vdim": int(ri["vdim"]), "gate_cap": float(ri["gate_cap"])})
+    else:
+      raise ValueError(f"layer {i}: unknown layer type {kind!r}")
+    mlp = lc.get("mlp")
+    if mlp is None:
+      lay.update({"ff": 0, "ff_kind": "none"})
+    elif mlp.get("kind", "moe") == "moe":
+      rt, sh = mlp["router"], mlp.get("shared")
+      lay.update({"ff": int(mlp["expert"]["ff"]), "ff_kind": "moe", "ff_act": "relu2", "route_input": False, "ff_limit": 0.0,
+                  "experts": int(rt["experts"]), "top": int(rt["top"]), "identity": int(rt.get("identity") or 0), "groups": 0, "keep_groups": 0,
+                  "route_scale": 1.0, "route_score": "softmax", "route_norm": True, "route_bias": True,
+                  "shared_ff": int(sh["ff"]) if sh else 0, "shared_limit": 0.0, "shared_gate": bool(sh)})
+    else:
+      raise ValueError(f"layer {i}: unknown feed-forward kind {mlp.get('kind')!r}")
+    lay["weights_of"] = int(lc["weights_of"]) if lc.get("weights_of") is not None else -1
+    layers.append(lay)
+  return {
+    "family": "hybrid", "architecture": "Sizolorn", "block": "prenorm", "norm_kind": "layer", "streams": int(raw.get("streams") or 1), "tied_head": True,
+    "embed_dim": int(raw["width"]), "vocab_size": int(raw["vocab"]), "num_layers": len(layers),
+    "max_seq_len": int(raw.get("max_seq_len", 1 << 20)), "norm_eps": float(raw["norm"]["eps"]),
+    "taps": 0, "side_dim": 0, "logit_softcap": 0.0, "layers": layers,
     "torch_dtype": HF_PRECISION_STR_TO_DTYPE.get(raw.get("torch_dtype", "bfloat16"), torch.bfloat16),
   }
 

@@ -139,7 +139,8 @@ class StageRuntime:
       L.ff_kind = {"relu2": _cabi.FF_RELU2, "none": _cabi.FF_RELU2, "glu_clamp": _cabi.FF_GLU_CLAMP, "glu": _cabi.FF_GLU, "moe": _cabi.FF_MOE}[lc.get("ff_kind", "relu2")]
       L.ff_limit = lc.get("ff_limit", 0.0)
       if lc.get("ff_kind") in ("moe", "glu"):
-        L.ff_act = {"glu_clamp": _cabi.ACT_GLU_CLAMP, "swiglu": _cabi.ACT_SWIGLU, "gelu": _cabi.ACT_GELU, "geglu": _cabi.ACT_GEGLU}[lc.get("ff_act", "glu_clamp")]
+        L.ff_act = {"glu_clamp": _cabi.ACT_GLU_CLAMP, "swiglu": _cabi.ACT_SWIGLU, "gelu": _cabi.ACT_GELU, "geglu": _cabi.ACT_GEGLU,
+                    "relu2": _cabi.ACT_RELU2}[lc.get("ff_act", "glu_clamp")]
       if lc.get("ff_kind") == "moe":
         L.n_experts, L.top, L.groups, L.keep_groups = lc["experts"], lc["top"], lc["groups"], lc["keep_groups"]
         L.route_scale, L.shared_ff, L.shared_limit = lc["route_scale"], lc["shared_ff"], lc["shared_limit"]
@@ -148,6 +149,7 @@ class StageRuntime:
         L.route_score = {"sigmoid": _cabi.ROUTE_SIGMOID, "softmax": _cabi.ROUTE_SOFTMAX}[lc.get("route_score", "sigmoid")]
         L.group_score = {"top2": _cabi.GROUP_TOP2, "max": _cabi.GROUP_MAX}[lc.get("group_score", "top2")]
         L.route_norm = int(bool(lc.get("route_norm", False)))
+        L.identity, L.route_bias = lc.get("identity", 0), int(bool(lc.get("route_bias", False)))
       if lc["mixer"] == "softmax":
         L.mixer = _cabi.MIX_SOFTMAX
         L.s_heads, L.s_kv_heads, L.s_dim, L.s_vdim = lc["heads"], lc["kv_heads"], lc["dim"], lc["vdim"]
@@ -162,8 +164,16 @@ class StageRuntime:
         L.s_rot_mult = lc.get("rot_mult", 1.0)
         L.s_rot_base, L.s_rot_factor, L.s_rot_orig = lc.get("rot_base", 10000.0), lc.get("rot_factor", 1.0), lc.get("rot_orig", 1.0)
         L.s_rot_p0, L.s_rot_p1 = lc.get("rot_p0", 0.0), lc.get("rot_p1", 0.0)
-      elif lc["mixer"] in ("latent", "gdelta", "lightning", "gla"):
-        L.mixer = {"latent": _cabi.MIX_LATENT, "gdelta": _cabi.MIX_GDELTA, "lightning": _cabi.MIX_LIGHTNING, "gla": _cabi.MIX_GLA}[lc["mixer"]]
+        L.s_taps, L.s_head_norm, L.s_o_bias = lc.get("taps", 0), int(bool(lc.get("head_norm"))), int(bool(lc.get("o_bias")))
+        L.s_window, L.s_chunk = lc.get("window", 0), lc.get("chunk", 0)
+        if lc.get("second"):   # another mixer on the same input
+          ri = lc["second"]
+          L.second = {"mlstm": _cabi.MIX_MLSTM}[ri["mixer"]]
+          L.m_heads, L.m_dim, L.m_vdim, L.m_gate_cap = ri["heads"], ri["dim"], ri["vdim"], ri["gate_cap"]
+          L.left_scale, L.right_scale = lc["left_scale"], lc["right_scale"]
+      elif lc["mixer"] in ("latent", "gdelta", "lightning", "gla", "mlstm"):
+        L.mixer = {"latent": _cabi.MIX_LATENT, "gdelta": _cabi.MIX_GDELTA, "lightning": _cabi.MIX_LIGHTNING, "gla": _cabi.MIX_GLA,
+                   "mlstm": _cabi.MIX_MLSTM}[lc["mixer"]]
         L.m_heads, L.m_dim = lc["heads"], lc["dim"]
         if lc["mixer"] == "latent":
           L.m_vdim, L.m_rot_dim, L.m_kv_rank, L.m_rot_dims = lc["vdim"], lc["rot_dim"], lc["kv_rank"], lc["rot_dims"]
@@ -179,7 +189,7 @@ class StageRuntime:
           L.m_vdim, L.m_rank = lc.get("vdim", lc["dim"]), lc["rank"]
           L.m_tau = lc.get("tau", 1.0)
         else:
-          L.m_vdim = lc["vdim"]
+          L.m_vdim, L.m_gate_cap = lc["vdim"], lc.get("gate_cap", 0.0)
       elif lc["mixer"] == "delta":
         L.mixer = _cabi.MIX_DELTA
         L.d_heads, L.d_kv_heads, L.d_dim, L.d_vdim, L.d_taps = lc["heads"], lc["kv_heads"], lc["dim"], lc["vdim"], lc["taps"]
@@ -202,7 +212,8 @@ class StageRuntime:
       gated_residual=int(bool(config.get("gated_residual", False))),
       bigram_buckets=int(bg["buckets"]) if bg else 0, bigram_mul_prev=int(bg["mul_prev"]) if bg else 0,
       bigram_mul_cur=int(bg["mul_cur"]) if bg else 0, pos_rows=int(config.get("pos_rows", 0)),
-      norm_kind=_cabi.NORM_TANH if config.get("norm_kind") == "tanh" else _cabi.NORM_RMS)
+      norm_kind={"tanh": _cabi.NORM_TANH, "layer": _cabi.NORM_LAYER}.get(config.get("norm_kind"), _cabi.NORM_RMS),
+      streams=int(config.get("streams", 0)))
     self.first_from_mlp = self.last_to_attn = False
     self.is_first = self.is_last = True
     self.desc, self._layers = d, lays
