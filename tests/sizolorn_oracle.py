@@ -120,7 +120,8 @@ def attention(state, pre, mx, h, eps, kind):
   H, G, n, m = (int(mx[k]) for k in ("heads", "kv_heads", "dim", "vdim"))
   q, k, v = (project(state, pre + s, h) for s in "qkv")
   if kind == "filtered":
-    q, k, v = (short_filter(a, _t(state, f"{pre}{s}.conv")) for a, s in ((q, "q"), (k, "k"), (v, "v")))
+    if mx.get("conv"):
+      q, k, v = (short_filter(a, _t(state, f"{pre}{s}.conv")) for a, s in ((q, "q"), (k, "k"), (v, "v")))
     q, k = unit_rms(q, eps) * _t(state, pre + "q.norm"), unit_rms(k, eps) * _t(state, pre + "k.norm")
   pos = np.arange(T)
   q, k = (rotate(a.reshape(T, x, n), pos, mx.get("rot"), kind != "window") for a, x in ((q, H), (k, G)))

@@ -240,6 +240,46 @@ _RURUTAR_1B = _rurutar(2048, 128256, [
    ("gla", _gla(16, 128, 128, rank=32), {"kind": "dense", "ff": 8192} if i % 4 == 0 else _gated_experts(16, 4, 384, 2048)))
   for i in range(16)])
 
+def _sizolorn(width, vocab, layers, streams, eps=1e-6):
+  """A Sizolorn config.json: layers is a list of (type, mixer, mlp) or (type, mixer, mlp, layer whose tensors it uses) entries."""
+  return {"architecture": "Sizolorn", "width": width, "vocab": vocab, "streams": streams, "norm": {"eps": eps},
+          "layers": [{"type": x[0], "mixer": x[1], "mlp": x[2], **({"weights_of": x[3]} if len(x) > 3 else {})} for x in layers]}
+
+
+def _masked_attn(heads, kv, dim, vdim, size, rot_dims, base=10000.0, conv=None, scaling=None):
+  m = {"heads": heads, "kv_heads": kv, "dim": dim, "vdim": vdim, "scale": dim ** -0.5, "mask": {"size": size}, "rot": {"base": base, "dims": rot_dims}}
+  if conv:
+    m["conv"] = conv
+  if scaling:
+    m["rot"]["scaling"] = dict(zip(("factor", "low", "high", "original"), scaling))
+  return m
+
+
+def _attn_beside_memory(left, heads, dim, vdim, gate_cap=15.0, left_scale=0.7, right_scale=0.6):
+  return {"left": left, "right": {"heads": heads, "dim": dim, "vdim": vdim, "gate_cap": gate_cap}, "left_scale": left_scale, "right_scale": right_scale}
+
+
+def _identity_experts(n, identity, top, ff, shared_ff):
+  m = _gated_experts(n, top, ff, shared_ff)
+  m["router"]["identity"] = identity
+  return m
+
+
+_SIZOLORN_TINY = _sizolorn(160, 384, [
+  ("parallel", _attn_beside_memory(_masked_attn(6, 2, 24, 40, 21, 16), 3, 24, 40), _identity_experts(6, 1, 2, 48, 72)),
+  ("attention", _masked_attn(4, 2, 32, 24, 40, 32, base=20000.0, conv=4, scaling=(8.0, 1.0, 4.0, 256)), _identity_experts(8, 2, 3, 32, 40)),
+  ("attention_2", _masked_attn(5, 1, 40, 40, 33, 24), None),
+  ("parallel", _attn_beside_memory(_masked_attn(6, 2, 24, 40, 21, 16), 3, 24, 40), _identity_experts(6, 1, 2, 48, 72), 0),
+], streams=2)
+# 1B-class geometry for throughput runs (random weights): the width, depth and vocabulary of llama-3.2-1b, four copies of the stream; of every
+# four layers one in chunks of 2048 with unit heads, one windowed beside a matrix memory (16 heads of 128 x 128), two filtered in chunks
+# of 1024; 16 experts of 512 and two identity outputs of which a token uses four, beside a shared expert of 2048
+_SIZOLORN_1B = _sizolorn(2048, 128256, [
+  ("attention_2", _masked_attn(32, 8, 64, 64, 2048, 64), _identity_experts(16, 2, 4, 512, 2048)) if i % 4 == 0 else
+  ("parallel", _attn_beside_memory(_masked_attn(16, 4, 128, 128, 1024, 64), 16, 128, 128), _identity_experts(16, 2, 4, 512, 2048)) if i % 4 == 1 else
+  ("attention", _masked_attn(32, 8, 64, 64, 1024, 64, base=500000.0, conv=4, scaling=(8.0, 1.0, 4.0, 8192)), _identity_experts(16, 2, 4, 512, 2048))
+  for i in range(16)], streams=4)
+
 # model id -> {layers, repo:{EngineClassName: hf repo}, hf_config}
 model_cards = {
   "llama-3.2-1b": {"layers": 16, "repo": {ENGINE_CLASS_NAME: "unsloth/Llama-3.2-1B-Instruct"},
@@ -269,6 +309,8 @@ model_cards = {
   "vusenex-1b": {"layers": 16, "repo": {ENGINE_CLASS_NAME: "synthetic/vusenex-1b"}, "hf_config": _VUSENEX_1B},
   "rurutar-tiny": {"layers": 4, "repo": {ENGINE_CLASS_NAME: "synthetic/rurutar-tiny"}, "hf_config": _RURUTAR_TINY},
   "rurutar-1b": {"layers": 16, "repo": {ENGINE_CLASS_NAME: "synthetic/rurutar-1b"}, "hf_config": _RURUTAR_1B},
+  "sizolorn-tiny": {"layers": 4, "repo": {ENGINE_CLASS_NAME: "synthetic/sizolorn-tiny"}, "hf_config": _SIZOLORN_TINY},
+  "sizolorn-1b": {"layers": 16, "repo": {ENGINE_CLASS_NAME: "synthetic/sizolorn-1b"}, "hf_config": _SIZOLORN_1B},
   "mistral-tiny": {"layers": 4, "repo": {ENGINE_CLASS_NAME: "synthetic/mistral-tiny"},
                    "hf_config": _mistral(320, 5, 1, 640, 4, head_dim=64, vocab=1280)},
 }

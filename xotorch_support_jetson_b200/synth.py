@@ -392,6 +392,93 @@ def random_rurutar_state(cfg: dict, seed: int = 0, dtype: torch.dtype = torch.bf
   return out
 
 
+def sizolorn_param_shapes(cfg: dict) -> Dict[str, tuple]:
+  """name -> shape of every tensor of a Sizolorn config.json (layers with ``weights_of`` have none)."""
+  D, V, s = cfg["width"], cfg["vocab"], cfg["streams"]
+  sh = {"embed": (V, D), "final.norm": (D,)}
+
+  def attn(p, m, biases, gate):
+    H, G, n, dv = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+    rows = {"q": H * n, "k": G * n, "v": G * dv}
+    for t, r in rows.items():
+      sh[p + t] = (r, D)
+      if biases:
+        sh[p + t + ".b"] = (r,)
+      if m.get("conv"):
+        sh[p + t + ".conv"] = (r, m["conv"])
+    sh[p + "o"] = (D, H * dv)
+    if biases:
+      sh[p + "o.b"] = (D,)
+    if gate:
+      sh[p + "g"] = (H, D)
+
+  for i, lc in enumerate(cfg["layers"]):
+    if lc.get("weights_of") is not None:
+      continue
+    p, m = f"l{i}.", lc["mixer"]
+    for q in (1, 2) if lc.get("mlp") else (1,):
+      sh.update({f"{p}norm{q}": (D,), f"{p}hc{q}.in": (s,), f"{p}hc{q}.out": (s,), f"{p}hc{q}.mix": (s, s)})
+    if lc["type"] == "parallel":
+      attn(p + "mix.left.", m["left"], False, True)
+      H, n, dv = m["right"]["heads"], m["right"]["dim"], m["right"]["vdim"]
+      r = p + "mix.right."
+      sh.update({r + "q": (H * n, D), r + "k": (H * n, D), r + "v": (H * dv, D), r + "g": (H * dv, D), r + "o": (D, H * dv), r + "norm": (H * dv,),
+                 r + "i": (H, D), r + "i.b": (H,), r + "f": (H, D), r + "f.b": (H,)})
+    else:
+      attn(p + "mix.", m, True, lc["type"] == "attention")
+      if lc["type"] == "attention":
+        sh.update({p + "mix.q.norm": (m["heads"] * m["dim"],), p + "mix.k.norm": (m["kv_heads"] * m["dim"],)})
+    mlp = lc.get("mlp")
+    if not mlp:
+      continue
+    F, E = mlp["expert"]["ff"], mlp["router"]["experts"]
+    outs = E + (mlp["router"].get("identity") or 0)
+    sh.update({p + "mlp.router": (outs, D), p + "mlp.correction": (outs,)})
+    for e in range(E):
+      sh.update({f"{p}mlp.e{e}.up": (F, D), f"{p}mlp.e{e}.down": (D, F)})
+    if mlp.get("shared"):
+      S = mlp["shared"]["ff"]
+      sh.update({p + "mlp.shared.up": (S, D), p + "mlp.shared.down": (D, S), p + "mlp.shared.sg": (1, D)})
+  return sh
+
+
+def random_sizolorn_state(cfg: dict, seed: int = 0, dtype: torch.dtype = torch.bfloat16, gain: float = 1.0, device: str = "cpu") -> Dict[str, torch.Tensor]:
+  """Seeded random Sizolorn weights: matrices N(0, gain^2 / in), norm weights 1 + N(0, 0.1^2), biases N(0, 0.1^2), forget offsets
+  spread over (0, 6) so that some heads forget within tokens and others keep hundreds, copies read at about 1 / streams, written at about one
+  and mixed near the identity, filters around their newest tap, routers spread so that the logits differ, embedding rows N(0, 1)."""
+  out, s = {}, cfg["streams"]
+  for idx, (name, shape) in enumerate(sorted(sizolorn_param_shapes(cfg).items())):
+    g = torch.Generator(device=device).manual_seed(seed * 1000003 + idx)
+    rn = lambda: torch.randn(shape, generator=g, device=device)  # noqa: E731
+    leaf = name.split(".")[-1]
+    hc = ".hc1." in name or ".hc2." in name
+    if hc and leaf == "in":
+      t = (1.0 + 0.3 * rn()) / s
+    elif hc and leaf == "out":
+      t = 1.0 + 0.3 * rn()
+    elif hc:
+      t = 0.9 * torch.eye(s, device=device) + 0.1 * rn()
+    elif leaf.startswith("norm"):
+      t = 1.0 + 0.1 * rn()
+    elif name.endswith("right.f.b"):
+      t = 6.0 * torch.rand(shape, generator=g, device=device)
+    elif leaf == "b":
+      t = 0.1 * rn()
+    elif leaf == "conv":
+      t = 0.3 * rn()
+      t[:, -1] += 1.0
+    elif leaf == "correction":
+      t = 0.05 * rn()
+    elif name == "embed":
+      t = rn()
+    elif leaf == "router":
+      t = 2.0 * gain * rn() / (shape[-1] ** 0.5)
+    else:
+      t = gain * rn() / (shape[-1] ** 0.5)
+    out[name] = t.to(dtype)
+  return out
+
+
 def write_random_checkpoint(path: Path, cfg: dict, seed: int = 0, std: float = 0.02,
                             norm_jitter: float = 0.0, shard_bytes: int = 4 << 30,
                             peaked_head: float = 0.0) -> Path:
@@ -410,6 +497,8 @@ def write_random_checkpoint(path: Path, cfg: dict, seed: int = 0, std: float = 0
     state = random_vusenex_state(cfg, seed=seed)
   elif cfg.get("architecture") == "Rurutar":
     state = random_rurutar_state(cfg, seed=seed)
+  elif cfg.get("architecture") == "Sizolorn":
+    state = random_sizolorn_state(cfg, seed=seed)
   else:
     state = random_hf_state(cfg, seed=seed, std=std, norm_jitter=norm_jitter, peaked_head=peaked_head)
   files, cur, cur_bytes = [], {}, 0
