@@ -219,6 +219,12 @@ struct AttDecOpt {
   const float* r1;   // both or neither, one number per head: r1 * ln(1 + r2 * (position - key position)) is taken off the score
   const float* r2;
   int window, chunk;
+  // hg with data: head h's output is multiplied by sigmoid(hg[t, hg_off + h]); everything by out_scale (0 = 1).  out_row: entries
+  // between the rows of out (0 = H * out_head_stride).
+  LinOut hg;
+  int hg_off;
+  float out_scale;
+  long long out_row;
 };
 struct QkvFin {
   const float* part;
@@ -253,6 +259,8 @@ __global__ void __launch_bounds__(160) xb_attn_decode_mma_kernel(
   const int t = blockIdx.x, kvh = opt.v_wide ? (int)blockIdx.y % KV : (int)blockIdx.y, sp = blockIdx.z;
   const int vh = opt.v_wide ? (int)blockIdx.y / KV : 0;
   const long long ohs = opt.out_head_stride > 0 ? opt.out_head_stride : (long long)HD;
+  const long long orow = (!FUSED && opt.out_row > 0) ? opt.out_row : H * ohs;
+  __shared__ float head_mult[G];   // what the group's finished heads are multiplied by
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   pdl_launch_dependents();
   // The batch metadata and page table were uploaded before the step's first kernel started, and
@@ -354,6 +362,11 @@ __global__ void __launch_bounds__(160) xb_attn_decode_mma_kernel(
         qf[ks][0] = lo; qf[ks][1] = 0u; qf[ks][2] = hi; qf[ks][3] = 0u;
       }
     }
+    if (!FUSED && threadIdx.x < G) {   // read behind the barriers of the merge
+      float g = opt.out_scale != 0.f ? opt.out_scale : 1.f;
+      if (opt.hg.f != nullptr || opt.hg.h != nullptr) g *= 1.0f / (1.0f + expf(-lin_at(opt.hg, t, opt.hg_off + kvh * G + threadIdx.x)));
+      head_mult[threadIdx.x] = g;
+    }
     float mrow[2] = {-INFINITY, -INFINITY}, lrow[2] = {0.f, 0.f};
     float o[DT][4];
 #pragma unroll
@@ -427,7 +440,7 @@ __global__ void __launch_bounds__(160) xb_attn_decode_mma_kernel(
       const int hh = kvh * G + g;
       if (n_splits == 1) {
         if (opt.sink != nullptr && M > -INFINITY) L += exp2f(opt.sink[hh] * 1.4426950408889634f - M);
-        out[((long long)t * H + hh) * ohs + (long long)vh * HD + d] = f2bf(L > 0.f ? A / L : 0.f);
+        out[(long long)t * orow + hh * ohs + (long long)vh * HD + d] = f2bf(L > 0.f ? A / L * (FUSED ? 1.f : head_mult[g]) : 0.f);
       } else if (cluster_merge) {
         xc_o[idx] = A;
         if (d == 0) { xc_ml[g * 2] = M; xc_ml[g * 2 + 1] = L; }       // M in log2 units
@@ -479,8 +492,8 @@ __global__ void __launch_bounds__(160) xb_attn_decode_mma_kernel(
             }
           }
         }
-        const float invL = L > 0.f ? 1.0f / L : 0.f;
-        bf16* dst = out + ((long long)t * H + kvh * G + g) * ohs + (long long)vh * HD + lane * VPL;
+        const float invL = L > 0.f ? (FUSED ? 1.0f : head_mult[g]) / L : 0.f;
+        bf16* dst = out + (long long)t * orow + (kvh * G + g) * ohs + (long long)vh * HD + lane * VPL;
 #pragma unroll
         for (int j = 0; j < VPL; j += 2)
           *reinterpret_cast<uint32_t*>(dst + j) = f2_to_bf2(acc[j] * invL, acc[j + 1] * invL);
@@ -626,6 +639,13 @@ struct AttIo {
   int p_split;   // 1: the softmax weights enter the value product as hi + lo bf16 pairs (fp32-grade weights): twice the PV MMAs
   const float* r1;   // both or neither, one number per head: r1 * ln(1 + r2 * (query position - key position)) is taken off
   const float* r2;   // the scaled (and capped) score
+  // EXT kernels.  hg != nullptr: head h's output is multiplied by sigmoid(hg[t * ld_hg + h] + hg_bias[h]) (bias optional); everything by
+  // out_scale (0 = 1).  out_row: entries between the rows of out (0 = H * out_head_stride).
+  const bf16* hg;
+  const float* hg_bias;
+  long long ld_hg;
+  float out_scale;
+  long long out_row;
 };
 
 // EXT = false compiles the plain causal / windowed kernel (the AttIo options below sink are ignored).
@@ -988,9 +1008,15 @@ __global__ void __launch_bounds__(192, 2) xb_attn_prefill_tc_kernel(
     mbar_wait(&o_done[(n_kt - 1) & 1], ((n_kt - 1) >> 1) & 1);
     tc_fence_after();
     if (EXT && io.sink != nullptr && m_used != -INFINITY) l_sum += exp2f(io.sink[kvh * G + gq] * 1.4426950408889634f - m_used);
-    const float inv = l_sum > 0.f ? 1.0f / l_sum : 0.f;
+    float inv = l_sum > 0.f ? 1.0f / l_sum : 0.f;
     const long long ohs = (EXT && io.out_head_stride > 0) ? io.out_head_stride : (long long)HD;
-    bf16* dst = out + ((long long)(t0 + (valid ? tq : 0)) * H + (kvh * G + gq)) * ohs + ((EXT && io.v_wide) ? (long long)blockIdx.z * HD : 0);
+    const long long orow = (EXT && io.out_row > 0) ? io.out_row : H * ohs;
+    if (EXT && io.hg != nullptr) {
+      const float z = bf2f(io.hg[(long long)(t0 + (valid ? tq : 0)) * io.ld_hg + kvh * G + gq]) + (io.hg_bias != nullptr ? io.hg_bias[kvh * G + gq] : 0.f);
+      inv *= 1.0f / (1.0f + expf(-z));
+    }
+    if (EXT && io.out_scale != 0.f) inv *= io.out_scale;
+    bf16* dst = out + (long long)(t0 + (valid ? tq : 0)) * orow + (kvh * G + gq) * ohs + ((EXT && io.v_wide) ? (long long)blockIdx.z * HD : 0);
     const bf16* gate = io.gate != nullptr ? io.gate + (long long)(t0 + (valid ? tq : 0)) * io.ld_gate + (long long)(kvh * G + gq) * HD : nullptr;
 #pragma unroll 1
     for (int c = 0; c < HD; c += 16) {

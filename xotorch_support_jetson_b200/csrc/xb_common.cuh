@@ -220,3 +220,28 @@ __host__ __device__ __forceinline__ int xb_n_segments(const SplitInfo& si, int c
   return ((tile + 1) * si.k_blocks - 1) / si.q - (tile * si.k_blocks) / si.q + 1;
 }
 
+// What a Linear left behind, whatever kernel ran it: one fp32 matrix, fp32 split-K planes, or a bf16 matrix.
+struct LinOut {
+  const float* f;      // fp32 [planes][T][ld] (planes summed per column, see SplitInfo), or nullptr
+  const bf16* h;       // bf16 [T][ld], or nullptr
+  SplitInfo si;        // si.splits == 0: one plane
+  long long plane;     // floats between planes
+  long long ld;
+  const float* bias;   // added on read (outputs of the tcgen05 Linear; the plain kernels add it themselves), or nullptr
+};
+
+__device__ __forceinline__ float lin_at(const LinOut& o, long long row, int col) {
+  const float b = o.bias != nullptr ? o.bias[col] : 0.f;
+  if (o.h != nullptr) return bf2f(o.h[row * o.ld + col]) + b;
+  const float* p = o.f + row * o.ld + col;
+  if (o.si.splits == 0) return *p + b;
+  const int n = xb_n_segments(o.si, col);
+  float s = 0.f;
+  int i = 0;
+  for (; i + 3 < n; i += 4) {   // four planes in flight
+    const float v0 = p[i * o.plane], v1 = p[(i + 1) * o.plane], v2 = p[(i + 2) * o.plane], v3 = p[(i + 3) * o.plane];
+    s += (v0 + v1) + (v2 + v3);
+  }
+  for (; i < n; ++i) s += p[i * o.plane];
+  return s + b;
+}

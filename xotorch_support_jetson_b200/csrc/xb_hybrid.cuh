@@ -1190,6 +1190,8 @@ template <int NCH, int LPC, int MODE>
 static int hy_segments_n(xb_engine* e, const RecurIn& in, float* state, long long ss, float* o, long long ldo, const BatchMeta& m, int n_seqs,
                          int H, int dk, int dv, int T, cudaStream_t st) {
   HyModel* hy = e->hy;
+  const int cols = dv;                      // columns of the state
+  if (MODE == HY_REC_MLSTM) dv = in.dv;     // the value columns among them
   const int cb = (dv + HY_SEG_COLS - 1) / HY_SEG_COLS;
   SegArgs sg;
   sg.seg = hy->seg_len > 0 ? hy->seg_len : ((long long)(T / 128) * H * cb >= 4LL * e->num_sms ? 128 : HY_SEG_MIN);
@@ -1197,6 +1199,7 @@ static int hy_segments_n(xb_engine* e, const RecurIn& in, float* state, long lon
   sg.ws = hy->seg_ws;
   sg.decay = MODE == HY_REC_LIGHTNING ? nullptr : hy->seg_decay;
   sg.per_head = MODE == HY_REC_MLSTM ? 1 : 0;
+  sg.cols = cols;
   const dim3 grid(cb, H, n_seqs * sg.max_segs);
   constexpr size_t row = (size_t)2 * HY_SEG_TS * sizeof(float);
   constexpr int ex = MODE == HY_REC_MLSTM ? 4 : 0;
@@ -1204,16 +1207,13 @@ static int hy_segments_n(xb_engine* e, const RecurIn& in, float* state, long lon
   if (s0 > 48 * 1024) XB_SMEM_ATTR_ONCE((hy_seg_kernel<NCH, LPC, MODE, 0>), s0);
   if (s1 > 48 * 1024) XB_SMEM_ATTR_ONCE((hy_seg_kernel<NCH, LPC, MODE, 1>), s1);
   XB_TRY(hy_launch(e, hy_seg_kernel<NCH, LPC, MODE, 0>, grid, dim3(128), s0, st, in, sg, state, ss, o, ldo, m, H, dk, dv));
-  if (sg.per_head)
-    XB_TRY(hy_launch(e, hy_seg_decay_kernel, dim3((H + 255) / 256, n_seqs * sg.max_segs), dim3(256), 0, st, in.decay, (long long)H, 0LL, H, sg.seg, sg.max_segs,
-                     hy->seg_decay, m));
-  else if (sg.decay != nullptr)
+  if (sg.decay != nullptr && !sg.per_head)
     XB_TRY(hy_launch(e, hy_seg_decay_kernel, dim3((H * dk + 255) / 256, n_seqs * sg.max_segs), dim3(256), 0, st, in.c, in.ldc,
                      MODE == HY_REC_GLA ? in.xoff[0] : in.koff, H * dk, sg.seg, sg.max_segs, hy->seg_decay, m));
   if (dk % 4 == 0)
-    XB_TRY(hy_launch(e, hy_seg_scan_kernel<4>, dim3((dv * dk / 4 + 127) / 128, H, n_seqs), dim3(128), 0, st, sg, in.hdecay, (const float*)state, ss, m, H, dk, dv));
+    XB_TRY(hy_launch(e, hy_seg_scan_kernel<4>, dim3((cols * dk / 4 + 127) / 128, H, n_seqs), dim3(128), 0, st, sg, in.hdecay, (const float*)state, ss, m, H, dk, cols));
   else
-    XB_TRY(hy_launch(e, hy_seg_scan_kernel<1>, dim3((dv * dk + 127) / 128, H, n_seqs), dim3(128), 0, st, sg, in.hdecay, (const float*)state, ss, m, H, dk, dv));
+    XB_TRY(hy_launch(e, hy_seg_scan_kernel<1>, dim3((cols * dk + 127) / 128, H, n_seqs), dim3(128), 0, st, sg, in.hdecay, (const float*)state, ss, m, H, dk, cols));
   return hy_launch(e, hy_seg_kernel<NCH, LPC, MODE, 1>, grid, dim3(128), s1, st, in, sg, state, ss, o, ldo, m, H, dk, dv);
 }
 template <int MODE>
@@ -1566,6 +1566,19 @@ static int hy_router(xb_engine* e, const HyLayer& l, int T, const void* xin, int
     return hy_launch(e, hy_router_route_kernel<AT>, dim3(T), dim3(32 * (NE < 32 ? (NE < 8 ? 8 : NE) : 32)), rs1, st, x, (long long)D, (const bf16*)l.w_router, D, EI, c.top, c.groups,
                      c.keep_groups, c.route_scale, hy->gw, c.route_score, c.group_score, c.route_norm, sg, choice);
   }
+  if constexpr (std::is_same<AT, bf16>::value) {   // prompts: the logits on the tensor cores, routed where they were made
+    if (T > 64 && D % 8 == 0 && NE <= HY_ROUTER_MMA_MAX) {
+      const size_t sm = hy_router_mma_smem(NE, EI, ng);
+#define HY_ROUTER_CASE(N)                                                                                                              \
+  if (NE <= 8 * N)                                                                                                                     \
+    return hy_launch(e, hy_router_mma_kernel<N>, dim3((T + 15) / 16), dim3(256), sm, st, x, (long long)D, (const bf16*)l.w_router, D, T, EI, c.top, c.groups, \
+                     c.keep_groups, c.route_scale, hy->gw, c.route_score, c.group_score, c.route_norm, sg, choice);
+      HY_ROUTER_CASE(2)
+      HY_ROUTER_CASE(4)
+      HY_ROUTER_CASE(8)
+#undef HY_ROUTER_CASE
+    }
+  }
   if (T <= 64) {   // few rows: a warp per (token, expert)
     XB_TRY(hy_launch(e, hy_router_logits_kernel<AT, 1>, dim3((unsigned)(((long long)T * NE + 7) / 8)), dim3(256), 0, st, x, (long long)D,
                      (const bf16*)l.w_router, hy->m2, T, NE, D));
@@ -1730,6 +1743,34 @@ static int hy_heads_mix_bf16(xb_engine* e, const HyLayer& l, int T, const LinOut
                    c.s_gate ? l.off_g : -1, H, G, dv, a1, (long long)l.n_o, ohs, os);
 }
 
+template <typename KT>
+static int hy_qkv_prep(xb_engine* e, const HyLayer& l, int T, const LinOut& P, const QkvPrep& a, const BatchMeta& m, cudaStream_t st) {
+  KT *kp = (KT*)l.k_pool, *vp = (KT*)l.v_pool;
+  const int NH = a.H + a.G;
+  if constexpr (std::is_same<KT, bf16>::value) {
+    const size_t tile = (size_t)HY_PREP_ROWS * (NH * (a.dk + 1) + a.rot.dims) * sizeof(float);
+    const bool taps = a.taps == 0 || (a.taps >= 2 && a.taps <= 4);
+    if (T > 64 && a.qg != nullptr && a.qa == nullptr && P.h != nullptr && ((P.ld | a.dk | a.dv | a.off_q) & 7) == 0 && taps && tile <= 160 * 1024 &&
+        !(a.head_norm && (a.qn != nullptr || a.temp_every > 0))) {
+      const dim3 grid((T + HY_PREP_ROWS - 1) / HY_PREP_ROWS);
+#define HY_PREP_CASE(N)                                                                                    \
+  if (a.taps == N) {                                                                                       \
+    if (tile > 48 * 1024) XB_SMEM_ATTR_ONCE(hy_qkv_prep_tile_kernel<N>, 160 * 1024);                       \
+    return hy_launch(e, hy_qkv_prep_tile_kernel<N>, grid, dim3(256), tile, st, P, a, kp, vp, m, T);        \
+  }
+      HY_PREP_CASE(0)
+      HY_PREP_CASE(2)
+      HY_PREP_CASE(3)
+      HY_PREP_CASE(4)
+#undef HY_PREP_CASE
+    }
+  }
+  const int nb = T <= 64 ? (NH >= 8 ? 8 : NH) : 1;   // few rows: a cluster of blocks per row
+  const size_t sm = (size_t)((NH + nb - 1) / nb * (a.dk + 1) + a.rot.dims) * sizeof(float);
+  if (nb > 1) return launch_kc(e, hy_qkv_prep_kernel<KT, 256>, dim3(T, nb), dim3(256), sm, st, dim3(1, nb, 1), P, a, kp, vp, m);
+  return hy_launch(e, hy_qkv_prep_kernel<KT, 256>, dim3(T), dim3(256), sm, st, P, a, kp, vp, m);
+}
+
 template <typename AT>
 static int hy_softmax_mixer(xb_engine* e, const HyLayer& l, int T, int n_seqs, int n_tiles, const LinOut& P, const BatchMeta& m, cudaStream_t st) {
   HyModel* hy = e->hy;
@@ -1759,16 +1800,7 @@ static int hy_softmax_mixer(xb_engine* e, const HyLayer& l, int T, int n_seqs, i
     a.rot = r; a.head_norm = c.s_head_norm;
     a.qa = (tc || dec) ? (float*)nullptr : hy->qa;
     a.qg = (tc || dec) ? hy->qg : (bf16*)nullptr;
-    const size_t sm = (size_t)((H + G) * (dk + 1) + c.s_rot_dims) * sizeof(float);
-    bool vec8 = false;
-    if constexpr (std::is_same<KT, bf16>::value) vec8 = T > 64 && P.h != nullptr && P.ld % 8 == 0 && dk % 8 == 0 && dv % 8 == 0 && l.off_q % 8 == 0;
-    if (vec8) {
-      if constexpr (std::is_same<KT, bf16>::value)
-        XB_TRY(hy_launch(e, hy_qkv_prep_kernel<KT, 256, 8>, dim3(T), dim3(256), sm, st, P, a, (KT*)l.k_pool, (KT*)l.v_pool, m));
-    } else if (T <= 64)
-      XB_TRY(hy_launch(e, hy_qkv_prep_kernel<KT, 1024, 1>, dim3(T), dim3(1024), sm, st, P, a, (KT*)l.k_pool, (KT*)l.v_pool, m));
-    else
-      XB_TRY(hy_launch(e, hy_qkv_prep_kernel<KT, 256, 1>, dim3(T), dim3(256), sm, st, P, a, (KT*)l.k_pool, (KT*)l.v_pool, m));
+    XB_TRY(hy_qkv_prep<KT>(e, l, T, P, a, m, st));
     if (c.s_taps > 1 && !a.write_tail) {
       const int C = H * dk + G * (dk + dv);
       XB_TRY(hy_launch(e, hy_tail_update_kernel, dim3(n_seqs, (C + 255) / 256), dim3(256), 0, st, P, l.off_q, C, c.s_taps, a.tail, a.tail_stride, m));
@@ -1805,7 +1837,10 @@ static int hy_softmax_mixer(xb_engine* e, const HyLayer& l, int T, int n_seqs, i
   const int vch = dvo > 512 ? 512 : 0;   // wider value rows: blocks along z take 512 channels each
   const AttnOpt opt{c.s_sink ? l.sink : nullptr, c.s_softcap, l.v_all ? 1 : G, vch, c.s_dist_bias ? l.r1 : nullptr, c.s_dist_bias ? l.r2 : nullptr, c.s_chunk};
   // padded rows and a second mixer's columns beside this one's go through the head kernel as well
-  const bool post = c.s_talk != 0 || c.s_gate != 0 || c.second != 0 || ((tc || dec) && l.vp != dv);
+  bool post = c.s_talk != 0 || c.s_gate != 0 || c.second != 0 || ((tc || dec) && l.vp != dv);
+  // head gates and a mixer's scale in the tensor-core kernels' own epilogues (prompts: gates out of a bf16 projection)
+  const bool own_gate = !c.s_talk && l.vp == dv && (dec || (tc && (P.h != nullptr || !c.s_gate))) && l.n_o % 8 == 0;
+  if (own_gate) post = false;
   const int wide = l.v_all ? 1 : (l.vpieces > 1 ? 2 : 0);
   const long long ohs = l.v_all ? (long long)G * dv : l.vp;
   const int HD = l.kp;
@@ -1815,7 +1850,9 @@ static int hy_softmax_mixer(xb_engine* e, const HyLayer& l, int T, int n_seqs, i
     const int span = c.s_window > 0 && (c.s_chunk <= 0 || c.s_window < c.s_chunk) ? c.s_window : c.s_chunk;   // most keys a query sees, 0 = all
     if (span > 0 && ns > (span + XB_ATT_TILE - 2) / XB_ATT_TILE + 1) ns = (span + XB_ATT_TILE - 2) / XB_ATT_TILE + 1;
     ns = ns < 1 ? 1 : ns;
-    const AttDecOpt dopt{c.s_sink ? l.sink : nullptr, c.s_softcap, wide, ohs, hy->p_split, opt.r1, opt.r2, c.s_window, c.s_chunk};
+    AttDecOpt dopt{c.s_sink ? l.sink : nullptr, c.s_softcap, wide, ohs, hy->p_split, opt.r1, opt.r2, c.s_window, c.s_chunk};
+    dopt.hg = own_gate && c.s_gate ? P : hy_none();
+    dopt.hg_off = l.off_g; dopt.out_scale = own_gate && c.second ? c.left_scale : 0.f; dopt.out_row = own_gate ? l.n_o : 0;
     bf16* dst = post ? reinterpret_cast<bf16*>(hy->o) : reinterpret_cast<bf16*>(hy->a1);
     if (HD == 128) XB_TRY(hy_attn_dec<128>(e, l, m, T, hy->qg, dst, H, G, c.s_scale, ns, dopt, st));
     else XB_TRY(hy_attn_dec<64>(e, l, m, T, hy->qg, dst, H, G, c.s_scale, ns, dopt, st));
@@ -1826,6 +1863,9 @@ static int hy_softmax_mixer(xb_engine* e, const HyLayer& l, int T, int n_seqs, i
     HyAttnIn in;
     in.tile_start = m.tile_start; in.tile_len = m.tile_len; in.n_tiles = n_tiles; in.q = hy->qg;
     in.io = AttIo{(long long)H * l.kp, nullptr, nullptr, 0, c.s_sink ? l.sink : nullptr, c.s_softcap, wide, ohs, hy->p_split, opt.r1, opt.r2};
+    if (own_gate && c.s_gate) { in.io.hg = P.h + l.off_g; in.io.hg_bias = P.bias != nullptr ? P.bias + l.off_g : nullptr; in.io.ld_hg = P.ld; }
+    in.io.out_scale = own_gate && c.second ? c.left_scale : 0.f;
+    in.io.out_row = own_gate ? l.n_o : 0;
     bf16* dst = post ? reinterpret_cast<bf16*>(hy->o) : reinterpret_cast<bf16*>(hy->a1);
     if (HD == 128) XB_TRY(hy_attn_tc_any<128>(e, l, m, in, dst, H, G, c.s_scale, l.v_all ? G : l.vpieces, st));
     else XB_TRY(hy_attn_tc_any<64>(e, l, m, in, dst, H, G, c.s_scale, l.v_all ? G : l.vpieces, st));
@@ -1942,9 +1982,10 @@ static int hy_hyper(xb_engine* e, int T, const HyperArgs& a, cudaStream_t st) {
   const size_t sm = (size_t)D * sizeof(float);
   const bool plain = a.y.f == nullptr || a.y.si.splits == 0;
   const bool vec = D % 4 == 0 && plain && ((a.y.f == nullptr && a.y.h == nullptr) || a.y.ld % 4 == 0);
-  if (T <= 64 && D >= 1024 && !vec) {   // few rows out of split-K planes: more threads per row keep more loads in flight
-    if (n <= 4) return hy_launch(e, hy_hyper_kernel<AT, 1024, 4, 1>, dim3(T), dim3(1024), sm, st, a);
-    return hy_launch(e, hy_hyper_kernel<AT, 1024, HY_MAX_STREAMS, 1>, dim3(T), dim3(1024), sm, st, a);
+  if (T <= 64 && D >= 512 && (a.y.f != nullptr || a.y.h != nullptr)) {   // few rows: a cluster of blocks per row
+    const int nb = 8, per = (D + nb - 1) / nb;
+    if (n <= 4) return launch_kc(e, hy_hyper_cluster_kernel<AT, 4>, dim3(T, nb), dim3(256), (size_t)per * sizeof(float), st, dim3(1, nb, 1), a);
+    return launch_kc(e, hy_hyper_cluster_kernel<AT, HY_MAX_STREAMS>, dim3(T, nb), dim3(256), (size_t)per * sizeof(float), st, dim3(1, nb, 1), a);
   }
   if (n <= 4) {
     if (vec) return hy_launch(e, hy_hyper_kernel<AT, 256, 4, 4>, dim3(T), dim3(256), sm, st, a);
@@ -1967,7 +2008,7 @@ static int hy_mlstm_mixer(xb_engine* e, const HyLayer& l, int T, int n_seqs, con
   if (T == n_seqs && tsm <= 48 * 1024)   // single tokens
     return hy_launch(e, hy_mlstm_token_kernel<AT>, dim3(n_seqs, H), dim3(512), tsm, st, P, l.off_mq, l.off_mk, l.off_mv, l.off_mg, l.off_mi, l.off_mf, c.m_gate_cap,
                      scale, rec, ms, SS, (const float*)l.m_norm, eps, out_scale, out, (long long)l.n_o, m, H, n, dv);
-  XB_TRY(hy_launch(e, hy_mlstm_gates_kernel, dim3(H, n_seqs), dim3(256), 0, st, P, l.off_mi, l.off_mf, c.m_gate_cap, ms, SS, hy->decay, hy->beta, hy->qk, H, m));
+  XB_TRY(hy_launch(e, hy_mlstm_gates_kernel, dim3(H, n_seqs), dim3(HY_GATE_THREADS), 0, st, P, l.off_mi, l.off_mf, c.m_gate_cap, ms, SS, hy->decay, hy->beta, hy->qk, H, m));
   const bool vec = P.h != nullptr && ((P.ld | l.off_mq | l.off_mk | l.off_mv | n | dv) & 7) == 0;
   const int units = vec ? (2 * HK + H * dv) / 8 + H : 2 * HK + H * dv + H;
   auto prep = vec ? hy_mlstm_prep_kernel<8> : hy_mlstm_prep_kernel<1>;
@@ -1975,8 +2016,13 @@ static int hy_mlstm_mixer(xb_engine* e, const HyLayer& l, int T, int n_seqs, con
   RecurIn in;
   in.c = hy->c; in.ldc = ldc; in.qoff = 0; in.koff = HK; in.voff = 2LL * HK; in.q_heads = H;
   in.xoff[0] = in.xoff[1] = in.xoff[2] = 0;
-  in.beta = in.qk = in.hdecay = nullptr; in.decay = hy->decay;
+  in.beta = in.qk = in.hdecay = nullptr; in.decay = hy->decay; in.dv = dv;
   XB_TRY(hy_recur<HY_REC_MLSTM>(e, in, rec, SS, hy->o, ldo, m, n_seqs, H, n, dvp, T, st));
+  const int per = dv / 8;
+  if (P.h != nullptr && ((P.ld | l.off_mg | l.n_o | l.n_left | dv) & 7) == 0 && per <= 32 && (per & (per - 1)) == 0)
+    return hy_launch(e, hy_mlstm_out_vec_kernel<AT>, dim3((unsigned)(((long long)T * H * per + 255) / 256)), dim3(256), 0, st, (const float*)hy->o, (const float*)hy->qk,
+                     (const float*)l.m_norm, P.h + l.off_mg, P.ld, P.bias != nullptr ? P.bias + l.off_mg : (const float*)nullptr, eps, out_scale, out,
+                     (long long)l.n_o, T, H, dv);
   return hy_launch(e, hy_mlstm_out_kernel<AT>, dim3((unsigned)(((long long)T * H + 7) / 8)), dim3(256), 0, st, (const float*)hy->o, (const float*)hy->qk,
                    (const float*)l.m_norm, P, l.off_mg, eps, out_scale, out, (long long)l.n_o, T, H, dv);
 }

@@ -29,31 +29,6 @@
 #define HY_REC_GLA 4
 #define HY_REC_MLSTM 5
 
-struct LinOut {
-  const float* f;      // fp32 [planes][T][ld] (planes summed per column, see SplitInfo), or nullptr
-  const bf16* h;       // bf16 [T][ld], or nullptr
-  SplitInfo si;        // si.splits == 0: one plane
-  long long plane;     // floats between planes
-  long long ld;
-  const float* bias;   // added on read (outputs of the tcgen05 Linear; the plain kernels add it themselves), or nullptr
-};
-
-__device__ __forceinline__ float lin_at(const LinOut& o, long long row, int col) {
-  const float b = o.bias != nullptr ? o.bias[col] : 0.f;
-  if (o.h != nullptr) return bf2f(o.h[row * o.ld + col]) + b;
-  const float* p = o.f + row * o.ld + col;
-  if (o.si.splits == 0) return *p + b;
-  const int n = xb_n_segments(o.si, col);
-  float s = 0.f;
-  int i = 0;
-  for (; i + 3 < n; i += 4) {   // four planes in flight
-    const float v0 = p[i * o.plane], v1 = p[(i + 1) * o.plane], v2 = p[(i + 2) * o.plane], v3 = p[(i + 3) * o.plane];
-    s += (v0 + v1) + (v2 + v3);
-  }
-  for (; i < n; ++i) s += p[i * o.plane];
-  return s + b;
-}
-
 template <typename AT> __device__ __forceinline__ void act_store(AT* p, float v);
 template <> __device__ __forceinline__ void act_store<float>(float* p, float v) { *p = v; }
 template <> __device__ __forceinline__ void act_store<bf16>(bf16* p, float v) { *p = f2bf(v); }
@@ -747,6 +722,11 @@ __global__ void __launch_bounds__(256) hy_linear_tiled_kernel(const AT* __restri
       ws[kk][r] = wv;
     }
     __syncthreads();
+    float part[4][4];   // a slice's own sum joins the total at once: rounding grows with the slices, not with k
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) part[i][j] = 0.f;
 #pragma unroll
     for (int kk = 0; kk < 16; ++kk) {
       float a[4], b[4];
@@ -757,8 +737,12 @@ __global__ void __launch_bounds__(256) hy_linear_tiled_kernel(const AT* __restri
 #pragma unroll
       for (int i = 0; i < 4; ++i)
 #pragma unroll
-        for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(a[i], b[j], acc[i][j]);
+        for (int j = 0; j < 4; ++j) part[i][j] = fmaf(a[i], b[j], part[i][j]);
     }
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) acc[i][j] += part[i][j];
     __syncthreads();
   }
 #pragma unroll
@@ -836,6 +820,7 @@ struct RecurIn {
   int q_heads;           // delta rule: heads share q / k in groups (q head = h / (H / q_heads)); others: = H
   const float *beta, *decay, *qk;   // gated delta rule: [T, H], [T, H], [T, q_heads]; HY_REC_GDELTA: beta = r.(a*u), decay = r.k, [T, H]; HY_REC_MLSTM: decay = w [T, H]
   const float* hdecay;   // HY_REC_LIGHTNING: [H] constant decay per head
+  int dv;                // HY_REC_MLSTM: value columns (the normaliser's and the padding behind them are columns of the state, too)
 };
 __device__ __forceinline__ void hy_cp4(float* dst, const float* src) {
   asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
@@ -1139,9 +1124,11 @@ __device__ __forceinline__ hy_f2 hy_f2_mul(hy_f2 a, hy_f2 b) {
 }
 struct SegArgs {
   float* ws;              // [entries][H * dv * dk]
-  const float* decay;     // [entries][H * dk], [entries][H] (per_head), or nullptr (lightning)
+  float* decay;           // [entries][H * dk], [entries][H] (per_head: made by PASS 0 itself), or nullptr (lightning)
   int seg, max_segs;      // tokens per segment, segments of the longest sequence a step can hold
   int per_head;           // 1: a head's channels fade alike
+  int cols;               // columns of a head in state, workspace and o; > dv for the matrix memory, whose column dv is the normaliser (its
+                          // value is one): the first warp of a head's first block carries it beside its own columns
 };
 // row vectors staged per step: k (or f), w where it is a vector of its own, q in the output pass
 __host__ __device__ constexpr int hy_seg_vectors(int mode, int pass) { return 1 + (mode == HY_REC_GLA ? 1 : 0) + (pass == 1 ? 1 : 0); }
@@ -1158,7 +1145,8 @@ __global__ void __launch_bounds__(128) hy_seg_kernel(RecurIn in, SegArgs sg, flo
   const int nseg = (sp.len + sg.seg - 1) / sg.seg;
   if (c >= nseg || (PASS == 0 && c == nseg - 1)) return;
   const int row0 = sp.start + c * sg.seg, len = sp.len - c * sg.seg < sg.seg ? sp.len - c * sg.seg : sg.seg;
-  float* entry = sg.ws + (long long)(sp.start / sg.seg + s + c) * H * dv * dk;
+  const int cols = MODE == HY_REC_MLSTM ? sg.cols : dv;
+  float* entry = sg.ws + (long long)(sp.start / sg.seg + s + c) * H * cols * dk;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, sub = lane & (LPC - 1);
   const int jl = (warp * (32 / LPC) + lane / LPC) * NCOL, ncv = dv - j0 < NB ? dv - j0 : NB;
   // staged vectors in the order of the shared rows: k, (w), (q)
@@ -1166,7 +1154,9 @@ __global__ void __launch_bounds__(128) hy_seg_kernel(RecurIn in, SegArgs sg, flo
   src[0] = in.c + in.koff + (long long)h * dk;
   if (MODE == HY_REC_GLA) src[1] = in.c + in.xoff[0] + (long long)h * dk;
   if (PASS == 1) src[NV - 1] = in.c + in.qoff + (long long)h * dk;
-  const float* cv = in.c + in.voff + (long long)h * dv + j0;
+  const float* cv = in.c + in.voff + (long long)h * cols + j0;
+  const bool norm = MODE == HY_REC_MLSTM && blockIdx.x == 0 && warp == 0;   // both lane groups of the warp do the same work on it
+  float faded = 1.f;   // product of the segment's decays (per_head)
   const hy_f2 hd2 = MODE == HY_REC_LIGHTNING ? hy_f2_pack(in.hdecay[h], in.hdecay[h]) : 0ull;
   bool al = ((in.ldc | in.qoff | in.koff | in.voff | dk | dv) & 3) == 0 && (reinterpret_cast<uintptr_t>(in.c) & 15) == 0;
   if (MODE == HY_REC_GLA) al = al && (in.xoff[0] & 3) == 0;
@@ -1181,7 +1171,7 @@ __global__ void __launch_bounds__(128) hy_seg_kernel(RecurIn in, SegArgs sg, flo
 #pragma unroll
   for (int n = 0; n < NCOL; ++n) {
     const bool have = PASS == 1 && jl + n < ncv;
-    const float* st = entry + ((long long)h * dv + j0 + jl + n) * dk;
+    const float* st = entry + ((long long)h * cols + j0 + jl + n) * dk;
 #pragma unroll
     for (int ch = 0; ch < NCH; ++ch) {
       const int r = (ch * LPC + sub) * 4;
@@ -1194,6 +1184,18 @@ __global__ void __launch_bounds__(128) hy_seg_kernel(RecurIn in, SegArgs sg, flo
         for (int x = 0; x < 4; ++x) e[x] = (have && r + x < dk) ? st[r + x] : 0.f;
         S[n][2 * ch] = hy_f2_pack(e[0], e[1]); S[n][2 * ch + 1] = hy_f2_pack(e[2], e[3]);
       }
+    }
+  }
+  hy_f2 Sn[2 * NCH];
+  if (MODE == HY_REC_MLSTM) {
+    const float* st = entry + ((long long)h * cols + dv) * dk;
+#pragma unroll
+    for (int ch = 0; ch < NCH; ++ch) {
+      const int r = (ch * LPC + sub) * 4;
+      float e[4];
+#pragma unroll
+      for (int x = 0; x < 4; ++x) e[x] = (norm && PASS == 1 && r + x < dk) ? st[r + x] : 0.f;
+      Sn[2 * ch] = hy_f2_pack(e[0], e[1]); Sn[2 * ch + 1] = hy_f2_pack(e[2], e[3]);
     }
   }
   __syncthreads();
@@ -1241,6 +1243,8 @@ __global__ void __launch_bounds__(128) hy_seg_kernel(RecurIn in, SegArgs sg, flo
       const float* sr = buf + ts * STRIDE;
       hy_f2 vv[NCOL], acc[NCOL];
       const hy_f2 fade = MODE == HY_REC_MLSTM ? hy_f2_pack(sr[VO + NB], sr[VO + NB]) : hd2;
+      hy_f2 accn = 0ull;
+      if (MODE == HY_REC_MLSTM && PASS == 0) faded *= sr[VO + NB];
 #pragma unroll
       for (int n = 0; n < NCOL; n += 4) {
         const float4 v = *reinterpret_cast<const float4*>(sr + VO + jl + n);
@@ -1276,6 +1280,19 @@ __global__ void __launch_bounds__(128) hy_seg_kernel(RecurIn in, SegArgs sg, flo
             S[n][2 * ch + x] = hy_f2_fma(w2[x], S[n][2 * ch + x], hy_f2_mul(k2[x], vv[n]));
             if (PASS == 1) acc[n] = hy_f2_fma(q2[x], S[n][2 * ch + x], acc[n]);
           }
+        if (MODE == HY_REC_MLSTM && norm)
+#pragma unroll
+          for (int x = 0; x < 2; ++x) {
+            Sn[2 * ch + x] = hy_f2_fma(fade, Sn[2 * ch + x], k2[x]);
+            if (PASS == 1) accn = hy_f2_fma(q2[x], Sn[2 * ch + x], accn);
+          }
+      }
+      if (MODE == HY_REC_MLSTM && PASS == 1 && norm) {
+        const float2 a = hy_f2_unpack(accn);
+        float y = a.x + a.y;
+#pragma unroll
+        for (int off = 1; off < LPC; off <<= 1) y += __shfl_xor_sync(0xffffffffu, y, off);
+        if (lane == 0) o[(long long)(row0 + t0 + ts) * ldo + (long long)h * cols + dv] = y;
       }
       if (PASS == 1) {
         // sums over the lanes: partners swap halves of their columns, so that log2(LPC) rounds leave one column per lane pair
@@ -1296,7 +1313,7 @@ __global__ void __launch_bounds__(128) hy_seg_kernel(RecurIn in, SegArgs sg, flo
           }
         }
         const float mine = y[0] + __shfl_xor_sync(0xffffffffu, y[0], LPC / 2);
-        if (writer) o[(long long)(row0 + t0 + ts) * ldo + (long long)h * dv + j0 + jl + col] = mine;
+        if (writer) o[(long long)(row0 + t0 + ts) * ldo + (long long)h * cols + j0 + jl + col] = mine;
       }
     };
     if (idle) {
@@ -1314,7 +1331,7 @@ __global__ void __launch_bounds__(128) hy_seg_kernel(RecurIn in, SegArgs sg, flo
 #pragma unroll
   for (int n = 0; n < NCOL; ++n) {
     if (jl + n >= ncv) continue;
-    float* st = base + ((long long)h * dv + j0 + jl + n) * dk;
+    float* st = base + ((long long)h * cols + j0 + jl + n) * dk;
 #pragma unroll
     for (int ch = 0; ch < NCH; ++ch) {
       const int r = (ch * LPC + sub) * 4;
@@ -1328,6 +1345,19 @@ __global__ void __launch_bounds__(128) hy_seg_kernel(RecurIn in, SegArgs sg, flo
           if (r + x < dk) st[r + x] = e[x];
       }
     }
+  }
+  if (MODE == HY_REC_MLSTM && norm && lane < LPC) {
+    float* st = base + ((long long)h * cols + dv) * dk;
+#pragma unroll
+    for (int ch = 0; ch < NCH; ++ch) {
+      const int r = (ch * LPC + sub) * 4;
+      const float2 a = hy_f2_unpack(Sn[2 * ch]), b = hy_f2_unpack(Sn[2 * ch + 1]);
+      const float e[4] = {a.x, a.y, b.x, b.y};
+#pragma unroll
+      for (int x = 0; x < 4; ++x)
+        if (r + x < dk) st[r + x] = e[x];
+    }
+    if (PASS == 0 && lane == 0) sg.decay[(long long)(sp.start / sg.seg + s + c) * H + h] = faded;
   }
 }
 
@@ -2957,6 +2987,71 @@ __global__ void __launch_bounds__(1024) hy_router_route_kernel(const AT* __restr
   }
   __syncthreads();
   if (warp == 0) hy_route_token(rsm, rsm + NE, rsm + NE + E, rsm + NE + 2 * E, E, top, groups, keep, scale, gw + t * NE, score_mode, group_mode, renorm, shared_gate, choice);
+}
+
+// Prompts in bf16 serving: a block forms the logits of 16 tokens with m16n8k16 MMAs (bf16 products, fp32 sums), its eight warps sharing out the
+// channels, then routes them, two tokens per warp.  A lane's 16-byte loads of a token row and of a router row hold eight neighbouring
+// channels; pairs 0, 1 and 2, 3 of them stand for the k positions of one MMA, in both operands alike.
+// NT8: router rows in eights.  K a multiple of 8.  grid (ceil(T / 16)), 256 threads.
+#define HY_ROUTER_MMA_MAX 64
+__host__ __device__ constexpr size_t hy_router_mma_smem(int NE, int EI, int ng) {
+  return (size_t)(8 * 16 * ((NE + 7) / 8 * 8) + 8 * (2 * EI + ng)) * sizeof(float);
+}
+template <int NT8>
+__global__ void __launch_bounds__(256) hy_router_mma_kernel(const bf16* __restrict__ x, long long ldx, const bf16* __restrict__ w, int K, int T, int E, int top,
+                                                            int groups, int keep, float scale, float* __restrict__ gw, int score_mode, int group_mode,
+                                                            int renorm, int shared_gate, const float* __restrict__ choice) {
+  pdl_launch_dependents();
+  pdl_wait();
+  extern __shared__ __align__(16) float rsm[];
+  const int NE = E + (shared_gate ? 1 : 0), NP = (NE + 7) / 8 * 8;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, t0 = blockIdx.x * 16, r = lane >> 2, kc = (lane & 3) * 8;
+  const int ta = t0 + r < T ? t0 + r : T - 1, tb = t0 + r + 8 < T ? t0 + r + 8 : T - 1;
+  const bf16 *xa = x + ta * ldx, *xb = x + tb * ldx;
+  float acc[NT8][4];
+#pragma unroll
+  for (int j = 0; j < NT8; ++j) acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.f;
+  const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
+#pragma unroll 2
+  for (int kb = warp * 32; kb < K; kb += 256) {
+    const int k = kb + kc;
+    const bool in = k < K;
+    const uint4 a0 = in ? *reinterpret_cast<const uint4*>(xa + k) : zero, a1 = in ? *reinterpret_cast<const uint4*>(xb + k) : zero;
+    const uint32_t f0[4] = {a0.x, a1.x, a0.y, a1.y}, f1[4] = {a0.z, a1.z, a0.w, a1.w};
+#pragma unroll
+    for (int j = 0; j < NT8; ++j) {
+      const int e = j * 8 + r;
+      const uint4 b = (in && e < NE) ? *reinterpret_cast<const uint4*>(w + (long long)e * K + k) : zero;
+      mma_bf16_16816(acc[j], f0, b.x, b.y);
+      mma_bf16_16816(acc[j], f1, b.z, b.w);
+    }
+  }
+  float* mine = rsm + warp * 16 * NP;
+#pragma unroll
+  for (int j = 0; j < NT8; ++j) {
+    const int e = j * 8 + (lane & 3) * 2;
+    if (e >= NP) continue;
+    mine[r * NP + e] = acc[j][0]; mine[r * NP + e + 1] = acc[j][1];
+    mine[(r + 8) * NP + e] = acc[j][2]; mine[(r + 8) * NP + e + 1] = acc[j][3];
+  }
+  __syncthreads();
+  for (int i = threadIdx.x; i < 16 * NP; i += 256) {
+    float s = 0.f;
+#pragma unroll
+    for (int v = 0; v < 8; ++v) s += rsm[v * 16 * NP + i];
+    rsm[i] = s;   // only this thread reads or writes entry i of any warp's part
+  }
+  __syncthreads();
+  const int ng = groups > 0 ? groups : 1;
+  float* sc = rsm + 8 * 16 * NP + warp * (2 * E + ng);
+#pragma unroll
+  for (int j = 0; j < 2; ++j) {
+    const int t = t0 + warp * 2 + j;
+    if (t < T)
+      hy_route_token(rsm + (warp * 2 + j) * NP, sc, sc + E, sc + 2 * E, E, top, groups, keep, scale, gw + (long long)t * NE, score_mode, group_mode, renorm, shared_gate,
+                     choice);
+    __syncwarp();
+  }
 }
 
 // U carries, expert after expert, [gate_e (f) | up_e (f)], then the shared expert's [gate (sf) | up (sf)].

@@ -8,6 +8,7 @@
 // type a Linear reads (same may be the very buffer that ha overwrites: a thread reads the channels it writes).
 // tokens != nullptr: every copy starts as the token's embedding row (no y).  Everything is fp32.
 #pragma once
+#include <cooperative_groups.h>
 
 #define HY_MAX_STREAMS 16
 struct HyperArgs {
@@ -184,4 +185,81 @@ __global__ void hy_stream_sum_kernel(const float* __restrict__ x, float* __restr
   float v = 0.f;
   for (int s = 0; s < n; ++s) v += x[(t * n + s) * D + i];
   out[t * D + i] = v;
+}
+
+// The same for steps of few rows: a row's channels are shared out over the gridDim.y blocks of a thread-block cluster (more loads in flight while
+// split-K planes are summed); mean and squared deviations of the blocks' parts are merged across the cluster.
+// grid (T, blocks per row), 256 threads; dynamic shared memory: ceil(D / blocks) floats.
+template <typename AT, int SM>
+__global__ void __launch_bounds__(256) hy_hyper_cluster_kernel(HyperArgs a) {
+  namespace cg = cooperative_groups;
+  extern __shared__ __align__(16) float row[];
+  __shared__ float wm[SM * SM], wo[SM], wr[SM];
+  __shared__ float red[32], part[2];
+  const int n = a.n, D = a.D, nb = gridDim.y;
+  pdl_launch_dependents();
+  for (int i = threadIdx.x; i < SM * SM; i += 256) {
+    const int f = i / SM, t = i - f * SM;
+    wm[i] = (f < n && t < n) ? (a.mix != nullptr ? a.mix[f * n + t] : (f == t ? 1.f : 0.f)) : 0.f;
+  }
+  for (int i = threadIdx.x; i < SM; i += 256) {
+    wo[i] = i < n ? (a.out != nullptr ? a.out[i] : 1.f) : 0.f;
+    wr[i] = i < n ? (a.rd != nullptr ? a.rd[i] : 1.f) : 0.f;
+  }
+  pdl_wait();
+  __syncthreads();
+  const long long t = blockIdx.x;
+  const int per = (D + nb - 1) / nb, c0 = blockIdx.y * per, nc = D - c0 < per ? (D - c0 > 0 ? D - c0 : 0) : per;
+  float* x = a.x + t * n * D + c0;
+  float sw = 0.f;
+  for (int i = 0; i < a.same_n; ++i) sw += a.same_w[t * a.same_ld + i];
+  const AT* same = reinterpret_cast<const AT*>(a.same) + t * D + c0;
+  float sum = 0.f;
+  for (int i = threadIdx.x; i < nc; i += 256) {
+    float xs[SM], u = 0.f;
+#pragma unroll
+    for (int s = 0; s < SM; ++s)
+      if (s < n) xs[s] = x[(long long)s * D + i];
+    float y = lin_at(a.y, t, c0 + i);
+    if (sw != 0.f) y = fmaf(sw, act_load<AT>(same + i), y);
+#pragma unroll
+    for (int j = 0; j < SM; ++j) {
+      if (j >= n) break;
+      float v = wo[j] * y;
+#pragma unroll
+      for (int s = 0; s < SM; ++s) {
+        if (s >= n) break;
+        v = fmaf(wm[s * SM + j], xs[s], v);
+      }
+      x[(long long)j * D + i] = v;
+      u = fmaf(wr[j], v, u);
+    }
+    row[i] = u;
+    sum += u;
+  }
+  // mean and squared deviations of this block's channels, then of the row (every block merges the parts in the same order)
+  float mean = a.norm == XB_NORM_LAYER ? block_sum<256>(sum, red) / (float)(nc > 0 ? nc : 1) : 0.f, sq = 0.f;
+  for (int i = threadIdx.x; i < nc; i += 256) { const float d = row[i] - mean; sq = fmaf(d, d, sq); }
+  sq = block_sum<256>(sq, red);
+  cg::cluster_group cl = cg::this_cluster();
+  if (threadIdx.x == 0) { part[0] = mean; part[1] = sq; }
+  cl.sync();
+  float cnt = 0.f, mu = 0.f, m2 = 0.f;
+  for (int b = 0; b < nb; ++b) {
+    const float* p = cl.map_shared_rank(part, b);
+    const int left = D - b * per;
+    const float k = (float)(left < per ? (left > 0 ? left : 0) : per);
+    if (k == 0.f) continue;
+    const float d = p[0] - mu, tot = cnt + k;
+    m2 += p[1] + d * d * (cnt * k / tot);
+    mu += d * (k / tot);
+    cnt = tot;
+  }
+  cl.sync();   // no block leaves while its part may still be read
+  const float inv = 1.0f / sqrtf(m2 / (float)D + a.eps);
+  for (int i = threadIdx.x; i < nc; i += 256) {
+    const float v = (row[i] - mu) * inv * hy_norm_weight(a.nw, a.nw_mode, c0 + i);
+    if (a.hn != nullptr) a.hn[t * D + c0 + i] = v;
+    if (a.ha != nullptr) act_store<AT>(reinterpret_cast<AT*>(a.ha) + t * D + c0 + i, v);
+  }
 }

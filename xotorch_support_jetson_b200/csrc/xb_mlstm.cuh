@@ -15,18 +15,19 @@ __device__ __forceinline__ float hy_soft_cap(float z, float cap) { return cap * 
 // The scalar recurrence of one (sequence, head): w -> decay[t, h], b -> beta[t, h], e^-m -> em[t, h], the last m -> the slot.
 // m_t = max(F + m_0, I) where (F, I) composes the steps up to t, (f1, i1) then (f2, i2) = (f1 + f2, max(i1 + f2, i2)): the threads compose
 // stretches of the tokens, scan over the threads, then walk their stretch once more from its start.
-// grid (H, n_seqs), 256 threads.
-__global__ void __launch_bounds__(256) hy_mlstm_gates_kernel(LinOut P, int off_i, int off_f, float cap, float* __restrict__ mstate, long long state_stride,
+// grid (H, n_seqs), HY_GATE_THREADS threads.
+#define HY_GATE_THREADS 1024
+__global__ void __launch_bounds__(HY_GATE_THREADS) hy_mlstm_gates_kernel(LinOut P, int off_i, int off_f, float cap, float* __restrict__ mstate, long long state_stride,
                                                              float* __restrict__ decay, float* __restrict__ beta, float* __restrict__ em, int H,
                                                              BatchMeta m) {
   pdl_launch_dependents();
   pdl_wait();
-  __shared__ float sF[256], sI[256];
+  __shared__ float sF[HY_GATE_THREADS], sI[HY_GATE_THREADS];
   const int h = blockIdx.x, tid = threadIdx.x;
   const SeqSpan sp = seq_span(m, blockIdx.y);
   float* slot_m = mstate + (long long)sp.slot * state_stride + h;
   const float m0 = sp.pos0 > 0 ? *slot_m : 0.f;
-  const int per = (sp.len + 255) / 256, t0 = tid * per, t1 = t0 + per < sp.len ? t0 + per : sp.len;
+  const int per = (sp.len + HY_GATE_THREADS - 1) / HY_GATE_THREADS, t0 = tid * per, t1 = t0 + per < sp.len ? t0 + per : sp.len;
   float F = 0.f, I = -INFINITY;
   for (int t = t0; t < t1; ++t) {
     const long long r = sp.start + t;
@@ -38,7 +39,7 @@ __global__ void __launch_bounds__(256) hy_mlstm_gates_kernel(LinOut P, int off_i
   }
   sF[tid] = F; sI[tid] = I;
   __syncthreads();
-  for (int off = 1; off < 256; off <<= 1) {   // inclusive scan of the stretches
+  for (int off = 1; off < HY_GATE_THREADS; off <<= 1) {   // inclusive scan of the stretches
     float pf = 0.f, pi = -INFINITY;
     if (tid >= off) { pf = sF[tid - off]; pi = sI[tid - off]; }
     __syncthreads();
@@ -87,7 +88,7 @@ __global__ void __launch_bounds__(256) hy_mlstm_prep_kernel(LinOut P, int off_q,
 }
 
 // Read-out of the recurrence o [T][H][dvp] (column dv: n . q) -> out[t, h dv + j] = out_scale * unit(o / den) * nw * sigmoid(gate), a warp per
-// (token, head).  grid ceil(T * H / 8), 256 threads.  Lanes own four neighbouring channels when dv is a multiple of four.
+// (token, head).  grid ceil(T * H / 8), 256 threads.
 template <typename AT>
 __global__ void __launch_bounds__(256) hy_mlstm_out_kernel(const float* __restrict__ o, const float* __restrict__ em, const float* __restrict__ nw, LinOut P,
                                                            int off_g, float eps, float out_scale, AT* __restrict__ out, long long ld_out, int T, int H,
@@ -103,33 +104,40 @@ __global__ void __launch_bounds__(256) hy_mlstm_out_kernel(const float* __restri
   const float den = 1.0f / (fmaxf(fabsf(p[dv]), em[th]) + 1e-6f);
   AT* dst = out + t * ld_out + (long long)h * dv;
   float ss = 0.f;
-  const bool vec = (dv & 3) == 0 && P.h != nullptr && ((P.ld | off_g | ld_out) & 3) == 0 && (reinterpret_cast<uintptr_t>(out) & 15) == 0;
-  if (vec && dv <= 128) {
-    const int j = lane * 4;
-    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-    if (j < dv) v = *reinterpret_cast<const float4*>(p + j);
-    v.x *= den; v.y *= den; v.z *= den; v.w *= den;
-    ss = warp_sum(fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, v.w * v.w))));
-    if (j >= dv) return;
-    const float inv = out_scale / sqrtf(ss / (float)dv + eps);
-    HyVec<4> g = hy_ldv<4>(P.h + t * P.ld + off_g + h * dv + j);
-    if (P.bias != nullptr) {
-      const HyVec<4> b = hy_ldv<4>(P.bias + off_g + h * dv + j);
-#pragma unroll
-      for (int e = 0; e < 4; ++e) g.v[e] += b.v[e];
-    }
-    const HyVec<4> w = hy_ldv<4>(nw + h * dv + j);
-    HyVec<4> y;
-    y.v[0] = v.x; y.v[1] = v.y; y.v[2] = v.z; y.v[3] = v.w;
-#pragma unroll
-    for (int e = 0; e < 4; ++e) y.v[e] = y.v[e] * inv * w.v[e] * hy_sigmoid(g.v[e]);
-    hy_stv<4>(dst + j, y);
-    return;
-  }
   for (int j = lane; j < dv; j += 32) { const float v = p[j] * den; ss = fmaf(v, v, ss); }
   const float inv = out_scale / sqrtf(warp_sum(ss) / (float)dv + eps);
   for (int j = lane; j < dv; j += 32)
     act_store<AT>(dst + j, p[j] * den * inv * nw[h * dv + j] * hy_sigmoid(lin_at(P, t, off_g + h * dv + j)));
+}
+
+// The same on 32- and 16-byte accesses: eight neighbouring channels per thread, dv / 8 (a power of two up to 32) neighbouring lanes per head, gate from
+// one bf16 matrix.  off_g, the pitches and dv are multiples of 8.  grid ceil(T * H * dv / 8 / 256), 256 threads.
+template <typename AT>
+__global__ void __launch_bounds__(256) hy_mlstm_out_vec_kernel(const float* __restrict__ o, const float* __restrict__ em, const float* __restrict__ nw,
+                                                               const bf16* __restrict__ g, long long ldg, const float* __restrict__ gbias, float eps,
+                                                               float out_scale, AT* __restrict__ out, long long ld_out, int T, int H, int dv) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int per = dv >> 3, dvp = hy_mlstm_cols(dv);
+  const long long idx = (long long)blockIdx.x * 256 + threadIdx.x, n = (long long)T * H * per;
+  const bool live = idx < n;
+  const long long th = (live ? idx : n - 1) / per;
+  const int j = (int)((live ? idx : n - 1) - th * per) << 3;
+  const long long t = th / H;
+  const int h = (int)(th - t * H);
+  float v[8], wv[8], gv[8];
+  hy_ld8f(o + th * dvp + j, v);
+  const float den = 1.0f / (fmaxf(fabsf(o[th * dvp + dv]), em[th]) + 1e-6f);
+  hy_load8(g + t * ldg + (long long)h * dv + j, gbias != nullptr ? gbias + h * dv + j : nullptr, gv);
+  hy_ld8f(nw + (long long)h * dv + j, wv);
+  float ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < 8; ++i) { v[i] *= den; ss = fmaf(v[i], v[i], ss); }
+  for (int off = per >> 1; off > 0; off >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, off);   // per divides 32: lanes of a head stay together
+  const float inv = out_scale / sqrtf(ss / (float)dv + eps);
+#pragma unroll
+  for (int i = 0; i < 8; ++i) v[i] = v[i] * inv * wv[i] * hy_sigmoid(gv[i]);
+  if (live) hy_st8a<AT>(out + t * ld_out + (long long)h * dv + j, v);
 }
 
 // A step of single tokens: everything between the input and the output projection in one kernel, a block per (sequence, head).
