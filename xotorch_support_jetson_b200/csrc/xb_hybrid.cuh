@@ -1200,7 +1200,7 @@ static int hy_segments_n(xb_engine* e, const RecurIn& in, float* state, long lon
   sg.decay = MODE == HY_REC_LIGHTNING ? nullptr : hy->seg_decay;
   sg.per_head = MODE == HY_REC_MLSTM ? 1 : 0;
   sg.cols = cols;
-  const dim3 grid(cb, H, n_seqs * sg.max_segs);
+  const dim3 grid(cb + (MODE == HY_REC_MLSTM ? 1 : 0), H, n_seqs * sg.max_segs);
   constexpr size_t row = (size_t)2 * HY_SEG_TS * sizeof(float);
   constexpr int ex = MODE == HY_REC_MLSTM ? 4 : 0;
   constexpr size_t s0 = row * (hy_seg_vectors(MODE, 0) * 4 * LPC * NCH + HY_SEG_COLS + ex), s1 = row * (hy_seg_vectors(MODE, 1) * 4 * LPC * NCH + HY_SEG_COLS + ex);

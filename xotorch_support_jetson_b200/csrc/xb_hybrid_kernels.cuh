@@ -1128,13 +1128,84 @@ struct SegArgs {
   int seg, max_segs;      // tokens per segment, segments of the longest sequence a step can hold
   int per_head;           // 1: a head's channels fade alike
   int cols;               // columns of a head in state, workspace and o; > dv for the matrix memory, whose column dv is the normaliser (its
-                          // value is one): the first warp of a head's first block carries it beside its own columns
+                          // value is one): one more block per segment and four heads carries it (hy_seg_normaliser)
 };
 // row vectors staged per step: k (or f), w where it is a vector of its own, q in the output pass
 __host__ __device__ constexpr int hy_seg_vectors(int mode, int pass) { return 1 + (mode == HY_REC_GLA ? 1 : 0) + (pass == 1 ? 1 : 0); }
 
+
+// The normaliser of a matrix memory over one segment: n <- w n + k, in the output pass also q . n, by one warp whose lanes own four neighbouring
+// numbers of n (twice that beyond 128), straight from global memory with the next steps' rows in flight.  entry / out: start state and end state.
+template <int PASS>
+__device__ __forceinline__ void hy_seg_normaliser(const float* kp, const float* qp, const float* wp, long long ldc, int ldw, int len, int dk, bool al,
+                                                  const float* entry, float* out, float* o, long long ldo, float* decay) {
+  constexpr int U = 4;
+  const int lane = threadIdx.x & 31;
+  float S[2][4], faded = 1.f;
+  auto load = [&](const float* p, int c, float* v) {
+    const int r = (c * 32 + lane) * 4;
+    if (al && r < dk) {
+      const float4 f = *reinterpret_cast<const float4*>(p + r);
+      v[0] = f.x; v[1] = f.y; v[2] = f.z; v[3] = f.w;
+    } else {
+#pragma unroll
+      for (int e = 0; e < 4; ++e) v[e] = r + e < dk ? p[r + e] : 0.f;
+    }
+  };
+#pragma unroll
+  for (int c = 0; c < 2; ++c)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int r = (c * 32 + lane) * 4 + e;
+      S[c][e] = PASS == 1 && r < dk ? entry[r] : 0.f;
+    }
+  const bool two = dk > 128;
+  for (int t0 = 0; t0 < len; t0 += U) {
+    float k[U][2][4], q[U][2][4], w[U];
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      if (t0 + u >= len) break;
+      w[u] = wp[(long long)(t0 + u) * ldw];
+      load(kp + (long long)(t0 + u) * ldc, 0, k[u][0]);
+      if (PASS == 1) load(qp + (long long)(t0 + u) * ldc, 0, q[u][0]);
+      if (two) {
+        load(kp + (long long)(t0 + u) * ldc, 1, k[u][1]);
+        if (PASS == 1) load(qp + (long long)(t0 + u) * ldc, 1, q[u][1]);
+      }
+    }
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      if (t0 + u >= len) break;
+      float y = 0.f;
+      faded *= w[u];
+#pragma unroll
+      for (int c = 0; c < 2; ++c) {
+        if (c == 1 && !two) break;
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          S[c][e] = fmaf(w[u], S[c][e], k[u][c][e]);
+          if (PASS == 1) y = fmaf(q[u][c][e], S[c][e], y);
+        }
+      }
+      if (PASS == 1) {
+        y = warp_sum(y);
+        if (lane == 0) o[(long long)(t0 + u) * ldo] = y;
+      }
+    }
+  }
+  if (out != nullptr)
+#pragma unroll
+    for (int c = 0; c < 2; ++c)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int r = (c * 32 + lane) * 4 + e;
+        if (r < dk) out[r] = S[c][e];
+      }
+  if (PASS == 0 && lane == 0) *decay = faded;
+}
+
 template <int NCH, int LPC, int MODE, int PASS>
-__global__ void __launch_bounds__(128) hy_seg_kernel(RecurIn in, SegArgs sg, float* __restrict__ state, long long state_stride, float* __restrict__ o,
+__global__ void __launch_bounds__(128, MODE == HY_REC_MLSTM ? 4 : 0) hy_seg_kernel(RecurIn in, SegArgs sg, float* __restrict__ state, long long state_stride, float* __restrict__ o,
                                                      long long ldo, BatchMeta m, int H, int dk, int dv) {
   pdl_wait();
   extern __shared__ __align__(16) float stg[];
@@ -1155,11 +1226,20 @@ __global__ void __launch_bounds__(128) hy_seg_kernel(RecurIn in, SegArgs sg, flo
   if (MODE == HY_REC_GLA) src[1] = in.c + in.xoff[0] + (long long)h * dk;
   if (PASS == 1) src[NV - 1] = in.c + in.qoff + (long long)h * dk;
   const float* cv = in.c + in.voff + (long long)h * cols + j0;
-  const bool norm = MODE == HY_REC_MLSTM && blockIdx.x == 0 && warp == 0;   // both lane groups of the warp do the same work on it
-  float faded = 1.f;   // product of the segment's decays (per_head)
   const hy_f2 hd2 = MODE == HY_REC_LIGHTNING ? hy_f2_pack(in.hdecay[h], in.hdecay[h]) : 0ull;
   bool al = ((in.ldc | in.qoff | in.koff | in.voff | dk | dv) & 3) == 0 && (reinterpret_cast<uintptr_t>(in.c) & 15) == 0;
   if (MODE == HY_REC_GLA) al = al && (in.xoff[0] & 3) == 0;
+  if (MODE == HY_REC_MLSTM && blockIdx.x == gridDim.x - 1) {   // the block behind the value columns
+    const int hn = h + warp;   // a warp per head, four heads per block: the blocks of the other three heads have nothing to do
+    if ((h & 3) != 0 || hn >= H) return;
+    const long long at = ((long long)hn * cols + dv) * dk;
+    float* out = PASS == 0 ? entry + at : (c == nseg - 1 ? state + (long long)sp.slot * state_stride + at : nullptr);
+    const long long kq = (long long)row0 * in.ldc + (long long)warp * dk;
+    hy_seg_normaliser<PASS>(src[0] + kq, src[NV - 1] + kq, in.decay + (long long)row0 * H + hn, in.ldc, H, len, dk, al, entry + at, out,
+                            o + (long long)row0 * ldo + (long long)hn * cols + dv, ldo,
+                            PASS == 0 ? sg.decay + (long long)(sp.start / sg.seg + s + c) * H + hn : nullptr);
+    return;
+  }
   for (int i = threadIdx.x; i < 2 * HY_SEG_TS * STRIDE; i += 128) stg[i] = 0.f;   // padding rows / columns stay zero
   int col = 0;   // the column whose sum ends up in this lane
 #pragma unroll
@@ -1184,18 +1264,6 @@ __global__ void __launch_bounds__(128) hy_seg_kernel(RecurIn in, SegArgs sg, flo
         for (int x = 0; x < 4; ++x) e[x] = (have && r + x < dk) ? st[r + x] : 0.f;
         S[n][2 * ch] = hy_f2_pack(e[0], e[1]); S[n][2 * ch + 1] = hy_f2_pack(e[2], e[3]);
       }
-    }
-  }
-  hy_f2 Sn[2 * NCH];
-  if (MODE == HY_REC_MLSTM) {
-    const float* st = entry + ((long long)h * cols + dv) * dk;
-#pragma unroll
-    for (int ch = 0; ch < NCH; ++ch) {
-      const int r = (ch * LPC + sub) * 4;
-      float e[4];
-#pragma unroll
-      for (int x = 0; x < 4; ++x) e[x] = (norm && PASS == 1 && r + x < dk) ? st[r + x] : 0.f;
-      Sn[2 * ch] = hy_f2_pack(e[0], e[1]); Sn[2 * ch + 1] = hy_f2_pack(e[2], e[3]);
     }
   }
   __syncthreads();
@@ -1243,8 +1311,6 @@ __global__ void __launch_bounds__(128) hy_seg_kernel(RecurIn in, SegArgs sg, flo
       const float* sr = buf + ts * STRIDE;
       hy_f2 vv[NCOL], acc[NCOL];
       const hy_f2 fade = MODE == HY_REC_MLSTM ? hy_f2_pack(sr[VO + NB], sr[VO + NB]) : hd2;
-      hy_f2 accn = 0ull;
-      if (MODE == HY_REC_MLSTM && PASS == 0) faded *= sr[VO + NB];
 #pragma unroll
       for (int n = 0; n < NCOL; n += 4) {
         const float4 v = *reinterpret_cast<const float4*>(sr + VO + jl + n);
@@ -1280,19 +1346,6 @@ __global__ void __launch_bounds__(128) hy_seg_kernel(RecurIn in, SegArgs sg, flo
             S[n][2 * ch + x] = hy_f2_fma(w2[x], S[n][2 * ch + x], hy_f2_mul(k2[x], vv[n]));
             if (PASS == 1) acc[n] = hy_f2_fma(q2[x], S[n][2 * ch + x], acc[n]);
           }
-        if (MODE == HY_REC_MLSTM && norm)
-#pragma unroll
-          for (int x = 0; x < 2; ++x) {
-            Sn[2 * ch + x] = hy_f2_fma(fade, Sn[2 * ch + x], k2[x]);
-            if (PASS == 1) accn = hy_f2_fma(q2[x], Sn[2 * ch + x], accn);
-          }
-      }
-      if (MODE == HY_REC_MLSTM && PASS == 1 && norm) {
-        const float2 a = hy_f2_unpack(accn);
-        float y = a.x + a.y;
-#pragma unroll
-        for (int off = 1; off < LPC; off <<= 1) y += __shfl_xor_sync(0xffffffffu, y, off);
-        if (lane == 0) o[(long long)(row0 + t0 + ts) * ldo + (long long)h * cols + dv] = y;
       }
       if (PASS == 1) {
         // sums over the lanes: partners swap halves of their columns, so that log2(LPC) rounds leave one column per lane pair
@@ -1345,19 +1398,6 @@ __global__ void __launch_bounds__(128) hy_seg_kernel(RecurIn in, SegArgs sg, flo
           if (r + x < dk) st[r + x] = e[x];
       }
     }
-  }
-  if (MODE == HY_REC_MLSTM && norm && lane < LPC) {
-    float* st = base + ((long long)h * cols + dv) * dk;
-#pragma unroll
-    for (int ch = 0; ch < NCH; ++ch) {
-      const int r = (ch * LPC + sub) * 4;
-      const float2 a = hy_f2_unpack(Sn[2 * ch]), b = hy_f2_unpack(Sn[2 * ch + 1]);
-      const float e[4] = {a.x, a.y, b.x, b.y};
-#pragma unroll
-      for (int x = 0; x < 4; ++x)
-        if (r + x < dk) st[r + x] = e[x];
-    }
-    if (PASS == 0 && lane == 0) sg.decay[(long long)(sp.start / sg.seg + s + c) * H + h] = faded;
   }
 }
 
@@ -3012,18 +3052,26 @@ __global__ void __launch_bounds__(256) hy_router_mma_kernel(const bf16* __restri
 #pragma unroll
   for (int j = 0; j < NT8; ++j) acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.f;
   const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
-#pragma unroll 2
-  for (int kb = warp * 32; kb < K; kb += 256) {
-    const int k = kb + kc;
-    const bool in = k < K;
-    const uint4 a0 = in ? *reinterpret_cast<const uint4*>(xa + k) : zero, a1 = in ? *reinterpret_cast<const uint4*>(xb + k) : zero;
-    const uint32_t f0[4] = {a0.x, a1.x, a0.y, a1.y}, f1[4] = {a0.z, a1.z, a0.w, a1.w};
+  constexpr int U = NT8 <= 4 ? 4 : 2;   // k steps whose loads are in flight together
+  for (int kb = warp * 32; kb < K; kb += 256 * U) {
+    uint4 a0[U], a1[U], b[U][NT8];
 #pragma unroll
-    for (int j = 0; j < NT8; ++j) {
-      const int e = j * 8 + r;
-      const uint4 b = (in && e < NE) ? *reinterpret_cast<const uint4*>(w + (long long)e * K + k) : zero;
-      mma_bf16_16816(acc[j], f0, b.x, b.y);
-      mma_bf16_16816(acc[j], f1, b.z, b.w);
+    for (int u = 0; u < U; ++u) {
+      const int k = kb + u * 256 + kc;
+      const bool in = k < K;
+      a0[u] = in ? *reinterpret_cast<const uint4*>(xa + k) : zero;
+      a1[u] = in ? *reinterpret_cast<const uint4*>(xb + k) : zero;
+#pragma unroll
+      for (int j = 0; j < NT8; ++j) b[u][j] = (in && j * 8 + r < NE) ? *reinterpret_cast<const uint4*>(w + (long long)(j * 8 + r) * K + k) : zero;
+    }
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      const uint32_t f0[4] = {a0[u].x, a1[u].x, a0[u].y, a1[u].y}, f1[4] = {a0[u].z, a1[u].z, a0[u].w, a1[u].w};
+#pragma unroll
+      for (int j = 0; j < NT8; ++j) {
+        mma_bf16_16816(acc[j], f0, b[u][j].x, b[u][j].y);
+        mma_bf16_16816(acc[j], f1, b[u][j].z, b[u][j].w);
+      }
     }
   }
   float* mine = rsm + warp * 16 * NP;

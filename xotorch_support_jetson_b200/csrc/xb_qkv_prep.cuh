@@ -177,58 +177,64 @@ __global__ void __launch_bounds__(256) hy_qkv_prep_tile_kernel(LinOut P, QkvPrep
   float sq[RT], sk[RT];
 #pragma unroll
   for (int r = 0; r < RT; ++r) sq[r] = sk[r] = 0.f;
-  for (int c = threadIdx.x * 8; c < C; c += 256 * 8) {
-    float w[TAPS > 0 ? TAPS : 1][8], z[RT + BACK][8];
+  for (int c = threadIdx.x * 4; c < C; c += 256 * 4) {   // four channels per thread keep a filter's window in few registers
+    HyVec<4> z[RT + BACK], b;
+    float w[TAPS > 0 ? TAPS : 1][4];
+#pragma unroll
+    for (int e = 0; e < 4; ++e) b.v[e] = 0.f;
+    if (P.bias != nullptr) b = hy_ldv<4>(P.bias + a.off_q + c);
 #pragma unroll
     for (int i = 0; i < RT + BACK; ++i) {
       const int row = r0 - BACK + i;
-      if (row >= 0 && row < r0 + nr) hy_prep_load<8>(P, row, a.off_q + c, z[i]);
+      if (row >= 0 && row < r0 + nr) z[i] = hy_ldv<4>(P.h + (long long)row * P.ld + a.off_q + c);
       else
 #pragma unroll
-        for (int e = 0; e < 8; ++e) z[i][e] = 0.f;
+        for (int e = 0; e < 4; ++e) z[i].v[e] = 0.f;
     }
     if (TAPS > 0) {
 #pragma unroll
-      for (int x = 0; x < (TAPS > 0 ? TAPS : 1); ++x) {   // eight channels' taps are 8 TAPS neighbouring numbers
-        float t[8];
-        hy_ld8f(a.conv_w + (long long)c * TAPS + 8 * x, t);
+      for (int x = 0; x < (TAPS > 0 ? TAPS : 1); ++x) {   // four channels' taps are 4 TAPS neighbouring numbers
+        const HyVec<4> t = hy_ldv<4>(a.conv_w + (long long)c * TAPS + 4 * x);
 #pragma unroll
-        for (int e = 0; e < 8; ++e) w[(8 * x + e) % (TAPS > 0 ? TAPS : 1)][(8 * x + e) / (TAPS > 0 ? TAPS : 1)] = t[e];
+        for (int e = 0; e < 4; ++e) w[(4 * x + e) % (TAPS > 0 ? TAPS : 1)][(4 * x + e) / (TAPS > 0 ? TAPS : 1)] = t.v[e];
       }
     }
 #pragma unroll
+    for (int i = 0; i < RT + BACK; ++i)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) z[i].v[e] += b.v[e];
+#pragma unroll
     for (int r = 0; r < RT; ++r) {
       if (r >= nr) break;
-      float y[8];
+      HyVec<4> y;
       if (TAPS == 0) {
-#pragma unroll
-        for (int e = 0; e < 8; ++e) y[e] = z[r + BACK][e];
+        y = z[r + BACK];
       } else {
         const int row = r0 + r, pos = where[r][0], start = where[r][2];
 #pragma unroll
-        for (int e = 0; e < 8; ++e) y[e] = 0.f;
+        for (int e = 0; e < 4; ++e) y.v[e] = 0.f;
 #pragma unroll
         for (int j = 0; j < TAPS; ++j) {   // oldest first
           const int d = TAPS - 1 - j;
           if (row - d >= start) {
 #pragma unroll
-            for (int e = 0; e < 8; ++e) y[e] = fmaf(w[j][e], z[r + BACK - d][e], y[e]);
+            for (int e = 0; e < 4; ++e) y.v[e] = fmaf(w[j][e], z[r + BACK - d].v[e], y.v[e]);
           } else if (pos - d >= 0) {       // in front of this step's rows: the slot's tail
             const float* tl = a.tail + (long long)where[r][4] * a.tail_stride + (long long)(pos - d - (where[r][3] - (TAPS - 1))) * C + c;
 #pragma unroll
-            for (int e = 0; e < 8; ++e) y[e] = fmaf(w[j][e], tl[e], y[e]);
+            for (int e = 0; e < 4; ++e) y.v[e] = fmaf(w[j][e], tl[e], y.v[e]);
           }
         }
       }
       if (c < nqk) {
         float ss = 0.f;
 #pragma unroll
-        for (int e = 0; e < 8; ++e) ss = fmaf(y[e], y[e], ss);
+        for (int e = 0; e < 4; ++e) ss = fmaf(y.v[e], y.v[e], ss);
         if (c < nq) sq[r] += ss; else sk[r] += ss;
-        hy_st8f(qk + r * nqk + c, y);
+        hy_stv<4>(qk + r * nqk + c, y);
       } else {
         const int iv = c - nqk, g = iv / dv, d = iv - g * dv;
-        *reinterpret_cast<uint4*>(v_pool + ((page[r] * G + g) * m.page_tokens + where[r][1]) * a.vp + d) = hy_pack8(y);
+        hy_stv<4>(v_pool + ((page[r] * G + g) * m.page_tokens + where[r][1]) * a.vp + d, y);
       }
     }
   }
