@@ -478,6 +478,33 @@ def test_filter_tail_shows(lib, dtype):
   st.close()
 
 
+@pytest.mark.parametrize("conv", [2, 3, 4])
+def test_filter_in_long_bf16_prompts(lib, conv):
+  """Prompts long enough for the preparation kernel's eight-row tiles: alone, behind a portion of five tokens (the slot's tail), and three
+  sequences side by side whose borders fall inside a tile; a filter that reads mostly its oldest tap."""
+  cfg = config([(filtered(heads=4, kv=2, dim=64, vdim=48, rot=32, size=200, conv=conv), None)], width=64)
+  w = {k: v.float().clone() for k, v in weights(cfg, seed=55).items()}
+  for k in w:
+    if k.endswith(".conv"):
+      w[k] *= 0.2
+      w[k][:, 0] += 1.0
+  w = {k: v.to(torch.bfloat16) for k, v in w.items()}
+  ids, b, c = toks(1110, cfg["vocab"], seed=56), toks(37, cfg["vocab"], seed=57), toks(202, cfg["vocab"], seed=58)
+  ref, tol = logits(cfg, w, ids), TOL["bfloat16"]
+  st = stage(cfg, w, "bfloat16", cap=1400, page=64)
+  assert rows_off(run(st, 0, ids, 0), ref, tol) == 0
+  got = torch.cat([run(st, 1, ids[:5], 0), run(st, 1, ids[5:], 5)])
+  st.release_slot(0), st.release_slot(1)
+  assert rows_off(got, ref, tol) == 0
+  n = [1023, 35, 200]
+  o = st.forward([2, 0, 1], n, [0, 0, 0], tokens=torch.tensor(ids[:1023] + b[:35] + c[:200], dtype=torch.int32, device="cuda"), want_rows=list(range(sum(n)))).cpu().double()
+  o2 = st.forward([0, 2, 1], [2, 87, 2], [35, 1023, 200], tokens=torch.tensor(b[35:] + ids[1023:] + c[200:], dtype=torch.int32, device="cuda"), want_rows=list(range(91))).cpu().double()
+  st.close()
+  rb, rc = logits(cfg, w, b), logits(cfg, w, c)
+  for x, y in ((o[:1023], ref[:1023]), (o[1023:1058], rb[:35]), (o[1058:], rc[:200]), (o2[:2], rb[35:]), (o2[2:89], ref[1023:]), (o2[89:], rc[200:])):
+    assert float((x - y).pow(2).mean(dim=-1).sqrt().max() / ref.pow(2).mean().sqrt()) < tol
+
+
 # ----------------------------------------------------------------------------- the matrix memory
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 def test_memory_that_keeps_and_memory_that_forgets(lib, dtype):

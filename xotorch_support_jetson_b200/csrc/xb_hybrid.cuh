@@ -1748,20 +1748,24 @@ static int hy_qkv_prep(xb_engine* e, const HyLayer& l, int T, const LinOut& P, c
   KT *kp = (KT*)l.k_pool, *vp = (KT*)l.v_pool;
   const int NH = a.H + a.G;
   if constexpr (std::is_same<KT, bf16>::value) {
-    const size_t tile = (size_t)HY_PREP_ROWS * (NH * (a.dk + 1) + a.rot.dims) * sizeof(float);
+    const size_t row = (size_t)(NH * (a.dk + 1) + a.rot.dims) * sizeof(float);
     const bool taps = a.taps == 0 || (a.taps >= 2 && a.taps <= 4);
-    if (T > 64 && a.qg != nullptr && a.qa == nullptr && P.h != nullptr && ((P.ld | a.dk | a.dv | a.off_q) & 7) == 0 && taps && tile <= 160 * 1024 &&
+    if (T > 64 && a.qg != nullptr && a.qa == nullptr && P.h != nullptr && ((P.ld | a.dk | a.dv | a.off_q) & 7) == 0 && taps && 4 * row <= 110 * 1024 &&
         !(a.head_norm && (a.qn != nullptr || a.temp_every > 0))) {
-      const dim3 grid((T + HY_PREP_ROWS - 1) / HY_PREP_ROWS);
-#define HY_PREP_CASE(N)                                                                                    \
-  if (a.taps == N) {                                                                                       \
-    if (tile > 48 * 1024) XB_SMEM_ATTR_ONCE(hy_qkv_prep_tile_kernel<N>, 160 * 1024);                       \
-    return hy_launch(e, hy_qkv_prep_tile_kernel<N>, grid, dim3(256), tile, st, P, a, kp, vp, m, T);        \
+      // with a filter, long prompts take eight rows per block (fewer reads of its weights, one wave of two blocks per SM at 2048 tokens)
+      const bool eight = a.taps > 0 && T >= 1024 && 8 * row <= 110 * 1024;
+#define HY_PREP_CASE(N, R)                                                                                                                         \
+  if (a.taps == N && eight == (R == 8)) {                                                                                                          \
+    if (R * row > 48 * 1024) XB_SMEM_ATTR_ONCE((hy_qkv_prep_tile_kernel<N, R>), 110 * 1024);                                                       \
+    return hy_launch(e, hy_qkv_prep_tile_kernel<N, R>, dim3((T + R - 1) / R), dim3(256), R * row, st, P, a, kp, vp, m, T);                         \
   }
-      HY_PREP_CASE(0)
-      HY_PREP_CASE(2)
-      HY_PREP_CASE(3)
-      HY_PREP_CASE(4)
+      HY_PREP_CASE(0, 4)
+      HY_PREP_CASE(2, 4)
+      HY_PREP_CASE(3, 4)
+      HY_PREP_CASE(4, 4)
+      HY_PREP_CASE(2, 8)
+      HY_PREP_CASE(3, 8)
+      HY_PREP_CASE(4, 8)
 #undef HY_PREP_CASE
     }
   }

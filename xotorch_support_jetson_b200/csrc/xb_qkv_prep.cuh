@@ -145,15 +145,14 @@ __global__ void __launch_bounds__(NT) hy_qkv_prep_kernel(LinOut P, QkvPrep a, KT
   }
 }
 
-// Prompts whose projection came back as ONE bf16 matrix, bf16 pools: a block takes HY_PREP_ROWS token rows, so that a filter's weights and the rows
+// Prompts whose projection came back as ONE bf16 matrix, bf16 pools: a block takes RT token rows, so that a filter's weights and the rows
 // it looks back to are read once for all of them; unit heads without whole-projection norms and temperature; 16-byte accesses (dk, dv, kp, vp, off_q and the pitch are multiples of 8).  TAPS: 0 = no filter.
-// grid (ceil(T / HY_PREP_ROWS)), 256 threads; dynamic shared memory HY_PREP_ROWS * ((H + G) (dk + 1) + rot.dims) floats.
-#define HY_PREP_ROWS 4
-template <int TAPS>
-__global__ void __launch_bounds__(256) hy_qkv_prep_tile_kernel(LinOut P, QkvPrep a, bf16* __restrict__ k_pool, bf16* __restrict__ v_pool, BatchMeta m, int T) {
+// grid (ceil(T / RT)), 256 threads; dynamic shared memory RT * ((H + G) (dk + 1) + rot.dims) floats.
+template <int TAPS, int RT>
+__global__ void __launch_bounds__(256, TAPS > 0 ? 2 : 4) hy_qkv_prep_tile_kernel(LinOut P, QkvPrep a, bf16* __restrict__ k_pool, bf16* __restrict__ v_pool, BatchMeta m, int T) {
   pdl_launch_dependents();
   pdl_wait();
-  constexpr int RT = HY_PREP_ROWS, BACK = TAPS > 1 ? TAPS - 1 : 0;
+  constexpr int BACK = TAPS > 1 ? TAPS - 1 : 0;
   extern __shared__ __align__(16) float qk[];   // [RT][(H + G) dk], then 1 / rms per head, then cos / sin
   __shared__ float sums[8][2 * RT], scale[2 * RT];
   __shared__ long long page[RT];
@@ -177,7 +176,27 @@ __global__ void __launch_bounds__(256) hy_qkv_prep_tile_kernel(LinOut P, QkvPrep
   float sq[RT], sk[RT];
 #pragma unroll
   for (int r = 0; r < RT; ++r) sq[r] = sk[r] = 0.f;
-  for (int c = threadIdx.x * 4; c < C; c += 256 * 4) {   // four channels per thread keep a filter's window in few registers
+  // the tile lies in one sequence: what its rows look back to is one run of rows and, in front of the step, of the slot's tail
+  const bool one = where[0][2] == where[nr - 1][2];
+  const int pos0 = where[0][0], start0 = where[0][2], first0 = where[0][3];
+  const float* tail0 = TAPS > 1 ? a.tail + (long long)where[0][4] * a.tail_stride : nullptr;
+  if (TAPS > 0 && !one) {   // rows of several sequences: each looks back by itself
+#pragma unroll
+    for (int r = 0; r < RT; ++r) {
+      if (r >= nr) break;
+      for (int c = threadIdx.x; c < C; c += 256) {
+        const float y = hy_prep_channel(a, P, r0 + r, where[r][2], where[r][0], where[r][3], a.tail + (long long)where[r][4] * a.tail_stride, C, c);
+        if (c < nqk) {
+          if (c < nq) sq[r] = fmaf(y, y, sq[r]); else sk[r] = fmaf(y, y, sk[r]);
+          qk[r * nqk + c] = y;
+        } else {
+          const int iv = c - nqk, g = iv / dv, d = iv - g * dv;
+          v_pool[((page[r] * G + g) * m.page_tokens + where[r][1]) * a.vp + d] = f2bf(y);
+        }
+      }
+    }
+  }
+  for (int c = threadIdx.x * 4; c < ((TAPS == 0 || one) ? C : 0); c += 256 * 4) {   // four channels per thread keep a filter's window in few registers
     HyVec<4> z[RT + BACK], b;
     float w[TAPS > 0 ? TAPS : 1][4];
 #pragma unroll
@@ -186,10 +205,18 @@ __global__ void __launch_bounds__(256) hy_qkv_prep_tile_kernel(LinOut P, QkvPrep
 #pragma unroll
     for (int i = 0; i < RT + BACK; ++i) {
       const int row = r0 - BACK + i;
-      if (row >= 0 && row < r0 + nr) z[i] = hy_ldv<4>(P.h + (long long)row * P.ld + a.off_q + c);
-      else
+      if (i >= BACK ? row < r0 + nr : row >= start0) {
+        z[i] = hy_ldv<4>(P.h + (long long)row * P.ld + a.off_q + c);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) z[i].v[e] += b.v[e];
+      } else if (i < BACK && pos0 - (BACK - i) >= 0) {   // in front of this step's rows: the slot's tail
+        const float* tl = tail0 + (long long)(pos0 - (BACK - i) - (first0 - BACK)) * C + c;   // (a slot's state has no alignment of its own)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) z[i].v[e] = tl[e];
+      } else {
 #pragma unroll
         for (int e = 0; e < 4; ++e) z[i].v[e] = 0.f;
+      }
     }
     if (TAPS > 0) {
 #pragma unroll
@@ -200,30 +227,17 @@ __global__ void __launch_bounds__(256) hy_qkv_prep_tile_kernel(LinOut P, QkvPrep
       }
     }
 #pragma unroll
-    for (int i = 0; i < RT + BACK; ++i)
-#pragma unroll
-      for (int e = 0; e < 4; ++e) z[i].v[e] += b.v[e];
-#pragma unroll
     for (int r = 0; r < RT; ++r) {
       if (r >= nr) break;
       HyVec<4> y;
       if (TAPS == 0) {
         y = z[r + BACK];
       } else {
-        const int row = r0 + r, pos = where[r][0], start = where[r][2];
 #pragma unroll
-        for (int e = 0; e < 4; ++e) y.v[e] = 0.f;
+        for (int e = 0; e < 4; ++e) {
+          y.v[e] = 0.f;
 #pragma unroll
-        for (int j = 0; j < TAPS; ++j) {   // oldest first
-          const int d = TAPS - 1 - j;
-          if (row - d >= start) {
-#pragma unroll
-            for (int e = 0; e < 4; ++e) y.v[e] = fmaf(w[j][e], z[r + BACK - d].v[e], y.v[e]);
-          } else if (pos - d >= 0) {       // in front of this step's rows: the slot's tail
-            const float* tl = a.tail + (long long)where[r][4] * a.tail_stride + (long long)(pos - d - (where[r][3] - (TAPS - 1))) * C + c;
-#pragma unroll
-            for (int e = 0; e < 4; ++e) y.v[e] = fmaf(w[j][e], tl[e], y.v[e]);
-          }
+          for (int j = 0; j < TAPS; ++j) y.v[e] = fmaf(w[j][e], z[r + j].v[e], y.v[e]);   // oldest first
         }
       }
       if (c < nqk) {
