@@ -186,7 +186,7 @@ def test_bf16_prompt_kernels_at_wide_steps(lib):
   for cfg in (config([(pair(heads=8, kv=2, dim=64, vdim=64, rot=32, size=150, r_heads=4, r_dim=64, r_vdim=64, cap=15.0), None),
                       (filtered(heads=8, kv=2, dim=32, vdim=48, rot=32, size=100, conv=4), None)], width=128),
               config([(unit(heads=4, kv=1, dim=128, vdim=128, rot=64, size=200), None),
-                      (pair(heads=4, kv=4, dim=96, vdim=192, rot=24, size=90, r_heads=2, r_dim=128, r_vdim=128, cap=15.0), None)], width=128, streams=4)):
+                      (pair(heads=4, kv=4, dim=80, vdim=176, rot=48, size=90, r_heads=2, r_dim=128, r_vdim=128, cap=15.0), None)], width=128, streams=4)):
     w = weights(cfg, seed=8)
     ids = toks(620, cfg["vocab"], seed=3)
     ref = logits(cfg, w, ids)
